@@ -42,6 +42,9 @@ SIGNATURES = {
     "deepj_cuda_synth_fill": (ctypes.c_int, [ctypes.c_int32, ctypes.c_uint64, ctypes.c_uint64, ctypes.c_float, ctypes.c_int64, ctypes.c_int64]),
     "deepj_cuda_kv_alloc": (ctypes.c_int, [ctypes.c_int32] * 6),
     "deepj_cuda_kv_alloc_f16": (ctypes.c_int, [ctypes.c_int32] * 6),
+    "deepj_cuda_bf16_alloc": (ctypes.c_int, [ctypes.c_int32] * 3),
+    "deepj_cuda_bf16_store": (ctypes.c_int, [ctypes.c_int32] * 5 + [ctypes.c_int64] + [ctypes.c_int32] * 2),
+    "deepj_cuda_latent_alloc": (ctypes.c_int, [ctypes.c_int32] * 5),
     "deepj_cuda_tp_create": (ctypes.c_int, [ctypes.c_int32, ctypes.c_int32, ctypes.c_int64, ctypes.c_void_p]),
     "deepj_cuda_decode_plan": (ctypes.c_int, [ctypes.c_int32, ctypes.c_void_p, ctypes.c_int32]),
     "deepj_cuda_tp_configure": (ctypes.c_int, [ctypes.c_int64]),
@@ -60,16 +63,21 @@ class DeepJCudaError(RuntimeError):
     java.lang.RuntimeException in the same place)."""
 
 
-def load() -> ctypes.CDLL:
-    """Load the shared library and bind every declared symbol.  Does not touch a GPU."""
+def load(path: str = "") -> ctypes.CDLL:
+    """Load the shared library and bind every declared symbol.  Does not touch a GPU.  `path`: a library with only some of
+    the parts (deepj_b200/build.py), to be named before anything else loads the full one."""
     global _lib
     if _lib is not None:
         return _lib
-    if not os.path.exists(LIB_PATH):
+    full = path in ("", LIB_PATH)
+    path = path or LIB_PATH
+    if not os.path.exists(path):
         raise DeepJCudaError(
-            f"{LIB_PATH} is missing: build it with `python -m deepj_b200.build` (there is no CPU fallback)")
-    lib = ctypes.CDLL(LIB_PATH)
+            f"{path} is missing: build it with `python -m deepj_b200.build` (there is no CPU fallback)")
+    lib = ctypes.CDLL(path)
     for name, (res, args) in SIGNATURES.items():
+        if not full and not hasattr(lib, name):
+            continue
         fn = getattr(lib, name)
         fn.restype = res
         fn.argtypes = args

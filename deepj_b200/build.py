@@ -2,11 +2,13 @@
 
 `python -m deepj_b200.build` compiles every .cu under deepj_b200/csrc for
 `-gencode arch=compute_100a,code=sm_100a` and links them into
-deepj_b200/libdeepj_cuda_jni.so.  No GPU is needed to build.
+deepj_b200/libdeepj_cuda_jni.so.  No GPU is needed to build.  A command-line tool that serves one model in a checkout
+without a built library compiles only the parts that model needs (`ensure`).
 """
 from __future__ import annotations
 
 import concurrent.futures
+import fcntl
 import os
 import shutil
 import subprocess
@@ -63,24 +65,53 @@ def _compile(src: str, obj: str, headers: list[str], verbose: bool) -> str:
     return res.stderr if verbose else ""
 
 
-def build_cuda(verbose: bool = False) -> str:
+# Kernel files by what they serve.  `core` is the runtime itself; a library holds it and any of the other parts (the
+# interpreter refuses ops whose part is absent).  "*" = everything.
+PARTS = {
+    "core": ["runtime.cu", "misc.cu"],
+    "bf16": ["bf16_linear.cu", "bf16_gemm_tc.cu", "bf16_experts.cu", "delta_rule.cu", "attn_latent.cu"],
+}
+
+
+def _sources(parts: tuple[str, ...]) -> list[str]:
+    if "*" in parts:
+        return sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cu", ".cpp")))
+    return [os.path.join(CSRC, f) for part in ("core",) + parts for f in PARTS[part]]
+
+
+def _headers() -> list[str]:
+    return [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".h", ".cuh"))] + [os.path.join(ROOT, "include", "deepj_cuda.h")]
+
+
+def build_cuda(verbose: bool = False, parts: tuple[str, ...] = ("*",)) -> str:
+    """Compile and link the library of the given parts (default: all of them, LIB) and return its path."""
+    lib = LIB if "*" in parts else os.path.join(PKG_DIR, "libdeepj_cuda_" + "_".join(parts) + ".so")
     os.makedirs(BUILD, exist_ok=True)
-    sources = sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cu", ".cpp")))
-    headers = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".h", ".cuh"))]
-    headers.append(os.path.join(ROOT, "include", "deepj_cuda.h"))
-    objs = [os.path.join(BUILD, os.path.basename(s) + ".o") for s in sources]
-    with concurrent.futures.ThreadPoolExecutor(max_workers=8) as ex:
-        logs = list(ex.map(lambda so: _compile(so[0], so[1], headers, verbose), zip(sources, objs)))
-    if verbose:
-        for log in logs:
-            if log:
-                print(log)
-    if not _newer(LIB, objs):
-        cmd = [_nvcc(), "-shared", "-o", LIB, *objs, "-lcudart"]
-        res = subprocess.run(cmd, capture_output=True, text=True)
-        if res.returncode != 0:
-            raise RuntimeError(f"link failed:\n{res.stdout}\n{res.stderr}")
-    return LIB
+    with open(os.path.join(BUILD, ".lock"), "w") as lock:       # one builder at a time in this checkout
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        sources, headers = _sources(parts), _headers()
+        objs = [os.path.join(BUILD, os.path.basename(s) + ".o") for s in sources]
+        with concurrent.futures.ThreadPoolExecutor(max_workers=8) as ex:
+            logs = list(ex.map(lambda so: _compile(so[0], so[1], headers, verbose), zip(sources, objs)))
+        if verbose:
+            for log in logs:
+                if log:
+                    print(log)
+        if not _newer(lib, objs):
+            cmd = [_nvcc(), "-shared", "-o", lib + ".tmp", *objs, "-lcudart"]
+            res = subprocess.run(cmd, capture_output=True, text=True)
+            if res.returncode != 0:
+                raise RuntimeError(f"link failed:\n{res.stdout}\n{res.stderr}")
+            os.replace(lib + ".tmp", lib)
+    return lib
+
+
+def ensure(parts: tuple[str, ...] = ("*",)) -> str:
+    """Path of a library that holds `parts`: the full one when it is up to date, else one with just these parts, built now
+    if need be."""
+    if _newer(LIB, _sources(("*",)) + _headers()):
+        return LIB
+    return build_cuda(parts=parts)
 
 
 def build_oracle() -> str:

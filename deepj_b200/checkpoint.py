@@ -22,6 +22,7 @@ blocks/GPTTransformerBlock.java:61-63, norm/LayerNorm1D.java:80-82, layers/FNN.j
 """
 from __future__ import annotations
 
+import json
 import os
 from typing import Callable, Dict, List, Tuple, Union
 
@@ -119,3 +120,63 @@ def weight_getter(cfg: DecoderConfig, source: Union[PathLike, List[np.ndarray]])
         a = named[(name, layer if (name, layer) in named else -1)]
         return a.reshape(-1) if a.shape[0] == 1 and name[0] in "gbc" else a
     return get
+
+
+class SafetensorsFile:
+    """Named tensors of a .safetensors file (8-byte little-endian header length, a JSON header name → dtype, shape,
+    data_offsets, then the data).  `get(name)` widens BF16 / F16 / F32 to fp32 and returns I32 tables as they are."""
+
+    def __init__(self, path: PathLike):
+        self._map = np.memmap(path, dtype=np.uint8, mode="r")
+        if self._map.size < 8:
+            raise IOError("safetensors file is shorter than its header length")
+        n = int(self._map[:8].view("<u8")[0])
+        if 8 + n > self._map.size:
+            raise IOError("safetensors file ends inside its header")
+        header = json.loads(bytes(self._map[8:8 + n]))
+        self._base = 8 + n
+        self.header = {name: h for name, h in header.items() if name != "__metadata__"}
+
+    def shape(self, name: str) -> Tuple[int, ...]:
+        if name not in self.header:
+            raise IOError(f"checkpoint has no tensor {name!r}")
+        return tuple(self.header[name]["shape"])
+
+    def get(self, name: str) -> np.ndarray:
+        shape = self.shape(name)
+        h = self.header[name]
+        lo, hi = h["data_offsets"]
+        raw = bytes(self._map[self._base + lo:self._base + hi])
+        kind = h["dtype"]
+        size = {"BF16": 2, "F16": 2, "F32": 4, "I32": 4}.get(kind)
+        if size is None:
+            raise IOError(f"tensor {name!r} has unsupported dtype {kind}")
+        if len(raw) != size * int(np.prod(shape, dtype=np.int64)):
+            raise IOError(f"tensor {name!r} does not fill its shape")
+        if kind == "BF16":
+            a = (np.frombuffer(raw, dtype="<u2").astype(np.uint32) << 16).view(np.float32)
+        elif kind == "I32":
+            a = np.frombuffer(raw, dtype="<i4")
+        else:
+            a = np.frombuffer(raw, dtype="<f2" if kind == "F16" else "<f4").astype(np.float32)
+        return a.reshape(shape)
+
+
+def write_safetensors(path: PathLike, tensors: Dict[str, np.ndarray]) -> None:
+    """The inverse: floating tensors are rounded to BF16, integer ones stored as I32."""
+    header, blobs, at = {}, [], 0
+    for name, a in tensors.items():
+        a = np.asarray(a)
+        if np.issubdtype(a.dtype, np.integer):
+            kind, blob = "I32", a.astype("<i4").tobytes()
+        else:
+            u = a.astype(np.float32).reshape(-1).view(np.uint32)
+            kind, blob = "BF16", ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype("<u2").tobytes()
+        header[name] = {"dtype": kind, "shape": list(a.shape), "data_offsets": [at, at + len(blob)]}
+        blobs.append(blob)
+        at += len(blob)
+    text = json.dumps(header).encode()
+    with open(path, "wb") as f:
+        f.write(np.asarray([len(text)], dtype="<u8").tobytes() + text)
+        for blob in blobs:
+            f.write(blob)

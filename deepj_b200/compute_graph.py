@@ -34,6 +34,8 @@ OP_EMBED_GATHER, OP_Q8_LINEAR, OP_Q8_SWIGLU, OP_ATTN_DECODE = 64, 65, 66, 67
 OP_ARGMAX_ROWS, OP_ADD_SCALAR_INPLACE, OP_COPY = 68, 69, 70
 OP_TP_ALLREDUCE, OP_TP_ALLGATHER = 71, 72
 OP_ATTN_PREFILL, OP_SAMPLE_TOPK, OP_Q8_LINEAR_LN, OP_DECODE_STEP = 73, 74, 75, 76
+# ops over bf16 weights
+OP_BF16_LINEAR, OP_BF16_BLOCK_LINEAR, OP_DELTA_RULE, OP_ATTN_LATENT, OP_TABLE_EXPERTS = 77, 78, 79, 80, 81
 
 # op → (stride, offsets of the slots that hold buffer ids); ComputeGraph.java:89-147
 OP_METADATA: Dict[int, tuple] = {}
@@ -69,6 +71,11 @@ OP_METADATA[OP_ATTN_PREFILL] = (18, (1, 6, 8, 9, 10, 11))
 OP_METADATA[OP_SAMPLE_TOPK] = (8, (1, 2, 3))
 OP_METADATA[OP_Q8_LINEAR_LN] = (17, (1, 4, 5, 7, 8, 9, 12))
 OP_METADATA[OP_DECODE_STEP] = (3, (1,))
+OP_METADATA[OP_BF16_LINEAR] = (29, (1, 4, 7, 11, 14, 15, 18, 24))
+OP_METADATA[OP_BF16_BLOCK_LINEAR] = (12, (1, 5, 7))
+OP_METADATA[OP_DELTA_RULE] = (20, (1, 8, 9, 10, 11, 12, 13))
+OP_METADATA[OP_ATTN_LATENT] = (26, (1, 4, 7, 10, 12, 13, 14, 15, 16))
+OP_METADATA[OP_TABLE_EXPERTS] = (25, (1, 4, 7, 8, 12, 13, 16, 19))
 
 
 def float_bits(value: float) -> int:

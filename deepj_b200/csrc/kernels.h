@@ -1,6 +1,7 @@
 // Launcher declarations shared by the runtime (runtime.cu) and the kernel files.
 // Every launcher enqueues on the given stream and never synchronises.
 #pragma once
+#include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <cstdint>
 #include <cstdlib>
@@ -16,6 +17,10 @@
             throw std::runtime_error(std::string("CUDA error: ") + cudaGetErrorString(_e) + \
                                      " at " + __FILE__ + ":" + std::to_string(__LINE__));   \
     } while (0)
+
+// Launchers of kernel files that a library built for one model family may leave out (build.py); the interpreter
+// refuses their ops with a message when they are absent.
+#define DJ_PART __attribute__((weak))
 
 namespace dj {
 
@@ -46,28 +51,28 @@ struct Q8View {
 };
 
 // ── base ops (ComputeGraph op codes 1-42) ──
-void launch_binary(int op, const float* a, const float* b, float* out, int n, cudaStream_t s);
-void launch_unary(int op, const float* in, float* out, int n, cudaStream_t s);
-void launch_scalar(int op, const float* in, float* out, float v, int n, cudaStream_t s);
-void launch_clamp(const float* in, float* out, float lo, float hi, int n, cudaStream_t s);
-void launch_matmul_f32(const float* a, const float* b, float* out, int m, int n, int k, cudaStream_t s);
-void launch_transpose(const float* in, float* out, int rows, int cols, cudaStream_t s);
-void launch_row_broadcast(int op, const float* a, const float* v, float* out, int rows, int cols, cudaStream_t s);
-void launch_col_broadcast(int op, const float* a, const float* v, float* out, int rows, int cols, cudaStream_t s);
-void launch_row_reduce(int op, const float* in, float* out, int rows, int cols, cudaStream_t s);
-void launch_sum_rows(const float* in, float* out, int rows, int cols, cudaStream_t s);
-void launch_sum_scalar(const float* in, float* out, long long n, cudaStream_t s);
-void launch_softmax_rows(const float* in, float* out, int rows, int cols, cudaStream_t s);
-void launch_softmax_backward(const float* g, const float* sm, float* out, int rows, int cols, cudaStream_t s);
-void launch_layernorm_backward(const float* dxh, const float* xh, const float* sd, float* out, int rows, int cols, cudaStream_t s);
-void launch_adamw(float* w, const float* g, float* mt, float* vt, float lr, float b1, float b2, float eps,
+DJ_PART void launch_binary(int op, const float* a, const float* b, float* out, int n, cudaStream_t s);
+DJ_PART void launch_unary(int op, const float* in, float* out, int n, cudaStream_t s);
+DJ_PART void launch_scalar(int op, const float* in, float* out, float v, int n, cudaStream_t s);
+DJ_PART void launch_clamp(const float* in, float* out, float lo, float hi, int n, cudaStream_t s);
+DJ_PART void launch_matmul_f32(const float* a, const float* b, float* out, int m, int n, int k, cudaStream_t s);
+DJ_PART void launch_transpose(const float* in, float* out, int rows, int cols, cudaStream_t s);
+DJ_PART void launch_row_broadcast(int op, const float* a, const float* v, float* out, int rows, int cols, cudaStream_t s);
+DJ_PART void launch_col_broadcast(int op, const float* a, const float* v, float* out, int rows, int cols, cudaStream_t s);
+DJ_PART void launch_row_reduce(int op, const float* in, float* out, int rows, int cols, cudaStream_t s);
+DJ_PART void launch_sum_rows(const float* in, float* out, int rows, int cols, cudaStream_t s);
+DJ_PART void launch_sum_scalar(const float* in, float* out, long long n, cudaStream_t s);
+DJ_PART void launch_softmax_rows(const float* in, float* out, int rows, int cols, cudaStream_t s);
+DJ_PART void launch_softmax_backward(const float* g, const float* sm, float* out, int rows, int cols, cudaStream_t s);
+DJ_PART void launch_layernorm_backward(const float* dxh, const float* xh, const float* sd, float* out, int rows, int cols, cudaStream_t s);
+DJ_PART void launch_adamw(float* w, const float* g, float* mt, float* vt, float lr, float b1, float b2, float eps,
                   float wd, float bc1, float bc2, int n, cudaStream_t s);
-void launch_scatter_add_rows(float* target, const float* idx, const float* grad, int tRows, int tCols, int nIdx, cudaStream_t s);
-void launch_ce_loss(const float* logits, const float* targets, float* out, int rows, int cols, cudaStream_t s);
-void launch_ce_grad(const float* logits, const float* targets, float* out, int rows, int cols, cudaStream_t s);
+DJ_PART void launch_scatter_add_rows(float* target, const float* idx, const float* grad, int tRows, int tCols, int nIdx, cudaStream_t s);
+DJ_PART void launch_ce_loss(const float* logits, const float* targets, float* out, int rows, int cols, cudaStream_t s);
+DJ_PART void launch_ce_grad(const float* logits, const float* targets, float* out, int rows, int cols, cudaStream_t s);
 
 // ── Q8 ──
-void launch_q8_quantize(const float* src, int src_ld, int K, int n_cols, int8_t* codes, float* scales,
+DJ_PART void launch_q8_quantize(const float* src, int src_ld, int K, int n_cols, int8_t* codes, float* scales,
                         int Kp, int nb, cudaStream_t s);
 struct Q8LinearArgs {
     const float* x; int ldx;            // activations [M × K], row stride ldx
@@ -85,18 +90,18 @@ struct Q8LinearArgs {
     // normalising pass into ln_ws ([M × K] floats) before and an activation pass over `out` after.
     const float* beta = nullptr; int act = 0; float* ln_ws = nullptr;
 };
-void launch_q8_linear(const Q8LinearArgs& a, cudaStream_t s);
-bool launch_q8_gemv_i8(const Q8LinearArgs& a, cudaStream_t s);
-bool launch_q8_gemv_tma(const Q8LinearArgs& a, cudaStream_t s);     // K a multiple of 128; false = outside its domain
-bool q8_gemv_i8_fuses_gpt(const Q8LinearArgs& a);     // true when launch_q8_gemv_i8 can take beta / act itself
-void launch_layernorm_rows(const float* x, int ldx, const float* gamma, const float* beta, float eps, float* out, int K, int M, cudaStream_t s);
-void launch_gelu_rows(float* buf, int ld, int N, int M, cudaStream_t s);
-bool launch_q8_linear_batch(const Q8LinearArgs& a, int m0, int rows, float* ws, int* tickets, cudaStream_t s);
-bool launch_q8_linear_batch_tma(const Q8LinearArgs& a, int m0, int rows, float* ws, int* tickets, cudaStream_t s);   // K a multiple of 128; same workspace
-size_t q8_batch_ws_floats(int K, int N, bool swiglu);
-bool launch_q8_linear_tc(const Q8LinearArgs& a, float* ws, cudaStream_t s);
-size_t q8_tc_ws_floats(int M, int K, int N);     // activation tiles, row scales and, when the reduction is split, the partial outputs
-double q8_tc_estimate_us(int M, int K, int N);
+DJ_PART void launch_q8_linear(const Q8LinearArgs& a, cudaStream_t s);
+DJ_PART bool launch_q8_gemv_i8(const Q8LinearArgs& a, cudaStream_t s);
+DJ_PART bool launch_q8_gemv_tma(const Q8LinearArgs& a, cudaStream_t s);     // K a multiple of 128; false = outside its domain
+DJ_PART bool q8_gemv_i8_fuses_gpt(const Q8LinearArgs& a);     // true when launch_q8_gemv_i8 can take beta / act itself
+DJ_PART void launch_layernorm_rows(const float* x, int ldx, const float* gamma, const float* beta, float eps, float* out, int K, int M, cudaStream_t s);
+DJ_PART void launch_gelu_rows(float* buf, int ld, int N, int M, cudaStream_t s);
+DJ_PART bool launch_q8_linear_batch(const Q8LinearArgs& a, int m0, int rows, float* ws, int* tickets, cudaStream_t s);
+DJ_PART bool launch_q8_linear_batch_tma(const Q8LinearArgs& a, int m0, int rows, float* ws, int* tickets, cudaStream_t s);   // K a multiple of 128; same workspace
+DJ_PART size_t q8_batch_ws_floats(int K, int N, bool swiglu);
+DJ_PART bool launch_q8_linear_tc(const Q8LinearArgs& a, float* ws, cudaStream_t s);
+DJ_PART size_t q8_tc_ws_floats(int M, int K, int N);     // activation tiles, row scales and, when the reduction is split, the partial outputs
+DJ_PART double q8_tc_estimate_us(int M, int K, int N);
 constexpr int kTcMinRows = 17;            // from this many activation rows on, a Q8 linear runs on the tcgen05 path
 
 // ── decode attention ──
@@ -116,10 +121,83 @@ struct AttnDecodeArgs {
     int splits;
 };
 constexpr int kAttnTickets = 1 << 16;
-size_t attn_decode_ws_floats(int B, int H, int hd, int splits);
-int attn_decode_splits(int B, int H, int maxSeq);
-void launch_attn_decode(const AttnDecodeArgs& a, cudaStream_t s);
-bool launch_attn_prefill_mma(const AttnDecodeArgs& a, cudaStream_t s);     // prompt chunks on the tensor cores (head dim 64 / 128)
+DJ_PART size_t attn_decode_ws_floats(int B, int H, int hd, int splits);
+DJ_PART int attn_decode_splits(int B, int H, int maxSeq);
+DJ_PART void launch_attn_decode(const AttnDecodeArgs& a, cudaStream_t s);
+DJ_PART bool launch_attn_prefill_mma(const AttnDecodeArgs& a, cudaStream_t s);     // prompt chunks on the tensor cores (head dim 64 / 128)
+
+// ── projections with bf16 weights (bf16_linear.cu, bf16_gemm_tc.cu) ──
+// A bf16 weight as laid out in HBM: [N][Kp], Kp = K rounded up to 8, zero padded.
+struct Bf16View { const __nv_bfloat16* w; int K, N, Kp; };
+// One segment of an activation row: fp32 values, optionally RMS-normalised in groups and multiplied by sigmoid(gate).
+struct RowOperand {
+    const float* x = nullptr; int ldx = 0; int k = 0;                       // k == 0: no segment
+    const float* gamma = nullptr; int groups = 0; float eps = 0.0f;         // groups == 0: no norm
+    const float* gate = nullptr; int ldg = 0;
+};
+struct Bf16LinearArgs {
+    RowOperand a, b;                           // b starts at weight column pad8(a.k)
+    Bf16View w;
+    const float* residual = nullptr; int ldr = 0;
+    float* out = nullptr; int ldo = 0;         // weight rows [0, gluRow)
+    int gluRow = 0; float limit = 0.0f;        // weight rows [gluRow, N) are (gate, up) pairs → glu, one value per pair
+    float* glu = nullptr; int ldglu = 0;
+    float softcap = 0.0f;                      // > 0: out = softcap · tanh(out / softcap)
+    int M = 0;
+    int exact = 0;                             // 1: fp32 products throughout
+    float* ws = nullptr;                       // bf16_linear_ws_floats
+};
+DJ_PART void launch_bf16_store(const float* src, int rows, int cols, __nv_bfloat16* dst, long long dst_ld, cudaStream_t s);
+DJ_PART const char* bf16_linear_check(const Bf16LinearArgs& a);      // nullptr, or why the shape is not supported
+DJ_PART size_t bf16_linear_ws_floats(const Bf16LinearArgs& a);
+DJ_PART void launch_bf16_linear(const Bf16LinearArgs& a, cudaStream_t s);
+DJ_PART bool launch_bf16_gemm_tc(const Bf16LinearArgs& a, const int* tileExpert, const int* rowMap, cudaStream_t s);
+DJ_PART void launch_stage_rows(const RowOperand& a, const RowOperand& b, int Kp, int rows, const int* map, int div, void* out, bool bf16, cudaStream_t s);
+DJ_PART void launch_bf16_block_linear(const float* x, int ldx, int xstr, const Bf16View& w, int heads, float* out, int ldo, int ostr, int M, cudaStream_t s);
+// Table-routed experts: token id → `top` experts, each of weight 1/top.  up holds every expert's (gate, up) row pairs
+// [experts·2ff][x.k], down [experts·d][ff].
+struct Bf16ExpertArgs {
+    RowOperand x;
+    const float* tok; const float* table; int vocab, top, experts;
+    Bf16View up, down; int ff, d; float limit;
+    const float* residual; int ldr; float* out; int ldo;
+    int M, exact;
+    float* ws;                                 // bf16_experts_ws_floats
+};
+DJ_PART size_t bf16_experts_ws_floats(const Bf16ExpertArgs& e);
+DJ_PART void launch_bf16_experts(const Bf16ExpertArgs& e, cudaStream_t s);
+DJ_PART void launch_bf16_expert_gemv(const Bf16ExpertArgs& e, float* y, cudaStream_t s);
+
+// ── generalized delta rule (delta_rule.cu) ──
+struct DeltaRuleArgs {
+    const float* proj; int ld, r_off, k_off, v_off, a_off, low_off;      // one row per token, heads side by side in every field
+    const float* abias; Bf16View w2; const float* w0;                   // w2 [H·dim][rank]
+    float* state;                              // this layer's [B][H][dim][dim]
+    const float* pos;
+    float* out; int ldo;                       // [rows][H·dim]
+    int B, T, H, dim;
+    float* ws;                                 // delta_rule_ws_floats
+};
+DJ_PART bool delta_rule_fits(int dim, int rank);
+DJ_PART size_t delta_rule_ws_floats(int rows, int H, int dim);
+DJ_PART void launch_delta_rule(const DeltaRuleArgs& a, cudaStream_t s);
+
+// ── latent attention (attn_latent.cu) ──
+struct LatentAttnArgs {
+    const float* q; int ldq;                   // [rows][H·(dim + rot)]
+    const float* qc; int ldqc;                 // [rows][H·R]: the unrotated part taken into the latent space
+    const float* kv; int ldkv;                 // [rows][R + rot]: the new latents (not normed) and key parts (not rotated)
+    const float* gamma; float eps;
+    void* cache; int bf16; int maxSeq;         // this layer's rows [B][maxSeq][R + rot]
+    const float* pos; const float* cosT; const float* sinT;      // [maxSeq × rot/2]
+    float* out; int ldo;                       // [rows][H·R]
+    int B, T, H, dim, rot, R; float scale;
+    float* ws;                                 // latent_attn_ws_floats
+};
+DJ_PART bool latent_attn_fits(int R, int rot);
+DJ_PART int latent_attn_splits(int rows, int H, int maxSeq);
+DJ_PART size_t latent_attn_ws_floats(const LatentAttnArgs& a);
+DJ_PART void launch_latent_attn(const LatentAttnArgs& a, cudaStream_t s);
 
 // ── misc ──
 void launch_embed_gather(const float* table, const float* ids, float* out, int rows, int d, int vocab, cudaStream_t s);
@@ -137,10 +215,10 @@ void launch_synth_fill(float* out, unsigned long long seed, unsigned long long o
                        long long first, long long n, cudaStream_t s);
 
 // ── tensor-parallel exchange over peer memory (tp.cu) ──
-bool tp_ready();
-int tp_world();
+DJ_PART bool tp_ready();
+DJ_PART int tp_world();
 // mode 0: out = residual + bias + Σ_ranks in (all-reduce); mode 1: out[m][r·n_local + j] = in_r[m][j] (all-gather)
-void launch_tp_exchange(const float* in, const float* bias, const float* residual, float* out, int M, int n_local, int mode,
+DJ_PART void launch_tp_exchange(const float* in, const float* bias, const float* residual, float* out, int M, int n_local, int mode,
                         cudaStream_t s);
 
 // Read-only views of the runtime's buffer pool for entry points that live beside their kernels.
@@ -156,8 +234,8 @@ void pool_add_plan(int id, void* dev_ptr, size_t bytes);
 
 // ── whole-token decode kernel (decode_step.cu) ──
 // Validates the plan object behind op 76 and appends the (id, serial) of everything it references to `refs`.
-void decode_step_check(int plan_id, std::vector<std::pair<int, unsigned long long>>* refs);
-void launch_decode_step(int plan_id, int feed_back, cudaStream_t s);
+DJ_PART void decode_step_check(int plan_id, std::vector<std::pair<int, unsigned long long>>* refs);
+DJ_PART void launch_decode_step(int plan_id, int feed_back, cudaStream_t s);
 // The library's stream and device; the stream is null until the library has been initialised.
 cudaStream_t runtime_stream();
 int runtime_device();

@@ -18,8 +18,6 @@
 
 namespace dj {
 
-int g_gemv_mode = 2;   // 2: tensor-pipe kernels (TMA GEMV, cp.async GEMV, batched, tcgen05) with the FMA kernel as the fallback, 1: the same without the TMA GEMV, 0: FMA kernel only
-
 namespace {
 
 // ───────────── quantizer ─────────────

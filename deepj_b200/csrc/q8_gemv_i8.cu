@@ -27,19 +27,6 @@
 
 namespace dj {
 
-int* g_dev_error = nullptr;     // device int, 0 = no bounded wait has ever expired
-
-// Phase tracing (environment DEEPJ_CUDA_TRACE=1): every traced launch gets eight
-// 64-bit slots in a device ring; CTA 0 stamps %globaltimer at its phase boundaries.
-unsigned long long* g_trace = nullptr;
-long long g_trace_launches = 0;
-unsigned long long* trace_slot() {
-    if (!g_trace) return nullptr;
-    unsigned long long* p = g_trace + (size_t)(g_trace_launches % kTraceSlots) * 8;
-    g_trace_launches++;
-    return p;
-}
-
 namespace {
 
 constexpr int kWarps = kGemvWarps;

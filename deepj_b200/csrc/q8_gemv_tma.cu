@@ -237,25 +237,6 @@ void launch_tma(const GemvTmaParams& p, cudaStream_t s) {
 
 }  // namespace
 
-using EncodeTiledFn = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                   const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                   CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-// The driver's tensor-map encoder, looked up through the runtime so that the library carries no link-time
-// dependency on the driver (it must load on machines without one).
-static EncodeTiledFn encode_tiled_fn() {
-    static EncodeTiledFn fn = []() -> EncodeTiledFn {
-        void* sym = nullptr;
-        cudaDriverEntryPointQueryResult q;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &sym, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess) {
-            cudaGetLastError();
-            return nullptr;
-        }
-        return reinterpret_cast<EncodeTiledFn>(sym);
-    }();
-    return fn;
-}
-
 // Tensor maps over one Q8 weight: codes [N][Kp] bytes in boxes of 8 rows × 128 bytes (128-byte swizzle) and
 // scales [N][nb] floats in boxes of 8 rows × 4.
 bool q8_encode_weight_maps(const Q8View& w, CUtensorMap* codes, CUtensorMap* scales) {

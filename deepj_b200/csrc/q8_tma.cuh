@@ -34,6 +34,11 @@ __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) {
 // exact for |v| < 2^22: the integer lands in the mantissa of 1.5 · 2^23
 __device__ __forceinline__ float int_to_float_exact(int v) { return __int_as_float(v + 0x4B400000) - 12582912.0f; }
 
+using EncodeTiledFn = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                                   const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
+                                   CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+EncodeTiledFn encode_tiled_fn();      // nullptr when the driver has none (runtime.cu)
+
 // Tensor maps over one Q8 weight: codes [N][Kp] bytes in boxes of 8 rows × 128 bytes (128-byte swizzle) and scales
 // [N][nb] floats in boxes of 8 rows × 4.  False when the driver's encoder is missing or the layout does not qualify
 // (16-byte aligned bases and row pitches).

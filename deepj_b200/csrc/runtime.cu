@@ -7,6 +7,7 @@
 // native/deepj_metal_jni.mm:1554-2140.
 #include "../../include/deepj_cuda.h"
 #include "kernels.h"
+#include "q8_tma.cuh"
 
 #include <cmath>
 #include <cstring>
@@ -18,6 +19,34 @@ namespace dj {
 long long g_launches = 0;
 int g_num_sms = 148;
 bool g_use_pdl = true;
+int g_gemv_mode = 2;   // 2: tensor-pipe kernels (TMA GEMV, cp.async GEMV, batched, tcgen05) with the FMA kernel as the fallback, 1: the same without the TMA GEMV, 0: FMA kernel only
+int* g_dev_error = nullptr;     // device int, 0 = no bounded wait has ever expired
+
+// Phase tracing (environment DEEPJ_CUDA_TRACE=1): every traced launch gets eight
+// 64-bit slots in a device ring; CTA 0 stamps %globaltimer at its phase boundaries.
+unsigned long long* g_trace = nullptr;
+long long g_trace_launches = 0;
+unsigned long long* trace_slot() {
+    if (!g_trace) return nullptr;
+    unsigned long long* p = g_trace + (size_t)(g_trace_launches % kTraceSlots) * 8;
+    g_trace_launches++;
+    return p;
+}
+
+// The driver's tensor-map encoder, looked up through the runtime so that the library carries no link-time
+// dependency on the driver (it must load on machines without one).
+EncodeTiledFn encode_tiled_fn() {
+    static EncodeTiledFn fn = []() -> EncodeTiledFn {
+        void* sym = nullptr;
+        cudaDriverEntryPointQueryResult q;
+        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &sym, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess) {
+            cudaGetLastError();
+            return nullptr;
+        }
+        return reinterpret_cast<EncodeTiledFn>(sym);
+    }();
+    return fn;
+}
 }  // namespace dj
 
 namespace {
@@ -26,14 +55,14 @@ using namespace dj;
 
 thread_local std::string g_err;
 
-enum BufKind { kF32 = 0, kQ8 = 1, kKV = 2, kPlan = 3 };
+enum BufKind { kF32 = 0, kQ8 = 1, kKV = 2, kPlan = 3, kBf16 = 4, kLatent = 5 };
 struct Buf {
     BufKind kind = kF32;
     void* ptr = nullptr;
     size_t bytes = 0;
     size_t floats = 0;                 // kF32
-    int K = 0, N = 0, Kp = 0, nb = 0;  // kQ8
-    int layers = 0, B = 0, H = 0, maxSeq = 0, hd = 0, kvHalf = 0;   // kKV (kvHalf: fp16 elements)
+    int K = 0, N = 0, Kp = 0, nb = 0;  // kQ8, kBf16
+    int layers = 0, B = 0, H = 0, maxSeq = 0, hd = 0, kvHalf = 0;   // kKV (kvHalf: fp16 elements), kLatent (B, maxSeq, hd = row width; kvHalf: bf16 elements)
     unsigned long long serial = 0;
 };
 
@@ -148,6 +177,38 @@ Q8View q8view(const Buf& b) {
     return v;
 }
 
+Bf16View bf16view(const Buf& b) {
+    Bf16View v;
+    v.w = (const __nv_bfloat16*)b.ptr; v.K = b.K; v.N = b.N; v.Kp = b.Kp;
+    return v;
+}
+// A row operand of a bf16-weight projection: `rows` rows of k values at (id, off, ld), an optional norm and gate.
+RowOperand row_operand(Ctx& c, int rows, int k, int id, int off, int ld, int gamma, int groups, float eps, int gate, int g_off, int ldg, const char* what) {
+    require(k >= 1 && off >= 0 && g_off >= 0 && groups >= 0 && ld >= k, what, "bad activation row");
+    require((groups > 0) == (gamma >= 0), what, "a norm needs both a gain and a group count");
+    RowOperand o;
+    o.x = f32(c, id, (size_t)off + (size_t)(rows - 1) * ld + k, what) + off; o.ldx = ld; o.k = k;
+    o.gamma = f32_opt(c, gamma, k, what); o.groups = groups; o.eps = eps;
+    if (gate >= 0) {
+        require(ldg >= k, what, "gate stride smaller than the row");
+        o.gate = f32(c, gate, (size_t)g_off + (size_t)(rows - 1) * ldg + k, what) + g_off; o.ldg = ldg;
+    }
+    return o;
+}
+
+// Kernel files that a library built for one model family may leave out: their launchers are weak symbols.
+template <typename F> void part(F* launcher, const char* what) {
+    if (launcher == nullptr) throw std::runtime_error(std::string(what) + ": this library was built without these kernels (python -m deepj_b200.build builds all)");
+}
+void check_part(int op) {
+    if (op <= 42) part(launch_binary, "base op");
+    else if (op == DEEPJ_OP_Q8_LINEAR || op == DEEPJ_OP_Q8_LINEAR_LN || op == DEEPJ_OP_Q8_SWIGLU) part(launch_q8_linear, "Q8 projection");
+    else if (op == DEEPJ_OP_ATTN_DECODE || op == DEEPJ_OP_ATTN_PREFILL) part(launch_attn_decode, "attention");
+    else if (op == DEEPJ_OP_TP_ALLREDUCE || op == DEEPJ_OP_TP_ALLGATHER) part(launch_tp_exchange, "tensor-parallel exchange");
+    else if (op == DEEPJ_OP_DECODE_STEP) part(launch_decode_step, "whole-token kernel");
+    else if (op >= DEEPJ_OP_BF16_LINEAR) part(launch_bf16_linear, "bf16 projections and their mixers");
+}
+
 int op_stride(int op) {
     switch (op) {
         case 7: case 8: case 9: case 10: case 11: case 12: case 13: case 15: return 4;
@@ -170,6 +231,11 @@ int op_stride(int op) {
         case DEEPJ_OP_TP_ALLREDUCE: return 7;
         case DEEPJ_OP_TP_ALLGATHER: return 5;
         case DEEPJ_OP_DECODE_STEP: return 3;
+        case DEEPJ_OP_BF16_LINEAR: return 29;
+        case DEEPJ_OP_BF16_BLOCK_LINEAR: return 12;
+        case DEEPJ_OP_DELTA_RULE: return 20;
+        case DEEPJ_OP_ATTN_LATENT: return 26;
+        case DEEPJ_OP_TABLE_EXPERTS: return 25;
         default: return -1;
     }
 }
@@ -181,6 +247,11 @@ void do_op(Ctx& ctx, const int32_t* c) {
     const int op = c[0];
     cudaStream_t s = ctx.s;
     const bool go = ctx.execute;
+    check_part(op);
+    auto scratch = [&](size_t floats) {          // room in the shared workspace for this op
+        if (floats > ctx.ws_need) ctx.ws_need = floats;
+        return R.ws;
+    };
     switch (op) {
         case 1: case 2: case 3: case 4: case 14: case 16: {
             int n = c[4]; require(n >= 0, "binary op", "negative element count");
@@ -448,6 +519,125 @@ void do_op(Ctx& ctx, const int32_t* c) {
             decode_step_check(c[1], ctx.refs);
             if (tp_world() > 1) ctx.bounded_waits = true;
             if (go) launch_decode_step(c[1], c[2], s);
+            break;
+        }
+        case DEEPJ_OP_BF16_LINEAR: {
+            // [op, x, x_off, ldx, gamma, groups, epsBits, gate, g_off, ldg, k1, x2, x2_off, ldx2, w, residual, res_off, ldr, out, out_off, ldo, M,
+            //  glu_row, limitBits, glu, glu_off, ldglu, softcapBits, exact]
+            const char* what = "bf16Linear";
+            Buf& wb = find_buf(ctx, c[14], kBf16, what);
+            const int k1 = c[10], M = c[21], N = wb.N, k2 = c[11] >= 0 ? wb.K - (k1 + 7) / 8 * 8 : 0;
+            require(M >= 1 && k1 >= 1 && (c[11] >= 0 ? k2 >= 1 : wb.K == k1), what, "the segments do not add up to the reduction length");
+            Bf16LinearArgs a;
+            a.a = row_operand(ctx, M, k1, c[1], c[2], c[3], c[4], c[5], bits_to_float(c[6]), c[7], c[8], c[9], what);
+            if (c[11] >= 0) a.b = row_operand(ctx, M, k2, c[11], c[12], c[13], -1, 0, 0.0f, -1, 0, 0, what);
+            a.w = bf16view(wb);
+            a.gluRow = c[22]; a.limit = bits_to_float(c[23]); a.softcap = bits_to_float(c[27]); a.exact = c[28]; a.M = M;
+            require(a.gluRow >= 0 && a.gluRow <= N && (a.gluRow == N || (a.gluRow % 8 == 0 && (N - a.gluRow) % 2 == 0)), what, "bad first gated row");
+            require(a.exact == 0 || a.exact == 1, what, "exact must be 0 or 1");
+            if (a.gluRow > 0) {
+                require(c[20] >= a.gluRow && c[19] >= 0, what, "row stride smaller than the row");
+                a.out = f32(ctx, c[18], (size_t)c[19] + sz(M - 1, c[20]) + a.gluRow, what) + c[19]; a.ldo = c[20];
+                if (c[15] >= 0) {
+                    require(c[17] >= a.gluRow && c[16] >= 0, what, "residual stride smaller than the row");
+                    a.residual = f32(ctx, c[15], (size_t)c[16] + sz(M - 1, c[17]) + a.gluRow, what) + c[16]; a.ldr = c[17];
+                }
+            }
+            if (a.gluRow < N) {
+                const int n = (N - a.gluRow) / 2;
+                require(c[26] >= n && c[25] >= 0, what, "row stride smaller than the gated row");
+                a.glu = f32(ctx, c[24], (size_t)c[25] + sz(M - 1, c[26]) + n, what) + c[25]; a.ldglu = c[26];
+            }
+            if (const char* msg = bf16_linear_check(a)) require(false, what, msg);
+            a.ws = scratch(bf16_linear_ws_floats(a));
+            if (go) launch_bf16_linear(a, s);
+            break;
+        }
+        case DEEPJ_OP_BF16_BLOCK_LINEAR: {   // [op, x, x_off, ldx, xstr, w, heads, out, out_off, ldo, ostr, M]
+            const char* what = "bf16BlockLinear";
+            Buf& wb = find_buf(ctx, c[5], kBf16, what);
+            const int x_off = c[2], ldx = c[3], xstr = c[4], heads = c[6], out_off = c[8], ldo = c[9], ostr = c[10], M = c[11];
+            require(M >= 1 && heads >= 1 && wb.N % heads == 0 && x_off >= 0 && out_off >= 0 && xstr >= 0 && ostr >= 0, what, "bad dimension");
+            const size_t xrow = sz(heads - 1, xstr) + wb.K, orow = sz(heads - 1, ostr) + wb.N / heads;
+            require((size_t)ldx >= xrow && (size_t)ldo >= orow && ostr >= wb.N / heads, what, "row stride smaller than the row");
+            require(wb.Kp <= 3072 && heads <= 65535, what, "slice too long");
+            const float* x = f32(ctx, c[1], (size_t)x_off + sz(M - 1, ldx) + xrow, what) + x_off;
+            float* o = f32(ctx, c[7], (size_t)out_off + sz(M - 1, ldo) + orow, what) + out_off;
+            if (go) launch_bf16_block_linear(x, ldx, xstr, bf16view(wb), heads, o, ldo, ostr, M, s);
+            break;
+        }
+        case DEEPJ_OP_DELTA_RULE: {
+            // [op, proj, r_off, k_off, v_off, a_off, low_off, ld, abias, w2, w0, state, pos, out, out_off, ldo, B, T, H, dim]
+            const char* what = "deltaRule";
+            const int ld = c[7], B = c[16], T = c[17], H = c[18], dim = c[19];
+            require(B >= 1 && T >= 1 && H >= 1 && (long)B * T <= 65535 * 8L && H <= 65535 && B <= 65535, what, "bad dimension");
+            Buf& w2 = find_buf(ctx, c[9], kBf16, what);
+            require(delta_rule_fits(dim, w2.K), what, "head size or decay rank not supported");
+            require(w2.N == H * dim, what, "the decay projection does not match the heads");
+            const int rows = B * T, HD = H * dim;
+            int last = std::max(c[6] + w2.K, HD + std::max(std::max(c[2], c[3]), std::max(c[4], c[5])));
+            require(c[2] >= 0 && c[3] >= 0 && c[4] >= 0 && c[5] >= 0 && c[6] >= 0 && c[14] >= 0 && ld >= last && c[15] >= HD, what, "bad offset or stride");
+            DeltaRuleArgs a;
+            a.proj = f32(ctx, c[1], sz(rows - 1, ld) + last, what); a.ld = ld;
+            a.r_off = c[2]; a.k_off = c[3]; a.v_off = c[4]; a.a_off = c[5]; a.low_off = c[6];
+            a.abias = f32(ctx, c[8], HD, what); a.w2 = bf16view(w2); a.w0 = f32(ctx, c[10], HD, what);
+            a.state = f32(ctx, c[11], sz(B, HD) * dim, what); a.pos = f32(ctx, c[12], B, what);
+            a.out = f32(ctx, c[13], (size_t)c[14] + sz(rows - 1, c[15]) + HD, what) + c[14]; a.ldo = c[15];
+            a.B = B; a.T = T; a.H = H; a.dim = dim;
+            a.ws = scratch(delta_rule_ws_floats(rows, H, dim));
+            if (go) launch_delta_rule(a, s);
+            break;
+        }
+        case DEEPJ_OP_ATTN_LATENT: {
+            // [op, q, q_off, ldq, qc, qc_off, ldqc, kv, kv_off, ldkv, gamma, epsBits, cache, pos, cos, sin, out, out_off, ldo, B, T, H, dim, rot, R, scaleBits]
+            const char* what = "attnLatent";
+            LatentAttnArgs a;
+            a.B = c[19]; a.T = c[20]; a.H = c[21]; a.dim = c[22]; a.rot = c[23]; a.R = c[24]; a.scale = bits_to_float(c[25]);
+            require(a.B >= 1 && a.T >= 1 && a.H >= 1 && a.dim >= 1 && (long)a.B * a.T <= 65535, what, "bad dimension");
+            require(latent_attn_fits(a.R, a.rot), what, "latent or rotated size not supported");
+            Buf& lc = find_buf(ctx, c[12], kLatent, what);
+            require(lc.hd == a.R + a.rot && a.B <= lc.B, what, "shape does not match the cache");
+            const int rows = a.B * a.T, qw = a.H * (a.dim + a.rot), cw = a.H * a.R;
+            require(c[2] >= 0 && c[5] >= 0 && c[8] >= 0 && c[17] >= 0 && c[3] >= qw && c[6] >= cw && c[9] >= a.R + a.rot && c[18] >= cw, what, "bad offset or stride");
+            a.q = f32(ctx, c[1], (size_t)c[2] + sz(rows - 1, c[3]) + qw, what) + c[2]; a.ldq = c[3];
+            a.qc = f32(ctx, c[4], (size_t)c[5] + sz(rows - 1, c[6]) + cw, what) + c[5]; a.ldqc = c[6];
+            a.kv = f32(ctx, c[7], (size_t)c[8] + sz(rows - 1, c[9]) + a.R + a.rot, what) + c[8]; a.ldkv = c[9];
+            a.gamma = f32(ctx, c[10], a.R, what); a.eps = bits_to_float(c[11]);
+            a.cache = lc.ptr; a.bf16 = lc.kvHalf; a.maxSeq = lc.maxSeq;
+            a.pos = f32(ctx, c[13], a.B, what);
+            a.cosT = f32(ctx, c[14], sz(lc.maxSeq, a.rot / 2), what); a.sinT = f32(ctx, c[15], sz(lc.maxSeq, a.rot / 2), what);
+            a.out = f32(ctx, c[16], (size_t)c[17] + sz(rows - 1, c[18]) + cw, what) + c[17]; a.ldo = c[18];
+            a.ws = scratch(latent_attn_ws_floats(a));
+            if (go) launch_latent_attn(a, s);
+            break;
+        }
+        case DEEPJ_OP_TABLE_EXPERTS: {
+            // [op, x, x_off, ldx, gamma, groups, epsBits, tok, table, vocab, top, experts, w_up, w_down, ff, limitBits, residual, res_off, ldr,
+            //  out, out_off, ldo, d, M, exact]
+            const char* what = "tableExperts";
+            Bf16ExpertArgs e;
+            e.vocab = c[9]; e.top = c[10]; e.experts = c[11]; e.ff = c[14]; e.limit = bits_to_float(c[15]); e.d = c[22]; e.M = c[23]; e.exact = c[24];
+            Buf& up = find_buf(ctx, c[12], kBf16, what);
+            Buf& down = find_buf(ctx, c[13], kBf16, what);
+            require(e.M >= 1 && e.vocab >= 1 && e.top >= 1 && e.experts >= e.top && e.ff >= 1 && e.d >= 1, what, "bad dimension");
+            require((long long)e.experts * 2 * e.ff == up.N && (long long)e.experts * e.d == down.N && down.K == e.ff, what, "expert weights do not match");
+            require((long)e.M * e.top <= 65535, what, "too many entries");
+            e.x = row_operand(ctx, e.M, up.K, c[1], c[2], c[3], c[4], c[5], bits_to_float(c[6]), -1, 0, 0, what);
+            e.tok = f32(ctx, c[7], e.M, what); e.table = f32(ctx, c[8], sz(e.vocab, e.top), what);
+            e.up = bf16view(up); e.down = bf16view(down);
+            require(c[20] >= 0 && c[21] >= e.d, what, "row stride smaller than the row");
+            e.residual = nullptr; e.ldr = 0;
+            if (c[16] >= 0) {
+                require(c[17] >= 0 && c[18] >= e.d, what, "residual stride smaller than the row");
+                e.residual = f32(ctx, c[16], (size_t)c[17] + sz(e.M - 1, c[18]) + e.d, what) + c[17]; e.ldr = c[18];
+            }
+            e.out = f32(ctx, c[19], (size_t)c[20] + sz(e.M - 1, c[21]) + e.d, what) + c[20]; e.ldo = c[21];
+            Bf16LinearArgs probe;
+            probe.a = e.x; probe.w = e.up;
+            if (const char* msg = bf16_linear_check(probe)) require(false, what, msg);
+            require((size_t)e.top * (down.Kp + 255) / 256 * 1024 <= 200 * 1024, what, "expert feed-forward too wide");
+            e.ws = scratch(bf16_experts_ws_floats(e));
+            if (go) launch_bf16_experts(e, s);
             break;
         }
         default:
@@ -789,6 +979,7 @@ int deepj_cuda_q8_quantize_into(int32_t q8_id, int32_t dst_col0, int32_t src_id,
     Buf& q = find_buf(c, q8_id, kQ8, "q8_quantize_into");
     if (dst_col0 < 0 || n_cols < 0 || dst_col0 + n_cols > q.N) throw std::runtime_error("q8_quantize_into: destination columns out of range");
     if (src_row0 < 0 || src_col0 < 0 || src_ld < src_col0 + n_cols) throw std::runtime_error("q8_quantize_into: source window out of range");
+    part(launch_q8_quantize, "q8_quantize_into");
     const float* src = f32(c, src_id, (size_t)(src_row0 + q.K - 1) * src_ld + src_col0 + n_cols, "q8_quantize_into");
     Q8View v = q8view(q);
     launch_q8_quantize(src + (size_t)src_row0 * src_ld + src_col0, src_ld, q.K, n_cols,
@@ -840,6 +1031,48 @@ static int kv_alloc_impl(int32_t id, int32_t layers, int32_t batch, int32_t head
     b.kvHalf = half;
     if (half && head_dim % 16 != 0) throw std::runtime_error("kv_alloc: an fp16 cache needs a head dim that is a multiple of 16");
     b.bytes = plane * 2 * (half ? 2 : 4);
+    DJ_CUDA_CHECK(cudaMalloc(&b.ptr, b.bytes));
+    DJ_CUDA_CHECK(cudaMemsetAsync(b.ptr, 0, b.bytes, R.stream));
+    b.serial = R.next_serial++;
+    R.pool[id] = b;
+    DJ_CATCH
+}
+
+int deepj_cuda_bf16_alloc(int32_t id, int32_t K, int32_t N) {
+    DJ_TRY
+    ensure_init();
+    if (K <= 0 || N <= 0) throw std::runtime_error("bf16_alloc: K and N must be positive");
+    if (R.pool.count(id)) throw std::runtime_error("bf16_alloc: id " + std::to_string(id) + " already exists");
+    Buf b; b.kind = kBf16; b.K = K; b.N = N; b.Kp = (K + 7) / 8 * 8;
+    b.bytes = (size_t)N * b.Kp * 2;
+    DJ_CUDA_CHECK(cudaMalloc(&b.ptr, b.bytes));
+    DJ_CUDA_CHECK(cudaMemsetAsync(b.ptr, 0, b.bytes, R.stream));
+    b.serial = R.next_serial++;
+    R.pool[id] = b;
+    DJ_CATCH
+}
+
+int deepj_cuda_bf16_store(int32_t id, int32_t row0, int32_t row_step, int32_t col0, int32_t src_id, int64_t src_off, int32_t rows, int32_t cols) {
+    DJ_TRY
+    ensure_init();
+    Ctx c; c.execute = false; c.s = R.stream;
+    Buf& w = find_buf(c, id, kBf16, "bf16_store");
+    part(launch_bf16_store, "bf16_store");
+    if (rows < 0 || cols < 0 || row0 < 0 || row_step < 1 || col0 < 0 || src_off < 0 || col0 + cols > w.K ||
+        (rows > 0 && (long long)row0 + (long long)(rows - 1) * row_step >= w.N))
+        throw std::runtime_error("bf16_store: window out of range");
+    const float* src = f32(c, src_id, (size_t)src_off + (size_t)rows * cols, "bf16_store") + src_off;
+    launch_bf16_store(src, rows, cols, (__nv_bfloat16*)w.ptr + (size_t)row0 * w.Kp + col0, (long long)row_step * w.Kp, R.stream);
+    DJ_CATCH
+}
+
+int deepj_cuda_latent_alloc(int32_t id, int32_t batch, int32_t max_seq, int32_t width, int32_t bf16) {
+    DJ_TRY
+    ensure_init();
+    if (batch <= 0 || max_seq <= 0 || width <= 0 || (bf16 != 0 && bf16 != 1)) throw std::runtime_error("latent_alloc: bad dimensions");
+    if (R.pool.count(id)) throw std::runtime_error("latent_alloc: id " + std::to_string(id) + " already exists");
+    Buf b; b.kind = kLatent; b.B = batch; b.maxSeq = max_seq; b.hd = width; b.kvHalf = bf16;
+    b.bytes = (size_t)batch * max_seq * width * (bf16 ? 2 : 4);
     DJ_CUDA_CHECK(cudaMalloc(&b.ptr, b.bytes));
     DJ_CUDA_CHECK(cudaMemsetAsync(b.ptr, 0, b.bytes, R.stream));
     b.serial = R.next_serial++;

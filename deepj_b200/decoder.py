@@ -27,6 +27,7 @@ from typing import Tuple, Callable, Dict, List, Optional
 import numpy as np
 
 from . import _lib
+from .runner import StreamDecoder
 from .compute_graph import (OP_ADD, OP_DECODE_STEP, OP_Q8_LINEAR_LN, OP_ADD_SCALAR_INPLACE, OP_ARGMAX_ROWS, OP_ATTN_DECODE, OP_ATTN_PREFILL, OP_COPY, OP_EMBED_GATHER, OP_SAMPLE_TOPK,
                             OP_Q8_LINEAR, OP_Q8_SWIGLU, OP_TP_ALLGATHER, OP_TP_ALLREDUCE, float_bits)
 
@@ -113,6 +114,23 @@ def rope_tables(head_dim: int, max_seq: int):
     return cos, sin
 
 
+def scaled_rope_tables(dims: int, max_seq: int, base: float, scaling=None):
+    """cos/sin tables of rotary pairs (2i, 2i+1) with f_i = base^(-2i/dims); `scaling` (factor, original, fast, slow) blends
+    f_i with f_i / factor over the pairs between those that turn `fast` and `slow` times in `original` positions and
+    multiplies both tables by 0.1·ln(factor) + 1 (YaRN).  Angles are formed in double and rounded once."""
+    i = np.arange(dims // 2, dtype=np.float64)
+    f, gain = np.float64(base) ** (-2.0 * i / dims), 1.0
+    if scaling is not None:
+        def turning(turns):
+            return dims * math.log(scaling["original"] / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+        lo, hi = max(math.floor(turning(scaling["fast"])), 0), min(math.ceil(turning(scaling["slow"])), dims - 1)
+        ramp = np.clip((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+        f = f / scaling["factor"] * ramp + f * (1.0 - ramp)
+        gain = 0.1 * math.log(scaling["factor"]) + 1.0
+    angle = np.arange(max_seq, dtype=np.float64)[:, None] * f[None, :]
+    return (np.cos(angle) * gain).astype(np.float32), (np.sin(angle) * gain).astype(np.float32)
+
+
 def shard_plan(cfg: DecoderConfig, rank: int, world: int) -> List[tuple]:
     """(device object, K_local, [(reference name, first row, first column, columns)]) of one block for
     one tensor-parallel rank.  Megatron-style split: Wq/Wk/Wv (or MLA's up-projections), gate and up
@@ -135,12 +153,8 @@ def shard_plan(cfg: DecoderConfig, rank: int, world: int) -> List[tuple]:
                    ("Wu", d, [("Wu", 0, r * Fl, Fl)]), ("Wd", Fl, [("Wd", r * Fl, 0, d)])]
 
 
-class Q8Decoder:
-    """Owns the device-side weights, KV cache and the per-token command stream.
-
-    Buffer ids are taken from `id_base` upwards so they never collide with the ids a
-    `ComputeGraph` hands out (those start at 0).
-    """
+class Q8Decoder(StreamDecoder):
+    """The Q8 families (Llama, DeepSeek, GPT): weights, KV cache and the streams of a token step and a prompt chunk."""
 
     def __init__(self, cfg: DecoderConfig, batch: int = 1, device: int = 0, id_base: int = 1 << 24,
                  tp_rank: int = 0, tp_world: int = 1, tp_slot_floats: int = 0, share_weights: Optional["Q8Decoder"] = None,
@@ -154,8 +168,6 @@ class Q8Decoder:
         Under tensor parallelism the plan is made at the first step, after `tp.connect`.
         `kv_dtype`: "f32" (the reference's precision) or "f16" — keys rounded after the rotation, values rounded, fp32
         arithmetic; half the bytes a step's attention reads."""
-        self.cfg = cfg
-        self.B = int(batch)
         if kv_dtype not in ("f32", "f16"):
             raise ValueError("kv_dtype must be 'f32' or 'f16'")
         if kv_dtype == "f16" and (fused_step or cfg.head_dim % 16 != 0):
@@ -176,20 +188,7 @@ class Q8Decoder:
         self.v_local = cfg.vocab_size // tp_world
         self._ref_shapes = {n: (k, w) for n, k, w in cfg.matmul_shapes()}
         self._ref_shapes["Wlm"] = (cfg.d_model, cfg.vocab_size)
-        self.lib = _lib.load()
-        _lib.check(self.lib.deepj_cuda_init(device))
-        self._next_id = id_base
-        self._owned: List[int] = []
-        self.ids: Dict[str, int] = {}
-        self.loaded = False
-        self._stream_host: Optional[np.ndarray] = None
-        self._stream_dev: Optional[np.ndarray] = None
-        self._op_labels: List[str] = []
-        self._pin_ptr = None
-        self._prefill_ids: Dict[str, int] = {}
-        self._prefill_cap = 0
-        self._prefill_streams: Dict[int, np.ndarray] = {}
-        self.position = 0
+        super().__init__(cfg, batch, device, id_base)
         self._plan_id: Optional[int] = None
         if fused_step and not self.fused_step_eligible(cfg, self.B, tp_world):
             raise ValueError("this configuration does not qualify for the single-kernel token step")
@@ -212,40 +211,7 @@ class Q8Decoder:
         ks = (cfg.d_model, cfg.d_model // tp_world, cfg.d_ff // tp_world)
         return all(k % 32 == 0 for k in ks) and max(ks) <= 16384
 
-    # ── id / buffer helpers ──
-    def _new_id(self) -> int:
-        i = self._next_id
-        self._next_id += 1
-        self._owned.append(i)
-        return i
-
-    def _f32(self, name: str, n: int, data: Optional[np.ndarray] = None) -> int:
-        i = self._new_id()
-        ids = (ctypes.c_int32 * 1)(i)
-        sizes = (ctypes.c_int32 * 1)(n)
-        _lib.check(self.lib.deepj_cuda_alloc_buffers(ids, sizes, 1))
-        if data is not None:
-            self._upload(i, data)
-        if name:
-            self.ids[name] = i
-        return i
-
-    def _upload(self, buf_id: int, data: np.ndarray) -> None:
-        data = np.ascontiguousarray(data, dtype=np.float32)
-        _lib.check(self.lib.deepj_cuda_upload_buffer(buf_id, data.ctypes.data, data.size))
-
-    def _download(self, buf_id: int, n: int) -> np.ndarray:
-        out = np.empty(n, dtype=np.float32)
-        _lib.check(self.lib.deepj_cuda_download_buffer(buf_id, out.ctypes.data, n))
-        return out
-
-    def _release(self, ids: List[int]) -> None:
-        arr = (ctypes.c_int32 * len(ids))(*ids)
-        _lib.check(self.lib.deepj_cuda_release_buffers(arr, len(ids)))
-        for i in ids:
-            if i in self._owned:
-                self._owned.remove(i)
-
+    # ── buffers ──
     def _alloc_state(self) -> None:
         c, B = self.cfg, self.B
         d = c.d_model
@@ -471,15 +437,11 @@ class Q8Decoder:
     def _streams(self):
         if not self.loaded:
             raise RuntimeError("weights are not loaded")
-        if self._stream_host is None:
-            if self.fused_step:
-                plan = self._decode_plan()
-                self._stream_dev = np.asarray([OP_DECODE_STEP, plan, 1], dtype=np.int32)
-                self._stream_host = np.asarray([OP_DECODE_STEP, plan, 0], dtype=np.int32)
-            else:
-                self._stream_dev = self._build(feed_back=True)
-                self._stream_host = self._build(feed_back=False)
-        return self._stream_host, self._stream_dev
+        if self._stream_host is None and self.fused_step:
+            plan = self._decode_plan()
+            self._stream_dev = np.asarray([OP_DECODE_STEP, plan, 1], dtype=np.int32)
+            self._stream_host = np.asarray([OP_DECODE_STEP, plan, 0], dtype=np.int32)
+        return super()._streams()
 
     def _decode_plan(self) -> int:
         """The plan object behind op 76: every buffer and weight of a token step, resolved once by the library."""
@@ -499,79 +461,13 @@ class Q8Decoder:
         return self._plan_id
 
     # ── stepping ──
-    def reset(self) -> None:
-        """Start every sequence at position 0 (cache contents are overwritten as it refills)."""
-        self._upload(self.ids["pos"], np.zeros(self.B, dtype=np.float32))
-        self.position = 0
-
-    def set_position(self, position: int) -> None:
-        """Rewind (or advance) every sequence to `position`; cache rows at and beyond it are
-        overwritten by the following steps."""
-        if position < 0 or position > self.cfg.max_seq_len:
-            raise ValueError(f"position {position} outside 0..{self.cfg.max_seq_len}")
-        self._upload(self.ids["pos"], np.full(self.B, float(position), dtype=np.float32))
-        self.position = int(position)
-
-    def _pinned(self) -> Tuple[np.ndarray, np.ndarray]:
-        """Page-locked staging for the ids going up and the picks coming down each step ([B] floats each)."""
-        if self._pin_ptr is None:
-            ptr = ctypes.c_void_p()
-            _lib.check(self.lib.deepj_cuda_pinned_alloc(ctypes.byref(ptr), 8 * self.B))
-            self._pin_ptr = ptr
-            buf = (ctypes.c_float * (2 * self.B)).from_address(ptr.value)
-            arr = np.frombuffer(buf, dtype=np.float32)
-            self._pin_tok, self._pin_next = arr[:self.B], arr[self.B:]
-        return self._pin_tok, self._pin_next
-
-    def set_tokens(self, tokens) -> None:
-        t = np.asarray(tokens, dtype=np.int64).reshape(-1)
-        if t.size != self.B:
-            raise ValueError(f"expected {self.B} token ids, got {t.size}")
-        # Embedding.forward range check (transformer/embeddings/Embedding.java:30-32)
-        if t.min() < 0 or t.max() >= self.cfg.vocab_size:
-            bad = t[(t < 0) | (t >= self.cfg.vocab_size)][0]
-            raise ValueError(f"Token id out of range: {int(bad)}")
-        tok, _ = self._pinned()
-        tok[:] = t
-        _lib.check(self.lib.deepj_cuda_upload_buffer(self.ids["tok"], tok.ctypes.data, self.B))
-
-    def step(self, tokens) -> np.ndarray:
-        """One token per sequence through host buffers: upload the ids, flush the
-        stream (synchronous), download the greedy picks."""
-        if self.position >= self.cfg.max_seq_len:
-            raise ValueError(f"seqLen {self.position + 1} exceeds maxSeqLen {self.cfg.max_seq_len}")
-        host, _ = self._streams()
-        self.set_tokens(tokens)
-        # enqueue the stream behind the upload and let the download's synchronisation be the only one of the step
-        _lib.check(self.lib.deepj_cuda_flush_ops_async(host.ctypes.data, host.size))
-        self.position += 1
-        _, nxt = self._pinned()
-        _lib.check(self.lib.deepj_cuda_download_buffer(self.ids["next"], nxt.ctypes.data, self.B))
-        return nxt.astype(np.int64)
-
-    def step_device(self, n_steps: int = 1, sync: bool = True) -> None:
-        """n greedy steps with the picked token fed back on the device (no host copies)."""
-        if self.position + n_steps > self.cfg.max_seq_len:
-            raise ValueError(f"seqLen {self.position + n_steps} exceeds maxSeqLen {self.cfg.max_seq_len}")
-        _, dev = self._streams()
-        for _ in range(n_steps):
-            _lib.check(self.lib.deepj_cuda_flush_ops_async(dev.ctypes.data, dev.size))
-        self.position += n_steps
-        if sync:
-            _lib.check(self.lib.deepj_cuda_synchronize())
-
     def logits(self) -> np.ndarray:
         if self.fused_step and self.tp_world > 1:
             # the single-kernel step leaves this rank's vocabulary columns; gather the ranks' shards (every rank calls this)
             I = self.ids
             g = np.asarray([OP_TP_ALLGATHER, I["logits_local"], I["logits"], self.B, self.v_local], dtype=np.int32)
             _lib.check(self.lib.deepj_cuda_flush_ops(g.ctypes.data, g.size))
-        return self._download(self.ids["logits"], self.B * self.cfg.vocab_size).reshape(self.B, self.cfg.vocab_size)
-
-    def next_tokens(self) -> np.ndarray:
-        return self._download(self.ids["next"], self.B).astype(np.int64)
-
-    PREFILL_CHUNK = 2048     # prompt tokens per sequence and pass of the many-row path (enough 128 × 256 tiles for the GEMM to pair them)
+        return super().logits()
 
     def _build_prefill(self, T: int) -> np.ndarray:
         """The stream of one prompt chunk: T tokens of every sequence at once, B·T activation rows through the
@@ -618,68 +514,45 @@ class Q8Decoder:
         s.extend((OP_ADD_SCALAR_INPLACE, I["pos"], float_bits(float(T)), B))
         return np.asarray(s, dtype=np.int32)
 
-    def _head_stream(self) -> np.ndarray:
-        """Final norm + LM head + greedy pick on the hidden state in the decode buffer."""
-        c, B, I = self.cfg, self.B, self.ids
+    def _head_ops(self, x: int, logits: int, rows: int) -> List[int]:
+        c, I = self.cfg, self.ids
         if c.kind == "gpt":
-            s = [OP_Q8_LINEAR_LN, I["x"], 0, c.d_model, I["gF"], I["bF"], float_bits(LN_EPS), I["Wlm"], I["blm"], -1, 0, 0, I["logits"], 0,
-                 c.vocab_size, B, 0]
-        elif self.tp_world > 1:
-            s = [OP_Q8_LINEAR, I["x"], 0, c.d_model, I["gF"], float_bits(RMS_EPS), I["Wlm"], I["blm"], -1, 0, 0, I["logits_local"], 0, self.v_local, B,
-                 OP_TP_ALLGATHER, I["logits_local"], I["logits"], B, self.v_local]
-        else:
-            s = [OP_Q8_LINEAR, I["x"], 0, c.d_model, I["gF"], float_bits(RMS_EPS), I["Wlm"], I["blm"], -1, 0, 0, I["logits"], 0, c.vocab_size, B]
-        s += [OP_ARGMAX_ROWS, I["logits"], I["next"], B, c.vocab_size]
-        return np.asarray(s, dtype=np.int32)
+            return [OP_Q8_LINEAR_LN, x, 0, c.d_model, I["gF"], I["bF"], float_bits(LN_EPS), I["Wlm"], I["blm"], -1, 0, 0, logits, 0,
+                    c.vocab_size, rows, 0]
+        if self.tp_world > 1:
+            if rows != self.B:
+                raise ValueError("under tensor parallelism the head runs on one row per sequence")
+            return [OP_Q8_LINEAR, x, 0, c.d_model, I["gF"], float_bits(RMS_EPS), I["Wlm"], I["blm"], -1, 0, 0, I["logits_local"], 0, self.v_local, rows,
+                    OP_TP_ALLGATHER, I["logits_local"], logits, rows, self.v_local]
+        return [OP_Q8_LINEAR, x, 0, c.d_model, I["gF"], float_bits(RMS_EPS), I["Wlm"], I["blm"], -1, 0, 0, logits, 0, c.vocab_size, rows]
+
+    def _tp_rows(self) -> int:
+        """Tokens per sequence and chunk that the exchange slot has room for."""
+        return self.tp_slot_floats // self.cfg.d_model // self.B
+
+    def _chunk_tokens(self) -> int:
+        limit = super()._chunk_tokens()
+        return min(limit, self._tp_rows()) if self.tp_world > 1 else limit
 
     def prefill(self, prompts, chunked: Optional[bool] = None) -> np.ndarray:
-        """Feed the prompt (every sequence the same length); returns the greedy pick after its last token.
-        Prompts of 32 tokens or more go through the many-row path in chunks of PREFILL_CHUNK tokens per
-        sequence (tensor-core GEMMs, chunk attention); shorter ones one decode step per position.  Under tensor
-        parallelism a chunk's rows × dModel must fit the exchange slot (`tp_slot_floats`), which bounds the chunk."""
-        p = np.asarray(prompts, dtype=np.int64).reshape(self.B, -1)
-        T_all = p.shape[1]
-        tp_rows = self.tp_slot_floats // self.cfg.d_model // self.B if self.tp_world > 1 else 0      # tokens per sequence and chunk
-        if chunked is None:
-            chunked = T_all >= 32 and (self.tp_world == 1 or tp_rows >= 16)
-        if not chunked or T_all == 0:
-            nxt = None
-            for t in range(T_all):
-                nxt = self.step(p[:, t])
-            return nxt
-        if self.tp_world > 1 and tp_rows < 1:
-            raise ValueError("the exchange slot (tp_slot_floats) is smaller than one token per sequence")
-        if np.any(p < 0) or np.any(p >= self.cfg.vocab_size):
-            raise ValueError(f"Token id out of range: {int(p[(p < 0) | (p >= self.cfg.vocab_size)][0])}")
-        if self.position + T_all > self.cfg.max_seq_len:
-            raise ValueError(f"seqLen {self.position + T_all} exceeds maxSeqLen {self.cfg.max_seq_len}")
-        C = min(self.PREFILL_CHUNK, T_all, max(1, 65535 // self.B))
+        """Under tensor parallelism a chunk's rows × dModel must fit the exchange slot (`tp_slot_floats`), which bounds the
+        chunk; a slot with room for only a few tokens takes the prompt step by step."""
         if self.tp_world > 1:
-            C = min(C, tp_rows)
-        self._ensure_prefill_buffers(C)
-        done = 0
-        while done < T_all:
-            T = min(C, T_all - done)
-            if T not in self._prefill_streams:
-                self._prefill_streams[T] = self._build_prefill(T)
-            st = self._prefill_streams[T]
-            self._upload(self._prefill_ids["tok"], p[:, done:done + T].astype(np.float32).reshape(-1))
-            if self.cfg.kind == "gpt":       # row b·T + t sits at position (start of the chunk) + t
-                rows = np.tile(np.arange(self.position, self.position + T, dtype=np.float32), self.B)
-                self._upload(self._prefill_ids["ppos"], rows)
-            _lib.check(self.lib.deepj_cuda_flush_ops(st.ctypes.data, st.size))
-            done += T
-            self.position += T
-        hs = self._head_stream()
-        _lib.check(self.lib.deepj_cuda_flush_ops(hs.ctypes.data, hs.size))
-        return self.next_tokens()
+            T_all = np.asarray(prompts).size // self.B
+            if chunked is None:
+                chunked = T_all >= self.CHUNK_MIN and self._tp_rows() >= 16
+            if chunked and T_all > 0 and self._tp_rows() < 1:
+                raise ValueError("the exchange slot (tp_slot_floats) is smaller than one token per sequence")
+        return super().prefill(prompts, chunked)
 
-    def _ensure_prefill_buffers(self, C: int) -> None:
-        if self._prefill_cap >= C:
-            return
-        if self._prefill_ids:
-            self._release(list(self._prefill_ids.values()))
-        c, M = self.cfg, self.B * C
+    def _upload_chunk(self, tokens: np.ndarray) -> None:
+        super()._upload_chunk(tokens)
+        if self.cfg.kind == "gpt":       # row b·T + t sits at position (start of the chunk) + t
+            rows = np.tile(np.arange(self.position, self.position + tokens.shape[1], dtype=np.float32), self.B)
+            self._upload(self._prefill_ids["ppos"], rows)
+
+    def _prefill_sizes(self, M: int) -> Dict[str, int]:
+        c = self.cfg
         sizes = {"tok": M, "x": M * c.d_model, "x2": M * c.d_model, "qkv": M * 3 * self.d_local, "att": M * self.d_local,
                  "h": M * self.f_local}
         if c.kind == "deepseek":
@@ -688,103 +561,4 @@ class Q8Decoder:
             sizes["xp"], sizes["ppos"] = M * c.d_model, M
         if self.tp_world > 1:
             sizes["part"] = M * c.d_model
-        self._prefill_ids = {}
-        for name, n in sizes.items():
-            self._prefill_ids[name] = self._f32("", n)
-        self._prefill_cap = C
-        self._prefill_streams = {}
-
-    def generate(self, prompt, max_new_tokens: int, temperature: float = 1.0, top_k: int = 40, seed: int = 0) -> np.ndarray:
-        """TextGenerator.generate for batch 1 (models/TextGenerator.java:66-151) with the draw on the device:
-        temperature / top-k sampling, one `java.util.Random(seed).nextFloat()` per new token, the logits never
-        leave the GPU.  topK = 0 means the whole vocabulary, as in the reference (TextGenerator.java:111-115)."""
-        from .jrandom import JavaRandom
-        if max_new_tokens < 0:
-            raise ValueError("maxNewTokens must be >= 0")
-        if not temperature > 0.0:
-            raise ValueError("temperature must be > 0")
-        if top_k < 0:
-            raise ValueError("topK must be >= 0")
-        if self.B != 1:
-            raise ValueError("generate drives one sequence")
-        rnd = JavaRandom(seed)
-        c, I = self.cfg, self.ids
-        pick = np.asarray([OP_SAMPLE_TOPK, I["logits"], I["r"], I["next"], 1, c.vocab_size, top_k, float_bits(float(temperature))], dtype=np.int32)
-        step = self._build(feed_back=False, sampler=(top_k, float(temperature)))
-        self.reset()
-        self.prefill(np.asarray(prompt).reshape(1, -1))              # leaves the last prompt position's logits on the device
-        out = []
-        for i in range(max_new_tokens):
-            self._upload(I["r"], np.asarray([rnd.next_float()], dtype=np.float32))
-            if i == 0:
-                _lib.check(self.lib.deepj_cuda_flush_ops(pick.ctypes.data, pick.size))
-            else:
-                if self.position + 1 > c.max_seq_len:
-                    raise ValueError(f"seqLen {self.position + 1} exceeds maxSeqLen {c.max_seq_len}")
-                self._upload(I["tok"], np.asarray([out[-1]], dtype=np.float32))
-                _lib.check(self.lib.deepj_cuda_flush_ops(step.ctypes.data, step.size))
-                self.position += 1
-            out.append(int(self.next_tokens()[0]))
-        return np.asarray(out, dtype=np.int64)
-
-    def generate_greedy(self, prompt, max_new_tokens: int, keep_logits: bool = False):
-        """TextGenerator.generate with topK = 1 (models/TextGenerator.java:66-100)
-        for batch 1: returns the new token ids (and the logits row behind each)."""
-        if max_new_tokens < 0:
-            raise ValueError("maxNewTokens must be >= 0")
-        if self.B != 1:
-            raise ValueError("generate_greedy drives one sequence")
-        self.reset()
-        nxt = self.prefill(np.asarray(prompt).reshape(1, -1))
-        out, rows = [], []
-        for i in range(max_new_tokens):
-            if keep_logits:
-                rows.append(self.logits()[0].copy())
-            tok = int(nxt[0])
-            out.append(tok)
-            if i + 1 < max_new_tokens:
-                nxt = self.step([tok])
-        return (np.asarray(out, dtype=np.int64), np.stack(rows) if rows else None) if keep_logits else np.asarray(out, dtype=np.int64)
-
-    def profile_step(self):
-        """Device time of every op of one token step, run op by op as the per-operator stream (also when the
-        decoder itself steps with the single-kernel op): [(label, ms)]."""
-        if not self.loaded:
-            raise RuntimeError("weights are not loaded")
-        host = self._build(feed_back=False)
-        n = len(self._op_labels) + 1
-        ms = np.zeros(n, dtype=np.float32)
-        cnt = ctypes.c_int32(0)
-        _lib.check(self.lib.deepj_cuda_profile_ops(host.ctypes.data, host.size, ms.ctypes.data, n, ctypes.byref(cnt)))
-        self.position += 1
-        return list(zip(self._op_labels, ms[: cnt.value].tolist()))
-
-    def time_ops(self, labels, iters: int = 20, warmup: int = 3) -> Tuple[float, int]:
-        """Device time of the ops whose label is in `labels`, run back to back as their own stream
-        (graph-replayed like the full step, at the current position): (ms per pass, ops per pass)."""
-        full = self._build(feed_back=False)
-        keep = [full[a:b] for lbl, (a, b) in zip(self._op_labels, self._op_bounds) if lbl in labels]
-        if not keep:
-            return 0.0, 0
-        sub = np.ascontiguousarray(np.concatenate(keep))
-        for _ in range(max(warmup, 3)):
-            _lib.check(self.lib.deepj_cuda_flush_ops(sub.ctypes.data, sub.size))
-        _lib.check(self.lib.deepj_cuda_timer_begin())
-        for _ in range(iters):
-            _lib.check(self.lib.deepj_cuda_flush_ops_async(sub.ctypes.data, sub.size))
-        ms = ctypes.c_float(0)
-        _lib.check(self.lib.deepj_cuda_timer_end(ctypes.byref(ms)))
-        return ms.value / iters, len(keep)
-
-    def stats(self) -> Dict[str, int]:
-        v = (ctypes.c_int64 * 6)()
-        _lib.check(self.lib.deepj_cuda_stats(v, 6))
-        return {"eager_launches": v[0], "graph_replays": v[1], "graphs_captured": v[2],
-                "kernels_per_replay": v[3], "workspace_bytes": v[4], "device_error": v[5]}
-
-    def close(self) -> None:
-        if self._pin_ptr is not None:
-            self.lib.deepj_cuda_pinned_free(self._pin_ptr)
-            self._pin_ptr = None
-        if self._owned:
-            self._release(list(self._owned))
+        return sizes

@@ -190,6 +190,18 @@ int deepj_cuda_attn_decode_static(int32_t qkv, int32_t q_off, int32_t k_off, int
                                   int32_t kv, int32_t layer, int32_t pos, int32_t cos_table, int32_t sin_table,
                                   int32_t out, int32_t out_off, int32_t ldo, int32_t batch, int32_t heads, int32_t head_dim);
 
+/* bf16 weights (checkpoints that ship in bf16 keep their values).  W[N][K], one output row's K-vector contiguous and
+ * padded with zeros to a multiple of eight; zero-filled at allocation, which is what the padding rows and columns of
+ * concatenated weights rely on.  The object lives in the id space of the buffers. */
+int deepj_cuda_bf16_alloc(int32_t id, int32_t K, int32_t N);
+/* Rounds rows x cols floats (row-major at src_off of the float buffer src_id) to bf16 into rows row0, row0 + row_step, …
+ * and columns col0 … of the object: row_step = 2 interleaves the gate and up rows of a gated feed-forward. */
+int deepj_cuda_bf16_store(int32_t id, int32_t row0, int32_t row_step, int32_t col0, int32_t src_id, int64_t src_off,
+                          int32_t rows, int32_t cols);
+/* Cache of a latent-attention layer: [batch][max_seq][width] fp32 or bf16 values, zero-filled; a row is the normed latent
+ * followed by the rotated key part that all heads share. */
+int deepj_cuda_latent_alloc(int32_t id, int32_t batch, int32_t max_seq, int32_t width, int32_t bf16);
+
 /* ───────────── fused decode op codes (extend ComputeGraph.java:19-60) ─────────────
  * Buffer-id slots may hold -1 where an operand is optional.  Integers that the
  * reference would keep in an int[] (token ids, positions) travel as floats holding
@@ -221,6 +233,30 @@ int deepj_cuda_attn_decode_static(int32_t qkv, int32_t q_off, int32_t k_off, int
  *                        the GPT blocks' projection: out = act(layernorm(x; gamma, beta, eps) · W + bias) (+residual),
  *                        LayerNorm1D semantics (mean, biased variance); act 0 = none, 1 = GELU (tanh form);
  *                        gamma = beta = -1 skips the norm
+ *
+ * Ops over bf16 weights.  An activation row is staged in fp32: optionally RMS-normalised in `groups` equal parts
+ * (part / sqrt(mean(part^2) + eps), times gamma; groups = 0 and gamma = -1: no norm) and multiplied by sigmoid(gate).
+ * exact = 1 keeps every product in fp32; exact = 0 lets the many-row kernels round the staged operand to bf16.
+ *
+ *  77 BF16_LINEAR       [op, x, x_off, ldx, gamma, groups, epsBits, gate, gate_off, ldgate, k1, x2, x2_off, ldx2, w,
+ *                        residual, res_off, ldr, out, out_off, ldo, M, glu_row, limitBits, glu, glu_off, ldglu,
+ *                        softcapBits, exact]
+ *                        [stage(x), x2] times the weight (x2 = -1: one segment; a second one starts at the next multiple
+ *                        of eight columns).  Weight rows below glu_row: out = product (+ residual), softcap·tanh(out/softcap)
+ *                        when softcap > 0.  Rows from glu_row on are (gate, up) pairs: g = min(gate, limit),
+ *                        u = clamp(up, -limit, limit), glu = g·sigmoid(1.702 g)·(u + 1)
+ *  78 BF16_BLOCK_LINEAR [op, x, x_off, ldx, xstr, w, heads, out, out_off, ldo, ostr, M]
+ *                        block-diagonal: out[m][h·ostr + n] = w[h·(N/heads) + n] · x[m][h·xstr …]
+ *  79 DELTA_RULE        [op, proj, r_off, k_off, v_off, a_off, low_off, ld, abias, w2, w0, state, pos, out, out_off, ldo,
+ *                        B, T, H, dim]   generalized delta rule over T tokens of B sequences, state [B][H][dim][dim] carried
+ *                        in fp32; a sequence at position 0 starts from a zero state (csrc/delta_rule.cu)
+ *  80 ATTN_LATENT       [op, q, q_off, ldq, qc, qc_off, ldqc, kv, kv_off, ldkv, gamma, epsBits, cache, pos, cos, sin,
+ *                        out, out_off, ldo, B, T, H, dim, rot, R, scaleBits]
+ *                        appends the chunk's normed latents and rotated key parts, then every row attends causally in the
+ *                        latent space; out = softmax-weighted latents per head (csrc/attn_latent.cu)
+ *  81 TABLE_EXPERTS     [op, x, x_off, ldx, gamma, groups, epsBits, tok, table, vocab, top, experts, w_up, w_down, ff,
+ *                        limitBits, residual, res_off, ldr, out, out_off, ldo, d, M, exact]
+ *                        out = residual + (1/top) sum over the experts of table[token] of their gated feed-forward
  */
 #define DEEPJ_OP_EMBED_GATHER        64
 #define DEEPJ_OP_Q8_LINEAR           65
@@ -235,6 +271,11 @@ int deepj_cuda_attn_decode_static(int32_t qkv, int32_t q_off, int32_t k_off, int
 #define DEEPJ_OP_SAMPLE_TOPK         74
 #define DEEPJ_OP_Q8_LINEAR_LN       75
 #define DEEPJ_OP_DECODE_STEP        76
+#define DEEPJ_OP_BF16_LINEAR        77
+#define DEEPJ_OP_BF16_BLOCK_LINEAR  78
+#define DEEPJ_OP_DELTA_RULE         79
+#define DEEPJ_OP_ATTN_LATENT        80
+#define DEEPJ_OP_TABLE_EXPERTS      81
 
 #ifdef __cplusplus
 }
