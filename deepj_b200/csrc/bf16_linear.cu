@@ -402,7 +402,7 @@ void launch_bf16_linear(const Bf16LinearArgs& a, cudaStream_t s) {
         }
         return;
     }
-    if (!a.exact && launch_bf16_gemm_tc(a, nullptr, nullptr, s)) return;
+    if (!a.exact && launch_bf16_gemm_tc(a, nullptr, s)) return;
     launch_stage_rows(a.a, a.b, a.w.Kp, a.M, nullptr, 1, a.ws, false, s);
     F32GemmParams p = {a.ws, a.w.w, a.M, a.w.N, a.w.Kp, a.residual, a.ldr, a.out, a.ldo, a.gluRow, a.limit, a.glu, a.ldglu, a.softcap};
     launch_k(k_bf16_gemm_f32, dim3((a.w.N + 63) / 64, (a.M + 63) / 64), dim3(256), 0, s, true, p);

@@ -151,7 +151,9 @@ DJ_PART void launch_bf16_store(const float* src, int rows, int cols, __nv_bfloat
 DJ_PART const char* bf16_linear_check(const Bf16LinearArgs& a);      // nullptr, or why the shape is not supported
 DJ_PART size_t bf16_linear_ws_floats(const Bf16LinearArgs& a);
 DJ_PART void launch_bf16_linear(const Bf16LinearArgs& a, cudaStream_t s);
-DJ_PART bool launch_bf16_gemm_tc(const Bf16LinearArgs& a, const int* tileExpert, const int* rowMap, cudaStream_t s);
+// Grouped rows of a tensor-core product: the expert of every 128-row tile (−1: none), where output rows go, rows per expert.
+struct GroupedRows { const int* tileExpert; const int* rowMap; int rowsPerExpert; };
+DJ_PART bool launch_bf16_gemm_tc(const Bf16LinearArgs& a, const GroupedRows* g, cudaStream_t s);
 DJ_PART void launch_stage_rows(const RowOperand& a, const RowOperand& b, int Kp, int rows, const int* map, int div, void* out, bool bf16, cudaStream_t s);
 DJ_PART void launch_bf16_block_linear(const float* x, int ldx, int xstr, const Bf16View& w, int heads, float* out, int ldo, int ostr, int M, cudaStream_t s);
 // Table-routed experts: token id → `top` experts, each of weight 1/top.  up holds every expert's (gate, up) row pairs
