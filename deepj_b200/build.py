@@ -69,7 +69,7 @@ def _compile(src: str, obj: str, headers: list[str], verbose: bool) -> str:
 # interpreter refuses ops whose part is absent).  "*" = everything.
 PARTS = {
     "core": ["runtime.cu", "misc.cu"],
-    "bf16": ["bf16_linear.cu", "bf16_gemm_tc.cu", "bf16_experts.cu", "delta_rule.cu", "attn_latent.cu"],
+    "bf16": ["bf16_linear.cu", "bf16_gemm_tc.cu", "bf16_experts.cu", "delta_rule.cu", "attn_latent.cu", "attn_latent_mma.cu"],
 }
 
 

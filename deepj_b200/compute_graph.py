@@ -36,6 +36,7 @@ OP_TP_ALLREDUCE, OP_TP_ALLGATHER = 71, 72
 OP_ATTN_PREFILL, OP_SAMPLE_TOPK, OP_Q8_LINEAR_LN, OP_DECODE_STEP = 73, 74, 75, 76
 # ops over bf16 weights
 OP_BF16_LINEAR, OP_BF16_BLOCK_LINEAR, OP_DELTA_RULE, OP_ATTN_LATENT, OP_TABLE_EXPERTS = 77, 78, 79, 80, 81
+OP_ATTN_LATENT_CHUNK = 82
 
 # op → (stride, offsets of the slots that hold buffer ids); ComputeGraph.java:89-147
 OP_METADATA: Dict[int, tuple] = {}
@@ -76,6 +77,7 @@ OP_METADATA[OP_BF16_BLOCK_LINEAR] = (12, (1, 5, 7))
 OP_METADATA[OP_DELTA_RULE] = (20, (1, 8, 9, 10, 11, 12, 13))
 OP_METADATA[OP_ATTN_LATENT] = (26, (1, 4, 7, 10, 12, 13, 14, 15, 16))
 OP_METADATA[OP_TABLE_EXPERTS] = (25, (1, 4, 7, 8, 12, 13, 16, 19))
+OP_METADATA[OP_ATTN_LATENT_CHUNK] = (26, (1, 4, 7, 9, 10, 11, 12, 13, 14, 15))
 
 
 def float_bits(value: float) -> int:

@@ -9,6 +9,7 @@
 //   k_latent_append   RMS norm of the latent, rotation of the key part, cache write
 //   k_latent_attn     fp32 FMA form, any sizes: a warp per head, tiles of 32 keys in shared memory shared by eight heads
 //   k_latent_merge    adds the partial results of a split key range
+// With a bf16 cache the tensor-core kernels of attn_latent_mma.cu take over where the sizes allow.
 #include "row_operand.cuh"
 
 #include <algorithm>
@@ -181,10 +182,14 @@ void launch_la(const LaParams& p, int rows, cudaStream_t s) {
 }
 
 template <typename CT>
+void append(const LatentAttnArgs& a, cudaStream_t s) {
+    launch_k(k_latent_append<CT>, dim3((unsigned)(a.B * a.T)), dim3(128), 0, s, true, a.kv, a.ldkv, a.gamma, a.eps, (CT*)a.cache, a.maxSeq, a.R + a.rot, a.pos,
+             a.cosT, a.sinT, a.T, a.R, a.rot);
+}
+
+template <typename CT>
 void run(const LatentAttnArgs& a, cudaStream_t s) {
     const int rows = a.B * a.T, W = a.R + a.rot;
-    launch_k(k_latent_append<CT>, dim3((unsigned)rows), dim3(128), 0, s, true, a.kv, a.ldkv, a.gamma, a.eps, (CT*)a.cache, a.maxSeq, W, a.pos, a.cosT, a.sinT,
-             a.T, a.R, a.rot);
     LaParams p;
     p.q = a.q; p.ldq = a.ldq; p.dim = a.dim; p.qc = a.qc; p.ldqc = a.ldqc; p.cache = a.cache; p.maxSeq = a.maxSeq; p.W = W;
     p.pos = a.pos; p.cosT = a.cosT; p.sinT = a.sinT; p.out = a.out; p.ldo = a.ldo;
@@ -207,13 +212,20 @@ int latent_attn_splits(int rows, int H, int maxSeq) {
     return (int)std::max(1l, std::min((long)std::min(tiles, 64), 2l * g_num_sms / ctas));
 }
 size_t latent_attn_ws_floats(const LatentAttnArgs& a) {
-    const int rows = a.B * a.T, splits = latent_attn_splits(rows, a.H, a.maxSeq);
+    const int rows = a.B * a.T, splits = latent_mma_fits(a) ? latent_mma_splits(a) : latent_attn_splits(rows, a.H, a.maxSeq);
     return splits > 1 ? (size_t)rows * a.H * splits * (a.R + 2) : 0;
 }
 bool latent_attn_fits(int R, int rot) { return R >= 1 && R <= 1024 && rot >= 2 && rot % 2 == 0 && la_smem(R + rot) <= 226 * 1024; }
 
+void launch_latent_append(const LatentAttnArgs& a, cudaStream_t s) {
+    if (a.bf16) append<__nv_bfloat16>(a, s);
+    else append<float>(a, s);
+}
+
 void launch_latent_attn(const LatentAttnArgs& a, cudaStream_t s) {
-    if (a.bf16) run<__nv_bfloat16>(a, s);
+    launch_latent_append(a, s);
+    if (latent_mma_fits(a)) launch_latent_mma(a, s);
+    else if (a.bf16) run<__nv_bfloat16>(a, s);
     else run<float>(a, s);
 }
 

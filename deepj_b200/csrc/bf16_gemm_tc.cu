@@ -26,8 +26,9 @@ struct GemmTcParams {
     CUtensorMap a, w;
     int M, N, nK, mTiles, nTiles;
     const int* tileExpert; const int* rowMap;
+    const float* lenPos; int lenT;               // rows = lenPos[0] + lenT, at most M (device-side length)
     const float* residual; int ldr;
-    float* out; int ldo;
+    float* out; int ldo; __nv_bfloat16* outHalf; // outHalf: bf16 rows instead of fp32
     int gluRow; float limit; float* glu; int ldglu;
     float softcap;
     int* error;
@@ -72,12 +73,19 @@ __global__ void __launch_bounds__(kGThreads, 1) k_bf16_gemm_tc(const __grid_cons
     __syncthreads();
     tc_fence_after();
     const uint32_t tmem = s_tmem;
-    const int tiles = p.mTiles * p.nTiles;
+    int rows = p.M, mTiles = p.mTiles, tiles = p.mTiles * p.nTiles;
+    auto read_length = [&] {                         // after the dependency wait
+        if (p.lenPos != nullptr) {
+            rows = min(p.M, max((int)p.lenPos[0], 0) + p.lenT);
+            mTiles = (rows + kGM - 1) / kGM;
+            tiles = mTiles * p.nTiles;
+        }
+    };
 
     if (warp == 4) {
         if (lane == 0) {
             int early = 0;                                   // stages whose weights were requested before the wait
-            if (p.tileExpert == nullptr && (int)blockIdx.x < tiles) {
+            if (p.tileExpert == nullptr && p.lenPos == nullptr && (int)blockIdx.x < tiles) {
                 const int n0 = ((int)blockIdx.x / p.mTiles) * BN;
                 for (; early < S::kStages && early < p.nK; early++) {
                     mbar_arrive_expect_tx(full(early), S::kStageBytes);
@@ -86,11 +94,12 @@ __global__ void __launch_bounds__(kGThreads, 1) k_bf16_gemm_tc(const __grid_cons
             }
             pdl_wait();
             pdl_launch_dependents();
+            read_length();
             unsigned it = 0;
             bool ok = true;
             for (int t = blockIdx.x; t < tiles && ok; t += gridDim.x) {
-                const int mt = t % p.mTiles;
-                int wrow = (t / p.mTiles) * BN;
+                const int mt = t % mTiles;
+                int wrow = (t / mTiles) * BN;
                 if (p.tileExpert != nullptr) {
                     const int e = p.tileExpert[mt];
                     if (e < 0) continue;
@@ -118,10 +127,11 @@ __global__ void __launch_bounds__(kGThreads, 1) k_bf16_gemm_tc(const __grid_cons
         if (lane == 0) {
             pdl_wait();
             pdl_launch_dependents();
+            read_length();
             unsigned it = 0, n = 0;
             bool ok = true;
             for (int t = blockIdx.x; t < tiles && ok; t += gridDim.x) {
-                if (p.tileExpert != nullptr && p.tileExpert[t % p.mTiles] < 0) continue;
+                if (p.tileExpert != nullptr && p.tileExpert[t % mTiles] < 0) continue;
                 const int a = n & 1;
                 if (n >= 2 && !mbar_wait(accEmpty(a), (n / 2 - 1) & 1, &s_abort, p.error, 212)) break;
                 tc_fence_after();
@@ -143,15 +153,16 @@ __global__ void __launch_bounds__(kGThreads, 1) k_bf16_gemm_tc(const __grid_cons
     } else {
         pdl_wait();
         pdl_launch_dependents();
+        read_length();
         unsigned n = 0;
         for (int t = blockIdx.x; t < tiles; t += gridDim.x) {
-            const int mt = t % p.mTiles, n0 = (t / p.mTiles) * BN;
+            const int mt = t % mTiles, n0 = (t / mTiles) * BN;
             if (p.tileExpert != nullptr && p.tileExpert[mt] < 0) continue;
             const int a = n & 1;
             if (!__all_sync(0xffffffffu, mbar_wait(accFull(a), (n / 2) & 1, &s_abort, p.error, 214))) break;
             tc_fence_after();
             const int mBase = mt * kGM + warp * 32;
-            int myRow = mBase + lane < p.M ? mBase + lane : -1;      // output row of tile row `lane`
+            int myRow = mBase + lane < rows ? mBase + lane : -1;      // output row of tile row `lane`
             if (myRow >= 0 && p.rowMap != nullptr) myRow = p.rowMap[myRow];
 #pragma unroll 1
             for (int c0 = 0; c0 < BN && n0 + c0 < p.N; c0 += 32) {
@@ -161,6 +172,16 @@ __global__ void __launch_bounds__(kGThreads, 1) k_bf16_gemm_tc(const __grid_cons
                 for (int j = 0; j < 32; j++) stg[lane * 33 + j] = __uint_as_float(v[j]);
                 __syncwarp();
                 const int nb = n0 + c0, nn = nb + lane;
+                if (p.outHalf != nullptr) {
+#pragma unroll 8
+                    for (int i = 0; i < 32; i += 2) {
+                        const int r = i + (lane >> 4), row = __shfl_sync(0xffffffffu, myRow, r), c = 2 * (lane & 15);
+                        if (row >= 0 && nb + c < p.N)
+                            *reinterpret_cast<__nv_bfloat162*>(p.outHalf + (size_t)row * p.ldo + nb + c) = __floats2bfloat162_rn(stg[r * 33 + c], stg[r * 33 + c + 1]);
+                    }
+                    __syncwarp();
+                    continue;
+                }
                 if (nb < p.gluRow) {
 #pragma unroll 8
                     for (int i = 0; i < 32; i++) {
@@ -194,11 +215,11 @@ __global__ void __launch_bounds__(kGThreads, 1) k_bf16_gemm_tc(const __grid_cons
     if (warp == 4) { tc_fence_after(); tmem_dealloc(tmem, S::kTmem); }
 }
 
-bool encode_rows(CUtensorMap* map, const void* base, size_t K, size_t rows, int boxRows) {
+bool encode_rows(CUtensorMap* map, const void* base, size_t K, size_t pitch, size_t rows, int boxRows) {
     EncodeTiledFn enc = encode_tiled_fn();
     if (!enc) return false;
     const cuuint64_t dims[2] = {(cuuint64_t)K, (cuuint64_t)rows};
-    const cuuint64_t strides[1] = {(cuuint64_t)K * 2};
+    const cuuint64_t strides[1] = {(cuuint64_t)pitch * 2};
     const cuuint32_t box[2] = {(cuuint32_t)kGK, (cuuint32_t)boxRows};
     const cuuint32_t estr[2] = {1u, 1u};
     return enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
@@ -206,9 +227,9 @@ bool encode_rows(CUtensorMap* map, const void* base, size_t K, size_t rows, int 
 }
 
 template <int BN>
-bool run(GemmTcParams& p, const void* a, const __nv_bfloat16* w, int Kp, size_t aRows, size_t wRows, cudaStream_t s) {
+bool run(GemmTcParams& p, const void* a, int aK, int aPitch, size_t aRows, const Bf16View& w, cudaStream_t s) {
     using S = GemmShape<BN>;
-    if (!encode_rows(&p.a, a, Kp, aRows, kGM) || !encode_rows(&p.w, w, Kp, wRows, BN)) return false;
+    if (!encode_rows(&p.a, a, aK, aPitch, aRows, kGM) || !encode_rows(&p.w, w.w, w.Kp, w.Kp, w.N, BN)) return false;
     static bool attr = false;
     if (!attr) {
         DJ_CUDA_CHECK(cudaFuncSetAttribute(k_bf16_gemm_tc<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)S::kSmem));
@@ -218,6 +239,20 @@ bool run(GemmTcParams& p, const void* a, const __nv_bfloat16* w, int Kp, size_t 
     const int grid = std::min(p.mTiles * p.nTiles, g_num_sms);
     launch_k(k_bf16_gemm_tc<BN>, dim3((unsigned)grid), dim3(kGThreads), S::kSmem, s, true, p);
     return true;
+}
+
+// the tile width with the least work per SM, wider tiles first
+int pick_width(int mTiles, int N) {
+    int best = 256; double bestCost = 1e30;
+    for (int bn : {256, 128, 64}) {
+        const long tiles = (long)mTiles * ((N + bn - 1) / bn);
+        const double cost = (double)((tiles + g_num_sms - 1) / g_num_sms) * (bn + 24);
+        if (cost < bestCost) { bestCost = cost; best = bn; }
+    }
+    return best;
+}
+bool run_width(int bn, GemmTcParams& p, const void* a, int aK, int aPitch, size_t aRows, const Bf16View& w, cudaStream_t s) {
+    return bn == 256 ? run<256>(p, a, aK, aPitch, aRows, w, s) : bn == 128 ? run<128>(p, a, aK, aPitch, aRows, w, s) : run<64>(p, a, aK, aPitch, aRows, w, s);
 }
 
 }  // namespace
@@ -232,18 +267,18 @@ bool launch_bf16_gemm_tc(const Bf16LinearArgs& a, const GroupedRows* g, cudaStre
     p.residual = a.residual; p.ldr = a.ldr; p.out = a.out; p.ldo = a.ldo;
     p.gluRow = a.gluRow; p.limit = a.limit; p.glu = a.glu; p.ldglu = a.ldglu; p.softcap = a.softcap;
     p.error = g_dev_error;
-    // the tile width with the least work per SM, wider tiles first
-    int best = 256; double bestCost = 1e30;
-    for (int bn : {256, 128, 64}) {
-        const long tiles = (long)p.mTiles * ((p.N + bn - 1) / bn);
-        const double cost = (double)((tiles + g_num_sms - 1) / g_num_sms) * (bn + 24);
-        if (cost < bestCost) { bestCost = cost; best = bn; }
-    }
+    p.lenPos = nullptr; p.lenT = 0; p.outHalf = nullptr;
     if (!g) launch_stage_rows(a.a, a.b, a.w.Kp, a.M, nullptr, 1, a.ws, true, s);
-    const bool ok = best == 256 ? run<256>(p, a.ws, a.w.w, a.w.Kp, a.M, a.w.N, s)
-                  : best == 128 ? run<128>(p, a.ws, a.w.w, a.w.Kp, a.M, a.w.N, s)
-                                : run<64>(p, a.ws, a.w.w, a.w.Kp, a.M, a.w.N, s);
-    return ok;
+    return run_width(pick_width(p.mTiles, p.N), p, a.ws, a.w.Kp, a.w.Kp, a.M, a.w, s);
+}
+
+void launch_bf16_gemm_rows(const __nv_bfloat16* rows, int lda, int K, const float* pos, int T, int maxRows, const Bf16View& w, __nv_bfloat16* out, int ldo,
+                           cudaStream_t s) {
+    GemmTcParams p = {};
+    p.M = maxRows; p.N = w.N; p.nK = (K + kGK - 1) / kGK; p.mTiles = (maxRows + kGM - 1) / kGM;
+    p.lenPos = pos; p.lenT = T; p.outHalf = out; p.ldo = ldo; p.gluRow = w.N; p.error = g_dev_error;
+    if (lda % 8 != 0 || w.Kp % 8 != 0 || (w.N & 1) != 0 || g_dev_error == nullptr || !run_width(pick_width(p.mTiles, p.N), p, rows, K, lda, maxRows, w, s))
+        throw std::runtime_error("bf16 product over cached rows: the shape does not qualify");
 }
 
 }  // namespace dj

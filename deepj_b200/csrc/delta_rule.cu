@@ -8,8 +8,10 @@
 // prompt is cut changes nothing.
 //
 //   k_delta_prepare   per (token, head): w, and b = a ⊙ k / (Σk² + ε) — with b the removal term is b (kᵀS)
-//   k_delta_scan      one warp per (sequence, head, few value columns): a lane holds the key channels lane, lane + 32, …
-//                     of its columns in registers; u·S and o are warp reductions, the next token's vectors are in flight
+//   k_delta_scan      a block of four warps per (sequence, head, 16 value columns), a warp per four of them: a lane holds some
+//                     key channels of its columns in registers, kᵀS and o are warp reductions over all lanes, and the
+//                     tokens' vectors stream through a two-stage cp.async ring of shared memory.  A single token computes
+//                     its own w and b (no prepare launch) and reads the state before the dependency wait.
 #include "row_operand.cuh"
 
 namespace dj {
@@ -78,11 +80,11 @@ __global__ void __launch_bounds__(128) k_delta_prepare(const PrepParams p) {
 }
 
 struct ScanParams {
-    const float* proj; int ld, r_off, k_off, v_off;
-    const float* w; const float* b;
+    PrepParams in;                 // projections, decay weights; wOut / bOut are read here
+    int r_off, v_off;
     float* state; const float* pos;
     float* out; int ldo;
-    int T, H, dim;
+    int T, vec;                    // vec: every field can be copied in 16-byte pieces
 };
 
 // Sums C per-lane values over the warp; lane (group g of 32/C lanes) ends up with the sum of column g.  C a power of two.
@@ -102,46 +104,35 @@ __device__ __forceinline__ float reduce_columns(float (&v)[C], int lane) {
     return v[0];
 }
 
-// E key channels per lane, C value columns per warp.
-template <int E, int C>
+// E key channels per lane (lane·E …), C value columns per warp, TB tokens per stage of the ring.
+template <int E, int C, int TB, bool FUSED>
 __global__ void __launch_bounds__(128) k_delta_scan(const ScanParams p) {
-    pdl_wait();
-    pdl_launch_dependents();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int h = blockIdx.y, b = blockIdx.z, dim = p.dim;
-    const int c0 = (blockIdx.x * 4 + warp) * C;
-    if (c0 >= dim) return;
+    constexpr int P = 32 * E, ROW = 4 * P + 4 * C, STAGE = TB * ROW;        // a token: k, r, w, b of the head, v of the block's columns
+    extern __shared__ __align__(16) float ring[];                           // [2][TB][ROW]; FUSED: one token, then low [w2p]
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int h = blockIdx.y, b = blockIdx.z, dim = p.in.dim, H = p.in.H, HD = H * dim, hd = h * dim;
+    const int cb = blockIdx.x * 4 * C, c0 = cb + warp * C;                  // the block's and this warp's first column
+    const size_t row0 = (size_t)b * p.T;
+    if (P > dim)                                                            // channels past the head stay zero
+        for (int i = tid; i < (FUSED ? 1 : 2 * TB) * 4 * (P - dim); i += 128)
+            ring[(i / (4 * (P - dim))) * ROW + (i / (P - dim)) % 4 * P + dim + i % (P - dim)] = 0.0f;
+    // the state was last written several kernels ago: it may be read before the dependency wait
     const bool fresh = p.pos[b] == 0.0f;
-    float* st = p.state + (((size_t)b * p.H + h) * dim + c0) * dim;
+    float* st = p.state + (((size_t)b * H + h) * dim + c0) * dim;
     float S[C][E];
 #pragma unroll
     for (int c = 0; c < C; c++)
 #pragma unroll
         for (int e = 0; e < E; e++) {
-            const int i = e * 32 + lane;
+            const int i = lane * E + e;
             S[c][e] = (!fresh && i < dim && c0 + c < dim) ? st[(size_t)c * dim + i] : 0.0f;
         }
-    const size_t row0 = (size_t)b * p.T;
-    const int hd = h * dim, HD = p.H * dim;
-    float k[E], w[E], q[E], r[E], v;
-    auto load = [&](int t, float (&k)[E], float (&w)[E], float (&q)[E], float (&r)[E], float& v) {
-        const float* row = p.proj + (row0 + t) * p.ld + hd;
-        const size_t wi = (row0 + t) * HD + hd;
+    auto token = [&](const float* row, int t) {
+        float k[E], r[E], w[E], q[E], v[C];
 #pragma unroll
-        for (int e = 0; e < E; e++) {
-            const int i = e * 32 + lane;
-            const bool on = i < dim;
-            k[e] = on ? row[p.k_off + i] : 0.0f;
-            r[e] = on ? row[p.r_off + i] : 0.0f;
-            w[e] = on ? p.w[wi + i] : 0.0f;
-            q[e] = on ? p.b[wi + i] : 0.0f;
-        }
-        v = (lane < C && c0 + lane < dim) ? row[p.v_off + c0 + lane] : 0.0f;
-    };
-    load(0, k, w, q, r, v);
-    for (int t = 0; t < p.T; t++) {
-        float k2[E], w2[E], q2[E], r2[E], v2;
-        if (t + 1 < p.T) load(t + 1, k2, w2, q2, r2, v2);
+        for (int e = 0; e < E; e++) { k[e] = row[lane * E + e]; r[e] = row[P + lane * E + e]; w[e] = row[2 * P + lane * E + e]; q[e] = row[3 * P + lane * E + e]; }
+#pragma unroll
+        for (int c = 0; c < C; c++) v[c] = row[4 * P + warp * C + c];
         float d[C];
 #pragma unroll
         for (int c = 0; c < C; c++) {
@@ -153,36 +144,114 @@ __global__ void __launch_bounds__(128) k_delta_scan(const ScanParams p) {
         float o[C];
 #pragma unroll
         for (int c = 0; c < C; c++) {
-            const float dot = __shfl_sync(0xffffffffu, ks, c * (32 / C)), vc = __shfl_sync(0xffffffffu, v, c);
+            const float dot = __shfl_sync(0xffffffffu, ks, c * (32 / C));
             o[c] = 0.0f;
 #pragma unroll
             for (int e = 0; e < E; e++) {
-                S[c][e] = fmaf(w[e], S[c][e], fmaf(k[e], vc, -(q[e] * dot)));
+                S[c][e] = fmaf(w[e], S[c][e], fmaf(k[e], v[c], -(q[e] * dot)));
                 o[c] = fmaf(r[e], S[c][e], o[c]);
             }
         }
         const float os = reduce_columns<C>(o, lane);
         const int col = c0 + lane / (32 / C);
         if (lane % (32 / C) == 0 && col < dim) p.out[(row0 + t) * p.ldo + hd + col] = os;
-        if (t + 1 < p.T) {
+    };
+    if constexpr (FUSED) {
+        pdl_wait();
+        pdl_launch_dependents();
+        float* low = ring + ROW;
+        const float* x = p.in.proj + row0 * p.in.ld;
+        for (int j = tid; j < p.in.w2p; j += 128) low[j] = j < p.in.rank ? tanhf(x[p.in.low_off + j]) : 0.0f;
+        float ss = 0.0f;
+        for (int i = lane; i < dim; i += 32) { const float k = x[p.in.k_off + hd + i]; ss = fmaf(k, k, ss); }
+        for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        const float inv = 1.0f / (ss + kUnitEps), rate = expf(-0.5f);
+        __syncthreads();
+        for (int i = tid; i < dim; i += 128) {
+            const float k = x[p.in.k_off + hd + i];
+            ring[i] = k;
+            ring[P + i] = x[p.r_off + hd + i];
+            float acc = 0.0f;
+            const __nv_bfloat16* w = p.in.w2 + (size_t)(hd + i) * p.in.w2p;
+            for (int j = 0; j < p.in.w2p; j += 8) {
+                const uint4 u4 = __ldg(reinterpret_cast<const uint4*>(w + j));
+                const uint32_t u[4] = {u4.x, u4.y, u4.z, u4.w};
 #pragma unroll
-            for (int e = 0; e < E; e++) { k[e] = k2[e]; w[e] = w2[e]; q[e] = q2[e]; r[e] = r2[e]; }
-            v = v2;
+                for (int q = 0; q < 4; q++) {
+                    acc = fmaf(__uint_as_float(u[q] << 16), low[j + 2 * q], acc);
+                    acc = fmaf(__uint_as_float(u[q] & 0xffff0000u), low[j + 2 * q + 1], acc);
+                }
+            }
+            ring[2 * P + i] = expf(-rate * sigmoid_f(acc + p.in.w0[hd + i]));
+            ring[3 * P + i] = sigmoid_f(x[p.in.a_off + hd + i] + p.in.abias[hd + i]) * k * inv;
+        }
+        for (int i = tid; i < 4 * C; i += 128) ring[4 * P + i] = cb + i < dim ? x[p.v_off + hd + cb + i] : 0.0f;
+        __syncthreads();
+        token(ring, 0);
+    } else {
+        pdl_wait();
+        pdl_launch_dependents();
+        const int nv = min(4 * C, dim - cb);
+        auto load = [&](int t0, int stage) {
+            float* dst = ring + stage * STAGE;
+            const int n = min(TB, p.T - t0);
+            if (p.vec) {
+                const int per = dim / 4, all = 4 * per + nv / 4;
+                for (int i = tid; i < n * all; i += 128) {
+                    const int t = i / all, j = i - t * all;
+                    const float* row = p.in.proj + (row0 + t0 + t) * p.in.ld + hd;
+                    const size_t wi = (row0 + t0 + t) * HD + hd;
+                    float* d = dst + t * ROW;
+                    if (j < per) cp_async16(d + 4 * j, row + p.in.k_off + 4 * j);
+                    else if (j < 2 * per) cp_async16(d + P + 4 * (j - per), row + p.r_off + 4 * (j - per));
+                    else if (j < 3 * per) cp_async16(d + 2 * P + 4 * (j - 2 * per), p.in.wOut + wi + 4 * (j - 2 * per));
+                    else if (j < 4 * per) cp_async16(d + 3 * P + 4 * (j - 3 * per), p.in.bOut + wi + 4 * (j - 3 * per));
+                    else cp_async16(d + 4 * P + 4 * (j - 4 * per), row + p.v_off + cb + 4 * (j - 4 * per));
+                }
+            } else {
+                const int all = 4 * dim + nv;
+                for (int i = tid; i < n * all; i += 128) {
+                    const int t = i / all, j = i - t * all;
+                    const float* row = p.in.proj + (row0 + t0 + t) * p.in.ld + hd;
+                    const size_t wi = (row0 + t0 + t) * HD + hd;
+                    float* d = dst + t * ROW;
+                    const int f = j / dim, c = j - f * dim;
+                    cp_async4(d + f * P + c, f == 0 ? row + p.in.k_off + c : f == 1 ? row + p.r_off + c : f == 2 ? p.in.wOut + wi + c
+                                             : f == 3 ? p.in.bOut + wi + c : row + p.v_off + cb + c);
+                }
+            }
+            cp_async_commit();
+        };
+        load(0, 0);
+        for (int t0 = 0, stage = 0; t0 < p.T; t0 += TB, stage ^= 1) {
+            cp_async_wait<0>();
+            __syncthreads();                       // this stage has landed, nobody reads the other one any more
+            if (t0 + TB < p.T) load(t0 + TB, stage ^ 1);
+            const int n = min(TB, p.T - t0);
+            const float* rows = ring + stage * STAGE;
+            if (n == TB) {
+#pragma unroll 2
+                for (int t = 0; t < TB; t++) token(rows + t * ROW, t0 + t);
+            } else {
+                for (int t = 0; t < n; t++) token(rows + t * ROW, t0 + t);
+            }
         }
     }
 #pragma unroll
     for (int c = 0; c < C; c++)
 #pragma unroll
         for (int e = 0; e < E; e++) {
-            const int i = e * 32 + lane;
+            const int i = lane * E + e;
             if (i < dim && c0 + c < dim) st[(size_t)c * dim + i] = S[c][e];
         }
 }
 
-template <int E>
+template <int E, int TB>
 void launch_scan(const ScanParams& p, int B, cudaStream_t s) {
-    constexpr int C = 4;
-    launch_k(k_delta_scan<E, C>, dim3((unsigned)((p.dim + 4 * C - 1) / (4 * C)), (unsigned)p.H, (unsigned)B), dim3(128), 0, s, true, p);
+    constexpr int C = 4, ROW = 4 * 32 * E + 4 * C;
+    const dim3 grid((unsigned)((p.in.dim + 4 * C - 1) / (4 * C)), (unsigned)p.in.H, (unsigned)B);
+    if (p.T == 1) launch_k(k_delta_scan<E, C, TB, true>, grid, dim3(128), (size_t)(ROW + p.in.w2p) * 4, s, true, p);
+    else launch_k(k_delta_scan<E, C, TB, false>, grid, dim3(128), (size_t)2 * TB * ROW * 4, s, true, p);
 }
 
 }  // namespace
@@ -198,16 +267,17 @@ void launch_delta_rule(const DeltaRuleArgs& a, cudaStream_t s) {
     q.abias = a.abias; q.w2 = a.w2.w; q.w2p = a.w2.Kp; q.w0 = a.w0;
     q.wOut = a.ws; q.bOut = a.ws + (size_t)rows * a.H * a.dim;
     q.rows = rows; q.H = a.H; q.dim = a.dim;
-    launch_k(k_delta_prepare, dim3((unsigned)a.H, (unsigned)((rows + kPrepRows - 1) / kPrepRows)), dim3(128), (size_t)kPrepRows * (q.w2p + 1) * 4, s, true, q);
+    if (a.T > 1)
+        launch_k(k_delta_prepare, dim3((unsigned)a.H, (unsigned)((rows + kPrepRows - 1) / kPrepRows)), dim3(128), (size_t)kPrepRows * (q.w2p + 1) * 4, s, true, q);
     ScanParams p;
-    p.proj = a.proj; p.ld = a.ld; p.r_off = a.r_off; p.k_off = a.k_off; p.v_off = a.v_off;
-    p.w = q.wOut; p.b = q.bOut; p.state = a.state; p.pos = a.pos; p.out = a.out; p.ldo = a.ldo;
-    p.T = a.T; p.H = a.H; p.dim = a.dim;
-    if (a.dim <= 32) launch_scan<1>(p, a.B, s);
-    else if (a.dim <= 64) launch_scan<2>(p, a.B, s);
-    else if (a.dim <= 96) launch_scan<3>(p, a.B, s);
-    else if (a.dim <= 128) launch_scan<4>(p, a.B, s);
-    else launch_scan<8>(p, a.B, s);
+    p.in = q; p.r_off = a.r_off; p.v_off = a.v_off;
+    p.state = a.state; p.pos = a.pos; p.out = a.out; p.ldo = a.ldo; p.T = a.T;
+    p.vec = ((a.dim | a.ld | a.r_off | a.k_off | a.v_off) & 3) == 0 && (((uintptr_t)a.proj | (uintptr_t)a.ws) & 15) == 0;
+    if (a.dim <= 32) launch_scan<1, 8>(p, a.B, s);
+    else if (a.dim <= 64) launch_scan<2, 8>(p, a.B, s);
+    else if (a.dim <= 96) launch_scan<3, 8>(p, a.B, s);
+    else if (a.dim <= 128) launch_scan<4, 8>(p, a.B, s);
+    else launch_scan<8, 4>(p, a.B, s);
 }
 
 }  // namespace dj

@@ -154,6 +154,9 @@ DJ_PART void launch_bf16_linear(const Bf16LinearArgs& a, cudaStream_t s);
 // Grouped rows of a tensor-core product: the expert of every 128-row tile (−1: none), where output rows go, rows per expert.
 struct GroupedRows { const int* tileExpert; const int* rowMap; int rowsPerExpert; };
 DJ_PART bool launch_bf16_gemm_tc(const Bf16LinearArgs& a, const GroupedRows* g, cudaStream_t s);
+// out (bf16) = rows · Wᵀ for the first pos[0] + T bf16 rows (at most maxRows) of a row-major matrix with pitch lda.
+DJ_PART void launch_bf16_gemm_rows(const __nv_bfloat16* rows, int lda, int K, const float* pos, int T, int maxRows, const Bf16View& w, __nv_bfloat16* out, int ldo,
+                           cudaStream_t s);
 DJ_PART void launch_stage_rows(const RowOperand& a, const RowOperand& b, int Kp, int rows, const int* map, int div, void* out, bool bf16, cudaStream_t s);
 DJ_PART void launch_bf16_block_linear(const float* x, int ldx, int xstr, const Bf16View& w, int heads, float* out, int ldo, int ostr, int M, cudaStream_t s);
 // Table-routed experts: token id → `top` experts, each of weight 1/top.  up holds every expert's (gate, up) row pairs
@@ -194,12 +197,21 @@ struct LatentAttnArgs {
     const float* pos; const float* cosT; const float* sinT;      // [maxSeq × rot/2]
     float* out; int ldo;                       // [rows][H·R]
     int B, T, H, dim, rot, R; float scale;
-    float* ws;                                 // latent_attn_ws_floats
+    int vdim; Bf16View uk, uv;                 // prompt chunks over expanded keys and values only: [H·dim][R], [H·vdim][R]
+    float* ws;                                 // latent_attn_ws_floats / latent_prefill_ws_floats
 };
 DJ_PART bool latent_attn_fits(int R, int rot);
 DJ_PART int latent_attn_splits(int rows, int H, int maxSeq);
 DJ_PART size_t latent_attn_ws_floats(const LatentAttnArgs& a);
 DJ_PART void launch_latent_attn(const LatentAttnArgs& a, cudaStream_t s);
+DJ_PART void launch_latent_append(const LatentAttnArgs& a, cudaStream_t s);
+// tensor-core forms (attn_latent_mma.cu)
+DJ_PART bool latent_mma_fits(const LatentAttnArgs& a);
+DJ_PART int latent_mma_splits(const LatentAttnArgs& a);
+DJ_PART void launch_latent_mma(const LatentAttnArgs& a, cudaStream_t s);
+DJ_PART bool latent_prefill_fits(const LatentAttnArgs& a);
+DJ_PART size_t latent_prefill_ws_floats(const LatentAttnArgs& a);
+DJ_PART void launch_latent_prefill(const LatentAttnArgs& a, cudaStream_t s);
 
 // ── misc ──
 void launch_embed_gather(const float* table, const float* ids, float* out, int rows, int d, int vocab, cudaStream_t s);

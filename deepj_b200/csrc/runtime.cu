@@ -236,6 +236,7 @@ int op_stride(int op) {
         case DEEPJ_OP_DELTA_RULE: return 20;
         case DEEPJ_OP_ATTN_LATENT: return 26;
         case DEEPJ_OP_TABLE_EXPERTS: return 25;
+        case DEEPJ_OP_ATTN_LATENT_CHUNK: return 26;
         default: return -1;
     }
 }
@@ -591,7 +592,7 @@ void do_op(Ctx& ctx, const int32_t* c) {
         case DEEPJ_OP_ATTN_LATENT: {
             // [op, q, q_off, ldq, qc, qc_off, ldqc, kv, kv_off, ldkv, gamma, epsBits, cache, pos, cos, sin, out, out_off, ldo, B, T, H, dim, rot, R, scaleBits]
             const char* what = "attnLatent";
-            LatentAttnArgs a;
+            LatentAttnArgs a = {};
             a.B = c[19]; a.T = c[20]; a.H = c[21]; a.dim = c[22]; a.rot = c[23]; a.R = c[24]; a.scale = bits_to_float(c[25]);
             require(a.B >= 1 && a.T >= 1 && a.H >= 1 && a.dim >= 1 && (long)a.B * a.T <= 65535, what, "bad dimension");
             require(latent_attn_fits(a.R, a.rot), what, "latent or rotated size not supported");
@@ -609,6 +610,32 @@ void do_op(Ctx& ctx, const int32_t* c) {
             a.out = f32(ctx, c[16], (size_t)c[17] + sz(rows - 1, c[18]) + cw, what) + c[17]; a.ldo = c[18];
             a.ws = scratch(latent_attn_ws_floats(a));
             if (go) launch_latent_attn(a, s);
+            break;
+        }
+        case DEEPJ_OP_ATTN_LATENT_CHUNK: {
+            // [op, q, q_off, ldq, kv, kv_off, ldkv, gamma, epsBits, cache, pos, cos, sin, w_uk, w_uv, out, out_off, ldo, B, T, H, dim, rot, R, vdim, scaleBits]
+            const char* what = "attnLatentChunk";
+            LatentAttnArgs a = {};
+            a.B = c[18]; a.T = c[19]; a.H = c[20]; a.dim = c[21]; a.rot = c[22]; a.R = c[23]; a.vdim = c[24]; a.scale = bits_to_float(c[25]);
+            require(a.B >= 1 && a.T >= 1 && a.H >= 1 && a.H <= 65535 && a.dim >= 1 && a.rot >= 1 && a.R >= 1 && a.vdim >= 1 && (long)a.B * a.T <= 65535, what, "bad dimension");
+            Buf& lc = find_buf(ctx, c[9], kLatent, what);
+            require(lc.hd == a.R + a.rot && a.B <= lc.B, what, "shape does not match the cache");
+            a.cache = lc.ptr; a.bf16 = lc.kvHalf; a.maxSeq = lc.maxSeq;
+            require(latent_prefill_fits(a), what, "sizes not supported (bf16 cache, multiples of eight)");
+            Buf& uk = find_buf(ctx, c[13], kBf16, what);
+            Buf& uv = find_buf(ctx, c[14], kBf16, what);
+            require(uk.K == a.R && uk.N == a.H * a.dim && uv.K == a.R && uv.N == a.H * a.vdim, what, "weights do not match the heads");
+            a.uk = bf16view(uk); a.uv = bf16view(uv);
+            const int rows = a.B * a.T, qw = a.H * (a.dim + a.rot), ow = a.H * a.vdim;
+            require(c[2] >= 0 && c[2] % 2 == 0 && c[3] % 2 == 0 && c[5] >= 0 && c[16] >= 0 && c[3] >= qw && c[6] >= a.R + a.rot && c[17] >= ow, what, "bad offset or stride");
+            a.q = f32(ctx, c[1], (size_t)c[2] + sz(rows - 1, c[3]) + qw, what) + c[2]; a.ldq = c[3];
+            a.kv = f32(ctx, c[4], (size_t)c[5] + sz(rows - 1, c[6]) + a.R + a.rot, what) + c[5]; a.ldkv = c[6];
+            a.gamma = f32(ctx, c[7], a.R, what); a.eps = bits_to_float(c[8]);
+            a.pos = f32(ctx, c[10], a.B, what);
+            a.cosT = f32(ctx, c[11], sz(lc.maxSeq, a.rot / 2), what); a.sinT = f32(ctx, c[12], sz(lc.maxSeq, a.rot / 2), what);
+            a.out = f32(ctx, c[15], (size_t)c[16] + sz(rows - 1, c[17]) + ow, what) + c[16]; a.ldo = c[17];
+            a.ws = scratch(latent_prefill_ws_floats(a));
+            if (go) { launch_latent_append(a, s); launch_latent_prefill(a, s); }
             break;
         }
         case DEEPJ_OP_TABLE_EXPERTS: {

@@ -23,7 +23,7 @@ from typing import Any, Callable, Dict, List, Mapping, Optional, Tuple
 import numpy as np
 
 from . import _lib
-from .compute_graph import (OP_ADD_SCALAR_INPLACE, OP_ARGMAX_ROWS, OP_ATTN_LATENT, OP_BF16_BLOCK_LINEAR, OP_BF16_LINEAR, OP_COPY, OP_DELTA_RULE,
+from .compute_graph import (OP_ADD_SCALAR_INPLACE, OP_ARGMAX_ROWS, OP_ATTN_LATENT, OP_ATTN_LATENT_CHUNK, OP_BF16_BLOCK_LINEAR, OP_BF16_LINEAR, OP_COPY, OP_DELTA_RULE,
                             OP_EMBED_GATHER, OP_SAMPLE_TOPK, OP_TABLE_EXPERTS, float_bits)
 from .decoder import scaled_rope_tables
 from .runner import StreamDecoder
@@ -151,10 +151,22 @@ class LatentAttention:
         dec._f32(f"dqnorm.{l}", self.q_rank, get("mix.dq.norm"))
         dec._f32(f"dkvnorm.{l}", R, get("mix.dkv.norm"))
         dec._weight(f"uq.{l}", self.q_rank, H * (self.dim + self.rot_dim), [("mix.uq", 0, 1, 0)], get)
-        # queries enter the latent space: W_uk of every head transposed, [heads · kv_rank][dim]
-        dec._weight(f"ukT.{l}", self.dim, H * R, [("mix.uk", 0, 1, 0)],
-                    lambda name: np.ascontiguousarray(get(name).reshape(H, self.dim, R).transpose(0, 2, 1)).reshape(H * R, self.dim))
+
+        def transposed(name):            # queries enter the latent space: W_uk of every head transposed, [heads · kv_rank][dim]
+            a = get(name)
+            if isinstance(a, tuple):     # generated on the device: any order will do
+                return H * R, self.dim, a[2]
+            return np.ascontiguousarray(a.reshape(H, self.dim, R).transpose(0, 2, 1)).reshape(H * R, self.dim)
+
+        dec._weight(f"ukT.{l}", self.dim, H * R, [("mix.uk", 0, 1, 0)], transposed)
+        if self.expands(dec):
+            dec._weight(f"uk.{l}", R, H * self.dim, [("mix.uk", 0, 1, 0)], get)
         dec._weight(f"uv.{l}", R, H * self.vdim, [("mix.uv", 0, 1, 0)], get)
+
+    def expands(self, dec: "HybridDecoder") -> bool:
+        """Whether prompt chunks run over expanded keys and values (op 82)."""
+        return (dec.dtype == "bf16" and all(n % 8 == 0 for n in (self.dim, self.rot_dim, self.vdim, self.kv_rank)) and self.dim + self.rot_dim <= 256 and
+                self.vdim <= 128)
 
     def emit(self, op, dec: "HybridDecoder", l: int, buf: Dict[str, int], B: int, T: int) -> None:
         I, at, ld, M = dec.ids, dec._offsets[l], dec._in_rows[l], B * T
@@ -163,6 +175,11 @@ class LatentAttention:
         key = f"rot {self.rot_dim} {self.base} {self.scaling}"
         dec._linear(op, "q_up", [buf["proj"], at["mix.dq"], ld, I[f"dqnorm.{l}"], 1, eps, -1, 0, 0], self.q_rank, None, I[f"uq.{l}"],
                     None, (buf["q"], qw), M, qw)
+        if self.expands(dec) and T >= EXPAND_MIN_TOKENS:
+            op("attn", OP_ATTN_LATENT_CHUNK, buf["q"], 0, qw, buf["proj"], at["mix.dkv"], ld, I[f"dkvnorm.{l}"], eps, I[f"cache.{l}"], I["pos"],
+               I[key + " cos"], I[key + " sin"], I[f"uk.{l}"], I[f"uv.{l}"], buf["mix"], 0, self.out_width, B, T, H, self.dim, self.rot_dim, R, self.vdim,
+               float_bits(self.scale))
+            return
         op("q_latent", OP_BF16_BLOCK_LINEAR, buf["q"], 0, qw, self.dim + self.rot_dim, I[f"ukT.{l}"], H, buf["qc"], 0, H * R, R, M)
         op("attn", OP_ATTN_LATENT, buf["q"], 0, qw, buf["qc"], 0, H * R, buf["proj"], at["mix.dkv"], ld, I[f"dkvnorm.{l}"], eps, I[f"cache.{l}"],
            I["pos"], I[key + " cos"], I[key + " sin"], buf["ctx"], 0, H * R, B, T, H, self.dim, self.rot_dim, R, float_bits(self.scale))
@@ -172,6 +189,7 @@ class LatentAttention:
         return [buf["mix"], 0, self.out_width, -1, 0, 0, buf["proj"], dec._offsets[l]["mix.g"], dec._in_rows[l]]
 
 
+EXPAND_MIN_TOKENS = 48      # chunks from here on expand the context's keys and values; shorter ones attend in the latent space
 MIXERS = {"general_delta": GeneralDelta, "latent_attention": LatentAttention}
 RECURRENT = (GeneralDelta,)
 
@@ -262,6 +280,8 @@ class HybridDecoder(StreamDecoder):
             raise ValueError("dtype must be 'bf16' or 'f32'")
         super().__init__(cfg, batch, device, id_base)
         self.dtype = dtype
+        self.weight_dims: Dict[int, Tuple[int, int]] = {}         # bf16 object → (K, N)
+        self.tables: Dict[str, np.ndarray] = {}
         self.REWINDS = not any(isinstance(m, RECURRENT) for m, _ in cfg.layers)
         # the input projection's rows per layer: every field starts at a multiple of eight, the gated pairs come last
         self._offsets: List[Dict[str, int]] = []
@@ -309,6 +329,7 @@ class HybridDecoder(StreamDecoder):
             _lib.check(self.lib.deepj_cuda_bf16_store(i, row0, step, col0, tmp, 0, rows, cols))
             self._release([tmp])
         self.ids[name] = i
+        self.weight_dims[i] = (K, N)
 
     def _load(self, get: Callable[[str], Any], vec: Callable[[str], np.ndarray], table: Callable[[str], np.ndarray]) -> None:
         """`get` yields a matrix (or a recipe for one), `vec` a vector, `table` an integer table."""
@@ -336,6 +357,7 @@ class HybridDecoder(StreamDecoder):
                 if t.min() < 0 or t.max() >= ff.experts:
                     raise ValueError("the expert table names an expert that does not exist")
                 self._f32(f"table.{l}", t.size, t.astype(np.float32))
+                self.tables[f"table.{l}"] = t
                 self._weight(f"up.{l}", d, ff.experts * 2 * ff.ff,
                              [(f"mlp.e{e}.{k}", e * 2 * ff.ff + j, 2, 0) for e in range(ff.experts) for j, k in enumerate(("gate", "up"))], mine)
                 self._weight(f"down.{l}", ff.ff, ff.experts * d, [(f"mlp.e{e}.down", e * d, 1, 0) for e in range(ff.experts)], mine)

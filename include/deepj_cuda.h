@@ -257,6 +257,11 @@ int deepj_cuda_latent_alloc(int32_t id, int32_t batch, int32_t max_seq, int32_t 
  *  81 TABLE_EXPERTS     [op, x, x_off, ldx, gamma, groups, epsBits, tok, table, vocab, top, experts, w_up, w_down, ff,
  *                        limitBits, residual, res_off, ldr, out, out_off, ldo, d, M, exact]
  *                        out = residual + (1/top) sum over the experts of table[token] of their gated feed-forward
+ *  82 ATTN_LATENT_CHUNK [op, q, q_off, ldq, kv, kv_off, ldkv, gamma, epsBits, cache, pos, cos, sin, w_uk, w_uv,
+ *                        out, out_off, ldo, B, T, H, dim, rot, R, vdim, scaleBits]
+ *                        op 80 for prompt chunks over a bf16 cache: keys and values of the context are expanded per head
+ *                        (w_uk [H·dim][R], w_uv [H·vdim][R]); out = the heads' values.  Sizes multiples of eight,
+ *                        dim + rot <= 256, vdim <= 128
  */
 #define DEEPJ_OP_EMBED_GATHER        64
 #define DEEPJ_OP_Q8_LINEAR           65
@@ -276,6 +281,7 @@ int deepj_cuda_latent_alloc(int32_t id, int32_t batch, int32_t max_seq, int32_t 
 #define DEEPJ_OP_DELTA_RULE         79
 #define DEEPJ_OP_ATTN_LATENT        80
 #define DEEPJ_OP_TABLE_EXPERTS      81
+#define DEEPJ_OP_ATTN_LATENT_CHUNK  82
 
 #ifdef __cplusplus
 }

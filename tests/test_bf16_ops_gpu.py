@@ -4,7 +4,7 @@ import pytest
 
 import punilix_ref as ref
 from deepj_b200 import _lib
-from deepj_b200.compute_graph import (OP_ATTN_LATENT, OP_BF16_BLOCK_LINEAR, OP_BF16_LINEAR, OP_DELTA_RULE, OP_TABLE_EXPERTS, float_bits)
+from deepj_b200.compute_graph import (OP_ATTN_LATENT, OP_ATTN_LATENT_CHUNK, OP_BF16_BLOCK_LINEAR, OP_BF16_LINEAR, OP_DELTA_RULE, OP_TABLE_EXPERTS, float_bits)
 from deepj_b200.decoder import scaled_rope_tables
 from test_q8_gpu import Dev
 
@@ -255,3 +255,49 @@ def test_table_experts(dev, exact, M, d, ff, experts, top):
     for _ in range(2):
         dev.flush(cmd)
     near(want, dev.get(o, M * d).reshape(M, d) - res, 2e-5 if exact or M <= 16 else 2e-2)
+
+
+@pytest.mark.parametrize("B,H,dim,rot,R,vdim,portions,scaled", [
+    (1, 8, 64, 16, 64, 48, [150, 1, 70], True), (1, 3, 24, 8, 48, 16, [48, 200], False), (2, 5, 40, 24, 200, 72, [65, 64], True),
+    (1, 4, 128, 64, 512, 128, [300, 2, 129], True), (1, 2, 192, 64, 128, 104, [130, 1], False)])
+def test_latent_attention_of_prompt_chunks(dev, B, H, dim, rot, R, vdim, portions, scaled):
+    """Op 82 (expanded keys and values) between portions that op 80 would take: same cache, values against the reference."""
+    rng = np.random.default_rng(H * R + rot + vdim)
+    total, W, qw = sum(portions), R + rot, H * (dim + rot)
+    scaling = {"factor": 8.0, "original": 32, "fast": 16.0, "slow": 2.0} if scaled else None
+    base, scale, eps = 5000.0, 1.3 / np.sqrt(dim + rot), 1e-5
+    kv, q = rng.standard_normal((B, total, W)), rng.standard_normal((B, total, H, dim + rot))
+    gamma = 1 + 0.2 * rng.standard_normal(R)
+    uk, uv = bf16(rng.standard_normal((H, dim, R)) / np.sqrt(R)), bf16(rng.standard_normal((H, vdim, R)) / np.sqrt(R))
+    c = bf16(ref.rms_norm(kv[..., :R], gamma, eps)).astype(np.float64)
+    for t in range(total):                       # some queries look for their own key, the first key, or one in between
+        for h, j in ((0, t), (H - 1, 0), (H // 2, t * 2 // 3)):
+            if t % 3 == 0:
+                for b in range(B):
+                    k = uk[h] @ c[b, j]
+                    q[b, t, h, :dim] = k * 10.0 / scale / (k @ k)
+    want = np.zeros((B, total, H, vdim))
+    for b in range(B):
+        kr = bf16(ref.rotate_interleaved(kv[b, :, R:], np.arange(total), rot, base, scaling)).astype(np.float64)
+        qr = ref.rotate_interleaved(q[b][..., -rot:], np.arange(total), rot, base, scaling)
+        k_un, v = np.einsum("hdr,tr->thd", uk, c[b]), np.einsum("hdr,tr->thd", uv, c[b])
+        for t in range(total):
+            s = (np.einsum("hd,thd->ht", q[b, t, :, :dim], k_un[:t + 1]) + qr[t] @ kr[:t + 1].T) * scale
+            want[b, t] = np.einsum("ht,thd->hd", ref.softmax_rows(s), v[:t + 1])
+    max_seq = total + 5
+    cos, sin = scaled_rope_tables(rot, max_seq, base, scaling)
+    cb, sb, gb, pos = dev.buf(cos.size, cos), dev.buf(sin.size, sin), dev.buf(R, gamma), dev.buf(B)
+    cache = dev.latent(B, max_seq, W, 1)
+    wk, wv = dev.weight(R, H * dim, [(uk.reshape(-1, R), 0, 1, 0)]), dev.weight(R, H * vdim, [(uv.reshape(-1, R), 0, 1, 0)])
+    qb, kvb, out = dev.buf(B * total * qw), dev.buf(B * total * W), dev.buf(B * total * H * vdim)
+    lo = 0
+
+    def put(i, a):
+        a = np.ascontiguousarray(a, dtype=np.float32)
+        _lib.check(dev.lib.deepj_cuda_upload_buffer(i, a.ctypes.data, a.size))
+    for T in portions:
+        put(qb, q[:, lo:lo + T]); put(pos, np.full(B, lo)); put(kvb, kv[:, lo:lo + T])
+        dev.flush([OP_ATTN_LATENT_CHUNK, qb, 0, qw, kvb, 0, W, gb, float_bits(eps), cache, pos, cb, sb, wk, wv, out, 0, H * vdim, B, T, H, dim, rot, R, vdim,
+                   float_bits(scale)])
+        near(want[:, lo:lo + T], dev.get(out, B * T * H * vdim).reshape(B, T, H, vdim), 1.5e-2)
+        lo += T
