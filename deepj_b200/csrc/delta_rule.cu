@@ -7,39 +7,50 @@
 // 0 starts from zeros whatever the buffer holds.  Prompts and single tokens run the same scan, token by token, so how a
 // prompt is cut changes nothing.
 //
-//   k_delta_prepare   per (token, head): w, and b = a ⊙ k / (Σk² + ε) — with b the removal term is b (kᵀS)
+//   k_delta_prepare   per (token, head): w, b = a ⊙ k / (Σk² + ε) — with b the removal term is b (kᵀS) — and, per block of four
+//                     tokens, what relates them: with P_ij = Π_{i<l<j} w_l, the vectors k̃_j = k_j ⊙ Π_{l<j} w_l and the scalars
+//                     A_ij = k_jᵀ(P_ij ⊙ b_i), B_ij = k_jᵀ(P_ij ⊙ k_i)
 //   k_delta_scan      a block of four warps per (sequence, head, 16 value columns), a warp per four of them: a lane holds some
-//                     key channels of its columns in registers, kᵀS and o are warp reductions over all lanes, and the
-//                     tokens' vectors stream through a two-stage cp.async ring of shared memory.  A single token computes
-//                     its own w and b (no prepare launch) and reads the state before the dependency wait.
+//                     key channels of its columns in registers.  The four kᵀS of a token block come out of ONE warp reduction
+//                     against the state S_0 before it: k_jᵀS_{j-1} = k̃_jᵀS_0 − Σ_{i<j} A_ij k_iᵀS_{i-1} + Σ_{i<j} B_ij v_i;
+//                     then the four updates run on the registers and the four outputs share a second reduction.  Tokens
+//                     stream through a two-stage cp.async ring.  A single token (decode) computes its own w and b and reads
+//                     the state before the dependency wait.
 #include "row_operand.cuh"
+
+#include <algorithm>
 
 namespace dj {
 namespace {
 
 constexpr float kUnitEps = 1e-6f;
-constexpr int kPrepRows = 8;
+constexpr int kPrepRows = 8;           // tokens per block of k_delta_prepare: two token blocks
+constexpr int kBlk = 4, kPairs = 6;    // tokens per block, pairs i < j of them
 
 struct PrepParams {
     const float* proj; int ld, k_off, a_off, low_off, rank;
     const float* abias; const __nv_bfloat16* w2; int w2p; const float* w0;
-    float* wOut; float* bOut;        // [rows][H·dim]
-    int rows, H, dim;
+    float* wOut; float* bOut; float* ktOut;      // [rows][H·dim]
+    float* pairs;                                // [B][token blocks][H][2·kPairs]: A then B, pairs (0,1)(0,2)(1,2)(0,3)(1,3)(2,3)
+    int T, H, dim;
 };
+__device__ __forceinline__ int token_blocks(int T) { return (T + kBlk - 1) / kBlk; }
 
 __global__ void __launch_bounds__(128) k_delta_prepare(const PrepParams p) {
-    extern __shared__ float low[];                       // [kPrepRows][w2p], then [kPrepRows] 1 / (Σk² + ε)
+    extern __shared__ __align__(16) float low[];                       // [kPrepRows][w2p], then [kPrepRows] 1 / (Σk² + ε)
+    __shared__ float red[4][2 * 2 * kPairs];
     float* inv = low + kPrepRows * p.w2p;
     pdl_wait();
     pdl_launch_dependents();
-    const int h = blockIdx.x, r0 = blockIdx.y * kPrepRows, n = min(kPrepRows, p.rows - r0);
+    const int h = blockIdx.x, t0 = blockIdx.y * kPrepRows, n = min(kPrepRows, p.T - t0);
+    const size_t r0 = (size_t)blockIdx.z * p.T + t0;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     for (int i = threadIdx.x; i < kPrepRows * p.w2p; i += 128) {
         const int r = i / p.w2p, j = i - r * p.w2p;
-        low[i] = (r < n && j < p.rank) ? tanhf(p.proj[(size_t)(r0 + r) * p.ld + p.low_off + j]) : 0.0f;
+        low[i] = (r < n && j < p.rank) ? tanhf(p.proj[(r0 + r) * p.ld + p.low_off + j]) : 0.0f;
     }
     for (int r = warp; r < n; r += 4) {
-        const float* k = p.proj + (size_t)(r0 + r) * p.ld + p.k_off + h * p.dim;
+        const float* k = p.proj + (r0 + r) * p.ld + p.k_off + h * p.dim;
         float ss = 0.0f;
         for (int i = lane; i < p.dim; i += 32) ss = fmaf(k[i], k[i], ss);
         for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
@@ -47,6 +58,11 @@ __global__ void __launch_bounds__(128) k_delta_prepare(const PrepParams p) {
     }
     __syncthreads();
     const float rate = expf(-0.5f);
+    float pr[2][2 * kPairs];
+#pragma unroll
+    for (int q = 0; q < 2; q++)
+#pragma unroll
+        for (int j = 0; j < 2 * kPairs; j++) pr[q][j] = 0.0f;
     for (int i = threadIdx.x; i < p.dim; i += 128) {
         const int c = h * p.dim + i;
         float acc[kPrepRows];
@@ -61,22 +77,60 @@ __global__ void __launch_bounds__(128) k_delta_prepare(const PrepParams p) {
                 const float lo = __uint_as_float(u[q] << 16), hi = __uint_as_float(u[q] & 0xffff0000u);
 #pragma unroll
                 for (int r = 0; r < kPrepRows; r++) {
-                    acc[r] = fmaf(lo, low[r * p.w2p + j + 2 * q], acc[r]);
-                    acc[r] = fmaf(hi, low[r * p.w2p + j + 2 * q + 1], acc[r]);
+                    const float2 l = *reinterpret_cast<const float2*>(low + r * p.w2p + j + 2 * q);
+                    acc[r] = fmaf(lo, l.x, acc[r]);
+                    acc[r] = fmaf(hi, l.y, acc[r]);
                 }
             }
         }
         const float w0 = p.w0[c], ab = p.abias[c];
-        for (int r = 0; r < n; r++) {
-            const float* row = p.proj + (size_t)(r0 + r) * p.ld;
-            const size_t o = (size_t)(r0 + r) * p.H * p.dim + c;
-            float a8 = acc[0];
 #pragma unroll
-            for (int q = 1; q < kPrepRows; q++) a8 = r == q ? acc[q] : a8;
-            p.wOut[o] = expf(-rate * sigmoid_f(a8 + w0));
-            p.bOut[o] = sigmoid_f(row[p.a_off + c] + ab) * row[p.k_off + c] * inv[r];
+        for (int q = 0; q < 2; q++) {
+            float kv[kBlk], wv[kBlk], bv[kBlk];
+#pragma unroll
+            for (int j = 0; j < kBlk; j++) {
+                const int r = q * kBlk + j;
+                kv[j] = 0.0f; wv[j] = 1.0f; bv[j] = 0.0f;
+                if (r < n) {
+                    const float* row = p.proj + (r0 + r) * p.ld;
+                    kv[j] = row[p.k_off + c];
+                    wv[j] = expf(-rate * sigmoid_f(acc[r] + w0));
+                    bv[j] = sigmoid_f(row[p.a_off + c] + ab) * kv[j] * inv[r];
+                }
+            }
+            float run = 1.0f;
+            int pair = 0;
+#pragma unroll
+            for (int j = 0; j < kBlk; j++) {
+                if (q * kBlk + j < n) {
+                    const size_t o = (r0 + q * kBlk + j) * p.H * p.dim + c;
+                    p.wOut[o] = wv[j]; p.bOut[o] = bv[j]; p.ktOut[o] = kv[j] * run;
+                }
+                run *= wv[j];
+#pragma unroll
+                for (int e = 0; e < j; e++, pair++) {
+                    float x = kv[j];
+#pragma unroll
+                    for (int l = e + 1; l < j; l++) x *= wv[l];
+                    pr[q][pair] = fmaf(x, bv[e], pr[q][pair]);
+                    pr[q][kPairs + pair] = fmaf(x, kv[e], pr[q][kPairs + pair]);
+                }
+            }
         }
     }
+#pragma unroll
+    for (int q = 0; q < 2; q++)
+#pragma unroll
+        for (int j = 0; j < 2 * kPairs; j++) {
+            float v = pr[q][j];
+            for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+            if (lane == 0) red[warp][q * 2 * kPairs + j] = v;
+        }
+    __syncthreads();
+    const int tb = threadIdx.x / (2 * kPairs), j = threadIdx.x % (2 * kPairs), blk = t0 / kBlk + tb;
+    if (tb < 2 && blk < token_blocks(p.T))
+        p.pairs[(((size_t)blockIdx.z * token_blocks(p.T) + blk) * p.H + h) * 2 * kPairs + j] =
+            (red[0][threadIdx.x] + red[1][threadIdx.x]) + (red[2][threadIdx.x] + red[3][threadIdx.x]);
 }
 
 struct ScanParams {
@@ -104,18 +158,38 @@ __device__ __forceinline__ float reduce_columns(float (&v)[C], int lane) {
     return v[0];
 }
 
-// E key channels per lane (lane·E …), C value columns per warp, TB tokens per stage of the ring.
-template <int E, int C, int TB, bool FUSED>
+// E consecutive floats of a lane
+template <int E>
+__device__ __forceinline__ void lane_row(const float* row, int lane, float (&v)[E]) {
+    if constexpr (E % 4 == 0) {
+#pragma unroll
+        for (int j = 0; j < E / 4; j++) {
+            const float4 f = *reinterpret_cast<const float4*>(row + lane * E + 4 * j);
+            v[4 * j] = f.x; v[4 * j + 1] = f.y; v[4 * j + 2] = f.z; v[4 * j + 3] = f.w;
+        }
+    } else if constexpr (E == 2) {
+        const float2 f = *reinterpret_cast<const float2*>(row + lane * 2);
+        v[0] = f.x; v[1] = f.y;
+    } else {
+#pragma unroll
+        for (int e = 0; e < E; e++) v[e] = row[lane * E + e];
+    }
+}
+
+// E key channels per lane (lane·E …), four value columns per warp, TB tokens per stage of the ring.
+template <int E, int TB, bool FUSED>
 __global__ void __launch_bounds__(128) k_delta_scan(const ScanParams p) {
-    constexpr int P = 32 * E, ROW = 4 * P + 4 * C, STAGE = TB * ROW;        // a token: k, r, w, b of the head, v of the block's columns
-    extern __shared__ __align__(16) float ring[];                           // [2][TB][ROW]; FUSED: one token, then low [w2p]
+    constexpr int C = 4, P = 32 * E, ROW = 5 * P + 4 * C;                   // a token: k̃, k, w, b, r of the head, v of the block's columns
+    constexpr int STAGE = TB * ROW + TB / kBlk * 2 * kPairs;                // … and the pairs of its token blocks
+    extern __shared__ __align__(16) float ring[];                           // [2][STAGE]; FUSED: one token, then low [w2p]
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int h = blockIdx.y, b = blockIdx.z, dim = p.in.dim, H = p.in.H, HD = H * dim, hd = h * dim;
     const int cb = blockIdx.x * 4 * C, c0 = cb + warp * C;                  // the block's and this warp's first column
     const size_t row0 = (size_t)b * p.T;
     if (P > dim)                                                            // channels past the head stay zero
-        for (int i = tid; i < (FUSED ? 1 : 2 * TB) * 4 * (P - dim); i += 128)
-            ring[(i / (4 * (P - dim))) * ROW + (i / (P - dim)) % 4 * P + dim + i % (P - dim)] = 0.0f;
+        for (int t = 0; t < (FUSED ? 1 : 2 * TB); t++)
+            for (int i = tid; i < 5 * (P - dim); i += 128)
+                ring[(t / TB) * STAGE + (t % TB) * ROW + i / (P - dim) * P + dim + i % (P - dim)] = 0.0f;
     // the state was last written several kernels ago: it may be read before the dependency wait
     const bool fresh = p.pos[b] == 0.0f;
     float* st = p.state + (((size_t)b * H + h) * dim + c0) * dim;
@@ -127,35 +201,6 @@ __global__ void __launch_bounds__(128) k_delta_scan(const ScanParams p) {
             const int i = lane * E + e;
             S[c][e] = (!fresh && i < dim && c0 + c < dim) ? st[(size_t)c * dim + i] : 0.0f;
         }
-    auto token = [&](const float* row, int t) {
-        float k[E], r[E], w[E], q[E], v[C];
-#pragma unroll
-        for (int e = 0; e < E; e++) { k[e] = row[lane * E + e]; r[e] = row[P + lane * E + e]; w[e] = row[2 * P + lane * E + e]; q[e] = row[3 * P + lane * E + e]; }
-#pragma unroll
-        for (int c = 0; c < C; c++) v[c] = row[4 * P + warp * C + c];
-        float d[C];
-#pragma unroll
-        for (int c = 0; c < C; c++) {
-            d[c] = k[0] * S[c][0];
-#pragma unroll
-            for (int e = 1; e < E; e++) d[c] = fmaf(k[e], S[c][e], d[c]);
-        }
-        const float ks = reduce_columns<C>(d, lane);
-        float o[C];
-#pragma unroll
-        for (int c = 0; c < C; c++) {
-            const float dot = __shfl_sync(0xffffffffu, ks, c * (32 / C));
-            o[c] = 0.0f;
-#pragma unroll
-            for (int e = 0; e < E; e++) {
-                S[c][e] = fmaf(w[e], S[c][e], fmaf(k[e], v[c], -(q[e] * dot)));
-                o[c] = fmaf(r[e], S[c][e], o[c]);
-            }
-        }
-        const float os = reduce_columns<C>(o, lane);
-        const int col = c0 + lane / (32 / C);
-        if (lane % (32 / C) == 0 && col < dim) p.out[(row0 + t) * p.ldo + hd + col] = os;
-    };
     if constexpr (FUSED) {
         pdl_wait();
         pdl_launch_dependents();
@@ -168,9 +213,9 @@ __global__ void __launch_bounds__(128) k_delta_scan(const ScanParams p) {
         const float inv = 1.0f / (ss + kUnitEps), rate = expf(-0.5f);
         __syncthreads();
         for (int i = tid; i < dim; i += 128) {
-            const float k = x[p.in.k_off + hd + i];
-            ring[i] = k;
-            ring[P + i] = x[p.r_off + hd + i];
+            const float kk = x[p.in.k_off + hd + i];
+            ring[P + i] = kk;
+            ring[4 * P + i] = x[p.r_off + hd + i];
             float acc = 0.0f;
             const __nv_bfloat16* w = p.in.w2 + (size_t)(hd + i) * p.in.w2p;
             for (int j = 0; j < p.in.w2p; j += 8) {
@@ -183,42 +228,55 @@ __global__ void __launch_bounds__(128) k_delta_scan(const ScanParams p) {
                 }
             }
             ring[2 * P + i] = expf(-rate * sigmoid_f(acc + p.in.w0[hd + i]));
-            ring[3 * P + i] = sigmoid_f(x[p.in.a_off + hd + i] + p.in.abias[hd + i]) * k * inv;
+            ring[3 * P + i] = sigmoid_f(x[p.in.a_off + hd + i] + p.in.abias[hd + i]) * kk * inv;
         }
-        for (int i = tid; i < 4 * C; i += 128) ring[4 * P + i] = cb + i < dim ? x[p.v_off + hd + cb + i] : 0.0f;
+        for (int i = tid; i < 4 * C; i += 128) ring[5 * P + i] = cb + i < dim ? x[p.v_off + hd + cb + i] : 0.0f;
         __syncthreads();
-        token(ring, 0);
+        float k[E], w[E], q[E], r[E], d[C], o[C];
+        lane_row<E>(ring + P, lane, k); lane_row<E>(ring + 2 * P, lane, w); lane_row<E>(ring + 3 * P, lane, q); lane_row<E>(ring + 4 * P, lane, r);
+#pragma unroll
+        for (int c = 0; c < C; c++) {
+            d[c] = k[0] * S[c][0];
+#pragma unroll
+            for (int e = 1; e < E; e++) d[c] = fmaf(k[e], S[c][e], d[c]);
+        }
+        const float ks = reduce_columns<C>(d, lane);
+#pragma unroll
+        for (int c = 0; c < C; c++) {
+            const float dot = __shfl_sync(0xffffffffu, ks, c * (32 / C)), v = ring[5 * P + warp * C + c];
+            o[c] = 0.0f;
+#pragma unroll
+            for (int e = 0; e < E; e++) {
+                S[c][e] = fmaf(w[e], S[c][e], fmaf(k[e], v, -(q[e] * dot)));
+                o[c] = fmaf(r[e], S[c][e], o[c]);
+            }
+        }
+        const float os = reduce_columns<C>(o, lane);
+        const int col = c0 + lane / (32 / C);
+        if (lane % (32 / C) == 0 && col < dim) p.out[row0 * p.ldo + hd + col] = os;
     } else {
         pdl_wait();
         pdl_launch_dependents();
-        const int nv = min(4 * C, dim - cb);
-        auto load = [&](int t0, int stage) {
+        const int nv = min(4 * C, dim - cb), nBlk = token_blocks(p.T);
+        auto load = [&](int t0, int stage) {           // a warp copies tokens warp, warp + 4, … of the stage
             float* dst = ring + stage * STAGE;
             const int n = min(TB, p.T - t0);
-            if (p.vec) {
-                const int per = dim / 4, all = 4 * per + nv / 4;
-                for (int i = tid; i < n * all; i += 128) {
-                    const int t = i / all, j = i - t * all;
-                    const float* row = p.in.proj + (row0 + t0 + t) * p.in.ld + hd;
-                    const size_t wi = (row0 + t0 + t) * HD + hd;
-                    float* d = dst + t * ROW;
-                    if (j < per) cp_async16(d + 4 * j, row + p.in.k_off + 4 * j);
-                    else if (j < 2 * per) cp_async16(d + P + 4 * (j - per), row + p.r_off + 4 * (j - per));
-                    else if (j < 3 * per) cp_async16(d + 2 * P + 4 * (j - 2 * per), p.in.wOut + wi + 4 * (j - 2 * per));
-                    else if (j < 4 * per) cp_async16(d + 3 * P + 4 * (j - 3 * per), p.in.bOut + wi + 4 * (j - 3 * per));
-                    else cp_async16(d + 4 * P + 4 * (j - 4 * per), row + p.v_off + cb + 4 * (j - 4 * per));
+            for (int t = warp; t < n; t += 4) {
+                const size_t r = row0 + t0 + t;
+                const float* row = p.in.proj + r * p.in.ld + hd;
+                const float* src[5] = {p.in.ktOut + r * HD + hd, row + p.in.k_off, p.in.wOut + r * HD + hd, p.in.bOut + r * HD + hd, row + p.r_off};
+                float* d = dst + t * ROW;
+#pragma unroll
+                for (int f = 0; f < 5; f++) {
+                    if (p.vec) { for (int i = lane * 4; i < dim; i += 128) cp_async16(d + f * P + i, src[f] + i); }
+                    else { for (int i = lane; i < dim; i += 32) cp_async4(d + f * P + i, src[f] + i); }
                 }
-            } else {
-                const int all = 4 * dim + nv;
-                for (int i = tid; i < n * all; i += 128) {
-                    const int t = i / all, j = i - t * all;
-                    const float* row = p.in.proj + (row0 + t0 + t) * p.in.ld + hd;
-                    const size_t wi = (row0 + t0 + t) * HD + hd;
-                    float* d = dst + t * ROW;
-                    const int f = j / dim, c = j - f * dim;
-                    cp_async4(d + f * P + c, f == 0 ? row + p.in.k_off + c : f == 1 ? row + p.r_off + c : f == 2 ? p.in.wOut + wi + c
-                                             : f == 3 ? p.in.bOut + wi + c : row + p.v_off + cb + c);
-                }
+                if (p.vec) { if (lane * 4 < nv) cp_async16(d + 5 * P + lane * 4, row + p.v_off + cb + lane * 4); }
+                else if (lane < nv) cp_async4(d + 5 * P + lane, row + p.v_off + cb + lane);
+            }
+            for (int i = tid; i < TB / kBlk * 2 * kPairs; i += 128) {
+                const int blk = t0 / kBlk + i / (2 * kPairs);
+                if (blk < nBlk) cp_async4(dst + TB * ROW + i, p.in.pairs + (((size_t)b * nBlk + blk) * H + h) * 2 * kPairs + i % (2 * kPairs));
             }
             cp_async_commit();
         };
@@ -227,13 +285,68 @@ __global__ void __launch_bounds__(128) k_delta_scan(const ScanParams p) {
             cp_async_wait<0>();
             __syncthreads();                       // this stage has landed, nobody reads the other one any more
             if (t0 + TB < p.T) load(t0 + TB, stage ^ 1);
-            const int n = min(TB, p.T - t0);
-            const float* rows = ring + stage * STAGE;
-            if (n == TB) {
-#pragma unroll 2
-                for (int t = 0; t < TB; t++) token(rows + t * ROW, t0 + t);
-            } else {
-                for (int t = 0; t < n; t++) token(rows + t * ROW, t0 + t);
+#pragma unroll 1
+            for (int q = 0; q < TB / kBlk; q++) {
+                const int n = min(kBlk, p.T - t0 - q * kBlk);      // tokens of this block
+                if (n <= 0) break;
+                const float* rows = ring + stage * STAGE + q * kBlk * ROW;
+                const float* pr = ring + stage * STAGE + TB * ROW + q * 2 * kPairs;
+                float d[kBlk * C];
+#pragma unroll
+                for (int j = 0; j < kBlk; j++) {
+                    float kt[E];
+                    lane_row<E>(rows + j * ROW, lane, kt);
+#pragma unroll
+                    for (int c = 0; c < C; c++) {
+                        float x = kt[0] * S[c][0];
+#pragma unroll
+                        for (int e = 1; e < E; e++) x = fmaf(kt[e], S[c][e], x);
+                        d[j * C + c] = x;
+                    }
+                }
+                const float mine = reduce_columns<kBlk * C>(d, lane);          // lanes 2i, 2i + 1 hold value i
+                float dot[kBlk][C], v[kBlk][C];
+#pragma unroll
+                for (int j = 0; j < kBlk; j++) {
+                    const float4 f = *reinterpret_cast<const float4*>(rows + j * ROW + 5 * P + warp * C);
+                    v[j][0] = f.x; v[j][1] = f.y; v[j][2] = f.z; v[j][3] = f.w;
+#pragma unroll
+                    for (int c = 0; c < C; c++) dot[j][c] = __shfl_sync(0xffffffffu, mine, 2 * (j * C + c));
+                }
+                int pair = 0;
+#pragma unroll
+                for (int j = 1; j < kBlk; j++)
+#pragma unroll
+                    for (int i = 0; i < j; i++, pair++) {
+                        const float A = pr[pair], Bk = pr[kPairs + pair];
+#pragma unroll
+                        for (int c = 0; c < C; c++) dot[j][c] = fmaf(Bk, v[i][c], fmaf(-A, dot[i][c], dot[j][c]));
+                    }
+                float o[kBlk * C];
+#pragma unroll
+                for (int j = 0; j < kBlk; j++) {
+                    if (j < n) {
+                        float k[E], w[E], qv[E], r[E];
+                        const float* row = rows + j * ROW;
+                        lane_row<E>(row + P, lane, k); lane_row<E>(row + 2 * P, lane, w); lane_row<E>(row + 3 * P, lane, qv); lane_row<E>(row + 4 * P, lane, r);
+#pragma unroll
+                        for (int c = 0; c < C; c++) {
+                            float x = 0.0f;
+#pragma unroll
+                            for (int e = 0; e < E; e++) {
+                                S[c][e] = fmaf(w[e], S[c][e], fmaf(k[e], v[j][c], -(qv[e] * dot[j][c])));
+                                x = fmaf(r[e], S[c][e], x);
+                            }
+                            o[j * C + c] = x;
+                        }
+                    } else {
+#pragma unroll
+                        for (int c = 0; c < C; c++) o[j * C + c] = 0.0f;
+                    }
+                }
+                const float os = reduce_columns<kBlk * C>(o, lane);
+                const int j = lane / (2 * C), col = c0 + lane / 2 % C;
+                if ((lane & 1) == 0 && j < n && col < dim) p.out[(row0 + t0 + q * kBlk + j) * p.ldo + hd + col] = os;
             }
         }
     }
@@ -248,27 +361,44 @@ __global__ void __launch_bounds__(128) k_delta_scan(const ScanParams p) {
 
 template <int E, int TB>
 void launch_scan(const ScanParams& p, int B, cudaStream_t s) {
-    constexpr int C = 4, ROW = 4 * 32 * E + 4 * C;
+    constexpr int C = 4, ROW = 5 * 32 * E + 4 * C, STAGE = TB * ROW + TB / kBlk * 2 * kPairs;
     const dim3 grid((unsigned)((p.in.dim + 4 * C - 1) / (4 * C)), (unsigned)p.in.H, (unsigned)B);
-    if (p.T == 1) launch_k(k_delta_scan<E, C, TB, true>, grid, dim3(128), (size_t)(ROW + p.in.w2p) * 4, s, true, p);
-    else launch_k(k_delta_scan<E, C, TB, false>, grid, dim3(128), (size_t)2 * TB * ROW * 4, s, true, p);
+    if (p.T == 1) {
+        launch_k(k_delta_scan<E, TB, true>, grid, dim3(128), (size_t)(ROW + p.in.w2p) * 4, s, true, p);
+        return;
+    }
+    static bool attr = false;
+    if (!attr) {
+        DJ_CUDA_CHECK(cudaFuncSetAttribute(k_delta_scan<E, TB, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024));
+        attr = true;
+    }
+    // blocks that start while an earlier kernel drains would pile up on the SMs that are free first: when everything fits
+    // with one or two blocks per SM, ask for as much shared memory as keeps it that way
+    size_t smem = (size_t)2 * STAGE * 4;
+    const long blocks = (long)grid.x * grid.y * grid.z;
+    if (blocks <= g_num_sms) smem = std::max(smem, (size_t)112 * 1024);
+    else if (blocks <= 2l * g_num_sms) smem = std::max(smem, (size_t)80 * 1024);
+    launch_k(k_delta_scan<E, TB, false>, grid, dim3(128), smem, s, true, p);
 }
 
 }  // namespace
 
 constexpr int kDeltaMaxDim = 256;
-bool delta_rule_fits(int dim, int rank) { return dim >= 1 && dim <= kDeltaMaxDim && pad8(rank) * kPrepRows * 4 + 64 <= 48 * 1024; }
-size_t delta_rule_ws_floats(int rows, int H, int dim) { return 2 * (size_t)rows * H * dim; }
+bool delta_rule_fits(int dim, int rank) { return dim >= 1 && dim <= kDeltaMaxDim && pad8(rank) * kPrepRows * 4 + 64 <= 44 * 1024; }
+size_t delta_rule_ws_floats(int B, int T, int H, int dim) {
+    return T == 1 ? 0 : 3 * (size_t)B * T * H * dim + (size_t)B * ((T + kBlk - 1) / kBlk) * H * 2 * kPairs;
+}
 
 void launch_delta_rule(const DeltaRuleArgs& a, cudaStream_t s) {
-    const int rows = a.B * a.T;
+    const size_t n = (size_t)a.B * a.T * a.H * a.dim;
     PrepParams q;
     q.proj = a.proj; q.ld = a.ld; q.k_off = a.k_off; q.a_off = a.a_off; q.low_off = a.low_off; q.rank = a.w2.K;
     q.abias = a.abias; q.w2 = a.w2.w; q.w2p = a.w2.Kp; q.w0 = a.w0;
-    q.wOut = a.ws; q.bOut = a.ws + (size_t)rows * a.H * a.dim;
-    q.rows = rows; q.H = a.H; q.dim = a.dim;
+    q.wOut = a.ws; q.bOut = a.ws + n; q.ktOut = a.ws + 2 * n; q.pairs = a.ws + 3 * n;
+    q.T = a.T; q.H = a.H; q.dim = a.dim;
     if (a.T > 1)
-        launch_k(k_delta_prepare, dim3((unsigned)a.H, (unsigned)((rows + kPrepRows - 1) / kPrepRows)), dim3(128), (size_t)kPrepRows * (q.w2p + 1) * 4, s, true, q);
+        launch_k(k_delta_prepare, dim3((unsigned)a.H, (unsigned)((a.T + kPrepRows - 1) / kPrepRows), (unsigned)a.B), dim3(128), (size_t)kPrepRows * (q.w2p + 1) * 4, s,
+                 true, q);
     ScanParams p;
     p.in = q; p.r_off = a.r_off; p.v_off = a.v_off;
     p.state = a.state; p.pos = a.pos; p.out = a.out; p.ldo = a.ldo; p.T = a.T;

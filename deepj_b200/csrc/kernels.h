@@ -184,7 +184,7 @@ struct DeltaRuleArgs {
     float* ws;                                 // delta_rule_ws_floats
 };
 DJ_PART bool delta_rule_fits(int dim, int rank);
-DJ_PART size_t delta_rule_ws_floats(int rows, int H, int dim);
+DJ_PART size_t delta_rule_ws_floats(int B, int T, int H, int dim);
 DJ_PART void launch_delta_rule(const DeltaRuleArgs& a, cudaStream_t s);
 
 // ── latent attention (attn_latent.cu) ──

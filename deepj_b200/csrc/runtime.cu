@@ -585,7 +585,7 @@ void do_op(Ctx& ctx, const int32_t* c) {
             a.state = f32(ctx, c[11], sz(B, HD) * dim, what); a.pos = f32(ctx, c[12], B, what);
             a.out = f32(ctx, c[13], (size_t)c[14] + sz(rows - 1, c[15]) + HD, what) + c[14]; a.ldo = c[15];
             a.B = B; a.T = T; a.H = H; a.dim = dim;
-            a.ws = scratch(delta_rule_ws_floats(rows, H, dim));
+            a.ws = scratch(delta_rule_ws_floats(B, T, H, dim));
             if (go) launch_delta_rule(a, s);
             break;
         }

@@ -134,7 +134,7 @@ def test_block_diagonal_linear(dev, M, H, K, Nb):
 # ───────────── generalized delta rule ─────────────
 
 @pytest.mark.parametrize("B,H,dim,rank,portions", [(1, 2, 64, 16, [1] * 9), (1, 1, 16, 3, [5, 2, 1, 7]), (2, 3, 40, 9, [2, 3, 1, 11]), (1, 2, 96, 32, [40, 1, 2]),
-                                                   (1, 2, 128, 70, [33, 2, 1, 1]), (1, 1, 200, 8, [3, 1, 12])])
+                                                   (1, 2, 128, 70, [33, 2, 1, 1, 3, 4, 64]), (1, 1, 200, 8, [3, 1, 12])])
 def test_delta_rule(dev, B, H, dim, rank, portions):
     """Portions carry the state; the buffer holds garbage before position 0; one decay per channel runs close to each end
     of its range and one key is zero."""
