@@ -66,24 +66,27 @@ __global__ void __launch_bounds__(256, 1) k_latent_mma(const LmParams p) {
     };
     if (tLo < tHi) load_tile(tLo, 0);
     const int half = p.rot / 2;
-    for (int i = tid; i < kLmRows * (LD / 2); i += 256) {        // query rows: latent part, rotated part, zeros
-        const int r = i / (LD / 2), c = (i - r * (LD / 2)) * 2, row = r0 + r;
-        float a = 0.0f, v = 0.0f;
-        if (row < rows && c < p.W) {
-            const int t = row / p.H, h = row - t * p.H;
-            const size_t m = (size_t)b * p.T + t;
-            if (c < p.R) {
-                const float* src = p.qc + m * p.ldqc + (size_t)h * p.R + c;
-                a = src[0]; v = src[1];
-            } else {
-                const int j = (c - p.R) >> 1, at = min(pos0 + t, p.maxSeq - 1);
-                const float* src = p.q + m * p.ldq + (size_t)h * (p.dim + p.rot) + p.dim + (c - p.R);
-                const float co = p.cosT[(size_t)at * half + j], si = p.sinT[(size_t)at * half + j];
-                a = src[0] * co - src[1] * si;
-                v = src[1] * co + src[0] * si;
+#pragma unroll
+    for (int j = 0; j < kLmRows / 8; j++) {                      // query rows, four per warp: latent part, rotated part, zeros
+        const int r = warp + 8 * j, row = r0 + r, t = row / p.H, h = row - t * p.H;
+        const size_t m = (size_t)b * p.T + t;
+        const bool on = row < rows;
+        const float* qc = p.qc + m * p.ldqc + (size_t)h * p.R;
+#pragma unroll 8
+        for (int c = 2 * lane; c < p.R; c += 64)
+            *reinterpret_cast<uint32_t*>(Qs + r * LD + c) = on ? pack_bf16(qc[c], qc[c + 1]) : 0u;
+        const float* qr = p.q + m * p.ldq + (size_t)h * (p.dim + p.rot) + p.dim;
+        const size_t at = (size_t)min(pos0 + t, p.maxSeq - 1) * half;
+        for (int i = lane; i < half; i += 32) {
+            float a = 0.0f, v = 0.0f;
+            if (on) {
+                const float co = p.cosT[at + i], si = p.sinT[at + i], x = qr[2 * i], y = qr[2 * i + 1];
+                a = x * co - y * si;
+                v = y * co + x * si;
             }
+            *reinterpret_cast<uint32_t*>(Qs + r * LD + p.R + 2 * i) = pack_bf16(a, v);
         }
-        *reinterpret_cast<uint32_t*>(Qs + r * LD + c) = pack_bf16(a, v);
+        for (int c = p.W + 2 * lane; c < LD; c += 64) *reinterpret_cast<uint32_t*>(Qs + r * LD + c) = 0u;
     }
     const int mt = warp & 1, ng = warp >> 1;                     // Q·Kᵀ: 16 rows × 16 keys per warp
     const int row0 = r0 + mt * 16 + g, row1 = row0 + 8;
@@ -218,20 +221,29 @@ __global__ void __launch_bounds__(128) k_latent_mma_merge(const float* __restric
     pdl_launch_dependents();
     const int h = blockIdx.x, row = blockIdx.y;
     const float* p = part + ((size_t)row * H + h) * splits * (R + 2);
-    float mx = -INFINITY, l = 0.0f;
-    for (int s = threadIdx.x; s < splits; s += 128) wgt[s] = p[(size_t)s * (R + 2) + R];
+    if (threadIdx.x < 32) {                              // at most 256 splits: eight per lane
+        float m[8], l[8], mx = -INFINITY, sum = 0.0f;
+#pragma unroll
+        for (int j = 0; j < 8; j++) {
+            const int s = threadIdx.x + 32 * j;
+            m[j] = s < splits ? p[(size_t)s * (R + 2) + R] : -INFINITY;
+            l[j] = s < splits ? p[(size_t)s * (R + 2) + R + 1] : 0.0f;
+            mx = fmaxf(mx, m[j]);
+        }
+        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+#pragma unroll
+        for (int j = 0; j < 8; j++) { m[j] = m[j] > -INFINITY ? exp2f(m[j] - mx) : 0.0f; sum = fmaf(l[j], m[j], sum); }
+        for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+#pragma unroll
+        for (int j = 0; j < 8; j++)
+            if (threadIdx.x + 32 * j < splits) wgt[threadIdx.x + 32 * j] = m[j] / sum;
+    }
     __syncthreads();
-    for (int s = 0; s < splits; s++) mx = fmaxf(mx, wgt[s]);
-    __syncthreads();
-    for (int s = threadIdx.x; s < splits; s += 128) wgt[s] = wgt[s] > -INFINITY ? exp2f(wgt[s] - mx) : 0.0f;
-    __syncthreads();
-    for (int s = 0; s < splits; s++) l = fmaf(p[(size_t)s * (R + 2) + R + 1], wgt[s], l);
-    const float inv = 1.0f / l;
     for (int i = threadIdx.x; i < R; i += 128) {
         float v = 0.0f;
-#pragma unroll 8
+#pragma unroll 16
         for (int s = 0; s < splits; s++) v = fmaf(p[(size_t)s * (R + 2) + i], wgt[s], v);
-        out[(size_t)row * ldo + (size_t)h * R + i] = v * inv;
+        out[(size_t)row * ldo + (size_t)h * R + i] = v;
     }
 }
 
@@ -430,7 +442,7 @@ bool latent_mma_fits(const LatentAttnArgs& a) {
 int latent_mma_splits(const LatentAttnArgs& a) {
     const long ctas = (long)a.B * ((a.T * a.H + kLmRows - 1) / kLmRows);
     const int tiles = (a.maxSeq + kLmKeys - 1) / kLmKeys;
-    return (int)std::max(1l, std::min((long)tiles, g_num_sms / ctas));
+    return (int)std::max(1l, std::min((long)std::min(tiles, 256), g_num_sms / ctas));
 }
 void launch_latent_mma(const LatentAttnArgs& a, cudaStream_t s) {
     LmParams p;

@@ -39,8 +39,9 @@ struct GvParams {
     const float* tok; const float* table; int top, vocab, expertRows;
 };
 
-template <int MR>
-__global__ void __launch_bounds__(kGvThreads, 2) k_bf16_gemv(const GvParams p) {
+// MR activation rows; DEPTH K-steps of four weight rows in flight per warp
+template <int MR, int DEPTH>
+__global__ void __launch_bounds__(kGvThreads, MR == 1 && DEPTH == 2 ? 3 : 2) k_bf16_gemv(const GvParams p) {
     extern __shared__ __align__(16) float xs[];          // [MR][row]
     __shared__ RowScratch sc;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -49,7 +50,7 @@ __global__ void __launch_bounds__(kGvThreads, 2) k_bf16_gemv(const GvParams p) {
     int task = blockIdx.x * kGvWarps + warp;
     const __nv_bfloat16* w = p.w;
 
-    uint4 buf[2][kGvRows];
+    uint4 buf[DEPTH][kGvRows];
     auto fetch = [&](uint4 (&d)[kGvRows], int t, int it) {
         const int k = (it * 32 + lane) * 8;
 #pragma unroll
@@ -59,7 +60,15 @@ __global__ void __launch_bounds__(kGvThreads, 2) k_bf16_gemv(const GvParams p) {
             if (n < p.N && k < p.Kp) d[r] = ld_weight(w + (size_t)n * p.Kp + k);
         }
     };
-    if (p.table == nullptr && task < tasks) fetch(buf[0], task, 0);
+    // step i of a warp's walk over its tasks is (task + (i / nIt)·stride, i % nIt)
+    auto begin = [&] {
+#pragma unroll
+        for (int j = 0; j < DEPTH - 1; j++) {
+            const int t = task + j / nIt * stride;
+            if (t < tasks) fetch(buf[j], t, j % nIt);
+        }
+    };
+    if (p.table == nullptr) begin();
     pdl_wait();
     pdl_launch_dependents();
     int xrow = blockIdx.y, orow = blockIdx.y;
@@ -67,7 +76,7 @@ __global__ void __launch_bounds__(kGvThreads, 2) k_bf16_gemv(const GvParams p) {
         xrow = blockIdx.y / p.top;
         const int id = min(max((int)p.tok[xrow], 0), p.vocab - 1);
         w += (size_t)(int)p.table[(size_t)id * p.top + (blockIdx.y - xrow * p.top)] * p.expertRows * p.Kp;
-        if (task < tasks) fetch(buf[0], task, 0);
+        begin();
     }
 #pragma unroll
     for (int m = 0; m < MR; m++) {
@@ -81,12 +90,17 @@ __global__ void __launch_bounds__(kGvThreads, 2) k_bf16_gemv(const GvParams p) {
     }
     __syncthreads();
 
-    for (; task < tasks; task += stride) {
-        float acc[MR][kGvRows];
+    float acc[MR][kGvRows];
+    int it = 0, ahead = (DEPTH - 1) % nIt, aheadTask = task + (DEPTH - 1) / nIt * stride;      // the step being multiplied, the step to request
+    while (task < tasks) {
 #pragma unroll
-        for (int m = 0; m < MR; m++)
+      for (int slot = 0; slot < DEPTH; slot++) {
+        if (it == 0) {
 #pragma unroll
-            for (int r = 0; r < kGvRows; r++) acc[m][r] = 0.0f;
+            for (int m = 0; m < MR; m++)
+#pragma unroll
+                for (int r = 0; r < kGvRows; r++) acc[m][r] = 0.0f;
+        }
         auto multiply = [&](const uint4 (&d)[kGvRows], int it) {
 #pragma unroll
             for (int m = 0; m < MR; m++) {
@@ -103,13 +117,11 @@ __global__ void __launch_bounds__(kGvThreads, 2) k_bf16_gemv(const GvParams p) {
                 }
             }
         };
-        for (int it = 0; it < nIt; it += 2) {
-            if (it + 1 < nIt) fetch(buf[1], task, it + 1);
-            multiply(buf[0], it);
-            if (it + 2 < nIt) fetch(buf[0], task, it + 2);
-            else if (task + stride < tasks) fetch(buf[0], task + stride, 0);
-            if (it + 1 < nIt) multiply(buf[1], it + 1);
-        }
+        if (aheadTask < tasks) fetch(buf[(slot + DEPTH - 1) % DEPTH], aheadTask, ahead);
+        if (++ahead == nIt) { ahead = 0; aheadTask += stride; }
+        multiply(buf[slot], it);
+        if (++it < nIt) continue;
+        it = 0;
         // lane i = r·MR + m ends up with the sum of (weight row r, activation row m)
         float mine = 0.0f;
 #pragma unroll
@@ -132,6 +144,9 @@ __global__ void __launch_bounds__(kGvThreads, 2) k_bf16_gemv(const GvParams p) {
                 p.out[(size_t)om * p.ldo + n] = softcap_f(v, p.softcap);
             }
         }
+        task += stride;
+        if (task >= tasks) break;
+      }
     }
 }
 
@@ -270,14 +285,24 @@ __global__ void __launch_bounds__(256) k_bf16_gemm_f32(const F32GemmParams p) {
     }
 }
 
-// Block-diagonal projection: out[m][h·os + n] = W[h·Nb + n] · x[m][h·xs …].  grid (heads, row tiles, groups of MR rows).
-constexpr int kBlkRows = 64;
+// Block-diagonal projection: out[m][h·os + n] = W[h·Nb + n] · x[m][h·xs …].  grid (heads, row tiles, groups of MR rows);
+// few rows take one weight row per lane group and block, its first chunk in flight before the dependency wait.
 template <int MR>
 __global__ void __launch_bounds__(256) k_bf16_block(const float* __restrict__ x, int ldx, int xstr, const __nv_bfloat16* __restrict__ w, int K, int Kp, int Nb,
-                                                    float* __restrict__ out, int ldo, int ostr, int M) {
+                                                    float* __restrict__ out, int ldo, int ostr, int M, int tile) {
     extern __shared__ __align__(16) float xs[];          // [MR][Kp]
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int h = blockIdx.x, m0 = blockIdx.z * MR;
+    const int chunks = Kp / 8;
+    int lpr = 1;
+    while (lpr < 32 && lpr < chunks) lpr <<= 1;          // lanes per weight row
+    const int rpw = 32 / lpr, sub = lane / lpr, l = lane - sub * lpr;
+    const int hi = min(Nb, ((int)blockIdx.y + 1) * tile);
+    uint4 first = make_uint4(0, 0, 0, 0);
+    {
+        const int n = blockIdx.y * tile + warp * rpw + sub;
+        if (n < hi && l < chunks) first = __ldg(reinterpret_cast<const uint4*>(w + ((size_t)h * Nb + n) * Kp + l * 8));
+    }
     pdl_wait();
     pdl_launch_dependents();
     for (int i = threadIdx.x; i < MR * Kp; i += 256) {
@@ -285,12 +310,7 @@ __global__ void __launch_bounds__(256) k_bf16_block(const float* __restrict__ x,
         xs[i] = (k < K && m0 + m < M) ? x[(size_t)(m0 + m) * ldx + (size_t)h * xstr + k] : 0.0f;
     }
     __syncthreads();
-    const int chunks = Kp / 8;
-    int lpr = 1;
-    while (lpr < 32 && lpr < chunks) lpr <<= 1;          // lanes per weight row
-    const int rpw = 32 / lpr, sub = lane / lpr, l = lane - sub * lpr;
-    const int hi = min(Nb, ((int)blockIdx.y + 1) * kBlkRows);
-    for (int base = blockIdx.y * kBlkRows + warp * rpw; base < hi; base += 8 * rpw) {
+    for (int base = blockIdx.y * tile + warp * rpw; base < hi; base += 8 * rpw) {
         const int n = base + sub;
         float acc[MR];
 #pragma unroll
@@ -298,7 +318,7 @@ __global__ void __launch_bounds__(256) k_bf16_block(const float* __restrict__ x,
         if (n < hi) {
             const __nv_bfloat16* wr = w + ((size_t)h * Nb + n) * Kp;
             for (int c = l; c < chunks; c += lpr) {
-                const uint4 d = __ldg(reinterpret_cast<const uint4*>(wr + c * 8));
+                const uint4 d = c == l && base == (int)blockIdx.y * tile + warp * rpw ? first : __ldg(reinterpret_cast<const uint4*>(wr + c * 8));
 #pragma unroll
                 for (int m = 0; m < MR; m++) {
                     const float4 x0 = *reinterpret_cast<const float4*>(xs + m * Kp + c * 8), x1 = *reinterpret_cast<const float4*>(xs + m * Kp + c * 8 + 4);
@@ -331,7 +351,7 @@ void raise_smem(const void* kernel, size_t bytes) {
         DJ_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kGvSmemMax));
 }
 
-template <int MR>
+template <int MR, int DEPTH = MR == 4 ? 2 : 4>
 void launch_gv(GvParams p, int m0, unsigned gy, cudaStream_t s) {
     p.a.x += (size_t)m0 * p.a.ldx;
     if (p.a.gate) p.a.gate += (size_t)m0 * p.a.ldg;
@@ -346,8 +366,8 @@ void launch_gv(GvParams p, int m0, unsigned gy, cudaStream_t s) {
     const int cap = 2 * g_num_sms;
     const int rounds = (tiles + cap - 1) / cap, gx = (tiles + rounds - 1) / rounds;
     const size_t smem = (size_t)MR * ((p.Kp + 255) / 256) * 1024;
-    raise_smem((const void*)k_bf16_gemv<MR>, smem);
-    launch_k(k_bf16_gemv<MR>, dim3((unsigned)gx, gy), dim3(kGvThreads), smem, s, true, p);
+    raise_smem((const void*)k_bf16_gemv<MR, DEPTH>, smem);
+    launch_k(k_bf16_gemv<MR, DEPTH>, dim3((unsigned)gx, gy), dim3(kGvThreads), smem, s, true, p);
 }
 
 }  // namespace
@@ -411,11 +431,14 @@ void launch_bf16_linear(const Bf16LinearArgs& a, cudaStream_t s) {
 void launch_bf16_block_linear(const float* x, int ldx, int xstr, const Bf16View& w, int heads, float* out, int ldo, int ostr, int M, cudaStream_t s) {
     const int Nb = w.N / heads;
     const dim3 block(256);
-    const unsigned tiles = (unsigned)((Nb + kBlkRows - 1) / kBlkRows);
+    int lpr = 1;
+    while (lpr < 32 && lpr < w.Kp / 8) lpr <<= 1;
+    const int tile = M <= 4 ? 8 * (32 / lpr) : 64;
+    const unsigned tiles = (unsigned)((Nb + tile - 1) / tile);
     auto go = [&](auto kernel, int MR) {
         const size_t smem = (size_t)MR * w.Kp * 4;
         raise_smem((const void*)kernel, smem);
-        launch_k(kernel, dim3((unsigned)heads, tiles, (unsigned)((M + MR - 1) / MR)), block, smem, s, true, x, ldx, xstr, w.w, w.K, w.Kp, Nb, out, ldo, ostr, M);
+        launch_k(kernel, dim3((unsigned)heads, tiles, (unsigned)((M + MR - 1) / MR)), block, smem, s, true, x, ldx, xstr, w.w, w.K, w.Kp, Nb, out, ldo, ostr, M, tile);
     };
     if (M == 1) go(k_bf16_block<1>, 1);
     else go(k_bf16_block<4>, 4);
@@ -426,7 +449,7 @@ void launch_bf16_expert_gemv(const Bf16ExpertArgs& e, float* y, cudaStream_t s) 
     p.a = e.x; p.w = e.up.w; p.N = 2 * e.ff; p.Kp = e.up.Kp; p.K1p = pad8(e.x.k);
     p.gluRow = 0; p.limit = e.limit; p.glu = y; p.ldglu = e.ff;
     p.tok = e.tok; p.table = e.table; p.top = e.top; p.vocab = e.vocab; p.expertRows = 2 * e.ff;
-    launch_gv<1>(p, 0, (unsigned)(e.M * e.top), s);
+    launch_gv<1, 2>(p, 0, (unsigned)(e.M * e.top), s);       // shallow: more blocks per SM, the entries are many and small
     const int row = (e.down.Kp + 255) / 256 * 256, tiles = (e.d + kGvRows * kGvWarps - 1) / (kGvRows * kGvWarps);
     const size_t smem = (size_t)e.top * row * 4;
     raise_smem((const void*)k_bf16_expert_down, smem);

@@ -10,11 +10,11 @@
 //   k_delta_prepare   per (token, head): w, b = a ⊙ k / (Σk² + ε) — with b the removal term is b (kᵀS) — and, per block of four
 //                     tokens, what relates them: with P_ij = Π_{i<l<j} w_l, the vectors k̃_j = k_j ⊙ Π_{l<j} w_l and the scalars
 //                     A_ij = k_jᵀ(P_ij ⊙ b_i), B_ij = k_jᵀ(P_ij ⊙ k_i)
-//   k_delta_scan      a block of four warps per (sequence, head, 16 value columns), a warp per four of them: a lane holds some
+//   k_delta_scan      a block of eight warps per (sequence, head, 16 value columns), a warp per two of them: a lane holds some
 //                     key channels of its columns in registers.  The four kᵀS of a token block come out of ONE warp reduction
 //                     against the state S_0 before it: k_jᵀS_{j-1} = k̃_jᵀS_0 − Σ_{i<j} A_ij k_iᵀS_{i-1} + Σ_{i<j} B_ij v_i;
-//                     then the four updates run on the registers and the four outputs share a second reduction.  Tokens
-//                     stream through a two-stage cp.async ring.  A single token (decode) computes its own w and b and reads
+//                     then the four updates run on the registers, two channels per instruction, and the outputs share the
+//                     next block's reduction.  Tokens stream through a two-stage cp.async ring.  A single token (decode) computes its own w and b and reads
 //                     the state before the dependency wait.
 #include "row_operand.cuh"
 
@@ -158,61 +158,85 @@ __device__ __forceinline__ float reduce_columns(float (&v)[C], int lane) {
     return v[0];
 }
 
-// E consecutive floats of a lane
-template <int E>
-__device__ __forceinline__ void lane_row(const float* row, int lane, float (&v)[E]) {
-    if constexpr (E % 4 == 0) {
+// two fp32 lanes per instruction
+typedef unsigned long long f2;
+__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) { f2 d; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c)); return d; }
+__device__ __forceinline__ f2 mul2(f2 a, f2 b) { f2 d; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b)); return d; }
+__device__ __forceinline__ f2 pack2(float a, float b) { f2 d; asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(a), "f"(b)); return d; }
+__device__ __forceinline__ float sum2(f2 v) { float a, b; asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); return a + b; }
+
+// The 2·EP channels of a lane.
+template <int EP>
+__device__ __forceinline__ void lane_row(const float* row, int lane, f2 (&v)[EP]) {
+    if constexpr (EP == 1) v[0] = *reinterpret_cast<const f2*>(row + lane * 2);
+    else {
 #pragma unroll
-        for (int j = 0; j < E / 4; j++) {
-            const float4 f = *reinterpret_cast<const float4*>(row + lane * E + 4 * j);
-            v[4 * j] = f.x; v[4 * j + 1] = f.y; v[4 * j + 2] = f.z; v[4 * j + 3] = f.w;
+        for (int j = 0; j < EP; j += 2) {
+            const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(row + lane * 2 * EP + 2 * j);
+            v[j] = f.x; v[j + 1] = f.y;
         }
-    } else if constexpr (E == 2) {
-        const float2 f = *reinterpret_cast<const float2*>(row + lane * 2);
-        v[0] = f.x; v[1] = f.y;
-    } else {
-#pragma unroll
-        for (int e = 0; e < E; e++) v[e] = row[lane * E + e];
     }
 }
+template <int EP>
+__device__ __forceinline__ float dot_row(const f2 (&a)[EP], const f2 (&S)[EP]) {
+    f2 x = mul2(a[0], S[0]);
+#pragma unroll
+    for (int e = 1; e < EP; e++) x = fma2(a[e], S[e], x);
+    return sum2(x);
+}
+// S ← w ⊙ S + k·v − q·dot for one column; returns the lane's part of rᵀS
+template <int EP>
+__device__ __forceinline__ float update_row(f2 (&S)[EP], const f2 (&w)[EP], const f2 (&k)[EP], const f2 (&q)[EP], const f2 (&r)[EP], float v, float dot) {
+    const f2 vv = pack2(v, v), nd = pack2(-dot, -dot);
+    f2 x = 0;
+#pragma unroll
+    for (int e = 0; e < EP; e++) {
+        S[e] = fma2(w[e], S[e], fma2(k[e], vv, mul2(q[e], nd)));
+        x = e == 0 ? mul2(r[e], S[e]) : fma2(r[e], S[e], x);
+    }
+    return sum2(x);
+}
 
-// E key channels per lane (lane·E …), four value columns per warp, TB tokens per stage of the ring.
-template <int E, int TB, bool FUSED>
-__global__ void __launch_bounds__(128) k_delta_scan(const ScanParams p) {
-    constexpr int C = 4, P = 32 * E, ROW = 5 * P + 4 * C;                   // a token: k̃, k, w, b, r of the head, v of the block's columns
+constexpr int kScanCols = 2, kScanWarps = 8, kScanThreads = 32 * kScanWarps, kBlockCols = kScanCols * kScanWarps;
+
+// 2·EP key channels per lane (lane·2EP …), kScanCols value columns per warp, TB tokens per stage of the ring.
+template <int EP, int TB, bool FUSED>
+__global__ void __launch_bounds__(kScanThreads) k_delta_scan(const ScanParams p) {
+    constexpr int C = kScanCols, NT = kScanThreads, P = 64 * EP, ROW = 5 * P + kBlockCols;                  // a token: k̃, k, w, b, r of the head, v of the block's columns
     constexpr int STAGE = TB * ROW + TB / kBlk * 2 * kPairs;                // … and the pairs of its token blocks
     extern __shared__ __align__(16) float ring[];                           // [2][STAGE]; FUSED: one token, then low [w2p]
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int h = blockIdx.y, b = blockIdx.z, dim = p.in.dim, H = p.in.H, HD = H * dim, hd = h * dim;
-    const int cb = blockIdx.x * 4 * C, c0 = cb + warp * C;                  // the block's and this warp's first column
+    const int cb = blockIdx.x * kBlockCols, c0 = cb + warp * C;                  // the block's and this warp's first column
     const size_t row0 = (size_t)b * p.T;
     if (P > dim)                                                            // channels past the head stay zero
         for (int t = 0; t < (FUSED ? 1 : 2 * TB); t++)
-            for (int i = tid; i < 5 * (P - dim); i += 128)
+            for (int i = tid; i < 5 * (P - dim); i += NT)
                 ring[(t / TB) * STAGE + (t % TB) * ROW + i / (P - dim) * P + dim + i % (P - dim)] = 0.0f;
     // the state was last written several kernels ago: it may be read before the dependency wait
     const bool fresh = p.pos[b] == 0.0f;
     float* st = p.state + (((size_t)b * H + h) * dim + c0) * dim;
-    float S[C][E];
+    f2 S[C][EP];
 #pragma unroll
     for (int c = 0; c < C; c++)
 #pragma unroll
-        for (int e = 0; e < E; e++) {
-            const int i = lane * E + e;
-            S[c][e] = (!fresh && i < dim && c0 + c < dim) ? st[(size_t)c * dim + i] : 0.0f;
+        for (int e = 0; e < EP; e++) {
+            const int i = (lane * EP + e) * 2;
+            const bool on = !fresh && c0 + c < dim;
+            S[c][e] = pack2(on && i < dim ? st[(size_t)c * dim + i] : 0.0f, on && i + 1 < dim ? st[(size_t)c * dim + i + 1] : 0.0f);
         }
     if constexpr (FUSED) {
         pdl_wait();
         pdl_launch_dependents();
         float* low = ring + ROW;
         const float* x = p.in.proj + row0 * p.in.ld;
-        for (int j = tid; j < p.in.w2p; j += 128) low[j] = j < p.in.rank ? tanhf(x[p.in.low_off + j]) : 0.0f;
+        for (int j = tid; j < p.in.w2p; j += NT) low[j] = j < p.in.rank ? tanhf(x[p.in.low_off + j]) : 0.0f;
         float ss = 0.0f;
         for (int i = lane; i < dim; i += 32) { const float k = x[p.in.k_off + hd + i]; ss = fmaf(k, k, ss); }
         for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
         const float inv = 1.0f / (ss + kUnitEps), rate = expf(-0.5f);
         __syncthreads();
-        for (int i = tid; i < dim; i += 128) {
+        for (int i = tid; i < dim; i += NT) {
             const float kk = x[p.in.k_off + hd + i];
             ring[P + i] = kk;
             ring[4 * P + i] = x[p.r_off + hd + i];
@@ -230,26 +254,18 @@ __global__ void __launch_bounds__(128) k_delta_scan(const ScanParams p) {
             ring[2 * P + i] = expf(-rate * sigmoid_f(acc + p.in.w0[hd + i]));
             ring[3 * P + i] = sigmoid_f(x[p.in.a_off + hd + i] + p.in.abias[hd + i]) * kk * inv;
         }
-        for (int i = tid; i < 4 * C; i += 128) ring[5 * P + i] = cb + i < dim ? x[p.v_off + hd + cb + i] : 0.0f;
+        for (int i = tid; i < kBlockCols; i += NT) ring[5 * P + i] = cb + i < dim ? x[p.v_off + hd + cb + i] : 0.0f;
         __syncthreads();
-        float k[E], w[E], q[E], r[E], d[C], o[C];
-        lane_row<E>(ring + P, lane, k); lane_row<E>(ring + 2 * P, lane, w); lane_row<E>(ring + 3 * P, lane, q); lane_row<E>(ring + 4 * P, lane, r);
+        f2 k[EP], w[EP], q[EP], r[EP];
+        lane_row<EP>(ring + P, lane, k); lane_row<EP>(ring + 2 * P, lane, w); lane_row<EP>(ring + 3 * P, lane, q); lane_row<EP>(ring + 4 * P, lane, r);
+        float d[C], o[C];
 #pragma unroll
-        for (int c = 0; c < C; c++) {
-            d[c] = k[0] * S[c][0];
-#pragma unroll
-            for (int e = 1; e < E; e++) d[c] = fmaf(k[e], S[c][e], d[c]);
-        }
+        for (int c = 0; c < C; c++) d[c] = dot_row<EP>(k, S[c]);
         const float ks = reduce_columns<C>(d, lane);
 #pragma unroll
         for (int c = 0; c < C; c++) {
-            const float dot = __shfl_sync(0xffffffffu, ks, c * (32 / C)), v = ring[5 * P + warp * C + c];
-            o[c] = 0.0f;
-#pragma unroll
-            for (int e = 0; e < E; e++) {
-                S[c][e] = fmaf(w[e], S[c][e], fmaf(k[e], v, -(q[e] * dot)));
-                o[c] = fmaf(r[e], S[c][e], o[c]);
-            }
+            const float dot = __shfl_sync(0xffffffffu, ks, c * (32 / C));
+            o[c] = update_row<EP>(S[c], w, k, q, r, ring[5 * P + warp * C + c], dot);
         }
         const float os = reduce_columns<C>(o, lane);
         const int col = c0 + lane / (32 / C);
@@ -257,11 +273,12 @@ __global__ void __launch_bounds__(128) k_delta_scan(const ScanParams p) {
     } else {
         pdl_wait();
         pdl_launch_dependents();
-        const int nv = min(4 * C, dim - cb), nBlk = token_blocks(p.T);
-        auto load = [&](int t0, int stage) {           // a warp copies tokens warp, warp + 4, … of the stage
+        const int nv = min(kBlockCols, dim - cb), nBlk = token_blocks(p.T);
+        constexpr int BPS = TB / kBlk;                 // token blocks per stage
+        auto load = [&](int t0, int stage) {           // a warp copies tokens warp, warp + 8, … of the stage
             float* dst = ring + stage * STAGE;
             const int n = min(TB, p.T - t0);
-            for (int t = warp; t < n; t += 4) {
+            for (int t = warp; t < n; t += kScanWarps) {
                 const size_t r = row0 + t0 + t;
                 const float* row = p.in.proj + r * p.in.ld + hd;
                 const float* src[5] = {p.in.ktOut + r * HD + hd, row + p.in.k_off, p.in.wOut + r * HD + hd, p.in.bOut + r * HD + hd, row + p.r_off};
@@ -274,102 +291,110 @@ __global__ void __launch_bounds__(128) k_delta_scan(const ScanParams p) {
                 if (p.vec) { if (lane * 4 < nv) cp_async16(d + 5 * P + lane * 4, row + p.v_off + cb + lane * 4); }
                 else if (lane < nv) cp_async4(d + 5 * P + lane, row + p.v_off + cb + lane);
             }
-            for (int i = tid; i < TB / kBlk * 2 * kPairs; i += 128) {
+            for (int i = tid; i < BPS * 2 * kPairs; i += NT) {
                 const int blk = t0 / kBlk + i / (2 * kPairs);
                 if (blk < nBlk) cp_async4(dst + TB * ROW + i, p.in.pairs + (((size_t)b * nBlk + blk) * H + h) * 2 * kPairs + i % (2 * kPairs));
             }
             cp_async_commit();
         };
-        load(0, 0);
-        for (int t0 = 0, stage = 0; t0 < p.T; t0 += TB, stage ^= 1) {
-            cp_async_wait<0>();
-            __syncthreads();                       // this stage has landed, nobody reads the other one any more
-            if (t0 + TB < p.T) load(t0 + TB, stage ^ 1);
-#pragma unroll 1
-            for (int q = 0; q < TB / kBlk; q++) {
-                const int n = min(kBlk, p.T - t0 - q * kBlk);      // tokens of this block
-                if (n <= 0) break;
-                const float* rows = ring + stage * STAGE + q * kBlk * ROW;
-                const float* pr = ring + stage * STAGE + TB * ROW + q * 2 * kPairs;
-                float d[kBlk * C];
+        constexpr int V = kBlk * C;                    // values per block
+        float red[2 * V];                              // [0, V): products of the coming block with S, [V, 2V): outputs of the last one
+        auto products = [&](const float* rows) {
 #pragma unroll
-                for (int j = 0; j < kBlk; j++) {
-                    float kt[E];
-                    lane_row<E>(rows + j * ROW, lane, kt);
+            for (int j = 0; j < kBlk; j++) {
+                f2 kt[EP];
+                lane_row<EP>(rows + j * ROW, lane, kt);
 #pragma unroll
-                    for (int c = 0; c < C; c++) {
-                        float x = kt[0] * S[c][0];
-#pragma unroll
-                        for (int e = 1; e < E; e++) x = fmaf(kt[e], S[c][e], x);
-                        d[j * C + c] = x;
-                    }
-                }
-                const float mine = reduce_columns<kBlk * C>(d, lane);          // lanes 2i, 2i + 1 hold value i
-                float dot[kBlk][C], v[kBlk][C];
-#pragma unroll
-                for (int j = 0; j < kBlk; j++) {
-                    const float4 f = *reinterpret_cast<const float4*>(rows + j * ROW + 5 * P + warp * C);
-                    v[j][0] = f.x; v[j][1] = f.y; v[j][2] = f.z; v[j][3] = f.w;
-#pragma unroll
-                    for (int c = 0; c < C; c++) dot[j][c] = __shfl_sync(0xffffffffu, mine, 2 * (j * C + c));
-                }
-                int pair = 0;
-#pragma unroll
-                for (int j = 1; j < kBlk; j++)
-#pragma unroll
-                    for (int i = 0; i < j; i++, pair++) {
-                        const float A = pr[pair], Bk = pr[kPairs + pair];
-#pragma unroll
-                        for (int c = 0; c < C; c++) dot[j][c] = fmaf(Bk, v[i][c], fmaf(-A, dot[i][c], dot[j][c]));
-                    }
-                float o[kBlk * C];
-#pragma unroll
-                for (int j = 0; j < kBlk; j++) {
-                    if (j < n) {
-                        float k[E], w[E], qv[E], r[E];
-                        const float* row = rows + j * ROW;
-                        lane_row<E>(row + P, lane, k); lane_row<E>(row + 2 * P, lane, w); lane_row<E>(row + 3 * P, lane, qv); lane_row<E>(row + 4 * P, lane, r);
-#pragma unroll
-                        for (int c = 0; c < C; c++) {
-                            float x = 0.0f;
-#pragma unroll
-                            for (int e = 0; e < E; e++) {
-                                S[c][e] = fmaf(w[e], S[c][e], fmaf(k[e], v[j][c], -(qv[e] * dot[j][c])));
-                                x = fmaf(r[e], S[c][e], x);
-                            }
-                            o[j * C + c] = x;
-                        }
-                    } else {
-#pragma unroll
-                        for (int c = 0; c < C; c++) o[j * C + c] = 0.0f;
-                    }
-                }
-                const float os = reduce_columns<kBlk * C>(o, lane);
-                const int j = lane / (2 * C), col = c0 + lane / 2 % C;
-                if ((lane & 1) == 0 && j < n && col < dim) p.out[(row0 + t0 + q * kBlk + j) * p.ldo + hd + col] = os;
+                for (int c = 0; c < C; c++) red[j * C + c] = dot_row<EP>(kt, S[c]);
             }
+        };
+        load(0, 0);
+        cp_async_wait<0>();
+        __syncthreads();
+        if (TB < p.T) load(TB, 1);
+        const float* rows = ring;
+        products(rows);
+#pragma unroll
+        for (int i = V; i < 2 * V; i++) red[i] = 0.0f;
+        constexpr int LPV = 32 / (2 * V);              // lanes per value
+        float mine = reduce_columns<2 * V>(red, lane);
+        const int oi = lane / LPV - V, oj = oi / C, ocol = c0 + oi % C;      // this lane's output, when oi ≥ 0
+        for (int blk = 0; blk < nBlk; blk++) {
+            const int slot = blk % BPS, stage = blk / BPS & 1;
+            const float* pr = ring + stage * STAGE + TB * ROW + slot * 2 * kPairs;
+            const int n = min(kBlk, p.T - blk * kBlk);             // tokens of this block
+            float dot[kBlk][C], v[kBlk][C], pair[2 * kPairs];
+#pragma unroll
+            for (int i = 0; i < kPairs / 2; i++) {                  // pairs: 12 floats, 16-byte aligned
+                const float4 f = *reinterpret_cast<const float4*>(pr + 4 * i);
+                pair[4 * i] = f.x; pair[4 * i + 1] = f.y; pair[4 * i + 2] = f.z; pair[4 * i + 3] = f.w;
+            }
+#pragma unroll
+            for (int j = 0; j < kBlk; j++) {
+                const float2 f = *reinterpret_cast<const float2*>(rows + j * ROW + 5 * P + warp * C);
+                v[j][0] = f.x; v[j][1] = f.y;
+#pragma unroll
+                for (int c = 0; c < C; c++) dot[j][c] = __shfl_sync(0xffffffffu, mine, (j * C + c) * LPV);
+            }
+            int at = 0;
+#pragma unroll
+            for (int j = 1; j < kBlk; j++)
+#pragma unroll
+                for (int i = 0; i < j; i++, at++)
+#pragma unroll
+                    for (int c = 0; c < C; c++) dot[j][c] = fmaf(pair[kPairs + at], v[i][c], fmaf(-pair[at], dot[i][c], dot[j][c]));
+            auto update = [&](int j) {
+                f2 k[EP], w[EP], q[EP], r[EP];
+                const float* row = rows + j * ROW;
+                lane_row<EP>(row + P, lane, k); lane_row<EP>(row + 2 * P, lane, w); lane_row<EP>(row + 3 * P, lane, q); lane_row<EP>(row + 4 * P, lane, r);
+#pragma unroll
+                for (int c = 0; c < C; c++) red[V + j * C + c] = update_row<EP>(S[c], w, k, q, r, v[j][c], dot[j][c]);
+            };
+            if (n == kBlk) {
+#pragma unroll
+                for (int j = 0; j < kBlk; j++) update(j);
+            } else {
+#pragma unroll
+                for (int j = 0; j < kBlk; j++)
+                    if (j < n) update(j);
+            }
+            if (blk + 1 < nBlk) {
+                if (slot == BPS - 1) {
+                    cp_async_wait<0>();
+                    __syncthreads();                   // the next stage has landed, and nobody reads this one any more
+                    const int t2 = (blk + 1) * kBlk + TB;
+                    if (t2 < p.T) load(t2, stage);
+                    rows = ring + (stage ^ 1) * STAGE;
+                } else rows += kBlk * ROW;
+                products(rows);
+            }
+            mine = reduce_columns<2 * V>(red, lane);
+            if (oi >= 0 && lane % LPV == 0 && oj < n && ocol < dim) p.out[(row0 + blk * kBlk + oj) * p.ldo + hd + ocol] = mine;
         }
     }
 #pragma unroll
     for (int c = 0; c < C; c++)
 #pragma unroll
-        for (int e = 0; e < E; e++) {
-            const int i = lane * E + e;
-            if (i < dim && c0 + c < dim) st[(size_t)c * dim + i] = S[c][e];
+        for (int e = 0; e < EP; e++) {
+            const int i = (lane * EP + e) * 2;
+            float a, b2;
+            asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b2) : "l"(S[c][e]));
+            if (i < dim && c0 + c < dim) st[(size_t)c * dim + i] = a;
+            if (i + 1 < dim && c0 + c < dim) st[(size_t)c * dim + i + 1] = b2;
         }
 }
 
-template <int E, int TB>
+template <int EP, int TB>
 void launch_scan(const ScanParams& p, int B, cudaStream_t s) {
-    constexpr int C = 4, ROW = 5 * 32 * E + 4 * C, STAGE = TB * ROW + TB / kBlk * 2 * kPairs;
-    const dim3 grid((unsigned)((p.in.dim + 4 * C - 1) / (4 * C)), (unsigned)p.in.H, (unsigned)B);
+    constexpr int ROW = 5 * 64 * EP + kBlockCols, STAGE = TB * ROW + TB / kBlk * 2 * kPairs;
+    const dim3 grid((unsigned)((p.in.dim + kBlockCols - 1) / kBlockCols), (unsigned)p.in.H, (unsigned)B);
     if (p.T == 1) {
-        launch_k(k_delta_scan<E, TB, true>, grid, dim3(128), (size_t)(ROW + p.in.w2p) * 4, s, true, p);
+        launch_k(k_delta_scan<EP, TB, true>, grid, dim3(kScanThreads), (size_t)(ROW + p.in.w2p) * 4, s, true, p);
         return;
     }
     static bool attr = false;
     if (!attr) {
-        DJ_CUDA_CHECK(cudaFuncSetAttribute(k_delta_scan<E, TB, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024));
+        DJ_CUDA_CHECK(cudaFuncSetAttribute(k_delta_scan<EP, TB, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024));
         attr = true;
     }
     // blocks that start while an earlier kernel drains would pile up on the SMs that are free first: when everything fits
@@ -378,7 +403,7 @@ void launch_scan(const ScanParams& p, int B, cudaStream_t s) {
     const long blocks = (long)grid.x * grid.y * grid.z;
     if (blocks <= g_num_sms) smem = std::max(smem, (size_t)112 * 1024);
     else if (blocks <= 2l * g_num_sms) smem = std::max(smem, (size_t)80 * 1024);
-    launch_k(k_delta_scan<E, TB, false>, grid, dim3(128), smem, s, true, p);
+    launch_k(k_delta_scan<EP, TB, false>, grid, dim3(kScanThreads), smem, s, true, p);
 }
 
 }  // namespace
@@ -403,11 +428,9 @@ void launch_delta_rule(const DeltaRuleArgs& a, cudaStream_t s) {
     p.in = q; p.r_off = a.r_off; p.v_off = a.v_off;
     p.state = a.state; p.pos = a.pos; p.out = a.out; p.ldo = a.ldo; p.T = a.T;
     p.vec = ((a.dim | a.ld | a.r_off | a.k_off | a.v_off) & 3) == 0 && (((uintptr_t)a.proj | (uintptr_t)a.ws) & 15) == 0;
-    if (a.dim <= 32) launch_scan<1, 8>(p, a.B, s);
-    else if (a.dim <= 64) launch_scan<2, 8>(p, a.B, s);
-    else if (a.dim <= 96) launch_scan<3, 8>(p, a.B, s);
-    else if (a.dim <= 128) launch_scan<4, 8>(p, a.B, s);
-    else launch_scan<8, 4>(p, a.B, s);
+    if (a.dim <= 64) launch_scan<1, 8>(p, a.B, s);
+    else if (a.dim <= 128) launch_scan<2, 8>(p, a.B, s);
+    else launch_scan<4, 8>(p, a.B, s);
 }
 
 }  // namespace dj
