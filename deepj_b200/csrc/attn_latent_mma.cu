@@ -239,7 +239,8 @@ __global__ void __launch_bounds__(128) k_latent_mma_merge(const float* __restric
             if (threadIdx.x + 32 * j < splits) wgt[threadIdx.x + 32 * j] = m[j] / sum;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < R; i += 128) {
+    const int i = blockIdx.z * 128 + threadIdx.x;
+    if (i < R) {
         float v = 0.0f;
 #pragma unroll 16
         for (int s = 0; s < splits; s++) v = fmaf(p[(size_t)s * (R + 2) + i], wgt[s], v);
@@ -453,7 +454,7 @@ void launch_latent_mma(const LatentAttnArgs& a, cudaStream_t s) {
     else if (a.R <= 256) launch_lm<4>(p, a.B, s);
     else launch_lm<8>(p, a.B, s);
     if (p.splits > 1)
-        launch_k(k_latent_mma_merge, dim3((unsigned)a.H, (unsigned)(a.B * a.T)), dim3(128), (size_t)p.splits * 4, s, true, (const float*)p.part, p.splits, a.R, a.H,
+        launch_k(k_latent_mma_merge, dim3((unsigned)a.H, (unsigned)(a.B * a.T), (unsigned)((a.R + 127) / 128)), dim3(128), (size_t)p.splits * 4, s, true, (const float*)p.part, p.splits, a.R, a.H,
                  a.out, a.ldo);
 }
 

@@ -4,8 +4,8 @@
 // their exact values this way.  Activations and accumulation are fp32 everywhere except in the many-row tensor-core
 // form (bf16_gemm_tc.cu), which rounds the staged operand to bf16.
 //
-//   k_bf16_gemv       1-16 rows, passes of up to four: HBM-bound, one warp per four weight rows, the weights of a
-//                     warp's first task in flight before the dependency wait
+//   k_bf16_gemv       1-16 rows, passes of up to four: HBM-bound, a warp takes four (or two) weight
+//                     rows at a time, the first of them in flight before the dependency wait
 //   k_bf16_gemm_f32   many rows, fp32 FMA arithmetic (models run in 32-bit)
 //   k_bf16_block      block-diagonal: head h's outputs read head h's slice of the row
 //   k_stage_rows      the staged operand of the many-row kernels, as fp32 or bf16 rows in the workspace
@@ -17,7 +17,8 @@
 namespace dj {
 namespace {
 
-constexpr int kGvThreads = 256, kGvWarps = kGvThreads / 32, kGvRows = 4;
+constexpr int kGvThreads = 256, kGvWarps = kGvThreads / 32;
+constexpr int kGvRows = 4;                       // weight rows per warp of the expert kernel below
 constexpr int kGvSmemMax = 200 * 1024;
 
 // Column k of a staged row: blocks of 256 columns, in which the first and the second half of every group of eight sit in
@@ -39,23 +40,23 @@ struct GvParams {
     const float* tok; const float* table; int top, vocab, expertRows;
 };
 
-// MR activation rows; DEPTH K-steps of four weight rows in flight per warp
-template <int MR, int DEPTH>
-__global__ void __launch_bounds__(kGvThreads, MR == 1 && DEPTH == 2 ? 3 : 2) k_bf16_gemv(const GvParams p) {
+// MR activation rows; a warp takes ROWS weight rows at a time and keeps DEPTH K-steps of them in flight
+template <int MR, int DEPTH, int ROWS>
+__global__ void __launch_bounds__(kGvThreads, MR == 1 && DEPTH * ROWS <= 8 ? 3 : 2) k_bf16_gemv(const GvParams p) {
     extern __shared__ __align__(16) float xs[];          // [MR][row]
     __shared__ RowScratch sc;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int nIt = (p.Kp + 255) / 256, row = nIt * 256;
-    const int tasks = (p.N + kGvRows - 1) / kGvRows, stride = gridDim.x * kGvWarps;
+    const int tasks = (p.N + ROWS - 1) / ROWS, stride = gridDim.x * kGvWarps;
     int task = blockIdx.x * kGvWarps + warp;
     const __nv_bfloat16* w = p.w;
 
-    uint4 buf[DEPTH][kGvRows];
-    auto fetch = [&](uint4 (&d)[kGvRows], int t, int it) {
+    uint4 buf[DEPTH][ROWS];
+    auto fetch = [&](uint4 (&d)[ROWS], int t, int it) {
         const int k = (it * 32 + lane) * 8;
 #pragma unroll
-        for (int r = 0; r < kGvRows; r++) {
-            const int n = t * kGvRows + r;
+        for (int r = 0; r < ROWS; r++) {
+            const int n = t * ROWS + r;
             d[r] = make_uint4(0, 0, 0, 0);
             if (n < p.N && k < p.Kp) d[r] = ld_weight(w + (size_t)n * p.Kp + k);
         }
@@ -78,7 +79,7 @@ __global__ void __launch_bounds__(kGvThreads, MR == 1 && DEPTH == 2 ? 3 : 2) k_b
         w += (size_t)(int)p.table[(size_t)id * p.top + (blockIdx.y - xrow * p.top)] * p.expertRows * p.Kp;
         begin();
     }
-#pragma unroll
+#pragma unroll 1
     for (int m = 0; m < MR; m++) {
         float* xr = xs + m * row;
         stage_segment(p.a, xrow + m, sc, [&](int k) -> float& { return xr[gv_index(k)]; });
@@ -90,7 +91,7 @@ __global__ void __launch_bounds__(kGvThreads, MR == 1 && DEPTH == 2 ? 3 : 2) k_b
     }
     __syncthreads();
 
-    float acc[MR][kGvRows];
+    float acc[MR][ROWS];
     int it = 0, ahead = (DEPTH - 1) % nIt, aheadTask = task + (DEPTH - 1) / nIt * stride;      // the step being multiplied, the step to request
     while (task < tasks) {
 #pragma unroll
@@ -99,15 +100,15 @@ __global__ void __launch_bounds__(kGvThreads, MR == 1 && DEPTH == 2 ? 3 : 2) k_b
 #pragma unroll
             for (int m = 0; m < MR; m++)
 #pragma unroll
-                for (int r = 0; r < kGvRows; r++) acc[m][r] = 0.0f;
+                for (int r = 0; r < ROWS; r++) acc[m][r] = 0.0f;
         }
-        auto multiply = [&](const uint4 (&d)[kGvRows], int it) {
+        auto multiply = [&](const uint4 (&d)[ROWS], int it) {
 #pragma unroll
             for (int m = 0; m < MR; m++) {
                 const float* xb = xs + m * row + it * 256 + lane * 4;
                 const float4 x0 = *reinterpret_cast<const float4*>(xb), x1 = *reinterpret_cast<const float4*>(xb + 128);
 #pragma unroll
-                for (int r = 0; r < kGvRows; r++) {
+                for (int r = 0; r < ROWS; r++) {
                     float s = acc[m][r];
                     s = fmaf(bf_lo(d[r].x), x0.x, s); s = fmaf(bf_hi(d[r].x), x0.y, s);
                     s = fmaf(bf_lo(d[r].y), x0.z, s); s = fmaf(bf_hi(d[r].y), x0.w, s);
@@ -125,7 +126,7 @@ __global__ void __launch_bounds__(kGvThreads, MR == 1 && DEPTH == 2 ? 3 : 2) k_b
         // lane i = r·MR + m ends up with the sum of (weight row r, activation row m)
         float mine = 0.0f;
 #pragma unroll
-        for (int r = 0; r < kGvRows; r++)
+        for (int r = 0; r < ROWS; r++)
 #pragma unroll
             for (int m = 0; m < MR; m++) {
                 float v = acc[m][r];
@@ -133,8 +134,8 @@ __global__ void __launch_bounds__(kGvThreads, MR == 1 && DEPTH == 2 ? 3 : 2) k_b
                 if (lane == r * MR + m) mine = v;
             }
         const float up = __shfl_down_sync(0xffffffffu, mine, MR);
-        const int r = lane / MR, m = lane - r * MR, n = task * kGvRows + r;
-        if (r < kGvRows && n < p.N) {
+        const int r = lane / MR, m = lane - r * MR, n = task * ROWS + r;
+        if (r < ROWS && n < p.N) {
             const int om = orow + m;
             if (n >= p.gluRow) {
                 if (((n - p.gluRow) & 1) == 0) p.glu[(size_t)om * p.ldglu + ((n - p.gluRow) >> 1)] = gated_clamp_f(mine, up, p.limit);
@@ -351,7 +352,7 @@ void raise_smem(const void* kernel, size_t bytes) {
         DJ_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kGvSmemMax));
 }
 
-template <int MR, int DEPTH = MR == 4 ? 2 : 4>
+template <int MR, int DEPTH, int ROWS>
 void launch_gv(GvParams p, int m0, unsigned gy, cudaStream_t s) {
     p.a.x += (size_t)m0 * p.a.ldx;
     if (p.a.gate) p.a.gate += (size_t)m0 * p.a.ldg;
@@ -362,12 +363,12 @@ void launch_gv(GvParams p, int m0, unsigned gy, cudaStream_t s) {
     if (p.residual) p.residual += (size_t)m0 * p.ldr;
     if (p.out) p.out += (size_t)m0 * p.ldo;
     if (p.glu) p.glu += (size_t)m0 * p.ldglu;
-    const int tiles = (p.N + kGvRows * kGvWarps - 1) / (kGvRows * kGvWarps);
+    const int tiles = (p.N + ROWS * kGvWarps - 1) / (ROWS * kGvWarps);
     const int cap = 2 * g_num_sms;
     const int rounds = (tiles + cap - 1) / cap, gx = (tiles + rounds - 1) / rounds;
     const size_t smem = (size_t)MR * ((p.Kp + 255) / 256) * 1024;
-    raise_smem((const void*)k_bf16_gemv<MR, DEPTH>, smem);
-    launch_k(k_bf16_gemv<MR, DEPTH>, dim3((unsigned)gx, gy), dim3(kGvThreads), smem, s, true, p);
+    raise_smem((const void*)k_bf16_gemv<MR, DEPTH, ROWS>, smem);
+    launch_k(k_bf16_gemv<MR, DEPTH, ROWS>, dim3((unsigned)gx, gy), dim3(kGvThreads), smem, s, true, p);
 }
 
 }  // namespace
@@ -415,9 +416,12 @@ void launch_bf16_linear(const Bf16LinearArgs& a, cudaStream_t s) {
             int rows = std::min(4, a.M - m0);
             if (rows == 3) rows = 2;
             while (rows > 1 && rows * perRow > (size_t)kGvSmemMax) rows >>= 1;
-            if (rows == 4) launch_gv<4>(p, m0, 1, s);
-            else if (rows == 2) launch_gv<2>(p, m0, 1, s);
-            else launch_gv<1>(p, m0, 1, s);
+            // fewer blocks than the SMs hold at a time: two weight rows per warp, twice the blocks
+            const bool narrow = (a.w.N + 4 * kGvWarps - 1) / (4 * kGvWarps) <= g_num_sms;
+            if (rows == 4) launch_gv<4, 2, 4>(p, m0, 1, s);
+            else if (rows == 2) { if (narrow) launch_gv<2, 6, 2>(p, m0, 1, s); else launch_gv<2, 4, 4>(p, m0, 1, s); }
+            else if (narrow) launch_gv<1, 8, 2>(p, m0, 1, s);
+            else launch_gv<1, 4, 4>(p, m0, 1, s);
             m0 += rows;
         }
         return;
@@ -449,7 +453,7 @@ void launch_bf16_expert_gemv(const Bf16ExpertArgs& e, float* y, cudaStream_t s) 
     p.a = e.x; p.w = e.up.w; p.N = 2 * e.ff; p.Kp = e.up.Kp; p.K1p = pad8(e.x.k);
     p.gluRow = 0; p.limit = e.limit; p.glu = y; p.ldglu = e.ff;
     p.tok = e.tok; p.table = e.table; p.top = e.top; p.vocab = e.vocab; p.expertRows = 2 * e.ff;
-    launch_gv<1, 2>(p, 0, (unsigned)(e.M * e.top), s);       // shallow: more blocks per SM, the entries are many and small
+    launch_gv<1, 2, 4>(p, 0, (unsigned)(e.M * e.top), s);       // shallow: more blocks per SM, the entries are many and small
     const int row = (e.down.Kp + 255) / 256 * 256, tiles = (e.d + kGvRows * kGvWarps - 1) / (kGvRows * kGvWarps);
     const size_t smem = (size_t)e.top * row * 4;
     raise_smem((const void*)k_bf16_expert_down, smem);

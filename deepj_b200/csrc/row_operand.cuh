@@ -24,28 +24,65 @@ __device__ __forceinline__ float softcap_f(float v, float cap) { return cap > 0.
 constexpr int kMaxNormGroups = 512;
 struct RowScratch { float part[kMaxNormGroups + 32]; float scale[kMaxNormGroups]; };
 
-// Stages one segment of row m with the whole block (blockDim.x a multiple of 32): put(k, v) receives every element
-// k < seg.k after norm and gate; raw(k) / get(k) address the same storage between the passes.  `Store` needs
-// operator()(int k) → float& (fp32 storage).  Ends with every element written, NOT with a barrier.
+// Stages one segment of row m with the whole block (blockDim.x a multiple of 32).  `at(k)` is the fp32 storage of column k;
+// four columns from a multiple of four on are contiguous in it.  Ends with every element written, NOT with a barrier.
+// The loads of a pass are issued in batches of four 16-byte pieces per thread: a block stages a row of thousands of
+// values, and what it waits for is the round trip to L2.
 template <typename Store>
 __device__ __forceinline__ void stage_segment(const RowOperand& seg, int m, RowScratch& sc, Store at) {
     const int tid = threadIdx.x, nt = blockDim.x, lane = tid & 31, warp = tid >> 5, nw = nt >> 5;
     const float* x = seg.x + (size_t)m * seg.ldx;
     const float* gate = seg.gate ? seg.gate + (size_t)m * seg.ldg : nullptr;
+    const int len = seg.groups > 0 ? seg.k / seg.groups : seg.k;
+    const bool vec = (((uintptr_t)x | (uintptr_t)gate | (uintptr_t)seg.gamma) & 15) == 0 && ((seg.k | len) & 3) == 0;
+    auto quad = [&](int k) -> float4& { return *reinterpret_cast<float4*>(&at(k)); };
+    auto ld4 = [](const float* p) { return *reinterpret_cast<const float4*>(p); };
+    auto gated = [](float4 v, float4 g) {
+        return make_float4(v.x * sigmoid_f(g.x), v.y * sigmoid_f(g.y), v.z * sigmoid_f(g.z), v.w * sigmoid_f(g.w));
+    };
     if (seg.groups == 0) {
-        for (int k = tid; k < seg.k; k += nt) {
-            const float v = x[k];
-            at(k) = gate ? v * sigmoid_f(gate[k]) : v;
+        if (vec) {
+            for (int k0 = tid * 4; k0 < seg.k; k0 += nt * 16) {
+                float4 v[4], g[4];
+#pragma unroll
+                for (int u = 0; u < 4; u++) {
+                    const int k = k0 + u * nt * 4;
+                    if (k < seg.k) { v[u] = ld4(x + k); if (gate) g[u] = ld4(gate + k); }
+                }
+#pragma unroll
+                for (int u = 0; u < 4; u++)
+                    if (k0 + u * nt * 4 < seg.k) quad(k0 + u * nt * 4) = gate ? gated(v[u], g[u]) : v[u];
+            }
+        } else {
+            for (int k = tid; k < seg.k; k += nt) {
+                const float v = x[k];
+                at(k) = gate ? v * sigmoid_f(gate[k]) : v;
+            }
         }
         return;
     }
-    const int len = seg.k / seg.groups;
     const int parts = seg.groups >= nw ? 1 : (nw + seg.groups - 1) / seg.groups;      // warps that share a group
     for (int u = warp; u < seg.groups * parts; u += nw) {
         const int g = u / parts, q = u - g * parts;
-        const int lo = g * len + (int)((long long)q * len / parts), hi = g * len + (int)((long long)(q + 1) * len / parts);
         float ss = 0.0f;
-        for (int k = lo + lane; k < hi; k += 32) { const float v = x[k]; at(k) = v; ss = fmaf(v, v, ss); }
+        if (vec) {
+            const int n4 = len / 4, lo = g * len + q * n4 / parts * 4, hi = g * len + (q + 1) * n4 / parts * 4;
+            for (int k0 = lo + lane * 4; k0 < hi; k0 += 512) {
+                float4 v[4];
+#pragma unroll
+                for (int j = 0; j < 4; j++)
+                    if (k0 + j * 128 < hi) v[j] = ld4(x + k0 + j * 128);
+#pragma unroll
+                for (int j = 0; j < 4; j++)
+                    if (k0 + j * 128 < hi) {
+                        quad(k0 + j * 128) = v[j];
+                        ss = fmaf(v[j].x, v[j].x, ss); ss = fmaf(v[j].y, v[j].y, ss); ss = fmaf(v[j].z, v[j].z, ss); ss = fmaf(v[j].w, v[j].w, ss);
+                    }
+            }
+        } else {
+            const int lo = g * len + (int)((long long)q * len / parts), hi = g * len + (int)((long long)(q + 1) * len / parts);
+            for (int k = lo + lane; k < hi; k += 32) { const float v = x[k]; at(k) = v; ss = fmaf(v, v, ss); }
+        }
         for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
         if (lane == 0) sc.part[u] = ss;
     }
@@ -56,10 +93,31 @@ __device__ __forceinline__ void stage_segment(const RowOperand& seg, int m, RowS
         sc.scale[g] = 1.0f / sqrtf(ss / (float)len + seg.eps);
     }
     __syncthreads();
-    for (int k = tid; k < seg.k; k += nt) {
-        float v = (at(k) * sc.scale[k / len]) * seg.gamma[k];
-        if (gate) v *= sigmoid_f(gate[k]);
-        at(k) = v;
+    if (vec) {
+        for (int k0 = tid * 4; k0 < seg.k; k0 += nt * 16) {
+            float4 w[4], g[4];
+#pragma unroll
+            for (int u = 0; u < 4; u++) {
+                const int k = k0 + u * nt * 4;
+                if (k < seg.k) { w[u] = ld4(seg.gamma + k); if (gate) g[u] = ld4(gate + k); }
+            }
+#pragma unroll
+            for (int u = 0; u < 4; u++) {
+                const int k = k0 + u * nt * 4;
+                if (k < seg.k) {
+                    const float s = sc.scale[k / len];
+                    float4 v = quad(k);
+                    v = make_float4((v.x * s) * w[u].x, (v.y * s) * w[u].y, (v.z * s) * w[u].z, (v.w * s) * w[u].w);
+                    quad(k) = gate ? gated(v, g[u]) : v;
+                }
+            }
+        }
+    } else {
+        for (int k = tid; k < seg.k; k += nt) {
+            float v = (at(k) * sc.scale[k / len]) * seg.gamma[k];
+            if (gate) v *= sigmoid_f(gate[k]);
+            at(k) = v;
+        }
     }
 }
 
