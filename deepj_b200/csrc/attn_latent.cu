@@ -223,8 +223,9 @@ void launch_latent_append(const LatentAttnArgs& a, cudaStream_t s) {
 }
 
 void launch_latent_attn(const LatentAttnArgs& a, cudaStream_t s) {
-    launch_latent_append(a, s);
-    if (latent_mma_fits(a)) launch_latent_mma(a, s);
+    const bool mma = latent_mma_fits(a);
+    if (!mma || a.T > 1) launch_latent_append(a, s);
+    if (mma) launch_latent_mma(a, s);
     else if (a.bf16) run<__nv_bfloat16>(a, s);
     else run<float>(a, s);
 }

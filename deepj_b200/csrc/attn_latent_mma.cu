@@ -2,7 +2,8 @@
 //
 //   k_latent_mma      few tokens: scores and sums in the latent space.  A block takes 32 (token, head) rows — all heads share
 //                     the cached rows — and walks its part of the keys in tiles of 64, streamed with cp.async into two
-//                     stages.  Eight warps split a tile's keys for Q·Kᵀ and the latent columns for P·V.
+//                     stages.  Eight warps split a tile's keys for Q·Kᵀ and the latent columns for P·V.  A single token
+//                     (decode) appends its own row: no append launch, and the older rows are fetched before the dependency wait.
 //   k_latent_prefill  prompt chunks: keys and values of the whole context are expanded per head by two projections (bf16,
 //                     in the workspace), then 128 query rows per block, 16 per warp, key tiles of 64 in two stages; the
 //                     rotated key part is read from the cache.  Per (query, key) pair this costs dim + rot + vdim products
@@ -28,11 +29,13 @@ struct LmParams {
     int T, H, R, rot; float scale;
     float* part; int splits;
     int Wp;                                        // shared-memory columns per row
+    // T == 1: the kernel appends the new row itself (norm, rotation, cache write); otherwise kv is null
+    const float* kv; int ldkv; const float* gamma; float eps; __nv_bfloat16* append;
 };
 
 constexpr int kLmRows = 32, kLmKeys = 64, kLmP = kLmKeys + 8;
 
-size_t lm_smem(int Wp) { return (size_t)(kLmRows + 2 * kLmKeys) * (Wp + 8) * 2 + (size_t)2 * kLmRows * kLmP * 2 + (4 * kLmRows + kLmRows) * 4; }
+size_t lm_smem(int Wp) { return (size_t)(kLmRows + 2 * kLmKeys + 1) * (Wp + 8) * 2 + (size_t)2 * kLmRows * kLmP * 2 + (4 * kLmRows + kLmRows) * 4; }
 
 // NT: output n-tiles (eight latent columns each) per warp
 template <int NT>
@@ -42,15 +45,17 @@ __global__ void __launch_bounds__(256, 1) k_latent_mma(const LmParams p) {
     __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(lm_raw);        // [32][LD]
     __nv_bfloat16* Ks = Qs + kLmRows * LD;                               // [2][64][LD]
     __nv_bfloat16* Ph = Ks + 2 * kLmKeys * LD;                           // [32][kLmP], then the low halves
-    float* s_max = reinterpret_cast<float*>(Ph + 2 * kLmRows * kLmP);    // [4][32]
+    __nv_bfloat16* s_new = Ph + 2 * kLmRows * kLmP;                      // the appended row
+    float* s_max = reinterpret_cast<float*>(s_new + LD);                 // [4][32]
     float* s_corr = s_max + 4 * kLmRows;                                 // [32]
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
     const int b = blockIdx.z, r0 = blockIdx.y * kLmRows, rows = p.T * p.H;
     const __nv_bfloat16* cache = p.cache + (size_t)b * p.maxSeq * p.W;
     // columns past the cached row stay zero
     for (int i = tid; i < 2 * kLmKeys * (LD - p.W); i += 256) Ks[(i / (LD - p.W)) * LD + p.W + i % (LD - p.W)] = __float2bfloat16_rn(0.0f);
-    pdl_wait();
-    pdl_launch_dependents();
+    // Positions and the cached rows below them were written several kernels ago: a block that appends its own row may read
+    // them before the dependency wait.
+    if (p.kv == nullptr) { pdl_wait(); pdl_launch_dependents(); }
     const int pos0 = max((int)p.pos[b], 0);
     const int lastKey = min(p.maxSeq - 1, pos0 + min(rows - 1, r0 + kLmRows - 1) / p.H);
     const int tiles = lastKey / kLmKeys + 1, per = (tiles + p.splits - 1) / p.splits;
@@ -58,13 +63,43 @@ __global__ void __launch_bounds__(256, 1) k_latent_mma(const LmParams p) {
     const int chunks = p.W / 8;
     auto load_tile = [&](int tile, int stage) {
         __nv_bfloat16* dst = Ks + stage * kLmKeys * LD;
-        for (int i = tid; i < kLmKeys * chunks; i += 256) {
-            const int key = i / chunks, c = i - key * chunks;
-            cp_async16(dst + key * LD + c * 8, cache + (size_t)min(tile * kLmKeys + key, p.maxSeq - 1) * p.W + c * 8);
+#pragma unroll 4
+        for (int key = warp; key < kLmKeys; key += 8) {
+            const __nv_bfloat16* src = cache + (size_t)min(tile * kLmKeys + key, p.maxSeq - 1) * p.W;
+            for (int c = lane; c < chunks; c += 32) cp_async16(dst + key * LD + c * 8, src + c * 8);
         }
         cp_async_commit();
     };
     if (tLo < tHi) load_tile(tLo, 0);
+    int newTile = -1;                                            // the tile that holds the row this block appends
+    if (p.kv != nullptr) {
+        pdl_wait();
+        pdl_launch_dependents();
+        if (pos0 < p.maxSeq && pos0 / kLmKeys >= tLo && pos0 / kLmKeys < tHi) newTile = pos0 / kLmKeys;
+    }
+    if (newTile >= 0) {
+        const float* x = p.kv + (size_t)b * p.ldkv;
+        __nv_bfloat16* dst = blockIdx.y == 0 ? p.append + ((size_t)b * p.maxSeq + pos0) * p.W : nullptr;
+        float ss = 0.0f;
+        for (int i = tid; i < p.R; i += 256) ss = fmaf(x[i], x[i], ss);
+        for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        if (lane == 0) s_max[warp] = ss;
+        __syncthreads();
+        ss = 0.0f;
+        for (int w = 0; w < 8; w++) ss += s_max[w];
+        const float inv = 1.0f / sqrtf(ss / (float)p.R + p.eps);
+        for (int i = tid; i < p.R; i += 256) {
+            const __nv_bfloat16 v = __float2bfloat16_rn((x[i] * inv) * p.gamma[i]);
+            s_new[i] = v;
+            if (dst) dst[i] = v;
+        }
+        for (int i = tid; i < p.rot / 2; i += 256) {
+            const float c = p.cosT[(size_t)pos0 * (p.rot / 2) + i], s = p.sinT[(size_t)pos0 * (p.rot / 2) + i], u = x[p.R + 2 * i], v = x[p.R + 2 * i + 1];
+            const __nv_bfloat16 a = __float2bfloat16_rn(u * c - v * s), e = __float2bfloat16_rn(v * c + u * s);
+            s_new[p.R + 2 * i] = a; s_new[p.R + 2 * i + 1] = e;
+            if (dst) { dst[p.R + 2 * i] = a; dst[p.R + 2 * i + 1] = e; }
+        }
+    }
     const int half = p.rot / 2;
 #pragma unroll
     for (int j = 0; j < kLmRows / 8; j++) {                      // query rows, four per warp: latent part, rotated part, zeros
@@ -109,6 +144,10 @@ __global__ void __launch_bounds__(256, 1) k_latent_mma(const LmParams p) {
         const int st = (tile - tLo) & 1;
         cp_async_wait<0>();
         __syncthreads();                                         // the tile is there; the other stage and P are free
+        if (tile == newTile) {
+            for (int c = tid; c < p.W; c += 256) Ks[(st * kLmKeys + pos0 % kLmKeys) * LD + c] = s_new[c];
+            __syncthreads();
+        }
         if (tile + 1 < tHi) load_tile(tile + 1, st ^ 1);
         float s[2][4] = {};
 #pragma unroll 4
@@ -209,7 +248,9 @@ __global__ void __launch_bounds__(256, 1) k_latent_mma(const LmParams p) {
 #pragma unroll
             for (int j = 0; j < NT; j++) {
                 const int c = warp * NT * 8 + j * 8 + 2 * t4;
-                if (c < p.R) { dst[c] = o[m][j][2 * e] * f; dst[c + 1] = o[m][j][2 * e + 1] * f; }
+                if (c >= p.R) continue;
+                if (p.splits > 1) *reinterpret_cast<float2*>(dst + c) = make_float2(o[m][j][2 * e], o[m][j][2 * e + 1]);      // R + 2 is even
+                else { dst[c] = o[m][j][2 * e] * f; dst[c + 1] = o[m][j][2 * e + 1] * f; }
             }
         }
 }
@@ -450,6 +491,7 @@ void launch_latent_mma(const LatentAttnArgs& a, cudaStream_t s) {
     p.q = a.q; p.ldq = a.ldq; p.dim = a.dim; p.qc = a.qc; p.ldqc = a.ldqc; p.cache = (const __nv_bfloat16*)a.cache; p.maxSeq = a.maxSeq; p.W = a.R + a.rot;
     p.pos = a.pos; p.cosT = a.cosT; p.sinT = a.sinT; p.out = a.out; p.ldo = a.ldo; p.T = a.T; p.H = a.H; p.R = a.R; p.rot = a.rot; p.scale = a.scale;
     p.part = a.ws; p.splits = latent_mma_splits(a); p.Wp = lm_width(a.R, p.W);
+    p.kv = a.T == 1 ? a.kv : nullptr; p.ldkv = a.ldkv; p.gamma = a.gamma; p.eps = a.eps; p.append = (__nv_bfloat16*)a.cache;
     if (a.R <= 128) launch_lm<2>(p, a.B, s);
     else if (a.R <= 256) launch_lm<4>(p, a.B, s);
     else launch_lm<8>(p, a.B, s);

@@ -42,7 +42,7 @@ struct GvParams {
 
 // MR activation rows; a warp takes ROWS weight rows at a time and keeps DEPTH K-steps of them in flight
 template <int MR, int DEPTH, int ROWS>
-__global__ void __launch_bounds__(kGvThreads, MR == 1 && DEPTH * ROWS <= 8 ? 3 : 2) k_bf16_gemv(const GvParams p) {
+__global__ void __launch_bounds__(kGvThreads, MR > 1 ? 1 : DEPTH * ROWS <= 8 ? 3 : 2) k_bf16_gemv(const GvParams p) {
     extern __shared__ __align__(16) float xs[];          // [MR][row]
     __shared__ RowScratch sc;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -306,10 +306,9 @@ __global__ void __launch_bounds__(256) k_bf16_block(const float* __restrict__ x,
     }
     pdl_wait();
     pdl_launch_dependents();
-    for (int i = threadIdx.x; i < MR * Kp; i += 256) {
-        const int m = i / Kp, k = i - m * Kp;
-        xs[i] = (k < K && m0 + m < M) ? x[(size_t)(m0 + m) * ldx + (size_t)h * xstr + k] : 0.0f;
-    }
+#pragma unroll
+    for (int m = 0; m < MR; m++)
+        for (int k = threadIdx.x; k < Kp; k += 256) xs[m * Kp + k] = (k < K && m0 + m < M) ? x[(size_t)(m0 + m) * ldx + (size_t)h * xstr + k] : 0.0f;
     __syncthreads();
     for (int base = blockIdx.y * tile + warp * rpw; base < hi; base += 8 * rpw) {
         const int n = base + sub;
