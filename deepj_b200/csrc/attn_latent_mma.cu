@@ -31,6 +31,7 @@ struct LmParams {
     int Wp;                                        // shared-memory columns per row
     // T == 1: the kernel appends the new row itself (norm, rotation, cache write); otherwise kv is null
     const float* kv; int ldkv; const float* gamma; float eps; __nv_bfloat16* append;
+    int early;                                     // … and may read positions and older rows before the dependency wait
 };
 
 constexpr int kLmRows = 32, kLmKeys = 64, kLmP = kLmKeys + 8;
@@ -53,9 +54,7 @@ __global__ void __launch_bounds__(256, 1) k_latent_mma(const LmParams p) {
     const __nv_bfloat16* cache = p.cache + (size_t)b * p.maxSeq * p.W;
     // columns past the cached row stay zero
     for (int i = tid; i < 2 * kLmKeys * (LD - p.W); i += 256) Ks[(i / (LD - p.W)) * LD + p.W + i % (LD - p.W)] = __float2bfloat16_rn(0.0f);
-    // Positions and the cached rows below them were written several kernels ago: a block that appends its own row may read
-    // them before the dependency wait.
-    if (p.kv == nullptr) { pdl_wait(); pdl_launch_dependents(); }
+    if (p.kv == nullptr || !p.early) { pdl_wait(); pdl_launch_dependents(); }
     const int pos0 = max((int)p.pos[b], 0);
     const int lastKey = min(p.maxSeq - 1, pos0 + min(rows - 1, r0 + kLmRows - 1) / p.H);
     const int tiles = lastKey / kLmKeys + 1, per = (tiles + p.splits - 1) / p.splits;
@@ -492,6 +491,7 @@ void launch_latent_mma(const LatentAttnArgs& a, cudaStream_t s) {
     p.pos = a.pos; p.cosT = a.cosT; p.sinT = a.sinT; p.out = a.out; p.ldo = a.ldo; p.T = a.T; p.H = a.H; p.R = a.R; p.rot = a.rot; p.scale = a.scale;
     p.part = a.ws; p.splits = latent_mma_splits(a); p.Wp = lm_width(a.R, p.W);
     p.kv = a.T == 1 ? a.kv : nullptr; p.ldkv = a.ldkv; p.gamma = a.gamma; p.eps = a.eps; p.append = (__nv_bfloat16*)a.cache;
+    p.early = a.early;
     if (a.R <= 128) launch_lm<2>(p, a.B, s);
     else if (a.R <= 256) launch_lm<4>(p, a.B, s);
     else launch_lm<8>(p, a.B, s);

@@ -138,7 +138,7 @@ struct ScanParams {
     int r_off, v_off;
     float* state; const float* pos;
     float* out; int ldo;
-    int T, vec;                    // vec: every field can be copied in 16-byte pieces
+    int T, vec, early;             // vec: every field can be copied in 16-byte pieces; early: the state may be read before the wait
 };
 
 // Sums C per-lane values over the warp; lane (group g of 32/C lanes) ends up with the sum of column g.  C a power of two.
@@ -213,7 +213,7 @@ __global__ void __launch_bounds__(kScanThreads) k_delta_scan(const ScanParams p)
         for (int t = 0; t < (FUSED ? 1 : 2 * TB); t++)
             for (int i = tid; i < 5 * (P - dim); i += NT)
                 ring[(t / TB) * STAGE + (t % TB) * ROW + i / (P - dim) * P + dim + i % (P - dim)] = 0.0f;
-    // the state was last written several kernels ago: it may be read before the dependency wait
+    if (!p.early) pdl_wait();
     const bool fresh = p.pos[b] == 0.0f;
     float* st = p.state + (((size_t)b * H + h) * dim + c0) * dim;
     f2 S[C][EP];
@@ -427,6 +427,7 @@ void launch_delta_rule(const DeltaRuleArgs& a, cudaStream_t s) {
     ScanParams p;
     p.in = q; p.r_off = a.r_off; p.v_off = a.v_off;
     p.state = a.state; p.pos = a.pos; p.out = a.out; p.ldo = a.ldo; p.T = a.T;
+    p.early = a.early || a.T > 1;             // k_delta_prepare comes before a scan of several tokens
     p.vec = ((a.dim | a.ld | a.r_off | a.k_off | a.v_off) & 3) == 0 && (((uintptr_t)a.proj | (uintptr_t)a.ws) & 15) == 0;
     if (a.dim <= 64) launch_scan<1, 8>(p, a.B, s);
     else if (a.dim <= 128) launch_scan<2, 8>(p, a.B, s);

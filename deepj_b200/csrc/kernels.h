@@ -181,6 +181,7 @@ struct DeltaRuleArgs {
     const float* pos;
     float* out; int ldo;                       // [rows][H·dim]
     int B, T, H, dim;
+    bool early;                                // the state may be read before the dependency wait
     float* ws;                                 // delta_rule_ws_floats
 };
 DJ_PART bool delta_rule_fits(int dim, int rank);
@@ -197,6 +198,7 @@ struct LatentAttnArgs {
     const float* pos; const float* cosT; const float* sinT;      // [maxSeq × rot/2]
     float* out; int ldo;                       // [rows][H·R]
     int B, T, H, dim, rot, R; float scale;
+    bool early;                                // cached rows and positions may be read before the dependency wait
     int vdim; Bf16View uk, uv;                 // prompt chunks over expanded keys and values only: [H·dim][R], [H·vdim][R]
     float* ws;                                 // latent_attn_ws_floats / latent_prefill_ws_floats
 };

@@ -142,6 +142,7 @@ struct Ctx {
     bool execute;
     cudaStream_t s;
     size_t ws_need = 0;
+    int prev_op = 0;                   // op code before this one in the stream
     bool bounded_waits = false;        // the stream holds an op whose kernel waits on a peer (tensor-parallel exchange)
     std::vector<std::pair<int, unsigned long long>>* refs = nullptr;
 };
@@ -249,6 +250,10 @@ void do_op(Ctx& ctx, const int32_t* c) {
     cudaStream_t s = ctx.s;
     const bool go = ctx.execute;
     check_part(op);
+    // An op that keeps a state or a cache may read what earlier steps left in it before the dependency wait only when the
+    // kernel right before it is a projection: that kernel has passed its own wait, so everything older is complete.
+    const bool early = ctx.prev_op == DEEPJ_OP_BF16_LINEAR || ctx.prev_op == DEEPJ_OP_BF16_BLOCK_LINEAR;
+    ctx.prev_op = op;
     auto scratch = [&](size_t floats) {          // room in the shared workspace for this op
         if (floats > ctx.ws_need) ctx.ws_need = floats;
         return R.ws;
@@ -584,7 +589,7 @@ void do_op(Ctx& ctx, const int32_t* c) {
             a.abias = f32(ctx, c[8], HD, what); a.w2 = bf16view(w2); a.w0 = f32(ctx, c[10], HD, what);
             a.state = f32(ctx, c[11], sz(B, HD) * dim, what); a.pos = f32(ctx, c[12], B, what);
             a.out = f32(ctx, c[13], (size_t)c[14] + sz(rows - 1, c[15]) + HD, what) + c[14]; a.ldo = c[15];
-            a.B = B; a.T = T; a.H = H; a.dim = dim;
+            a.B = B; a.T = T; a.H = H; a.dim = dim; a.early = early;
             a.ws = scratch(delta_rule_ws_floats(B, T, H, dim));
             if (go) launch_delta_rule(a, s);
             break;
@@ -608,6 +613,7 @@ void do_op(Ctx& ctx, const int32_t* c) {
             a.pos = f32(ctx, c[13], a.B, what);
             a.cosT = f32(ctx, c[14], sz(lc.maxSeq, a.rot / 2), what); a.sinT = f32(ctx, c[15], sz(lc.maxSeq, a.rot / 2), what);
             a.out = f32(ctx, c[16], (size_t)c[17] + sz(rows - 1, c[18]) + cw, what) + c[17]; a.ldo = c[18];
+            a.early = early;
             a.ws = scratch(latent_attn_ws_floats(a));
             if (go) launch_latent_attn(a, s);
             break;

@@ -473,5 +473,9 @@ class HybridDecoder(StreamDecoder):
         s.extend((OP_ADD_SCALAR_INPLACE, I["pos"], float_bits(float(T)), B))
         return np.asarray(s, dtype=np.int32)
 
+    def _chunk_tokens(self) -> int:
+        top = max([ff.top for _, ff in self.cfg.layers if isinstance(ff, TableExperts)] or [1])
+        return min(super()._chunk_tokens(), max(1, 65535 // (self.B * top)))
+
     def _prefill_sizes(self, M: int) -> Dict[str, int]:
         return dict(self._row_buffers(M), tok=M)
