@@ -64,6 +64,10 @@ CASES = {
 }
 
 
+# decode attention where the cache is long enough to be streamed: the context is taken as given (its rows are zeros)
+LONG = ("context32k", _stack(2048, 16, 128, 16, 128, 64, 128, 1024, 512, 5632, 4, 1), DecoderConfig("deepseek", 32000, 32832, 2048, 16, 4, 5632, 1024, 512), 32768)
+
+
 def split_ops(stream: np.ndarray) -> List[np.ndarray]:
     out, at = [], 0
     while at < stream.size:
@@ -184,6 +188,18 @@ def measure(dec, prompt: int, steps: int, warmup: int, seed: int, pk) -> Dict[st
             "device_error": dec.stats()["device_error"]}
 
 
+def measure_long(dec, context: int, steps: int, pk) -> Dict[str, Any]:
+    dec.reset()
+    dec.set_position(context)
+    dec.set_tokens([1])
+    dec.step_device(3)
+    step_ms = time_stream(dec.lib, dec._build(feed_back=False), max(4, min(steps, 40)))
+    dec.set_position(context)
+    return {"decode": {"context": context, "ms_per_step": round(step_ms, 4), "tokens_per_s": round(1e3 / step_ms, 1),
+                       "ops": by_op(dec, dec._build(feed_back=False), context, np.zeros(1, dtype=np.int64), pk, 20)},
+            "device_error": dec.stats()["device_error"]}
+
+
 def main(case: str = "", steps: int = 64, warmup: int = 8, clocks=None) -> None:
     pk = peaks()
     line: Dict[str, Any] = {"metric": "layers_prefill_and_decode", "peaks": pk, "data": "synthetic", "steps": steps, "warmup": max(3, warmup), "cases": {}}
@@ -207,5 +223,16 @@ def main(case: str = "", steps: int = 64, warmup: int = 8, clocks=None) -> None:
         q.close()
         if sampler:
             res["clocks"] = sampler.stop()
+        line["cases"][name] = res
+    name, rec, near, context = LONG
+    if case in ("", name):
+        dec = HybridDecoder(HybridConfig.parse(rec, near.max_seq_len, lambda _n: 64), dtype="bf16")
+        dec.load_synthetic(5, 0.02)
+        res = {"punilix": measure_long(dec, context, steps, pk)}
+        dec.close()
+        q = Q8Decoder(near, id_base=2 << 24)
+        q.load_synthetic(5, 0.02)
+        res[f"{near.kind}_q8"] = measure_long(q, context, steps, pk)
+        q.close()
         line["cases"][name] = res
     print(json.dumps(line), flush=True)
