@@ -36,7 +36,7 @@ OP_TP_ALLREDUCE, OP_TP_ALLGATHER = 71, 72
 OP_ATTN_PREFILL, OP_SAMPLE_TOPK, OP_Q8_LINEAR_LN, OP_DECODE_STEP = 73, 74, 75, 76
 # ops over bf16 weights
 OP_BF16_LINEAR, OP_BF16_BLOCK_LINEAR, OP_DELTA_RULE, OP_ATTN_LATENT, OP_TABLE_EXPERTS = 77, 78, 79, 80, 81
-OP_ATTN_LATENT_CHUNK = 82
+OP_ATTN_LATENT_CHUNK, OP_BF16_LINEAR_SUM, OP_NORM_ADD, OP_ATTN_GROUPED, OP_MLSTM = 82, 83, 84, 85, 86
 
 # op → (stride, offsets of the slots that hold buffer ids); ComputeGraph.java:89-147
 OP_METADATA: Dict[int, tuple] = {}
@@ -78,6 +78,10 @@ OP_METADATA[OP_DELTA_RULE] = (20, (1, 8, 9, 10, 11, 12, 13))
 OP_METADATA[OP_ATTN_LATENT] = (26, (1, 4, 7, 10, 12, 13, 14, 15, 16))
 OP_METADATA[OP_TABLE_EXPERTS] = (25, (1, 4, 7, 8, 12, 13, 16, 19))
 OP_METADATA[OP_ATTN_LATENT_CHUNK] = (26, (1, 4, 7, 9, 10, 11, 12, 13, 14, 15))
+OP_METADATA[OP_BF16_LINEAR_SUM] = (38, (1, 4, 7, 11, 14, 15, 18, 24, 29, 31, 35))
+OP_METADATA[OP_NORM_ADD] = (13, (1, 4, 6, 10))
+OP_METADATA[OP_ATTN_GROUPED] = (27, (1, 6, 7, 9, 10, 12, 13, 14, 15, 16))
+OP_METADATA[OP_MLSTM] = (22, (1, 10, 11, 12, 13))
 
 
 def float_bits(value: float) -> int:

@@ -1,0 +1,516 @@
+// Grouped attention on the tensor cores (bf16 cache); what a score is made of is described in attn_grouped.cu.
+//
+//   k_grouped_decode    one token per sequence.  grid (key splits, blocks of 16 query heads of a group, B·G): the heads of a group
+//                       are the rows of one 16-row operand, so a cached row is read once per group.  Four warps walk tiles
+//                       of 16 keys, each through a private three-stage cp.async ring that starts before the dependency wait; the
+//                       block that holds the newest position norms and appends it.  Queries enter as two bf16 halves.  Warps merge
+//                       in shared memory, blocks through partials that the last one to finish (a ticket) adds up.
+//   k_grouped_prefill   prompt chunks: 128 rows (token, head in the group) per block, 16 per warp, key tiles in two stages.
+// Softmax is fp32 and its weights enter the second product as two bf16 halves (16 bits).
+#include "mma_common.cuh"
+#include "row_operand.cuh"
+
+#include <algorithm>
+
+namespace dj {
+namespace {
+
+constexpr float kLog2e = 1.4426950408889634f;
+constexpr int kGdKeys = 16, kGdStages = 3, kGdWarps = 4, kGdThreads = 32 * kGdWarps;
+constexpr int kGpRows = 128, kGpThreads = 256;
+
+// 16 bytes to shared memory, or zeros
+__device__ __forceinline__ void cp_async16_or_zero(void* dst, const void* src, bool on) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(on ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ float quad_max(float v) {
+    v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 1));
+    return fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 2));
+}
+__device__ __forceinline__ float quad_sum(float v) {
+    v += __shfl_xor_sync(0xffffffffu, v, 1);
+    return v + __shfl_xor_sync(0xffffffffu, v, 2);
+}
+__device__ __forceinline__ float warp_sum(float v) {
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+
+// Bias of query rows (table row `rel`, fp32) at distance d, in the exponent's base-2 units.
+__device__ __forceinline__ float bias_at(const float* rel, int d, int len) { return __ldg(rel + min(d, len - 1)) * kLog2e; }
+
+struct GdShape { int Dp, LDK, LDV, stage; };       // padded head size, row pitches (halves), bytes of a stage
+__host__ __device__ __forceinline__ GdShape gd_shape(int kw, int vw, bool shared, int keys) {
+    GdShape g;
+    g.Dp = kw; g.LDK = kw + 8; g.LDV = shared ? 0 : vw + 8;
+    g.stage = keys * (g.LDK + g.LDV) * 2 + (shared ? keys * 4 : 0);
+    return g;
+}
+size_t gd_smem(const GroupedAttnArgs& a) {
+    const bool shared = a.vcache == nullptr;
+    const GdShape g = gd_shape(a.kw, a.vw, shared, kGdKeys);
+    const size_t ring = (size_t)kGdWarps * kGdStages * g.stage, merge = (size_t)kGdWarps * 16 * ((shared ? a.kw : a.vw) + 2) * 4;
+    return 2 * 16 * g.LDK * 2 + (size_t)(g.LDK + (shared ? 8 : g.LDV)) * 2 + std::max(ring, merge);
+}
+
+// VN: most output n-tiles (eight value columns each)
+template <int VN>
+__global__ void __launch_bounds__(kGdThreads) k_grouped_decode(const GroupedAttnArgs a, int splits) {
+    extern __shared__ __align__(16) unsigned char gd_raw[];
+    __shared__ float s_newScale;
+    __shared__ int s_last;
+    const bool shared = a.vcache == nullptr;
+    const GdShape S = gd_shape(a.kw, a.vw, shared, kGdKeys);
+    const int Vp = shared ? a.kw : a.vw, vt = Vp / 8;
+    __nv_bfloat16* Qh = reinterpret_cast<__nv_bfloat16*>(gd_raw);        // [16][LDK], then the low halves
+    __nv_bfloat16* newK = Qh + 2 * 16 * S.LDK;
+    __nv_bfloat16* newV = newK + S.LDK;
+    unsigned char* ring = reinterpret_cast<unsigned char*>(newV + (shared ? 8 : S.LDV));
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, rl = lane >> 2, t4 = lane & 3;
+    unsigned char* mine = ring + warp * kGdStages * S.stage;
+    const int rep = a.H / a.G, b = blockIdx.z / a.G, g = blockIdx.z - b * a.G, h0 = g * rep + blockIdx.y * 16, nrow = min(16, rep - (int)blockIdx.y * 16);
+    if (!a.early) { pdl_wait(); pdl_launch_dependents(); }
+    const int pos = (int)a.pos[b];
+    const bool valid = pos >= 0 && pos < a.maxSeq;
+    const int tiles = valid ? pos / kGdKeys + 1 : 0, per = max(kGdWarps, (tiles + splits - 1) / splits), active = (tiles + per - 1) / per;
+    const int tLo = blockIdx.x * per, tHi = min(tiles, tLo + per);
+    const __nv_bfloat16* kc = (const __nv_bfloat16*)a.kcache + (size_t)blockIdx.z * a.maxSeq * a.kw;
+    const __nv_bfloat16* vc = (const __nv_bfloat16*)a.vcache + (size_t)blockIdx.z * a.maxSeq * a.vw;
+    const float* ksc = a.kscale + (size_t)blockIdx.z * a.kpitch;
+    auto load = [&](int tile, int stage) {
+        const int k0 = tile * kGdKeys, kq = a.kw / 8, vq = a.vw / 8;
+        __nv_bfloat16* K = reinterpret_cast<__nv_bfloat16*>(mine + stage * S.stage);
+        for (int i = lane; i < kGdKeys * kq; i += 32) {
+            const int j = i / kq, c = i - j * kq;
+            cp_async16_or_zero(K + j * S.LDK + c * 8, kc + (size_t)min(k0 + j, pos) * a.kw + c * 8, k0 + j <= pos);
+        }
+        if (!shared) {
+            __nv_bfloat16* V = K + kGdKeys * S.LDK;
+            for (int i = lane; i < kGdKeys * vq; i += 32) {
+                const int j = i / vq, c = i - j * vq;
+                cp_async16_or_zero(V + j * S.LDV + c * 8, vc + (size_t)min(k0 + j, pos) * a.vw + c * 8, k0 + j <= pos);
+            }
+        } else if (lane < kGdKeys / 4) cp_async16_or_zero(K + kGdKeys * S.LDK + lane * 8, ksc + k0 + lane * 4, true);      // kpitch covers whole tiles
+    };
+#pragma unroll
+    for (int i = 0; i < kGdStages - 1; i++) {
+        if (tLo + warp + i * kGdWarps < tHi) load(tLo + warp + i * kGdWarps, i);
+        cp_async_commit();
+    }
+    if (a.early) { pdl_wait(); pdl_launch_dependents(); }
+    if (tLo >= tHi) { cp_async_wait<0>(); return; }
+
+    const float* x = a.proj + (size_t)b * a.ld;
+    const float qf = a.scale * (a.qtab ? a.qtab[pos] : 1.0f) * kLog2e;
+    for (int r = warp; r < 16; r += kGdWarps) {
+        float inv = 0.0f;
+        const float* q = x + a.q_off + (size_t)(h0 + r) * a.dim;
+        if (r < nrow) {
+            float ss = 0.0f;
+            for (int i = lane; i < a.dim; i += 32) ss = fmaf(q[i], q[i], ss);
+            inv = 1.0f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
+        }
+        for (int i = lane; i < a.kw; i += 32) {
+            float v = 0.0f;
+            if (r < nrow && i < a.dim) {
+                v = (q[i] * inv) * a.qgamma[i] * qf;
+                if (shared) v *= a.kgamma[i];
+            }
+            const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+            Qh[r * S.LDK + i] = hi;
+            Qh[(16 + r) * S.LDK + i] = __float2bfloat16_rn(v - __bfloat162float(hi));
+        }
+    }
+    const bool append = a.k_off >= 0 && pos / kGdKeys >= tLo && pos / kGdKeys < tHi;
+    if (append && warp == kGdWarps - 1) {
+        const float* k = x + a.k_off + (size_t)g * a.dim;
+        float ss = 0.0f;
+        for (int i = lane; i < a.dim; i += 32) ss = fmaf(k[i], k[i], ss);
+        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
+        __nv_bfloat16* kd = (__nv_bfloat16*)a.kcache + ((size_t)blockIdx.z * a.maxSeq + pos) * a.kw;
+        for (int i = lane; i < a.kw; i += 32) {
+            const __nv_bfloat16 v = __float2bfloat16_rn(i >= a.dim ? 0.0f : shared ? k[i] : (k[i] * inv) * a.kgamma[i]);
+            newK[i] = v;
+            if (blockIdx.y == 0) kd[i] = v;
+        }
+        if (shared) {
+            if (lane == 0) {
+                s_newScale = inv;
+                if (blockIdx.y == 0) a.kscale[(size_t)blockIdx.z * a.kpitch + pos] = inv;
+            }
+        } else {
+            const float* v = x + a.v_off + (size_t)g * a.vdim;
+            __nv_bfloat16* vd = (__nv_bfloat16*)a.vcache + ((size_t)blockIdx.z * a.maxSeq + pos) * a.vw;
+            for (int i = lane; i < a.vw; i += 32) {
+                const __nv_bfloat16 u = __float2bfloat16_rn(i < a.vdim ? v[i] : 0.0f);
+                newV[i] = u;
+                if (blockIdx.y == 0) vd[i] = u;
+            }
+        }
+    }
+    __syncthreads();
+
+    const uint32_t qAddr = smem_u32(Qh) + (uint32_t)(((lane & 15) * S.LDK + (lane >> 4) * 8) * 2), qlDelta = (uint32_t)(16 * S.LDK * 2);
+    const uint32_t kLane = (uint32_t)((((lane & 7) + ((lane >> 4) << 3)) * S.LDK + ((lane >> 3) & 1) * 8) * 2);
+    const int ldv = shared ? S.LDK : S.LDV;
+    const uint32_t vLane = (uint32_t)((((lane & 7) + (((lane >> 3) & 1) << 3)) * ldv + (lane >> 4) * 8) * 2);
+    const float* rel0 = a.rel ? a.rel + (size_t)(h0 + min(rl, nrow - 1)) * a.relLen : nullptr;
+    const float* rel1 = a.rel ? a.rel + (size_t)(h0 + min(rl + 8, nrow - 1)) * a.relLen : nullptr;
+    const float far0 = a.rel ? bias_at(rel0, a.relLen - 1, a.relLen) : 0.0f, far1 = a.rel ? bias_at(rel1, a.relLen - 1, a.relLen) : 0.0f;
+    float o[VN][4];
+#pragma unroll
+    for (int j = 0; j < VN; j++) { o[j][0] = 0.0f; o[j][1] = 0.0f; o[j][2] = 0.0f; o[j][3] = 0.0f; }
+    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;
+    int stage = 0;
+    for (int tile = tLo + warp; tile < tHi; tile += kGdWarps) {
+        cp_async_wait<kGdStages - 2>();
+        __syncwarp();
+        const int k0 = tile * kGdKeys;
+        __nv_bfloat16* K = reinterpret_cast<__nv_bfloat16*>(mine + stage * S.stage);
+        __nv_bfloat16* V = shared ? K : K + kGdKeys * S.LDK;
+        float* sc = reinterpret_cast<float*>(K + kGdKeys * S.LDK);
+        if (append && tile == pos / kGdKeys) {               // what was fetched predates the append
+            for (int i = lane; i < a.kw; i += 32) K[(pos - k0) * S.LDK + i] = newK[i];
+            if (shared) { if (lane == 0) sc[pos - k0] = s_newScale; }
+            else { for (int i = lane; i < a.vw; i += 32) V[(pos - k0) * S.LDV + i] = newV[i]; }
+            __syncwarp();
+        }
+        {
+            const int next = tile + (kGdStages - 1) * kGdWarps;
+            if (next < tHi) load(next, stage == 0 ? kGdStages - 1 : stage - 1);
+            cp_async_commit();
+        }
+        float s[2][4];
+#pragma unroll
+        for (int j = 0; j < 2; j++) { s[j][0] = 0.0f; s[j][1] = 0.0f; s[j][2] = 0.0f; s[j][3] = 0.0f; }
+        const uint32_t kAddr = smem_u32(K) + kLane;
+        for (int kk = 0; kk < S.Dp / 16; kk++) {
+            uint32_t ah[4], al[4], bk[4];
+            ldm_x4(ah, qAddr + kk * 32);
+            ldm_x4(al, qAddr + qlDelta + kk * 32);
+            ldm_x4(bk, kAddr + kk * 32);
+            mma_bf16(s[0], ah, bk[0], bk[1]); mma_bf16(s[1], ah, bk[2], bk[3]);
+            mma_bf16(s[0], al, bk[0], bk[1]); mma_bf16(s[1], al, bk[2], bk[3]);
+        }
+        const bool far = a.rel == nullptr || pos - (k0 + kGdKeys - 1) >= a.relLen - 1;
+        float mx0 = -INFINITY, mx1 = -INFINITY;
+#pragma unroll
+        for (int j = 0; j < 2; j++)
+#pragma unroll
+            for (int e = 0; e < 2; e++) {
+                const int i = j * 8 + 2 * t4 + e, d = pos - k0 - i;
+                if (shared) { s[j][e] *= sc[i]; s[j][2 + e] *= sc[i]; }
+                if (d < 0) { s[j][e] = -INFINITY; s[j][2 + e] = -INFINITY; }
+                else {
+                    s[j][e] += far ? far0 : bias_at(rel0, d, a.relLen);
+                    s[j][2 + e] += far ? far1 : bias_at(rel1, d, a.relLen);
+                }
+                mx0 = fmaxf(mx0, s[j][e]); mx1 = fmaxf(mx1, s[j][2 + e]);
+            }
+        mx0 = fmaxf(m0, quad_max(mx0)); mx1 = fmaxf(m1, quad_max(mx1));      // finite: a tile's first key is always seen
+        const float c0 = exp2f(m0 - mx0), c1 = exp2f(m1 - mx1);
+        m0 = mx0; m1 = mx1;
+        float ps0 = 0.0f, ps1 = 0.0f;
+#pragma unroll
+        for (int j = 0; j < 2; j++)
+#pragma unroll
+            for (int e = 0; e < 2; e++) {
+                s[j][e] = exp2f(s[j][e] - m0); s[j][2 + e] = exp2f(s[j][2 + e] - m1);
+                ps0 += s[j][e]; ps1 += s[j][2 + e];
+            }
+        l0 = l0 * c0 + ps0; l1 = l1 * c1 + ps1;
+        uint32_t ph[4], pl[4];
+        split_bf16(s[0][0], s[0][1], ph[0], pl[0]); split_bf16(s[0][2], s[0][3], ph[1], pl[1]);
+        split_bf16(s[1][0], s[1][1], ph[2], pl[2]); split_bf16(s[1][2], s[1][3], ph[3], pl[3]);
+        const uint32_t vAddr = smem_u32(V) + vLane;
+#pragma unroll
+        for (int c = 0; c < VN; c += 2) {
+            if (c >= vt) break;
+            uint32_t bv[4];
+            ldm_x4_t(bv, vAddr + c * 16);
+#pragma unroll
+            for (int q = 0; q < 2; q++) {
+                o[c + q][0] *= c0; o[c + q][1] *= c0; o[c + q][2] *= c1; o[c + q][3] *= c1;
+                mma_bf16(o[c + q], ph, bv[2 * q], bv[2 * q + 1]);
+                mma_bf16(o[c + q], pl, bv[2 * q], bv[2 * q + 1]);
+            }
+        }
+        if (++stage == kGdStages) stage = 0;
+        __syncwarp();
+    }
+    l0 = quad_sum(l0); l1 = quad_sum(l1);
+    cp_async_wait<0>();
+    __syncthreads();                                         // the ring becomes the merge buffer: [warp][16][Vp + 2]
+    float* mg = reinterpret_cast<float*>(ring);
+    const int mrow = Vp + 2;
+    {
+        float* d0 = mg + (warp * 16 + rl) * mrow; float* d1 = d0 + 8 * mrow;
+#pragma unroll
+        for (int c = 0; c < VN; c++)
+            if (c < vt) {
+                d0[c * 8 + 2 * t4] = o[c][0]; d0[c * 8 + 2 * t4 + 1] = o[c][1];
+                d1[c * 8 + 2 * t4] = o[c][2]; d1[c * 8 + 2 * t4 + 1] = o[c][3];
+            }
+        if (t4 == 0) { d0[Vp] = m0; d0[Vp + 1] = l0; d1[Vp] = m1; d1[Vp + 1] = l1; }
+    }
+    __syncthreads();
+    const int pw = a.vdim + 2;
+    float* part = a.ws + ((size_t)blockIdx.z * rep + blockIdx.y * 16) * splits * pw;      // [row][split][pw]
+    for (int r = warp; r < nrow; r += kGdWarps) {
+        float m = active == 1 && a.sink ? 0.0f : -INFINITY;
+#pragma unroll
+        for (int w = 0; w < kGdWarps; w++) m = fmaxf(m, mg[(w * 16 + r) * mrow + Vp]);
+        float f[kGdWarps], l = active == 1 && a.sink ? exp2f(-m) : 0.0f;
+#pragma unroll
+        for (int w = 0; w < kGdWarps; w++) {
+            f[w] = exp2f(mg[(w * 16 + r) * mrow + Vp] - m);
+            l = fmaf(f[w], mg[(w * 16 + r) * mrow + Vp + 1], l);
+        }
+        float* dst = active == 1 ? a.out + (size_t)b * a.ldo + (size_t)(h0 + r) * a.vdim : part + ((size_t)r * splits + blockIdx.x) * pw;
+        const float norm = active == 1 ? 1.0f / l : 1.0f;
+        for (int i = lane; i < a.vdim; i += 32) {
+            float v = 0.0f;
+#pragma unroll
+            for (int w = 0; w < kGdWarps; w++) v = fmaf(f[w], mg[(w * 16 + r) * mrow + i], v);
+            dst[i] = v * norm;
+        }
+        if (active > 1 && lane == 0) { dst[a.vdim] = m; dst[a.vdim + 1] = l; }
+    }
+    if (active == 1) return;
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) {
+        int* ticket = a.tickets + blockIdx.z * gridDim.y + blockIdx.y;
+        s_last = atomicAdd(ticket, 1) == active - 1;
+        if (s_last) *ticket = 0;
+    }
+    __syncthreads();
+    if (!s_last) return;
+    __threadfence();
+    float* wts = mg;                                         // [warp][active]
+    for (int r = warp; r < nrow; r += kGdWarps) {
+        const float* src = part + (size_t)r * splits * pw;
+        float* w = wts + warp * splits;
+        float m = a.sink ? 0.0f : -INFINITY;
+        for (int s = lane; s < active; s += 32) { w[s] = src[s * pw + a.vdim]; m = fmaxf(m, w[s]); }
+        for (int o2 = 16; o2 > 0; o2 >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o2));
+        float l = 0.0f;
+        for (int s = lane; s < active; s += 32) { w[s] = exp2f(w[s] - m); l = fmaf(w[s], src[s * pw + a.vdim + 1], l); }
+        l = warp_sum(l);
+        if (a.sink) l += exp2f(-m);
+        __syncwarp();
+        float* dst = a.out + (size_t)b * a.ldo + (size_t)(h0 + r) * a.vdim;
+        for (int i = lane; i < a.vdim; i += 32) {
+            float v = 0.0f;
+#pragma unroll 8
+            for (int s = 0; s < active; s++) v = fmaf(w[s], src[(size_t)s * pw + i], v);
+            dst[i] = v / l;
+        }
+        __syncwarp();
+    }
+}
+
+size_t gp_smem(const GroupedAttnArgs& a, int keys) {
+    const GdShape g = gd_shape(a.kw, a.vw, a.vcache == nullptr, keys);
+    return (size_t)kGpRows * g.LDK * 2 + 2 * (size_t)g.stage;
+}
+
+// VN: most output n-tiles, KEYS: keys per tile
+template <int VN, int KEYS>
+__global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const GroupedAttnArgs a, const __nv_bfloat16* __restrict__ qp) {
+    extern __shared__ __align__(16) unsigned char gd_raw[];
+    constexpr int NT = KEYS / 8;
+    const bool shared = a.vcache == nullptr;
+    const GdShape S = gd_shape(a.kw, a.vw, shared, KEYS);
+    const int vt = (shared ? a.kw : a.vw) / 8;
+    __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(gd_raw);
+    unsigned char* ring = gd_raw + (size_t)kGpRows * S.LDK * 2;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, rl = lane >> 2, t4 = lane & 3;
+    const int rep = a.H / a.G, rows = a.T * rep, b = blockIdx.y / a.G, g = blockIdx.y - b * a.G;
+    const int r0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * kGpRows;         // the rows with the most keys first
+    pdl_wait();
+    pdl_launch_dependents();
+    const int pos0 = (int)a.pos[b];
+    if (pos0 < 0 || pos0 + a.T > a.maxSeq) return;
+    const int lastKey = pos0 + (min(rows, r0 + kGpRows) - 1) / rep;
+    const __nv_bfloat16* kc = (const __nv_bfloat16*)a.kcache + (size_t)blockIdx.y * a.maxSeq * a.kw;
+    const __nv_bfloat16* vc = (const __nv_bfloat16*)a.vcache + (size_t)blockIdx.y * a.maxSeq * a.vw;
+    const float* ksc = a.kscale + (size_t)blockIdx.y * a.kpitch;
+    const int kq = a.kw / 8, vq = a.vw / 8;
+    auto load = [&](int tile, int stage) {
+        const int k0 = tile * KEYS;
+        __nv_bfloat16* K = reinterpret_cast<__nv_bfloat16*>(ring + stage * S.stage);
+        for (int i = tid; i < KEYS * kq; i += kGpThreads) {
+            const int j = i / kq, c = i - j * kq;
+            cp_async16_or_zero(K + j * S.LDK + c * 8, kc + (size_t)min(k0 + j, lastKey) * a.kw + c * 8, k0 + j <= lastKey);
+        }
+        if (!shared) {
+            __nv_bfloat16* V = K + KEYS * S.LDK;
+            for (int i = tid; i < KEYS * vq; i += kGpThreads) {
+                const int j = i / vq, c = i - j * vq;
+                cp_async16_or_zero(V + j * S.LDV + c * 8, vc + (size_t)min(k0 + j, lastKey) * a.vw + c * 8, k0 + j <= lastKey);
+            }
+        } else if (tid < KEYS / 4) cp_async16_or_zero(K + KEYS * S.LDK + tid * 8, ksc + k0 + tid * 4, true);
+        cp_async_commit();
+    };
+    load(0, 0);
+    const __nv_bfloat16* q0 = qp + ((size_t)blockIdx.y * rows + r0) * a.kw;
+    for (int i = tid; i < kGpRows * kq; i += kGpThreads) {
+        const int r = i / kq, c = i - r * kq;
+        *reinterpret_cast<uint4*>(Qs + r * S.LDK + c * 8) =
+            r0 + r < rows ? *reinterpret_cast<const uint4*>(q0 + (size_t)r * a.kw + c * 8) : make_uint4(0, 0, 0, 0);
+    }
+    const int w0 = r0 + warp * 16, ra = w0 + rl, rb = ra + 8;
+    const int limA = ra < rows ? pos0 + ra / rep : -1, limB = rb < rows ? pos0 + rb / rep : -1;      // newest key of a row
+    const int warpLast = w0 < rows ? pos0 + (min(rows, w0 + 16) - 1) / rep : -1, warpFirst = pos0 + w0 / rep;
+    const float* relA = a.rel ? a.rel + (size_t)(g * rep + ra % rep) * a.relLen : nullptr;
+    const float* relB = a.rel ? a.rel + (size_t)(g * rep + rb % rep) * a.relLen : nullptr;
+    const float farA = a.rel ? bias_at(relA, a.relLen - 1, a.relLen) : 0.0f, farB = a.rel ? bias_at(relB, a.relLen - 1, a.relLen) : 0.0f;
+    const uint32_t qAddr = smem_u32(Qs) + (uint32_t)(((warp * 16 + (lane & 15)) * S.LDK + (lane >> 4) * 8) * 2);
+    const uint32_t kLane = (uint32_t)((((lane & 7) + ((lane >> 4) << 3)) * S.LDK + ((lane >> 3) & 1) * 8) * 2);
+    const int ldv = shared ? S.LDK : S.LDV;
+    const uint32_t vLane = (uint32_t)((((lane & 7) + (((lane >> 3) & 1) << 3)) * ldv + (lane >> 4) * 8) * 2);
+    float o[VN][4];
+#pragma unroll
+    for (int j = 0; j < VN; j++) { o[j][0] = 0.0f; o[j][1] = 0.0f; o[j][2] = 0.0f; o[j][3] = 0.0f; }
+    float mA = -INFINITY, mB = -INFINITY, lA = 0.0f, lB = 0.0f;
+    const int tiles = lastKey / KEYS + 1;
+    for (int tile = 0; tile < tiles; tile++) {
+        cp_async_wait<0>();
+        __syncthreads();                                     // this tile has landed, nobody reads the other stage any more
+        if (tile + 1 < tiles) load(tile + 1, (tile + 1) & 1);
+        const int k0 = tile * KEYS;
+        if (k0 > warpLast) continue;
+        const __nv_bfloat16* K = reinterpret_cast<const __nv_bfloat16*>(ring + (tile & 1) * S.stage);
+        const float* sc = reinterpret_cast<const float*>(K + KEYS * S.LDK);
+        float s[NT][4];
+#pragma unroll
+        for (int j = 0; j < NT; j++) { s[j][0] = 0.0f; s[j][1] = 0.0f; s[j][2] = 0.0f; s[j][3] = 0.0f; }
+        const uint32_t kAddr = smem_u32(K) + kLane;
+        for (int kk = 0; kk < S.Dp / 16; kk++) {
+            uint32_t aq[4];
+            ldm_x4(aq, qAddr + kk * 32);
+#pragma unroll
+            for (int n = 0; n < NT; n += 2) {
+                uint32_t bk[4];
+                ldm_x4(bk, kAddr + (uint32_t)(n * 8 * S.LDK * 2) + kk * 32);
+                mma_bf16(s[n], aq, bk[0], bk[1]); mma_bf16(s[n + 1], aq, bk[2], bk[3]);
+            }
+        }
+        const bool edge = k0 + KEYS - 1 > warpFirst;         // some row of the warp does not see the whole tile
+        const bool far = a.rel == nullptr || warpFirst - (k0 + KEYS - 1) >= a.relLen - 1;
+        float xA = -INFINITY, xB = -INFINITY;
+#pragma unroll
+        for (int j = 0; j < NT; j++)
+#pragma unroll
+            for (int e = 0; e < 2; e++) {
+                const int i = j * 8 + 2 * t4 + e, dA = limA - k0 - i, dB = limB - k0 - i;
+                float vA = s[j][e], vB = s[j][2 + e];
+                if (shared) { vA *= sc[i]; vB *= sc[i]; }
+                vA = fmaf(vA, kLog2e, far ? farA : dA >= 0 ? bias_at(relA, dA, a.relLen) : 0.0f);
+                vB = fmaf(vB, kLog2e, far ? farB : dB >= 0 ? bias_at(relB, dB, a.relLen) : 0.0f);
+                if (edge && dA < 0) vA = -INFINITY;
+                if (edge && dB < 0) vB = -INFINITY;
+                s[j][e] = vA; s[j][2 + e] = vB;
+                xA = fmaxf(xA, vA); xB = fmaxf(xB, vB);
+            }
+        xA = fmaxf(mA, quad_max(xA)); xB = fmaxf(mB, quad_max(xB));
+        const float uA = xA > -INFINITY ? xA : 0.0f, uB = xB > -INFINITY ? xB : 0.0f;      // a row that has seen no key yet
+        const float cA = exp2f(mA - uA), cB = exp2f(mB - uB);
+        mA = xA; mB = xB;
+        float pA = 0.0f, pB = 0.0f;
+#pragma unroll
+        for (int j = 0; j < NT; j++)
+#pragma unroll
+            for (int e = 0; e < 2; e++) {
+                s[j][e] = exp2f(s[j][e] - uA); s[j][2 + e] = exp2f(s[j][2 + e] - uB);
+                pA += s[j][e]; pB += s[j][2 + e];
+            }
+        lA = lA * cA + pA; lB = lB * cB + pB;
+        if (__any_sync(0xffffffffu, cA != 1.0f || cB != 1.0f)) {
+#pragma unroll
+            for (int c = 0; c < VN; c++) { o[c][0] *= cA; o[c][1] *= cA; o[c][2] *= cB; o[c][3] *= cB; }
+        }
+        const uint32_t vAddr = smem_u32(shared ? K : K + KEYS * S.LDK) + vLane;
+#pragma unroll
+        for (int kk = 0; kk < KEYS / 16; kk++) {
+            uint32_t ph[4], pl[4];
+            split_bf16(s[2 * kk][0], s[2 * kk][1], ph[0], pl[0]); split_bf16(s[2 * kk][2], s[2 * kk][3], ph[1], pl[1]);
+            split_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1], ph[2], pl[2]); split_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3], ph[3], pl[3]);
+#pragma unroll
+            for (int c = 0; c < VN; c += 2) {
+                if (c >= vt) break;
+                uint32_t bv[4];
+                ldm_x4_t(bv, vAddr + (uint32_t)(kk * 16 * ldv * 2) + c * 16);
+                mma_bf16(o[c], ph, bv[0], bv[1]); mma_bf16(o[c + 1], ph, bv[2], bv[3]);
+                mma_bf16(o[c], pl, bv[0], bv[1]); mma_bf16(o[c + 1], pl, bv[2], bv[3]);
+            }
+        }
+    }
+    lA = quad_sum(lA); lB = quad_sum(lB);
+    auto finish = [&](int r, float m, float l, int e) {
+        if (r >= rows) return;
+        float f = 1.0f;
+        if (a.sink) {
+            const float u = fmaxf(m, 0.0f);
+            f = exp2f(m - u);
+            l = l * f + exp2f(-u);
+        }
+        f /= l;
+        float* dst = a.out + (size_t)(b * a.T + r / rep) * a.ldo + (size_t)(g * rep + r % rep) * a.vdim;
+#pragma unroll
+        for (int c = 0; c < VN; c++) {
+            const int i = c * 8 + 2 * t4;
+            if (i < a.vdim) dst[i] = o[c][e] * f;
+            if (i + 1 < a.vdim) dst[i + 1] = o[c][e + 1] * f;
+        }
+    };
+    finish(ra, mA, lA, 0);
+    finish(rb, mB, lB, 2);
+}
+
+template <typename K>
+void raise(K kernel, size_t bytes, bool& done) {
+    if (!done) DJ_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - 64));
+    done = true;
+    (void)bytes;
+}
+template <int VN>
+void decode(const GroupedAttnArgs& a, cudaStream_t s) {
+    static bool done = false;
+    raise(k_grouped_decode<VN>, 0, done);
+    const int splits = grouped_mma_splits(a);
+    launch_k(k_grouped_decode<VN>, dim3((unsigned)splits, (unsigned)((a.H / a.G + 15) / 16), (unsigned)(a.B * a.G)), dim3(kGdThreads), gd_smem(a), s, true, a, splits);
+}
+template <int VN, int KEYS>
+void prefill(const GroupedAttnArgs& a, const __nv_bfloat16* q, cudaStream_t s) {
+    static bool done = false;
+    raise(k_grouped_prefill<VN, KEYS>, 0, done);
+    const unsigned blocks = (unsigned)((a.T * (a.H / a.G) + kGpRows - 1) / kGpRows);
+    launch_k(k_grouped_prefill<VN, KEYS>, dim3(blocks, (unsigned)(a.B * a.G)), dim3(kGpThreads), gp_smem(a, KEYS), s, true, a, q);
+}
+
+}  // namespace
+
+bool grouped_mma_fits(const GroupedAttnArgs& a) {
+    return a.bf16 && a.kw <= 256 && a.vw <= 256 && a.kw % 16 == 0 && a.vw % 16 == 0 && (a.vcache != nullptr || a.kpitch % 64 == 0);
+}
+int grouped_mma_splits(const GroupedAttnArgs& a) {
+    const int blocks = a.B * a.G * ((a.H / a.G + 15) / 16), tiles = (a.maxSeq + kGdKeys - 1) / kGdKeys;
+    return std::max(1, std::min({2 * g_num_sms / blocks, (tiles + kGdWarps - 1) / kGdWarps, 512}));
+}
+void launch_grouped_decode(const GroupedAttnArgs& a, cudaStream_t s) {
+    const int vw = a.vcache ? a.vw : a.kw;
+    if (vw <= 64) decode<8>(a, s);
+    else if (vw <= 128) decode<16>(a, s);
+    else decode<32>(a, s);
+}
+void launch_grouped_prefill(const GroupedAttnArgs& a, const __nv_bfloat16* q, int qw, cudaStream_t s) {
+    if (qw != a.kw) throw std::runtime_error("grouped attention: query rows do not match the cache");
+    const int vw = a.vcache ? a.vw : a.kw;
+    if (vw <= 64) prefill<8, 64>(a, q, s);
+    else if (vw <= 128) prefill<16, 64>(a, q, s);
+    else prefill<32, 32>(a, q, s);
+}
+
+}  // namespace dj

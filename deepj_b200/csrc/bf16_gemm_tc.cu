@@ -30,7 +30,7 @@ struct GemmTcParams {
     const float* residual; int ldr;
     float* out; int ldo; __nv_bfloat16* outHalf; // outHalf: bf16 rows instead of fp32
     int gluRow; float limit; float* glu; int ldglu;
-    float softcap;
+    float softcap; const float* bias; int pair;
     int* error;
 };
 
@@ -183,11 +183,12 @@ __global__ void __launch_bounds__(kGThreads, 1) k_bf16_gemm_tc(const __grid_cons
                     continue;
                 }
                 if (nb < p.gluRow) {
+                    const float myBias = p.bias != nullptr && nn < p.gluRow ? p.bias[nn] : 0.0f;
 #pragma unroll 8
                     for (int i = 0; i < 32; i++) {
                         const int row = __shfl_sync(0xffffffffu, myRow, i);
                         if (row >= 0 && nn < p.gluRow) {
-                            float val = stg[i * 33 + lane];
+                            float val = stg[i * 33 + lane] + myBias;
                             if (p.residual) val += p.residual[(size_t)row * p.ldr + nn];
                             p.out[(size_t)row * p.ldo + nn] = softcap_f(val, p.softcap);
                         }
@@ -200,7 +201,7 @@ __global__ void __launch_bounds__(kGThreads, 1) k_bf16_gemm_tc(const __grid_cons
                         const int r = i + (lane >> 4), row = __shfl_sync(0xffffffffu, myRow, r);
                         if (row >= 0 && pair >= p.gluRow && pair < p.N) {
                             const float g = stg[r * 33 + 2 * (lane & 15)], u = stg[r * 33 + 2 * (lane & 15) + 1];
-                            p.glu[(size_t)row * p.ldglu + ((pair - p.gluRow) >> 1)] = gated_clamp_f(g, u, p.limit);
+                            p.glu[(size_t)row * p.ldglu + ((pair - p.gluRow) >> 1)] = pair_f(g, u, p.limit, p.pair);
                         }
                     }
                 }
@@ -265,7 +266,7 @@ bool launch_bf16_gemm_tc(const Bf16LinearArgs& a, const GroupedRows* g, cudaStre
     p.M = a.M; p.N = g ? g->rowsPerExpert : a.w.N; p.nK = (a.w.Kp + kGK - 1) / kGK; p.mTiles = (a.M + kGM - 1) / kGM;
     p.tileExpert = g ? g->tileExpert : nullptr; p.rowMap = g ? g->rowMap : nullptr;
     p.residual = a.residual; p.ldr = a.ldr; p.out = a.out; p.ldo = a.ldo;
-    p.gluRow = a.gluRow; p.limit = a.limit; p.glu = a.glu; p.ldglu = a.ldglu; p.softcap = a.softcap;
+    p.gluRow = a.gluRow; p.limit = a.limit; p.glu = a.glu; p.ldglu = a.ldglu; p.softcap = a.softcap; p.bias = a.bias; p.pair = a.pair;
     p.error = g_dev_error;
     p.lenPos = nullptr; p.lenT = 0; p.outHalf = nullptr;
     if (!g) launch_stage_rows(a.a, a.b, a.w.Kp, a.M, nullptr, 1, a.ws, true, s);

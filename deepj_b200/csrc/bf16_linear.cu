@@ -35,7 +35,7 @@ struct GvParams {
     const float* residual; int ldr;
     float* out; int ldo;
     int gluRow; float limit; float* glu; int ldglu;
-    float softcap;
+    float softcap; const float* bias; int pair;
     // table-routed experts: blockIdx.y is an entry (token row, slot); the weight rows are those of the entry's expert
     const float* tok; const float* table; int top, vocab, expertRows;
 };
@@ -82,7 +82,7 @@ __global__ void __launch_bounds__(kGvThreads, MR > 1 ? 1 : DEPTH * ROWS <= 8 ? 3
 #pragma unroll 1
     for (int m = 0; m < MR; m++) {
         float* xr = xs + m * row;
-        stage_segment(p.a, xrow + m, sc, [&](int k) -> float& { return xr[gv_index(k)]; });
+        stage_segment(p.a, xrow + m, sc, [&](int k) -> float& { return xr[gv_index(k)]; }, blockIdx.x == 0);
         if (p.b.k > 0) stage_segment(p.b, xrow + m, sc, [&](int k) -> float& { return xr[gv_index(p.K1p + k)]; });
         for (int k = p.a.k + (int)threadIdx.x; k < (p.b.k > 0 ? p.K1p : row); k += kGvThreads) xr[gv_index(k)] = 0.0f;
         if (p.b.k > 0)
@@ -138,9 +138,10 @@ __global__ void __launch_bounds__(kGvThreads, MR > 1 ? 1 : DEPTH * ROWS <= 8 ? 3
         if (r < ROWS && n < p.N) {
             const int om = orow + m;
             if (n >= p.gluRow) {
-                if (((n - p.gluRow) & 1) == 0) p.glu[(size_t)om * p.ldglu + ((n - p.gluRow) >> 1)] = gated_clamp_f(mine, up, p.limit);
+                if (((n - p.gluRow) & 1) == 0) p.glu[(size_t)om * p.ldglu + ((n - p.gluRow) >> 1)] = pair_f(mine, up, p.limit, p.pair);
             } else {
                 float v = mine;
+                if (p.bias) v += p.bias[n];
                 if (p.residual) v += p.residual[(size_t)om * p.ldr + n];
                 p.out[(size_t)om * p.ldo + n] = softcap_f(v, p.softcap);
             }
@@ -222,7 +223,7 @@ __global__ void __launch_bounds__(256) k_stage_rows(const RowOperand a, const Ro
         }
         m /= div;
     }
-    stage_segment(a, m, sc, [&](int k) -> float& { return xs[k]; });
+    stage_segment(a, m, sc, [&](int k) -> float& { return xs[k]; }, true);
     if (b.k > 0) {
         __syncthreads();
         stage_segment(b, m, sc, [&](int k) -> float& { return xs[K1p + k]; });
@@ -237,10 +238,22 @@ __global__ void __launch_bounds__(256) k_stage_rows(const RowOperand a, const Ro
     }
 }
 
+// out[m] = base[m] + mult · norm(x[m])·gamma, one row per block; out may be base
+__global__ void __launch_bounds__(256) k_norm_add(const RowOperand x, float* out, int ldo) {
+    extern __shared__ __align__(16) float xs[];
+    __shared__ RowScratch sc;
+    pdl_wait();
+    pdl_launch_dependents();
+    stage_segment(x, blockIdx.x, sc, [&](int k) -> float& { return xs[k]; });
+    __syncthreads();
+    for (int k = threadIdx.x; k < x.k; k += 256) out[(size_t)blockIdx.x * ldo + k] = xs[k];
+}
+
 // out[M × N] = A[M][Kp] (fp32) · W[N][Kp]ᵀ in fp32 FMAs: 64 × 64 tiles, 4 × 4 outputs per thread.
 struct F32GemmParams {
     const float* a; const __nv_bfloat16* w; int M, N, Kp;
     const float* residual; int ldr; float* out; int ldo; int gluRow; float limit; float* glu; int ldglu; float softcap;
+    const float* bias; int pair;
 };
 __global__ void __launch_bounds__(256) k_bf16_gemm_f32(const F32GemmParams p) {
     __shared__ float As[16][68], Ws[16][68];
@@ -276,9 +289,10 @@ __global__ void __launch_bounds__(256) k_bf16_gemm_f32(const F32GemmParams p) {
             const int n = n0 + tn + j;
             if (n >= p.N) continue;
             if (n >= p.gluRow) {                         // gluRow is even and so is tn: a pair never leaves the thread
-                if (((n - p.gluRow) & 1) == 0 && j < 3) p.glu[(size_t)m * p.ldglu + ((n - p.gluRow) >> 1)] = gated_clamp_f(acc[i][j], acc[i][j + 1], p.limit);
+                if (((n - p.gluRow) & 1) == 0 && j < 3) p.glu[(size_t)m * p.ldglu + ((n - p.gluRow) >> 1)] = pair_f(acc[i][j], acc[i][j + 1], p.limit, p.pair);
             } else {
                 float v = acc[i][j];
+                if (p.bias) v += p.bias[n];
                 if (p.residual) v += p.residual[(size_t)m * p.ldr + n];
                 p.out[(size_t)m * p.ldo + n] = softcap_f(v, p.softcap);
             }
@@ -355,6 +369,8 @@ template <int MR, int DEPTH, int ROWS>
 void launch_gv(GvParams p, int m0, unsigned gy, cudaStream_t s) {
     p.a.x += (size_t)m0 * p.a.ldx;
     if (p.a.gate) p.a.gate += (size_t)m0 * p.a.ldg;
+    if (p.a.base) p.a.base += (size_t)m0 * p.a.ldbase;
+    if (p.a.sum) p.a.sum += (size_t)m0 * p.a.ldsum;
     if (p.b.k > 0) {
         p.b.x += (size_t)m0 * p.b.ldx;
         if (p.b.gate) p.b.gate += (size_t)m0 * p.b.ldg;
@@ -390,6 +406,12 @@ void launch_stage_rows(const RowOperand& a, const RowOperand& b, int Kp, int row
     }
 }
 
+void launch_norm_add(const RowOperand& x, float* out, int ldo, int rows, cudaStream_t s) {
+    const size_t smem = (size_t)pad8(x.k) * 4;
+    raise_smem((const void*)k_norm_add, smem);
+    launch_k(k_norm_add, dim3((unsigned)rows), dim3(256), smem, s, true, x, out, ldo);
+}
+
 constexpr int kGvMaxM = 16;      // up to here passes of the GEMV
 
 size_t bf16_linear_ws_floats(const Bf16LinearArgs& a) {
@@ -409,7 +431,7 @@ void launch_bf16_linear(const Bf16LinearArgs& a, cudaStream_t s) {
         GvParams p = {};
         p.a = a.a; p.b = a.b; p.w = a.w.w; p.N = a.w.N; p.Kp = a.w.Kp; p.K1p = pad8(a.a.k);
         p.residual = a.residual; p.ldr = a.ldr; p.out = a.out; p.ldo = a.ldo;
-        p.gluRow = a.gluRow; p.limit = a.limit; p.glu = a.glu; p.ldglu = a.ldglu; p.softcap = a.softcap;
+        p.gluRow = a.gluRow; p.limit = a.limit; p.glu = a.glu; p.ldglu = a.ldglu; p.softcap = a.softcap; p.bias = a.bias; p.pair = a.pair;
         const size_t perRow = (size_t)((a.w.Kp + 255) / 256) * 1024;
         for (int m0 = 0; m0 < a.M;) {
             int rows = std::min(4, a.M - m0);
@@ -427,7 +449,8 @@ void launch_bf16_linear(const Bf16LinearArgs& a, cudaStream_t s) {
     }
     if (!a.exact && launch_bf16_gemm_tc(a, nullptr, s)) return;
     launch_stage_rows(a.a, a.b, a.w.Kp, a.M, nullptr, 1, a.ws, false, s);
-    F32GemmParams p = {a.ws, a.w.w, a.M, a.w.N, a.w.Kp, a.residual, a.ldr, a.out, a.ldo, a.gluRow, a.limit, a.glu, a.ldglu, a.softcap};
+    F32GemmParams p = {a.ws, a.w.w, a.M, a.w.N, a.w.Kp, a.residual, a.ldr, a.out, a.ldo, a.gluRow, a.limit, a.glu, a.ldglu, a.softcap,
+                       a.bias, a.pair};
     launch_k(k_bf16_gemm_f32, dim3((a.w.N + 63) / 64, (a.M + 63) / 64), dim3(256), 0, s, true, p);
 }
 

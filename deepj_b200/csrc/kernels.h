@@ -134,7 +134,13 @@ struct RowOperand {
     const float* x = nullptr; int ldx = 0; int k = 0;                       // k == 0: no segment
     const float* gamma = nullptr; int groups = 0; float eps = 0.0f;         // groups == 0: no norm
     const float* gate = nullptr; int ldg = 0;
+    // base != nullptr: the staged row is base + mult · norm(x), a sublayer's normed output added to the residual stream; the
+    // sum is also written to `sum` (another buffer than base and x)
+    const float* base = nullptr; int ldbase = 0; float mult = 0.0f; float* sum = nullptr; int ldsum = 0;
 };
+// What becomes of a (gate, up) pair of a gated feed-forward.
+constexpr int kPairClamp = 0;     // g·sigmoid(1.702 g)·(u + 1) with g and u clamped
+constexpr int kPairSilu = 1;      // g·sigmoid(g)·u
 struct Bf16LinearArgs {
     RowOperand a, b;                           // b starts at weight column pad8(a.k)
     Bf16View w;
@@ -143,6 +149,8 @@ struct Bf16LinearArgs {
     int gluRow = 0; float limit = 0.0f;        // weight rows [gluRow, N) are (gate, up) pairs → glu, one value per pair
     float* glu = nullptr; int ldglu = 0;
     float softcap = 0.0f;                      // > 0: out = softcap · tanh(out / softcap)
+    const float* bias = nullptr;               // [gluRow], added to the product
+    int pair = kPairClamp;
     int M = 0;
     int exact = 0;                             // 1: fp32 products throughout
     float* ws = nullptr;                       // bf16_linear_ws_floats
@@ -158,6 +166,8 @@ DJ_PART bool launch_bf16_gemm_tc(const Bf16LinearArgs& a, const GroupedRows* g, 
 DJ_PART void launch_bf16_gemm_rows(const __nv_bfloat16* rows, int lda, int K, const float* pos, int T, int maxRows, const Bf16View& w, __nv_bfloat16* out, int ldo,
                            cudaStream_t s);
 DJ_PART void launch_stage_rows(const RowOperand& a, const RowOperand& b, int Kp, int rows, const int* map, int div, void* out, bool bf16, cudaStream_t s);
+// out[m] = base[m] + mult · norm(x[m])·gamma, one group; out may be base
+DJ_PART void launch_norm_add(const RowOperand& x, float* out, int ldo, int rows, cudaStream_t s);
 DJ_PART void launch_bf16_block_linear(const float* x, int ldx, int xstr, const Bf16View& w, int heads, float* out, int ldo, int ostr, int M, cudaStream_t s);
 // Table-routed experts: token id → `top` experts, each of weight 1/top.  up holds every expert's (gate, up) row pairs
 // [experts·2ff][x.k], down [experts·d][ff].
@@ -214,6 +224,43 @@ DJ_PART void launch_latent_mma(const LatentAttnArgs& a, cudaStream_t s);
 DJ_PART bool latent_prefill_fits(const LatentAttnArgs& a);
 DJ_PART size_t latent_prefill_ws_floats(const LatentAttnArgs& a);
 DJ_PART void launch_latent_prefill(const LatentAttnArgs& a, cudaStream_t s);
+
+// ── grouped attention over cached keys and values (attn_grouped.cu, attn_grouped_mma.cu) ──
+struct GroupedAttnArgs {
+    const float* proj; int ld, q_off, k_off, v_off;      // one row per token, heads side by side in every field; k_off < 0: nothing is appended
+    const float* qgamma; const float* kgamma; float eps; // per head, over dim
+    const float* qtab;                         // [maxSeq] factor of the queries by position, or null
+    const float* rel; int relLen;              // [H][relLen] bias by distance (the last entry stands for everything beyond), or null
+    void* kcache; void* vcache;                // [B·G][maxSeq][kw], [B·G][maxSeq][vw]; vcache null: the keys as projected are cached and are the values
+    float* kscale; int kpitch;                 // … and their norms [B·G][kpitch]: 1 / root mean square of each key
+    int kw, vw, bf16, maxSeq;
+    const float* pos; float* out; int ldo;
+    int B, T, H, G, dim, vdim; float scale; int sink;
+    bool early;                                // cached rows and positions may be read before the dependency wait
+    float* ws; int* tickets;
+};
+DJ_PART const char* grouped_attn_check(const GroupedAttnArgs& a);
+DJ_PART size_t grouped_attn_ws_floats(const GroupedAttnArgs& a);
+DJ_PART void launch_grouped_attn(const GroupedAttnArgs& a, cudaStream_t s);
+DJ_PART bool grouped_mma_fits(const GroupedAttnArgs& a);
+DJ_PART int grouped_mma_splits(const GroupedAttnArgs& a);
+DJ_PART void launch_grouped_decode(const GroupedAttnArgs& a, cudaStream_t s);
+DJ_PART void launch_grouped_prefill(const GroupedAttnArgs& a, const __nv_bfloat16* q, int qw, cudaStream_t s);
+
+// ── matrix-memory recurrence with exponential gates (mlstm.cu) ──
+struct MlstmArgs {
+    const float* proj; int ld, q_off, k_off, v_off, i_off, f_off;
+    float cap, qscale;
+    float* state;                              // [B][H][vdim][dim]
+    float* norm;                               // [2][B][H][dim + 1]: normaliser and running maximum, by parity of the position
+    const float* pos; float* out; int ldo;
+    int B, T, H, dim, vdim, exact;
+    bool early;
+    float* ws;
+};
+DJ_PART const char* mlstm_check(const MlstmArgs& a);
+DJ_PART size_t mlstm_ws_floats(const MlstmArgs& a);
+DJ_PART void launch_mlstm(const MlstmArgs& a, cudaStream_t s);
 
 // ── misc ──
 void launch_embed_gather(const float* table, const float* ids, float* out, int rows, int d, int vocab, cudaStream_t s);

@@ -2,7 +2,8 @@
 //
 // A projection reads one or two segments per row; a segment is a slice of an fp32 buffer that may be RMS-normalised in
 // groups (the slice is cut into `groups` equal consecutive parts, each divided by its own sqrt(mean(part²) + eps), the
-// whole multiplied by `gamma`) and multiplied by sigmoid(gate).  Everything here is fp32.  The second segment starts at
+// whole multiplied by `gamma`) and multiplied by sigmoid(gate), or added to a row of the residual stream (`base`).
+// Everything here is fp32.  The second segment starts at
 // the next multiple of eight columns of the weight; the columns between hold zeros on both sides.
 #pragma once
 #include <cuda_bf16.h>
@@ -19,6 +20,7 @@ __device__ __forceinline__ float gated_clamp_f(float g, float u, float limit) {
     u = fminf(fmaxf(u, -limit), limit);
     return (g * sigmoid_f(1.702f * g)) * (u + 1.0f);
 }
+__device__ __forceinline__ float pair_f(float g, float u, float limit, int pair) { return pair == kPairSilu ? (g * sigmoid_f(g)) * u : gated_clamp_f(g, u, limit); }
 __device__ __forceinline__ float softcap_f(float v, float cap) { return cap > 0.0f ? cap * tanhf(v / cap) : v; }
 
 constexpr int kMaxNormGroups = 512;
@@ -27,14 +29,16 @@ struct RowScratch { float part[kMaxNormGroups + 32]; float scale[kMaxNormGroups]
 // Stages one segment of row m with the whole block (blockDim.x a multiple of 32).  `at(k)` is the fp32 storage of column k;
 // four columns from a multiple of four on are contiguous in it.  Ends with every element written, NOT with a barrier.
 // The loads of a pass are issued in batches of four 16-byte pieces per thread: a block stages a row of thousands of
-// values, and what it waits for is the round trip to L2.
+// values, and what it waits for is the round trip to L2.  `keep`: this block writes the sum of a row with a base.
 template <typename Store>
-__device__ __forceinline__ void stage_segment(const RowOperand& seg, int m, RowScratch& sc, Store at) {
+__device__ __forceinline__ void stage_segment(const RowOperand& seg, int m, RowScratch& sc, Store at, bool keep = false) {
     const int tid = threadIdx.x, nt = blockDim.x, lane = tid & 31, warp = tid >> 5, nw = nt >> 5;
     const float* x = seg.x + (size_t)m * seg.ldx;
     const float* gate = seg.gate ? seg.gate + (size_t)m * seg.ldg : nullptr;
+    const float* base = seg.base ? seg.base + (size_t)m * seg.ldbase : nullptr;
+    float* sum = keep && seg.sum ? seg.sum + (size_t)m * seg.ldsum : nullptr;
     const int len = seg.groups > 0 ? seg.k / seg.groups : seg.k;
-    const bool vec = (((uintptr_t)x | (uintptr_t)gate | (uintptr_t)seg.gamma) & 15) == 0 && ((seg.k | len) & 3) == 0;
+    const bool vec = (((uintptr_t)x | (uintptr_t)gate | (uintptr_t)seg.gamma | (uintptr_t)base | (uintptr_t)sum) & 15) == 0 && ((seg.k | len) & 3) == 0;
     auto quad = [&](int k) -> float4& { return *reinterpret_cast<float4*>(&at(k)); };
     auto ld4 = [](const float* p) { return *reinterpret_cast<const float4*>(p); };
     auto gated = [](float4 v, float4 g) {
@@ -99,7 +103,7 @@ __device__ __forceinline__ void stage_segment(const RowOperand& seg, int m, RowS
 #pragma unroll
             for (int u = 0; u < 4; u++) {
                 const int k = k0 + u * nt * 4;
-                if (k < seg.k) { w[u] = ld4(seg.gamma + k); if (gate) g[u] = ld4(gate + k); }
+                if (k < seg.k) { w[u] = ld4(seg.gamma + k); if (gate) g[u] = ld4(gate + k); else if (base) g[u] = ld4(base + k); }
             }
 #pragma unroll
             for (int u = 0; u < 4; u++) {
@@ -108,6 +112,10 @@ __device__ __forceinline__ void stage_segment(const RowOperand& seg, int m, RowS
                     const float s = sc.scale[k / len];
                     float4 v = quad(k);
                     v = make_float4((v.x * s) * w[u].x, (v.y * s) * w[u].y, (v.z * s) * w[u].z, (v.w * s) * w[u].w);
+                    if (base) {
+                        v = make_float4(fmaf(seg.mult, v.x, g[u].x), fmaf(seg.mult, v.y, g[u].y), fmaf(seg.mult, v.z, g[u].z), fmaf(seg.mult, v.w, g[u].w));
+                        if (sum) *reinterpret_cast<float4*>(sum + k) = v;
+                    }
                     quad(k) = gate ? gated(v, g[u]) : v;
                 }
             }
@@ -116,6 +124,10 @@ __device__ __forceinline__ void stage_segment(const RowOperand& seg, int m, RowS
         for (int k = tid; k < seg.k; k += nt) {
             float v = (at(k) * sc.scale[k / len]) * seg.gamma[k];
             if (gate) v *= sigmoid_f(gate[k]);
+            if (base) {
+                v = fmaf(seg.mult, v, base[k]);
+                if (sum) sum[k] = v;
+            }
             at(k) = v;
         }
     }

@@ -9,6 +9,7 @@
 #include "kernels.h"
 #include "q8_tma.cuh"
 
+#include <algorithm>
 #include <cmath>
 #include <cstring>
 #include <memory>
@@ -197,6 +198,17 @@ RowOperand row_operand(Ctx& c, int rows, int k, int id, int off, int ld, int gam
     return o;
 }
 
+// The residual row that a normed sublayer output is added to: t = [base, base_off, ldbase, multBits, sum, sum_off, ldsum].
+void add_base(Ctx& c, RowOperand& o, int rows, const int32_t* t, const char* what) {
+    require(o.groups > 0 && o.gate == nullptr, what, "only a normed row without a gate is added to a base");
+    require(t[1] >= 0 && t[2] >= o.k, what, "base stride smaller than the row");
+    o.base = f32(c, t[0], (size_t)t[1] + (size_t)(rows - 1) * t[2] + o.k, what) + t[1]; o.ldbase = t[2];
+    o.mult = bits_to_float(t[3]);
+    if (t[4] < 0) return;
+    require(t[5] >= 0 && t[6] >= o.k && t[4] != t[0], what, "the sum goes to rows of another buffer than the base's");
+    o.sum = f32(c, t[4], (size_t)t[5] + (size_t)(rows - 1) * t[6] + o.k, what) + t[5]; o.ldsum = t[6];
+}
+
 // Kernel files that a library built for one model family may leave out: their launchers are weak symbols.
 template <typename F> void part(F* launcher, const char* what) {
     if (launcher == nullptr) throw std::runtime_error(std::string(what) + ": this library was built without these kernels (python -m deepj_b200.build builds all)");
@@ -238,6 +250,10 @@ int op_stride(int op) {
         case DEEPJ_OP_ATTN_LATENT: return 26;
         case DEEPJ_OP_TABLE_EXPERTS: return 25;
         case DEEPJ_OP_ATTN_LATENT_CHUNK: return 26;
+        case DEEPJ_OP_BF16_LINEAR_SUM: return 38;
+        case DEEPJ_OP_NORM_ADD: return 13;
+        case DEEPJ_OP_ATTN_GROUPED: return 27;
+        case DEEPJ_OP_MLSTM: return 22;
         default: return -1;
     }
 }
@@ -252,7 +268,7 @@ void do_op(Ctx& ctx, const int32_t* c) {
     check_part(op);
     // An op that keeps a state or a cache may read what earlier steps left in it before the dependency wait only when the
     // kernel right before it is a projection: that kernel has passed its own wait, so everything older is complete.
-    const bool early = ctx.prev_op == DEEPJ_OP_BF16_LINEAR || ctx.prev_op == DEEPJ_OP_BF16_BLOCK_LINEAR;
+    const bool early = ctx.prev_op == DEEPJ_OP_BF16_LINEAR || ctx.prev_op == DEEPJ_OP_BF16_LINEAR_SUM || ctx.prev_op == DEEPJ_OP_BF16_BLOCK_LINEAR;
     ctx.prev_op = op;
     auto scratch = [&](size_t floats) {          // room in the shared workspace for this op
         if (floats > ctx.ws_need) ctx.ws_need = floats;
@@ -527,9 +543,10 @@ void do_op(Ctx& ctx, const int32_t* c) {
             if (go) launch_decode_step(c[1], c[2], s);
             break;
         }
-        case DEEPJ_OP_BF16_LINEAR: {
+        case DEEPJ_OP_BF16_LINEAR:
+        case DEEPJ_OP_BF16_LINEAR_SUM: {
             // [op, x, x_off, ldx, gamma, groups, epsBits, gate, g_off, ldg, k1, x2, x2_off, ldx2, w, residual, res_off, ldr, out, out_off, ldo, M,
-            //  glu_row, limitBits, glu, glu_off, ldglu, softcapBits, exact]
+            //  glu_row, limitBits, glu, glu_off, ldglu, softcapBits, exact]; 83 adds [bias, pair, base, base_off, ldbase, multBits, sum, sum_off, ldsum]
             const char* what = "bf16Linear";
             Buf& wb = find_buf(ctx, c[14], kBf16, what);
             const int k1 = c[10], M = c[21], N = wb.N, k2 = c[11] >= 0 ? wb.K - (k1 + 7) / 8 * 8 : 0;
@@ -554,9 +571,93 @@ void do_op(Ctx& ctx, const int32_t* c) {
                 require(c[26] >= n && c[25] >= 0, what, "row stride smaller than the gated row");
                 a.glu = f32(ctx, c[24], (size_t)c[25] + sz(M - 1, c[26]) + n, what) + c[25]; a.ldglu = c[26];
             }
+            if (op == DEEPJ_OP_BF16_LINEAR_SUM) {
+                if (a.gluRow > 0) a.bias = f32_opt(ctx, c[29], a.gluRow, what);
+                a.pair = c[30];
+                require(a.pair == kPairClamp || a.pair == kPairSilu, what, "unknown pair function");
+                if (c[31] >= 0) add_base(ctx, a.a, M, c + 31, what);
+            }
             if (const char* msg = bf16_linear_check(a)) require(false, what, msg);
             a.ws = scratch(bf16_linear_ws_floats(a));
             if (go) launch_bf16_linear(a, s);
+            break;
+        }
+        case DEEPJ_OP_NORM_ADD: {   // [op, x, x_off, ldx, gamma, epsBits, base, base_off, ldbase, multBits, out, d, M]: out rows are dense
+            const char* what = "normAdd";
+            const int d = c[11], M = c[12];
+            require(d >= 1 && M >= 1 && (size_t)d * 4 <= 190 * 1024, what, "bad dimension");
+            RowOperand x = row_operand(ctx, M, d, c[1], c[2], c[3], c[4], 1, bits_to_float(c[5]), -1, 0, 0, what);
+            const int32_t tail[7] = {c[6], c[7], c[8], c[9], -1, 0, 0};
+            add_base(ctx, x, M, tail, what);
+            float* o = f32(ctx, c[10], sz(M, d), what);
+            if (go) launch_norm_add(x, o, d, M, s);
+            break;
+        }
+        case DEEPJ_OP_ATTN_GROUPED: {
+            // [op, proj, q_off, k_off, v_off, ld, qgamma, kgamma, epsBits, qtab, rel, rel_len, kcache, vcache, kscale, pos, out, out_off, ldo,
+            //  B, T, H, G, dim, vdim, scaleBits, sink]
+            const char* what = "attnGrouped";
+            GroupedAttnArgs a = {};
+            a.B = c[19]; a.T = c[20]; a.H = c[21]; a.G = c[22]; a.dim = c[23]; a.vdim = c[24]; a.scale = bits_to_float(c[25]); a.sink = c[26];
+            require(a.B >= 1 && a.T >= 1 && a.H >= 1 && a.G >= 1 && a.dim >= 1 && a.vdim >= 1 && (a.sink == 0 || a.sink == 1), what, "bad dimension");
+            if (const char* msg = grouped_attn_check(a)) require(false, what, msg);
+            const bool shared = c[13] < 0, append = c[3] >= 0;
+            require(!shared || a.dim == a.vdim, what, "values that are the keys have their size");
+            require(shared == (c[14] >= 0), what, "a cache of projected keys needs their norms beside it, another one does not");
+            Buf& kc = find_buf(ctx, c[12], kLatent, what);
+            a.kcache = kc.ptr; a.kw = kc.hd; a.bf16 = kc.kvHalf; a.maxSeq = kc.maxSeq;
+            require(a.B * a.G <= kc.B && kc.hd >= a.dim, what, "shape does not match the key cache");
+            if (!shared) {
+                Buf& vc = find_buf(ctx, c[13], kLatent, what);
+                require(a.B * a.G <= vc.B && vc.hd >= a.vdim && vc.maxSeq == kc.maxSeq && vc.kvHalf == kc.kvHalf, what, "shape does not match the value cache");
+                a.vcache = vc.ptr; a.vw = vc.hd;
+            } else {
+                a.kpitch = (a.maxSeq + 63) / 64 * 64;
+                a.kscale = f32(ctx, c[14], sz(kc.B, a.kpitch), what);
+            }
+            const int rows = a.B * a.T;
+            a.q_off = c[2]; a.k_off = append ? c[3] : -1; a.v_off = c[4]; a.ld = c[5];
+            require(a.q_off >= 0 && (!append || shared || a.v_off >= 0), what, "bad offset");
+            int last = a.q_off + a.H * a.dim;
+            if (append) last = std::max(last, a.k_off + a.G * a.dim);
+            if (append && !shared) last = std::max(last, a.v_off + a.G * a.vdim);
+            require(a.ld >= last && c[17] >= 0 && c[18] >= a.H * a.vdim, what, "bad offset or stride");
+            a.proj = f32(ctx, c[1], sz(rows - 1, a.ld) + last, what);
+            a.qgamma = f32(ctx, c[6], a.dim, what); a.eps = bits_to_float(c[8]);
+            require((append || shared) == (c[7] >= 0), what, "the key gain goes with appended or projected keys");
+            a.kgamma = f32_opt(ctx, c[7], a.dim, what);
+            a.qtab = f32_opt(ctx, c[9], a.maxSeq, what);
+            a.relLen = c[11];
+            require(c[10] < 0 || a.relLen >= 1, what, "empty bias table");
+            a.rel = f32_opt(ctx, c[10], sz(a.H, std::max(1, a.relLen)), what);
+            a.pos = f32(ctx, c[15], a.B, what);
+            a.out = f32(ctx, c[16], (size_t)c[17] + sz(rows - 1, c[18]) + a.H * a.vdim, what) + c[17]; a.ldo = c[18];
+            a.early = early; a.tickets = R.tickets;
+            a.ws = scratch(grouped_attn_ws_floats(a));
+            if (go) launch_grouped_attn(a, s);
+            break;
+        }
+        case DEEPJ_OP_MLSTM: {
+            // [op, proj, q_off, k_off, v_off, i_off, f_off, ld, capBits, qscaleBits, state, norm, pos, out, out_off, ldo, B, T, H, dim, vdim, exact]
+            const char* what = "mlstm";
+            MlstmArgs a = {};
+            a.q_off = c[2]; a.k_off = c[3]; a.v_off = c[4]; a.i_off = c[5]; a.f_off = c[6]; a.ld = c[7];
+            a.cap = bits_to_float(c[8]); a.qscale = bits_to_float(c[9]);
+            a.B = c[16]; a.T = c[17]; a.H = c[18]; a.dim = c[19]; a.vdim = c[20]; a.exact = c[21];
+            require(a.B >= 1 && a.T >= 1 && a.H >= 1 && a.H <= 65535 && a.B <= 65535 && a.dim >= 1 && a.vdim >= 1 && (a.exact == 0 || a.exact == 1) && a.cap > 0.0f,
+                    what, "bad dimension");
+            if (const char* msg = mlstm_check(a)) require(false, what, msg);
+            const int rows = a.B * a.T, HD = a.H * a.dim, HV = a.H * a.vdim;
+            const int last = std::max({a.q_off + HD, a.k_off + HD, a.v_off + HV, a.i_off + a.H, a.f_off + a.H});
+            require(std::min({a.q_off, a.k_off, a.v_off, a.i_off, a.f_off, (int)c[14]}) >= 0 && a.ld >= last && c[15] >= HV, what, "bad offset or stride");
+            a.proj = f32(ctx, c[1], sz(rows - 1, a.ld) + last, what);
+            a.state = f32(ctx, c[10], sz(a.B, HV) * a.dim, what);
+            a.norm = f32(ctx, c[11], 2 * sz(a.B, a.H) * (a.dim + 1), what);
+            a.pos = f32(ctx, c[12], a.B, what);
+            a.out = f32(ctx, c[13], (size_t)c[14] + sz(rows - 1, c[15]) + HV, what) + c[14]; a.ldo = c[15];
+            a.early = early;
+            a.ws = scratch(mlstm_ws_floats(a));
+            if (go) launch_mlstm(a, s);
             break;
         }
         case DEEPJ_OP_BF16_BLOCK_LINEAR: {   // [op, x, x_off, ldx, xstr, w, heads, out, out_off, ldo, ostr, M]

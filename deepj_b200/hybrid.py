@@ -1,30 +1,40 @@
-"""Decoders whose configuration lists their layers one by one (Punilix): every layer names its mixer and its feed-forward.
+"""Decoders whose configuration lists their layers one by one: every layer names its mixer and its feed-forward.
 
-A layer is parallel: with h = norm(x), x ← x + mixer(h) + feed_forward(h).  All projections that read h are one bf16
-weight and one launch (op 77: the norm is staged with the row, the gated feed-forward's pairs are finished in the
-epilogue), and so are the two that write the residual: [W_o ‖ W_down] over [mixed heads, gated values].  Between them the
-mixer runs its own ops:
+`DESIGNS` says, per architecture, what the layer types mean, how a feed-forward's (gate, up) pairs are joined and how a
+layer is put together:
 
-  general_delta      op 79 (the recurrence); its head norm and output gate are part of the output projection's staging
-  latent_attention   W_uq on the normed query latent, the queries taken into the latent space (op 78), op 80, values (op 78)
+  parallel (Punilix)    with h = norm(x), x ← x + mixer(h) + feed_forward(h).  All projections that read h are one bf16
+                        weight and one launch (op 77: the norm is staged with the row, the gated feed-forward's pairs are
+                        finished in the epilogue), and so are the two that write the residual: [W_o ‖ W_down] over [mixed
+                        heads, gated values].
+  post_norm (Somipel)   x ← x + c·norm1(mixer(x)), then x ← x + c·norm2(feed_forward(x)).  A sublayer's output is normed
+                        and added where the next sublayer's projection stages its row (op 83), which also leaves the new
+                        residual row for the one after it; only the last sum of a pass is a launch of its own (op 84).
+
+Between its projections a mixer runs its own ops; head norms and output gates are part of the output projection's staging:
+
+  GeneralDelta       op 79 (the recurrence)
+  LatentAttention    W_uq on the normed query latent, the queries taken into the latent space (op 78), op 80, values (op 78)
+  GroupedAttention   op 85: norms, cache append and attention over grouped heads
+  MatrixLstm         op 86 (the recurrence)
 
 A feed-forward is dense or table-routed experts (op 81), or absent.  A token step and a prompt chunk record the same
-sequence of ops with different row counts.  `MIXERS` maps a configuration's layer type to its class: another mechanism is
-another class with the same five methods.
+sequence of ops with different row counts.  Another mechanism is another class with the same methods.
 
 dtype "bf16": bf16 weights and latent cache; rows are fp32 between ops, the many-row kernels round their operand to bf16.
 dtype "f32": the same weights, every product in fp32, fp32 cache.
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
-from typing import Any, Callable, Dict, List, Mapping, Optional, Tuple
+from typing import Any, Callable, Dict, List, Mapping, NamedTuple, Optional, Tuple
 
 import numpy as np
 
 from . import _lib
-from .compute_graph import (OP_ADD_SCALAR_INPLACE, OP_ARGMAX_ROWS, OP_ATTN_LATENT, OP_ATTN_LATENT_CHUNK, OP_BF16_BLOCK_LINEAR, OP_BF16_LINEAR, OP_COPY, OP_DELTA_RULE,
-                            OP_EMBED_GATHER, OP_SAMPLE_TOPK, OP_TABLE_EXPERTS, float_bits)
+from .compute_graph import (OP_ADD_SCALAR_INPLACE, OP_ARGMAX_ROWS, OP_ATTN_GROUPED, OP_ATTN_LATENT, OP_ATTN_LATENT_CHUNK, OP_BF16_BLOCK_LINEAR, OP_BF16_LINEAR,
+                            OP_BF16_LINEAR_SUM, OP_COPY, OP_DELTA_RULE, OP_EMBED_GATHER, OP_MLSTM, OP_NORM_ADD, OP_SAMPLE_TOPK, OP_TABLE_EXPERTS, float_bits)
 from .decoder import scaled_rope_tables
 from .runner import StreamDecoder
 
@@ -53,8 +63,9 @@ class GeneralDelta:
     rank: int            # of the decay's low-rank projection
 
     @classmethod
-    def parse(cls, rec: Mapping[str, Any], rank: Optional[int]) -> "GeneralDelta":
+    def parse(cls, rec: Mapping[str, Any], rows_of: Callable[[str], Optional[int]]) -> "GeneralDelta":
         heads, dim = _positive(rec, "heads", "dim")
+        rank = rows_of("mix.w1")
         if rank is None:
             raise ValueError("the decay rank of a general_delta layer comes from its weights")
         return cls(heads, dim, rank)
@@ -110,7 +121,7 @@ class LatentAttention:
     scaling: Optional[Tuple[Tuple[str, float], ...]]
 
     @classmethod
-    def parse(cls, rec: Mapping[str, Any], rank: Optional[int]) -> "LatentAttention":
+    def parse(cls, rec: Mapping[str, Any], rows_of: Callable[[str], Optional[int]]) -> "LatentAttention":
         heads, dim, rot_dim, vdim, q_rank, kv_rank = _positive(rec, "heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank")
         rot = rec["rot"]
         if rot["dims"] != rot_dim or rot_dim % 2 != 0:
@@ -190,14 +201,214 @@ class LatentAttention:
 
 
 EXPAND_MIN_TOKENS = 48      # chunks from here on expand the context's keys and values; shorter ones attend in the latent space
-MIXERS = {"general_delta": GeneralDelta, "latent_attention": LatentAttention}
-RECURRENT = (GeneralDelta,)
+
+
+def distance_buckets(rows: int, far: float, limit: int) -> np.ndarray:
+    """Table row for distances 0, 1, … up to the first that has the last row, or `limit` of them: one row per distance in
+    the first half, logarithmic up to `far` in the second."""
+    half = rows // 2
+    if rows < 2 or far <= half:
+        raise ValueError("the distance table needs two rows and a largest distance beyond its first half")
+    out: List[int] = []
+    while len(out) < limit and (not out or out[-1] < rows - 1):
+        n = len(out)
+        # the quotient of logarithms can come out just below a whole number it equals
+        out.append(n if n < half else min(rows - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (rows - half) + 1e-9)))
+    return np.asarray(out, dtype=np.int64)
+
+
+@dataclass(frozen=True)
+class GroupedAttention:
+    """Causal attention of grouped query heads, queries and keys RMS-normed per head.  Options: projection biases, a sigmoid
+    output gate, a learned bias by distance, a query factor by position, a sink in the softmax's denominator, values that are
+    the keys as projected, another layer's keys and values."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    biases: bool = False
+    gated: bool = False
+    keys_are_values: bool = False
+    sink: bool = False
+    rel_rows: int = 0                                   # rows of the distance bias table, 0 = none
+    rel_far: float = 0.0
+    q_temp: Optional[Tuple[float, float]] = None        # (coefficient, positions per step of the logarithm's argument)
+    kv_from: Optional[int] = None
+
+    @classmethod
+    def parse(cls, rec: Mapping[str, Any], rows_of: Callable[[str], Optional[int]], distance_bias: bool = False, **options: bool) -> "GroupedAttention":
+        heads, kv_heads, dim = _positive(rec, "heads", "kv_heads", "dim")
+        vdim = dim if options.get("keys_are_values") and "vdim" not in rec else _positive(rec, "vdim")[0]
+        if heads % kv_heads:
+            raise ValueError("kv_heads must divide heads")
+        if options.get("keys_are_values") and vdim != dim:
+            raise ValueError("values that are the keys have the keys' size")
+        rel_rows, far = 0, 0.0
+        if distance_bias:
+            rel_rows, far = rows_of("mix.rel") or 0, float(rec["bias_max"])
+            distance_buckets(rel_rows, far, 1)
+        temp = rec.get("q_temp")
+        if temp is not None:
+            temp = (float(temp["coef"]), float(temp["every"]))
+            if not temp[1] > 0:
+                raise ValueError("q_temp.every must be positive")
+        return cls(heads, kv_heads, dim, vdim, float(rec["scale"]), rel_rows=rel_rows, rel_far=far, q_temp=temp, kv_from=rec.get("kv_from"), **options)
+
+    def check_source(self, l: int, layers) -> None:
+        """The layer whose keys and values this one reads comes earlier, has its own, and the same shapes."""
+        if self.kv_from is None:
+            return
+        src = layers[self.kv_from][0] if isinstance(self.kv_from, int) and 0 <= self.kv_from < l else None
+        same = ("kv_heads", "dim", "vdim", "keys_are_values")
+        if not isinstance(src, GroupedAttention) or src.kv_from is not None or any(getattr(src, k) != getattr(self, k) for k in same):
+            raise ValueError(f"layer {l}: kv_from must name an earlier layer with keys and values of its own and the same head sizes")
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    def tensors(self, d: int) -> Dict[str, Tuple[int, ...]]:
+        own = {"q": self.heads * self.dim}
+        t: Dict[str, Tuple[int, ...]] = {"mix.q.norm": (self.dim,), "mix.o": (d, self.out_width)}
+        if self.kv_from is None:
+            t["mix.k.norm"] = (self.dim,)
+            own["k"] = self.kv_heads * self.dim
+            if not self.keys_are_values:
+                own["v"] = self.kv_heads * self.vdim
+        for name, n in own.items():
+            t[f"mix.{name}"] = (n, d)
+            if self.biases:
+                t[f"mix.{name}.b"] = (n,)
+        if self.rel_rows:
+            t["mix.rel"] = (self.rel_rows, self.heads)
+        if self.gated:
+            t["mix.g"] = (self.out_width, d)
+        return t
+
+    def fields(self) -> List[Tuple[str, int]]:
+        t = self.tensors(1)
+        return [(n, t[n][0]) for n in ("mix.q", "mix.k", "mix.v", "mix.g") if n in t]
+
+    def field_biases(self) -> List[str]:
+        return [n for n in ("mix.q", "mix.k", "mix.v") if n + ".b" in self.tensors(1)]
+
+    def buffers(self, M: int) -> Dict[str, int]:
+        return {"mix": M * self.out_width}
+
+    def alloc(self, dec: "HybridDecoder", l: int) -> None:
+        if self.kv_from is None:
+            half, n, S = int(dec.dtype == "bf16"), dec.B * self.kv_heads, dec.cfg.max_seq_len
+            for name, width in (("keys", self.dim),) + (() if self.keys_are_values else (("values", self.vdim),)):
+                i = dec._new_id()
+                _lib.check(dec.lib.deepj_cuda_latent_alloc(i, n, S, (width + 15) // 16 * 16, half))
+                dec.ids[f"{name}.{l}"] = i
+            if self.keys_are_values:
+                dec._f32(f"kscale.{l}", n * ((S + 63) // 64 * 64))
+        if self.q_temp and f"temp {self.q_temp}" not in dec.ids:
+            coef, every = self.q_temp
+            steps = np.floor((np.arange(dec.cfg.max_seq_len, dtype=np.float64) + 1.0) / every)
+            dec._f32(f"temp {self.q_temp}", steps.size, 1.0 + coef * np.log(steps + 1.0))
+
+    def load(self, dec: "HybridDecoder", l: int, get) -> None:
+        dec._f32(f"qnorm.{l}", self.dim, get("mix.q.norm"))
+        if self.kv_from is None:
+            dec._f32(f"knorm.{l}", self.dim, get("mix.k.norm"))
+        if self.rel_rows:
+            rows = distance_buckets(self.rel_rows, self.rel_far, dec.cfg.max_seq_len)
+            table = get("mix.rel")
+            by_distance = np.zeros((rows.size, self.heads)) if isinstance(table, tuple) else np.asarray(table)[rows]
+            dec._f32(f"rel.{l}", by_distance.size, np.ascontiguousarray(by_distance.T))
+
+    def emit(self, op, dec: "HybridDecoder", l: int, buf: Dict[str, int], B: int, T: int) -> None:
+        I, at, own = dec.ids, dec._offsets[l], self.kv_from is None
+        src = l if own else self.kv_from
+        rel_len = distance_buckets(self.rel_rows, self.rel_far, dec.cfg.max_seq_len).size if self.rel_rows else 0
+        op("attn", OP_ATTN_GROUPED, buf["proj"], at["mix.q"], at["mix.k"] if own else -1, at.get("mix.v", -1), dec._in_rows[l], I[f"qnorm.{l}"],
+           I[f"knorm.{src}"] if own or self.keys_are_values else -1, float_bits(dec.cfg.eps), I[f"temp {self.q_temp}"] if self.q_temp else -1,
+           I[f"rel.{l}"] if self.rel_rows else -1, rel_len, I[f"keys.{src}"], -1 if self.keys_are_values else I[f"values.{src}"],
+           I[f"kscale.{src}"] if self.keys_are_values else -1, I["pos"], buf["mix"], 0, self.out_width, B, T, self.heads, self.kv_heads, self.dim, self.vdim,
+           float_bits(self.scale), int(self.sink))
+
+    def out_operand(self, dec: "HybridDecoder", l: int, buf: Dict[str, int]) -> List[int]:
+        gate = [buf["proj"], dec._offsets[l]["mix.g"], dec._in_rows[l]] if self.gated else [-1, 0, 0]
+        return [buf["mix"], 0, self.out_width, -1, 0, 0] + gate
+
+
+@dataclass(frozen=True)
+class MatrixLstm:
+    """Matrix memory per head with exponential input and forget gates and a running maximum."""
+    heads: int
+    dim: int
+    vdim: int
+    cap: float
+
+    @classmethod
+    def parse(cls, rec: Mapping[str, Any], rows_of: Callable[[str], Optional[int]]) -> "MatrixLstm":
+        cap = float(rec["gate_cap"])
+        if not cap > 0:
+            raise ValueError("gate_cap must be positive")
+        return cls(*_positive(rec, "heads", "dim", "vdim"), cap)
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    def tensors(self, d: int) -> Dict[str, Tuple[int, ...]]:
+        H, n = self.heads, self.out_width
+        return {"mix.q": (H * self.dim, d), "mix.k": (H * self.dim, d), "mix.v": (n, d), "mix.g": (n, d), "mix.i": (H, d), "mix.f": (H, d),
+                "mix.i.b": (H,), "mix.f.b": (H,), "mix.norm": (n,), "mix.o": (d, n)}
+
+    def fields(self) -> List[Tuple[str, int]]:
+        t = self.tensors(1)
+        return [(f"mix.{n}", t[f"mix.{n}"][0]) for n in "qkvgif"]
+
+    def field_biases(self) -> List[str]:
+        return ["mix.i", "mix.f"]
+
+    def buffers(self, M: int) -> Dict[str, int]:
+        return {"mix": M * self.out_width}
+
+    def alloc(self, dec: "HybridDecoder", l: int) -> None:
+        dec._f32(f"state.{l}", dec.B * self.out_width * self.dim)
+        dec._f32(f"normaliser.{l}", 2 * dec.B * self.heads * (self.dim + 1))
+
+    def load(self, dec: "HybridDecoder", l: int, get) -> None:
+        dec._f32(f"onorm.{l}", self.out_width, get("mix.norm"))
+
+    def emit(self, op, dec: "HybridDecoder", l: int, buf: Dict[str, int], B: int, T: int) -> None:
+        I, at = dec.ids, dec._offsets[l]
+        op("mlstm", OP_MLSTM, buf["proj"], *(at[f"mix.{n}"] for n in "qkvif"), dec._in_rows[l], float_bits(self.cap), float_bits(self.dim ** -0.5),
+           I[f"state.{l}"], I[f"normaliser.{l}"], I["pos"], buf["mix"], 0, self.out_width, B, T, self.heads, self.dim, self.vdim, int(dec.dtype == "f32"))
+
+    def out_operand(self, dec: "HybridDecoder", l: int, buf: Dict[str, int]) -> List[int]:
+        return [buf["mix"], 0, self.out_width, dec.ids[f"onorm.{l}"], self.heads, float_bits(dec.cfg.eps), buf["proj"], dec._offsets[l]["mix.g"], dec._in_rows[l]]
+
+
+RECURRENT = (GeneralDelta, MatrixLstm)
+PAIR_CLAMP, PAIR_SILU = 0, 1            # how a feed-forward joins its (gate, up) pairs (op 83)
+
+
+class Design(NamedTuple):
+    """What an architecture's configuration means."""
+    block: str                          # "parallel" | "post_norm"
+    pair: int
+    mixers: Mapping[str, Callable[[Mapping[str, Any], Callable[[str], Optional[int]]], Any]]      # layer type → parser
+
+
+DESIGNS = {
+    "Punilix": Design("parallel", PAIR_CLAMP, {"general_delta": GeneralDelta.parse, "latent_attention": LatentAttention.parse}),
+    "Somipel": Design("post_norm", PAIR_SILU, {
+        "attention": lambda rec, rows_of: GroupedAttention.parse(rec, rows_of, distance_bias=True, biases=True, gated=True),
+        "attention_2": lambda rec, rows_of: GroupedAttention.parse(rec, rows_of, keys_are_values=True, sink=True),
+        "mlstm": MatrixLstm.parse}),
+}
 
 
 @dataclass(frozen=True)
 class DenseFF:
     ff: int
-    limit: float
+    limit: float             # of the clamped pair
 
     def tensors(self, d: int) -> Dict[str, Tuple[int, ...]]:
         return {"mlp.gate": (self.ff, d), "mlp.up": (self.ff, d), "mlp.down": (d, self.ff)}
@@ -218,12 +429,12 @@ class TableExperts:
         return t
 
 
-def parse_ff(rec: Optional[Mapping[str, Any]], vocab: int):
+def parse_ff(rec: Optional[Mapping[str, Any]], vocab: int, pair: int = PAIR_CLAMP):
     if rec is None:
         return None
     if rec["kind"] == "dense":
-        return DenseFF(*_positive(rec, "ff"), limit=float(rec["limit"]))
-    if rec["kind"] == "moe":
+        return DenseFF(*_positive(rec, "ff"), limit=float(rec["limit"]) if pair == PAIR_CLAMP else 0.0)
+    if rec["kind"] == "moe" and pair == PAIR_CLAMP:
         experts, top = _positive(rec["router"], "experts", "top")
         if top > experts:
             raise ValueError("a token cannot use more experts than there are")
@@ -240,22 +451,30 @@ class HybridConfig:
     logit_softcap: float                 # 0 = none
     max_seq_len: int
     layers: Tuple[Tuple[Any, Any], ...] = field(default=())      # (mixer, feed-forward or None)
+    block: str = "parallel"
+    pair: int = PAIR_CLAMP
+    residual_mult: float = 1.0           # of a sublayer's output, post_norm blocks
 
     @classmethod
     def parse(cls, rec: Mapping[str, Any], max_seq_len: int, rank_of: Callable[[str], Optional[int]]) -> "HybridConfig":
         """From a config.json record; `rank_of(tensor)` gives the first dimension of a weight that only its shape tells."""
+        design = DESIGNS[rec["architecture"]]
         vocab, width = _positive(rec, "vocab", "width")
-        groups, = _positive(rec["norm"], "groups")
+        groups, = _positive(dict(rec["norm"], groups=rec["norm"].get("groups", 1)), "groups")
         if width % groups:
             raise ValueError("norm.groups must divide width")
         if max_seq_len <= 0:
             raise ValueError("maxSeqLen must be > 0")
         layers = []
         for i, L in enumerate(rec["layers"]):
-            if L["type"] not in MIXERS:
+            if L["type"] not in design.mixers:
                 raise ValueError(f"unknown layer type {L['type']!r}")
-            layers.append((MIXERS[L["type"]].parse(L["mixer"], rank_of(f"l{i}.mix.w1")), parse_ff(L["mlp"], vocab)))
-        return cls(vocab, width, groups, float(rec["norm"]["eps"]), float(rec.get("logit_softcap") or 0.0), int(max_seq_len), tuple(layers))
+            mixer = design.mixers[L["type"]](L["mixer"], lambda name, i=i: rank_of(f"l{i}.{name}"))
+            if isinstance(mixer, GroupedAttention):
+                mixer.check_source(i, layers)
+            layers.append((mixer, parse_ff(L["mlp"], vocab, design.pair)))
+        return cls(vocab, width, groups, float(rec["norm"]["eps"]), float(rec.get("logit_softcap") or 0.0), int(max_seq_len), tuple(layers),
+                   design.block, design.pair, float(rec["residual_mult"]) if design.block == "post_norm" else 1.0)
 
     def tensors(self) -> Dict[str, Tuple[int, ...]]:
         """Every tensor of a checkpoint and its shape."""
@@ -263,6 +482,8 @@ class HybridConfig:
         out: Dict[str, Tuple[int, ...]] = {"embed": (self.vocab_size, d)}
         for i, (mixer, ff) in enumerate(self.layers):
             out[f"l{i}.norm1"] = (d,)
+            if self.block == "post_norm" and ff is not None:
+                out[f"l{i}.norm2"] = (d,)
             for part in (mixer, ff):
                 if part is not None:
                     out.update({f"l{i}.{n}": s for n, s in part.tensors(d).items()})
@@ -304,6 +525,8 @@ class HybridDecoder(StreamDecoder):
         sizes = {"x": M * self.cfg.d_model}
         for l, (mixer, ff) in enumerate(self.cfg.layers):
             need = dict(mixer.buffers(M), proj=M * self._in_rows[l])
+            if self.cfg.block == "post_norm":
+                need.update(x2=M * self.cfg.d_model, s=M * self.cfg.d_model)
             if isinstance(ff, DenseFF):
                 need["y"] = M * ff.ff
             if isinstance(ff, TableExperts):
@@ -340,6 +563,9 @@ class HybridDecoder(StreamDecoder):
                 shape = self._shapes[f"l{l}.{name}"]
                 return vec(f"l{l}.{name}") if len(shape) == 1 else get(f"l{l}.{name}")
             self._f32(f"norm.{l}", d, mine("norm1"))
+            if c.block == "post_norm":
+                self._load_post_norm(l, mixer, ff, mine)
+                continue
             at, n = self._offsets[l], self._in_rows[l]
             parts = [(name, at[name], 1, 0) for name, _ in mixer.fields()]
             out = [("mix.o", 0, 1, 0)]
@@ -364,6 +590,22 @@ class HybridDecoder(StreamDecoder):
         self._f32("gF", d, vec("final.norm"))
         self._weight("head", d, c.vocab_size, [("head", 0, 1, 0)], get)
         self.loaded = True
+
+    def _load_post_norm(self, l: int, mixer, ff: Optional[DenseFF], get) -> None:
+        d, at, n = self.cfg.d_model, self._offsets[l], self._in_rows[l]
+        self._weight(f"in.{l}", d, n, [(name, at[name], 1, 0) for name, _ in mixer.fields()], get)
+        if mixer.field_biases():
+            bias = np.zeros(n, dtype=np.float32)
+            for name in mixer.field_biases():
+                b = get(name + ".b")
+                bias[at[name]:at[name] + b.size] = b
+            self._f32(f"inbias.{l}", n, bias)
+        self._weight(f"out.{l}", mixer.out_width, d, [("mix.o", 0, 1, 0)], get)
+        mixer.load(self, l, get)
+        if ff is not None:
+            self._f32(f"norm2.{l}", d, get("norm2"))
+            self._weight(f"up.{l}", d, 2 * ff.ff, [("mlp.gate", 0, 2, 0), ("mlp.up", 1, 2, 0)], get)
+            self._weight(f"down.{l}", ff.ff, d, [("mlp.down", 0, 1, 0)], get)
 
     @property
     def _shapes(self) -> Dict[str, Tuple[int, ...]]:
@@ -400,22 +642,32 @@ class HybridDecoder(StreamDecoder):
 
         emb = self._f32("embed", self.cfg.vocab_size * self.cfg.d_model)
         filler("embed")(emb, self.cfg.vocab_size * self.cfg.d_model)
-        self._load(lambda n: (*shapes[n], filler(n)), lambda n: (np.ones if n.endswith(("norm", "norm1")) else np.zeros)(shapes[n], dtype=np.float32), table)
+        self._load(lambda n: (*shapes[n], filler(n)), lambda n: (np.ones if n.endswith(("norm", "norm1", "norm2")) else np.zeros)(shapes[n], dtype=np.float32), table)
 
     # ── streams ──
     def _linear(self, op, label, operand: List[int], k1: int, second: Optional[Tuple[int, int]], w: int, residual: Optional[Tuple[int, int]],
-                out: Tuple[int, int], M: int, glu_row: int, glu: Optional[Tuple[int, int, float]] = None, softcap: float = 0.0) -> None:
+                out: Tuple[int, int], M: int, glu_row: int, glu: Optional[Tuple[int, int, float]] = None, softcap: float = 0.0,
+                bias: int = -1, pair: int = PAIR_CLAMP, base: Optional[Tuple[int, int, float, int]] = None) -> None:
+        """`operand`: x … ldgate of op 77; `second`, `residual`, `out`: (buffer, row stride); `glu` adds the clamp's limit; `base`:
+        (residual buffer, row stride, factor, buffer of the sum), the staged row being base + factor · norm(x)."""
         x2, ldx2 = second if second else (-1, 0)
         res, ldr = residual if residual else (-1, 0)
         gb, ldg, limit = glu if glu else (-1, 0, 0.0)
-        op(label, OP_BF16_LINEAR, *operand, k1, x2, 0, ldx2, w, res, 0, ldr, out[0], 0, out[1], M, glu_row, float_bits(limit), gb, 0, ldg,
-           float_bits(softcap), int(self.dtype == "f32"))
+        ints = [*operand, k1, x2, 0, ldx2, w, res, 0, ldr, out[0], 0, out[1], M, glu_row, float_bits(limit), gb, 0, ldg, float_bits(softcap), int(self.dtype == "f32")]
+        if bias < 0 and pair == PAIR_CLAMP and base is None:
+            op(label, OP_BF16_LINEAR, *ints)
+        else:
+            tail = [base[0], 0, base[1], float_bits(base[2]), base[3], 0, base[1]] if base else [-1, 0, 0, 0, -1, 0, 0]
+            op(label, OP_BF16_LINEAR_SUM, *ints, bias, pair, *tail)
 
     def _blocks(self, op, buf: Dict[str, int], tok: int, B: int, T: int) -> None:
         """Embedding and every layer for B·T rows (row b·T + t is token pos[b] + t of sequence b)."""
         c, I, M, d = self.cfg, self.ids, B * T, self.cfg.d_model
         eps = float_bits(c.eps)
         op("embed", OP_EMBED_GATHER, I["embed"], tok, buf["x"], M, d, c.vocab_size)
+        if c.block == "post_norm":
+            self._post_norm_blocks(op, buf, B, T)
+            return
         for l, (mixer, ff) in enumerate(c.layers):
             x = [buf["x"], 0, d, I[f"norm.{l}"], c.norm_groups, eps]
             n = self._in_rows[l]
@@ -430,6 +682,36 @@ class HybridDecoder(StreamDecoder):
             else:
                 self._linear(op, "out", mixer.out_operand(self, l, buf), mixer.out_width, (buf["y"], ff.ff) if dense else None, I[f"out.{l}"],
                              (buf["x"], d), (buf["x"], d), M, d)
+
+    def _post_norm_blocks(self, op, buf: Dict[str, int], B: int, T: int) -> None:
+        """The residual rows alternate between two buffers: a projection reads one, adds the normed sublayer output in "s" that
+        is still pending, and leaves the sum in the other."""
+        c, I, M, d = self.cfg, self.ids, B * T, self.cfg.d_model
+        eps, mult = float_bits(c.eps), c.residual_mult
+        x, other = buf["x"], buf["x2"]
+        pending: Optional[int] = None            # gain of the norm of what is in "s"
+
+        def read(label, w, out, n, **more):
+            nonlocal x, other
+            if pending is None:
+                operand, base = [x, 0, d, -1, 0, 0, -1, 0, 0], None
+            else:
+                operand, base = [buf["s"], 0, d, pending, c.norm_groups, eps, -1, 0, 0], (x, d, mult, other)
+                x, other = other, x
+            self._linear(op, label, operand, d, None, w, None, out, M, n, base=base, **more)
+
+        for l, (mixer, ff) in enumerate(c.layers):
+            n = self._in_rows[l]
+            read("in", I[f"in.{l}"], (buf["proj"], n), n, bias=I.get(f"inbias.{l}", -1))
+            mixer.emit(op, self, l, buf, B, T)
+            self._linear(op, "out", mixer.out_operand(self, l, buf), mixer.out_width, None, I[f"out.{l}"], None, (buf["s"], d), M, d)
+            pending = I[f"norm.{l}"]
+            if ff is not None:
+                read("up", I[f"up.{l}"], (-1, 0), 0, glu=(buf["y"], ff.ff, ff.limit), pair=c.pair)
+                self._linear(op, "down", [buf["y"], 0, ff.ff, -1, 0, 0, -1, 0, 0], ff.ff, None, I[f"down.{l}"], None, (buf["s"], d), M, d)
+                pending = I[f"norm2.{l}"]
+        if pending is not None:
+            op("sum", OP_NORM_ADD, buf["s"], 0, d, pending, eps, x, 0, d, float_bits(mult), buf["x"], d, M)
 
     def _head_ops(self, x: int, logits: int, rows: int) -> List[int]:
         s: List[int] = []

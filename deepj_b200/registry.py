@@ -4,7 +4,7 @@ parts it needs.
   "llama", "deepseek", "gpt"   {"architecture", "vocab_size", "max_seq_len", "d_model", "n_heads", "n_layers", "d_ff",
                                "q_rank", "kv_rank"} with a DeepJ checkpoint model.bin (persistence/ModelSerializer.java),
                                quantized to Q8 on load; dtype "q8"
-  "Punilix"                    layers listed one by one (hybrid.py) with model.safetensors; dtype "bf16" or "f32"
+  "Punilix", "Somipel"         layers listed one by one (hybrid.py) with model.safetensors; dtype "bf16" or "f32"
 """
 from __future__ import annotations
 
@@ -14,7 +14,7 @@ from typing import Any, Dict, Optional
 
 from . import _lib, build
 
-HYBRID = ("Punilix",)
+HYBRID = ("Punilix", "Somipel")
 Q8_KINDS = ("llama", "deepseek", "gpt")
 DTYPES = {"bfloat16": "bf16", "float32": "f32", "bf16": "bf16", "f32": "f32", "q8": "q8"}
 

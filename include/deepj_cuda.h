@@ -198,8 +198,9 @@ int deepj_cuda_bf16_alloc(int32_t id, int32_t K, int32_t N);
  * and columns col0 … of the object: row_step = 2 interleaves the gate and up rows of a gated feed-forward. */
 int deepj_cuda_bf16_store(int32_t id, int32_t row0, int32_t row_step, int32_t col0, int32_t src_id, int64_t src_off,
                           int32_t rows, int32_t cols);
-/* Cache of a latent-attention layer: [batch][max_seq][width] fp32 or bf16 values, zero-filled; a row is the normed latent
- * followed by the rotated key part that all heads share. */
+/* Row cache of an attention layer: [batch][max_seq][width] fp32 or bf16 values, zero-filled.  Latent attention: a row is the
+ * normed latent followed by the rotated key part that all heads share.  Grouped attention: one object for keys and one for
+ * values, batch = sequences x key/value heads, width = the head size rounded up to sixteen. */
 int deepj_cuda_latent_alloc(int32_t id, int32_t batch, int32_t max_seq, int32_t width, int32_t bf16);
 
 /* ───────────── fused decode op codes (extend ComputeGraph.java:19-60) ─────────────
@@ -262,6 +263,25 @@ int deepj_cuda_latent_alloc(int32_t id, int32_t batch, int32_t max_seq, int32_t 
  *                        op 80 for prompt chunks over a bf16 cache: keys and values of the context are expanded per head
  *                        (w_uk [H·dim][R], w_uv [H·vdim][R]); out = the heads' values.  Sizes multiples of eight,
  *                        dim + rot <= 256, vdim <= 128
+ *  83 BF16_LINEAR_SUM   [the 29 ints of op 77, bias, pair, base, base_off, ldbase, multBits, sum, sum_off, ldsum]
+ *                        op 77 with: a bias per plain output (or -1); pair = 1: glu = g·sigmoid(g)·u; base >= 0: the staged
+ *                        row is base + mult·norm(x), a sublayer's normed output added to the residual stream, also written
+ *                        to `sum` (>= 0, another buffer than base)
+ *  84 NORM_ADD          [op, x, x_off, ldx, gamma, epsBits, base, base_off, ldbase, multBits, out, d, M]
+ *                        out = base + mult·norm(x)·gamma, rows of d values; out may be base
+ *  85 ATTN_GROUPED      [op, proj, q_off, k_off, v_off, ld, qgamma, kgamma, epsBits, qtab, rel, rel_len, kcache, vcache, kscale, pos,
+ *                        out, out_off, ldo, B, T, H, G, dim, vdim, scaleBits, sink]
+ *                        causal attention of H query heads over G key/value heads, queries and keys RMS-normed per head; the
+ *                        chunk's keys and values are appended to the row caches [B·G][max_seq][width >= dim, vdim] first
+ *                        (k_off = -1: another layer has done so).  qtab: factor of the queries by position; rel [H][rel_len]:
+ *                        bias by distance, the last entry for everything beyond; both may be -1.  vcache = -1: the values are
+ *                        the keys as projected; kcache then holds those and kscale [B·G][max_seq rounded up to 64] their
+ *                        1 / root mean square.  sink = 1: one more score of 0 in the softmax's denominator
+ *                        (csrc/attn_grouped.cu)
+ *  86 MLSTM             [op, proj, q_off, k_off, v_off, i_off, f_off, ld, capBits, qscaleBits, state, norm, pos, out, out_off, ldo,
+ *                        B, T, H, dim, vdim, exact]   matrix-memory recurrence with exponential gates over T tokens of B
+ *                        sequences; state [B][H][vdim][dim] and norm [2][B][H][dim + 1] carried in fp32; a sequence at
+ *                        position 0 starts from zeros (csrc/mlstm.cu)
  */
 #define DEEPJ_OP_EMBED_GATHER        64
 #define DEEPJ_OP_Q8_LINEAR           65
@@ -282,6 +302,10 @@ int deepj_cuda_latent_alloc(int32_t id, int32_t batch, int32_t max_seq, int32_t 
 #define DEEPJ_OP_ATTN_LATENT        80
 #define DEEPJ_OP_TABLE_EXPERTS      81
 #define DEEPJ_OP_ATTN_LATENT_CHUNK  82
+#define DEEPJ_OP_BF16_LINEAR_SUM    83
+#define DEEPJ_OP_NORM_ADD           84
+#define DEEPJ_OP_ATTN_GROUPED       85
+#define DEEPJ_OP_MLSTM              86
 
 #ifdef __cplusplus
 }
