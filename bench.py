@@ -310,7 +310,7 @@ def main():
     ap.add_argument("--no-parity", action="store_true", help="skip the reduced-depth check against the CPU oracle")
     ap.add_argument("--no-batch16", action="store_true", help="skip the 16-sequence sub-record of the 7B workload")
     ap.add_argument("--fused-step", action="store_true", help="the single whole-token kernel (op 76) instead of one kernel per operator")
-    ap.add_argument("--layers", action="store_true", help="instead: layers at real widths, Punilix beside the closest Q8 model (deepj_b200/layerbench.py)")
+    ap.add_argument("--layers", action="store_true", help="instead: layers at real widths, the layer-list models beside the closest Q8 model (deepj_b200/layerbench.py)")
     ap.add_argument("--layers-case", default="", help="one case of --layers")
     args = ap.parse_args()
     if args.layers:

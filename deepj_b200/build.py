@@ -70,7 +70,7 @@ def _compile(src: str, obj: str, headers: list[str], verbose: bool) -> str:
 PARTS = {
     "core": ["runtime.cu", "misc.cu"],
     "bf16": ["bf16_linear.cu", "bf16_gemm_tc.cu", "bf16_experts.cu", "delta_rule.cu", "attn_latent.cu", "attn_latent_mma.cu",
-             "attn_grouped.cu", "attn_grouped_mma.cu", "mlstm.cu"],
+             "attn_grouped.cu", "attn_grouped_mma.cu", "mlstm.cu", "mlstm_mma.cu"],
 }
 
 

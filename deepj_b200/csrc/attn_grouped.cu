@@ -222,7 +222,7 @@ const char* grouped_attn_check(const GroupedAttnArgs& a) {
 // the queries as rows, then partials
 size_t grouped_attn_ws_floats(const GroupedAttnArgs& a) {
     const size_t rows = (size_t)a.B * a.T * a.H;
-    if (grouped_mma_fits(a)) return a.T == 1 ? rows * grouped_mma_splits(a) * (a.vdim + 2) : query_floats(a);
+    if (grouped_mma_fits(a)) return a.T == 1 ? rows * grouped_mma_splits(a) * ((a.vcache ? a.vw : a.kw) + 4) : query_floats(a);
     const int splits = fma_splits(a);
     return query_floats(a) + (splits > 1 ? rows * splits * (a.vdim + 2) : 0);
 }

@@ -1,7 +1,7 @@
 // Grouped attention on the tensor cores (bf16 cache); what a score is made of is described in attn_grouped.cu.
 //
 //   k_grouped_decode    one token per sequence.  grid (key splits, blocks of 16 query heads of a group, B·G): the heads of a group
-//                       are the rows of one 16-row operand, so a cached row is read once per group.  Four warps walk tiles
+//                       are the rows of one 16-row operand, so a cached row is read once per group.  Eight (or four) warps walk tiles
 //                       of 16 keys, each through a private three-stage cp.async ring that starts before the dependency wait; the
 //                       block that holds the newest position norms and appends it.  Queries enter as two bf16 halves.  Warps merge
 //                       in shared memory, blocks through partials that the last one to finish (a ticket) adds up.
@@ -16,7 +16,7 @@ namespace dj {
 namespace {
 
 constexpr float kLog2e = 1.4426950408889634f;
-constexpr int kGdKeys = 16, kGdStages = 3, kGdWarps = 4, kGdThreads = 32 * kGdWarps;
+constexpr int kGdKeys = 16, kGdStages = 3;
 constexpr int kGpRows = 128, kGpThreads = 256;
 
 // 16 bytes to shared memory, or zeros
@@ -46,16 +46,16 @@ __host__ __device__ __forceinline__ GdShape gd_shape(int kw, int vw, bool shared
     g.stage = keys * (g.LDK + g.LDV) * 2 + (shared ? keys * 4 : 0);
     return g;
 }
-size_t gd_smem(const GroupedAttnArgs& a) {
+size_t gd_smem(const GroupedAttnArgs& a, int warps) {
     const bool shared = a.vcache == nullptr;
     const GdShape g = gd_shape(a.kw, a.vw, shared, kGdKeys);
-    const size_t ring = (size_t)kGdWarps * kGdStages * g.stage, merge = (size_t)kGdWarps * 16 * ((shared ? a.kw : a.vw) + 2) * 4;
+    const size_t ring = (size_t)warps * kGdStages * g.stage, merge = (size_t)warps * 16 * ((shared ? a.kw : a.vw) + 4) * 4;
     return 2 * 16 * g.LDK * 2 + (size_t)(g.LDK + (shared ? 8 : g.LDV)) * 2 + std::max(ring, merge);
 }
 
-// VN: most output n-tiles (eight value columns each)
-template <int VN>
-__global__ void __launch_bounds__(kGdThreads) k_grouped_decode(const GroupedAttnArgs a, int splits) {
+// VN: most output n-tiles (eight value columns each), NW: warps
+template <int VN, int NW>
+__global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArgs a, int splits) {
     extern __shared__ __align__(16) unsigned char gd_raw[];
     __shared__ float s_newScale;
     __shared__ int s_last;
@@ -72,7 +72,7 @@ __global__ void __launch_bounds__(kGdThreads) k_grouped_decode(const GroupedAttn
     if (!a.early) { pdl_wait(); pdl_launch_dependents(); }
     const int pos = (int)a.pos[b];
     const bool valid = pos >= 0 && pos < a.maxSeq;
-    const int tiles = valid ? pos / kGdKeys + 1 : 0, per = max(kGdWarps, (tiles + splits - 1) / splits), active = (tiles + per - 1) / per;
+    const int tiles = valid ? pos / kGdKeys + 1 : 0, per = max(NW, (tiles + splits - 1) / splits), active = (tiles + per - 1) / per;
     const int tLo = blockIdx.x * per, tHi = min(tiles, tLo + per);
     const __nv_bfloat16* kc = (const __nv_bfloat16*)a.kcache + (size_t)blockIdx.z * a.maxSeq * a.kw;
     const __nv_bfloat16* vc = (const __nv_bfloat16*)a.vcache + (size_t)blockIdx.z * a.maxSeq * a.vw;
@@ -94,58 +94,72 @@ __global__ void __launch_bounds__(kGdThreads) k_grouped_decode(const GroupedAttn
     };
 #pragma unroll
     for (int i = 0; i < kGdStages - 1; i++) {
-        if (tLo + warp + i * kGdWarps < tHi) load(tLo + warp + i * kGdWarps, i);
+        if (tLo + warp + i * NW < tHi) load(tLo + warp + i * NW, i);
         cp_async_commit();
     }
     if (a.early) { pdl_wait(); pdl_launch_dependents(); }
     if (tLo >= tHi) { cp_async_wait<0>(); return; }
 
+    // A warp norms query rows warp, warp + NW, …; the warp after those with a first row norms the new key.  Rows are loaded to
+    // registers together with the gains: one round trip to L2.
+    constexpr int NE = 8;                                    // channels per lane, head size up to 256
     const float* x = a.proj + (size_t)b * a.ld;
-    const float qf = a.scale * (a.qtab ? a.qtab[pos] : 1.0f) * kLog2e;
-    for (int r = warp; r < 16; r += kGdWarps) {
-        float inv = 0.0f;
-        const float* q = x + a.q_off + (size_t)(h0 + r) * a.dim;
-        if (r < nrow) {
-            float ss = 0.0f;
-            for (int i = lane; i < a.dim; i += 32) ss = fmaf(q[i], q[i], ss);
-            inv = 1.0f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
+    const float qf = a.scale * (a.qtab ? __ldg(a.qtab + pos) : 1.0f) * kLog2e;
+    const bool append = a.k_off >= 0 && pos / kGdKeys >= tLo && pos / kGdKeys < tHi;
+    auto inverse_rms = [&](const float (&v)[NE]) {
+        float ss = 0.0f;
+#pragma unroll
+        for (int e = 0; e < NE; e++) ss = fmaf(v[e], v[e], ss);
+        return 1.0f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
+    };
+    auto fetch = [&](const float* src, int n, float (&v)[NE]) {
+#pragma unroll
+        for (int e = 0; e < NE; e++) v[e] = e * 32 + lane < n ? src[e * 32 + lane] : 0.0f;
+    };
+    if (append && warp == min(nrow, NW - 1)) {
+        float k[NE], kg[NE], v[NE];
+        fetch(x + a.k_off + (size_t)g * a.dim, a.dim, k);
+        fetch(a.kgamma, a.dim, kg);
+        if (!shared) fetch(x + a.v_off + (size_t)g * a.vdim, a.vdim, v);
+        const float inv = inverse_rms(k);
+        __nv_bfloat16* kd = (__nv_bfloat16*)a.kcache + ((size_t)blockIdx.z * a.maxSeq + pos) * a.kw;
+        __nv_bfloat16* vd = (__nv_bfloat16*)a.vcache + ((size_t)blockIdx.z * a.maxSeq + pos) * a.vw;
+#pragma unroll
+        for (int e = 0; e < NE; e++) {
+            const int i = e * 32 + lane;
+            const __nv_bfloat16 kv = __float2bfloat16_rn(shared ? k[e] : (k[e] * inv) * kg[e]);
+            if (i < a.kw) { newK[i] = kv; if (blockIdx.y == 0) kd[i] = kv; }
+            if (!shared && i < a.vw) {
+                const __nv_bfloat16 vv = __float2bfloat16_rn(v[e]);
+                newV[i] = vv;
+                if (blockIdx.y == 0) vd[i] = vv;
+            }
         }
-        for (int i = lane; i < a.kw; i += 32) {
+        if (shared && lane == 0) {
+            s_newScale = inv;
+            if (blockIdx.y == 0) a.kscale[(size_t)blockIdx.z * a.kpitch + pos] = inv;
+        }
+    }
+    for (int r = warp; r < 16; r += NW) {
+        float q[NE], w[NE], kg[NE], inv = 0.0f;
+        if (r < nrow) {
+            fetch(x + a.q_off + (size_t)(h0 + r) * a.dim, a.dim, q);
+            fetch(a.qgamma, a.dim, w);
+            if (shared) fetch(a.kgamma, a.dim, kg);
+            inv = inverse_rms(q);
+        }
+#pragma unroll
+        for (int e = 0; e < NE; e++) {
+            const int i = e * 32 + lane;
+            if (i >= a.kw) break;
             float v = 0.0f;
-            if (r < nrow && i < a.dim) {
-                v = (q[i] * inv) * a.qgamma[i] * qf;
-                if (shared) v *= a.kgamma[i];
+            if (r < nrow) {
+                v = (q[e] * inv) * w[e] * qf;
+                if (shared) v *= kg[e];
             }
             const __nv_bfloat16 hi = __float2bfloat16_rn(v);
             Qh[r * S.LDK + i] = hi;
             Qh[(16 + r) * S.LDK + i] = __float2bfloat16_rn(v - __bfloat162float(hi));
-        }
-    }
-    const bool append = a.k_off >= 0 && pos / kGdKeys >= tLo && pos / kGdKeys < tHi;
-    if (append && warp == kGdWarps - 1) {
-        const float* k = x + a.k_off + (size_t)g * a.dim;
-        float ss = 0.0f;
-        for (int i = lane; i < a.dim; i += 32) ss = fmaf(k[i], k[i], ss);
-        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
-        __nv_bfloat16* kd = (__nv_bfloat16*)a.kcache + ((size_t)blockIdx.z * a.maxSeq + pos) * a.kw;
-        for (int i = lane; i < a.kw; i += 32) {
-            const __nv_bfloat16 v = __float2bfloat16_rn(i >= a.dim ? 0.0f : shared ? k[i] : (k[i] * inv) * a.kgamma[i]);
-            newK[i] = v;
-            if (blockIdx.y == 0) kd[i] = v;
-        }
-        if (shared) {
-            if (lane == 0) {
-                s_newScale = inv;
-                if (blockIdx.y == 0) a.kscale[(size_t)blockIdx.z * a.kpitch + pos] = inv;
-            }
-        } else {
-            const float* v = x + a.v_off + (size_t)g * a.vdim;
-            __nv_bfloat16* vd = (__nv_bfloat16*)a.vcache + ((size_t)blockIdx.z * a.maxSeq + pos) * a.vw;
-            for (int i = lane; i < a.vw; i += 32) {
-                const __nv_bfloat16 u = __float2bfloat16_rn(i < a.vdim ? v[i] : 0.0f);
-                newV[i] = u;
-                if (blockIdx.y == 0) vd[i] = u;
-            }
         }
     }
     __syncthreads();
@@ -162,7 +176,7 @@ __global__ void __launch_bounds__(kGdThreads) k_grouped_decode(const GroupedAttn
     for (int j = 0; j < VN; j++) { o[j][0] = 0.0f; o[j][1] = 0.0f; o[j][2] = 0.0f; o[j][3] = 0.0f; }
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;
     int stage = 0;
-    for (int tile = tLo + warp; tile < tHi; tile += kGdWarps) {
+    for (int tile = tLo + warp; tile < tHi; tile += NW) {
         cp_async_wait<kGdStages - 2>();
         __syncwarp();
         const int k0 = tile * kGdKeys;
@@ -176,22 +190,29 @@ __global__ void __launch_bounds__(kGdThreads) k_grouped_decode(const GroupedAttn
             __syncwarp();
         }
         {
-            const int next = tile + (kGdStages - 1) * kGdWarps;
+            const int next = tile + (kGdStages - 1) * NW;
             if (next < tHi) load(next, stage == 0 ? kGdStages - 1 : stage - 1);
             cp_async_commit();
         }
-        float s[2][4];
+        float s[2][4], sl[2][4];                             // by the queries' high and low halves
 #pragma unroll
-        for (int j = 0; j < 2; j++) { s[j][0] = 0.0f; s[j][1] = 0.0f; s[j][2] = 0.0f; s[j][3] = 0.0f; }
+        for (int j = 0; j < 2; j++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) { s[j][e] = 0.0f; sl[j][e] = 0.0f; }
         const uint32_t kAddr = smem_u32(K) + kLane;
+#pragma unroll 4
         for (int kk = 0; kk < S.Dp / 16; kk++) {
             uint32_t ah[4], al[4], bk[4];
             ldm_x4(ah, qAddr + kk * 32);
             ldm_x4(al, qAddr + qlDelta + kk * 32);
             ldm_x4(bk, kAddr + kk * 32);
             mma_bf16(s[0], ah, bk[0], bk[1]); mma_bf16(s[1], ah, bk[2], bk[3]);
-            mma_bf16(s[0], al, bk[0], bk[1]); mma_bf16(s[1], al, bk[2], bk[3]);
+            mma_bf16(sl[0], al, bk[0], bk[1]); mma_bf16(sl[1], al, bk[2], bk[3]);
         }
+#pragma unroll
+        for (int j = 0; j < 2; j++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) s[j][e] += sl[j][e];
         const bool far = a.rel == nullptr || pos - (k0 + kGdKeys - 1) >= a.relLen - 1;
         float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
@@ -222,27 +243,31 @@ __global__ void __launch_bounds__(kGdThreads) k_grouped_decode(const GroupedAttn
         uint32_t ph[4], pl[4];
         split_bf16(s[0][0], s[0][1], ph[0], pl[0]); split_bf16(s[0][2], s[0][3], ph[1], pl[1]);
         split_bf16(s[1][0], s[1][1], ph[2], pl[2]); split_bf16(s[1][2], s[1][3], ph[3], pl[3]);
+        if (__any_sync(0xffffffffu, c0 != 1.0f || c1 != 1.0f)) {
+#pragma unroll
+            for (int c = 0; c < VN; c++) { o[c][0] *= c0; o[c][1] *= c0; o[c][2] *= c1; o[c][3] *= c1; }
+        }
         const uint32_t vAddr = smem_u32(V) + vLane;
 #pragma unroll
-        for (int c = 0; c < VN; c += 2) {
+        for (int c = 0; c < VN; c += 4) {
             if (c >= vt) break;
-            uint32_t bv[4];
-            ldm_x4_t(bv, vAddr + c * 16);
-#pragma unroll
-            for (int q = 0; q < 2; q++) {
-                o[c + q][0] *= c0; o[c + q][1] *= c0; o[c + q][2] *= c1; o[c + q][3] *= c1;
-                mma_bf16(o[c + q], ph, bv[2 * q], bv[2 * q + 1]);
-                mma_bf16(o[c + q], pl, bv[2 * q], bv[2 * q + 1]);
-            }
+            uint32_t bv[2][4];
+            const bool two = c + 2 < vt;                     // value columns come in pairs of tiles
+            ldm_x4_t(bv[0], vAddr + c * 16);
+            ldm_x4_t(bv[1], vAddr + (two ? c + 2 : c) * 16);
+            mma_bf16(o[c], ph, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], ph, bv[0][2], bv[0][3]);
+            if (two) { mma_bf16(o[c + 2], ph, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], ph, bv[1][2], bv[1][3]); }
+            mma_bf16(o[c], pl, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], pl, bv[0][2], bv[0][3]);
+            if (two) { mma_bf16(o[c + 2], pl, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], pl, bv[1][2], bv[1][3]); }
         }
         if (++stage == kGdStages) stage = 0;
         __syncwarp();
     }
     l0 = quad_sum(l0); l1 = quad_sum(l1);
     cp_async_wait<0>();
-    __syncthreads();                                         // the ring becomes the merge buffer: [warp][16][Vp + 2]
+    __syncthreads();                                         // the ring becomes the merge buffer: [warp][16][Vp + 4]
     float* mg = reinterpret_cast<float*>(ring);
-    const int mrow = Vp + 2;
+    const int mrow = Vp + 4;
     {
         float* d0 = mg + (warp * 16 + rl) * mrow; float* d1 = d0 + 8 * mrow;
 #pragma unroll
@@ -254,27 +279,28 @@ __global__ void __launch_bounds__(kGdThreads) k_grouped_decode(const GroupedAttn
         if (t4 == 0) { d0[Vp] = m0; d0[Vp + 1] = l0; d1[Vp] = m1; d1[Vp + 1] = l1; }
     }
     __syncthreads();
-    const int pw = a.vdim + 2;
-    float* part = a.ws + ((size_t)blockIdx.z * rep + blockIdx.y * 16) * splits * pw;      // [row][split][pw]
-    for (int r = warp; r < nrow; r += kGdWarps) {
-        float m = active == 1 && a.sink ? 0.0f : -INFINITY;
+    // partials: [row][split][pw], the maximum and the sum in the last four floats, the values padded to whole 16-byte pieces
+    const int pw = Vp + 4;
+    float* part = a.ws + ((size_t)blockIdx.z * rep + blockIdx.y * 16) * splits * pw;
+    for (int r = warp; r < nrow; r += NW) {
+        float mw[NW], m = active == 1 && a.sink ? 0.0f : -INFINITY;
 #pragma unroll
-        for (int w = 0; w < kGdWarps; w++) m = fmaxf(m, mg[(w * 16 + r) * mrow + Vp]);
-        float f[kGdWarps], l = active == 1 && a.sink ? exp2f(-m) : 0.0f;
+        for (int w = 0; w < NW; w++) { mw[w] = mg[(w * 16 + r) * mrow + Vp]; m = fmaxf(m, mw[w]); }
+        float l = active == 1 && a.sink ? exp2f(-m) : 0.0f;
 #pragma unroll
-        for (int w = 0; w < kGdWarps; w++) {
-            f[w] = exp2f(mg[(w * 16 + r) * mrow + Vp] - m);
-            l = fmaf(f[w], mg[(w * 16 + r) * mrow + Vp + 1], l);
+        for (int w = 0; w < NW; w++) {
+            mw[w] = exp2f(mw[w] - m);
+            l = fmaf(mw[w], mg[(w * 16 + r) * mrow + Vp + 1], l);
         }
         float* dst = active == 1 ? a.out + (size_t)b * a.ldo + (size_t)(h0 + r) * a.vdim : part + ((size_t)r * splits + blockIdx.x) * pw;
         const float norm = active == 1 ? 1.0f / l : 1.0f;
-        for (int i = lane; i < a.vdim; i += 32) {
+        for (int i = lane; i < (active == 1 ? a.vdim : Vp); i += 32) {
             float v = 0.0f;
 #pragma unroll
-            for (int w = 0; w < kGdWarps; w++) v = fmaf(f[w], mg[(w * 16 + r) * mrow + i], v);
+            for (int w = 0; w < NW; w++) v = fmaf(mw[w], mg[(w * 16 + r) * mrow + i], v);
             dst[i] = v * norm;
         }
-        if (active > 1 && lane == 0) { dst[a.vdim] = m; dst[a.vdim + 1] = l; }
+        if (active > 1 && lane == 0) { dst[Vp] = m; dst[Vp + 1] = l; }
     }
     if (active == 1) return;
     __threadfence();
@@ -287,26 +313,48 @@ __global__ void __launch_bounds__(kGdThreads) k_grouped_decode(const GroupedAttn
     __syncthreads();
     if (!s_last) return;
     __threadfence();
-    float* wts = mg;                                         // [warp][active]
-    for (int r = warp; r < nrow; r += kGdWarps) {
-        const float* src = part + (size_t)r * splits * pw;
-        float* w = wts + warp * splits;
+    float* wts = mg;                                         // [16][splits]: weight of every part, all over the row's sum
+    for (int r = warp; r < nrow; r += NW) {
+        const float* src = part + (size_t)r * splits * pw + Vp;
+        float* w = wts + r * splits;
         float m = a.sink ? 0.0f : -INFINITY;
-        for (int s = lane; s < active; s += 32) { w[s] = src[s * pw + a.vdim]; m = fmaxf(m, w[s]); }
+        for (int s = lane; s < active; s += 32) { w[s] = __ldcg(src + (size_t)s * pw); m = fmaxf(m, w[s]); }
         for (int o2 = 16; o2 > 0; o2 >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o2));
         float l = 0.0f;
-        for (int s = lane; s < active; s += 32) { w[s] = exp2f(w[s] - m); l = fmaf(w[s], src[s * pw + a.vdim + 1], l); }
+        for (int s = lane; s < active; s += 32) { w[s] = exp2f(w[s] - m); l = fmaf(w[s], __ldcg(src + (size_t)s * pw + 1), l); }
         l = warp_sum(l);
         if (a.sink) l += exp2f(-m);
-        __syncwarp();
-        float* dst = a.out + (size_t)b * a.ldo + (size_t)(h0 + r) * a.vdim;
-        for (int i = lane; i < a.vdim; i += 32) {
-            float v = 0.0f;
+        const float inv = 1.0f / l;
+        for (int s = lane; s < active; s += 32) w[s] *= inv;
+    }
+    __syncthreads();
+    // a thread: four columns of a row over every `share`-th part; the shares of a column sit in neighbouring lanes
+    const int items = nrow * (Vp / 4);
+    int share = 1;
+    while (share < 8 && items * share * 2 <= 32 * NW) share <<= 1;
+    for (int u = tid / share; u < (items + 31) / 32 * 32; u += 32 * NW / share) {
+        const int r = u / (Vp / 4), c = u - r * (Vp / 4), first = tid & (share - 1);
+        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (u < items) {
+            const float4* src = reinterpret_cast<const float4*>(part + (size_t)r * splits * pw) + c;
+            const float* w = wts + r * splits;
 #pragma unroll 8
-            for (int s = 0; s < active; s++) v = fmaf(w[s], src[(size_t)s * pw + i], v);
-            dst[i] = v / l;
+            for (int s = first; s < active; s += share) {
+                const float4 p4 = __ldcg(src + (size_t)s * (pw / 4));
+                v.x = fmaf(w[s], p4.x, v.x); v.y = fmaf(w[s], p4.y, v.y); v.z = fmaf(w[s], p4.z, v.z); v.w = fmaf(w[s], p4.w, v.w);
+            }
         }
-        __syncwarp();
+        for (int o2 = 1; o2 < share; o2 <<= 1) {
+            v.x += __shfl_xor_sync(0xffffffffu, v.x, o2); v.y += __shfl_xor_sync(0xffffffffu, v.y, o2);
+            v.z += __shfl_xor_sync(0xffffffffu, v.z, o2); v.w += __shfl_xor_sync(0xffffffffu, v.w, o2);
+        }
+        if (u < items && first == 0) {
+            float* dst = a.out + (size_t)b * a.ldo + (size_t)(h0 + r) * a.vdim + 4 * c;
+            const float e[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+            for (int i = 0; i < 4; i++)
+                if (4 * c + i < a.vdim) dst[i] = e[i];
+        }
     }
 }
 
@@ -469,23 +517,30 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const Grouped
     finish(rb, mB, lB, 2);
 }
 
+constexpr size_t kSmemMax = 227 * 1024 - 64;
 template <typename K>
-void raise(K kernel, size_t bytes, bool& done) {
-    if (!done) DJ_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - 64));
+void raise(K kernel, bool& done) {
+    if (!done) DJ_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax));
     done = true;
-    (void)bytes;
+}
+// warps of a decode block: eight where their rings fit
+int gd_warps(const GroupedAttnArgs& a) { return gd_smem(a, 8) <= kSmemMax ? 8 : 4; }
+template <int VN, int NW>
+void decode_with(const GroupedAttnArgs& a, cudaStream_t s) {
+    static bool done = false;
+    raise(k_grouped_decode<VN, NW>, done);
+    const int splits = grouped_mma_splits(a);
+    launch_k(k_grouped_decode<VN, NW>, dim3((unsigned)splits, (unsigned)((a.H / a.G + 15) / 16), (unsigned)(a.B * a.G)), dim3(32 * NW), gd_smem(a, NW), s, true, a, splits);
 }
 template <int VN>
 void decode(const GroupedAttnArgs& a, cudaStream_t s) {
-    static bool done = false;
-    raise(k_grouped_decode<VN>, 0, done);
-    const int splits = grouped_mma_splits(a);
-    launch_k(k_grouped_decode<VN>, dim3((unsigned)splits, (unsigned)((a.H / a.G + 15) / 16), (unsigned)(a.B * a.G)), dim3(kGdThreads), gd_smem(a), s, true, a, splits);
+    if (gd_warps(a) == 8) decode_with<VN, 8>(a, s);
+    else decode_with<VN, 4>(a, s);
 }
 template <int VN, int KEYS>
 void prefill(const GroupedAttnArgs& a, const __nv_bfloat16* q, cudaStream_t s) {
     static bool done = false;
-    raise(k_grouped_prefill<VN, KEYS>, 0, done);
+    raise(k_grouped_prefill<VN, KEYS>, done);
     const unsigned blocks = (unsigned)((a.T * (a.H / a.G) + kGpRows - 1) / kGpRows);
     launch_k(k_grouped_prefill<VN, KEYS>, dim3(blocks, (unsigned)(a.B * a.G)), dim3(kGpThreads), gp_smem(a, KEYS), s, true, a, q);
 }
@@ -496,8 +551,9 @@ bool grouped_mma_fits(const GroupedAttnArgs& a) {
     return a.bf16 && a.kw <= 256 && a.vw <= 256 && a.kw % 16 == 0 && a.vw % 16 == 0 && (a.vcache != nullptr || a.kpitch % 64 == 0);
 }
 int grouped_mma_splits(const GroupedAttnArgs& a) {
-    const int blocks = a.B * a.G * ((a.H / a.G + 15) / 16), tiles = (a.maxSeq + kGdKeys - 1) / kGdKeys;
-    return std::max(1, std::min({2 * g_num_sms / blocks, (tiles + kGdWarps - 1) / kGdWarps, 512}));
+    const int blocks = a.B * a.G * ((a.H / a.G + 15) / 16), tiles = (a.maxSeq + kGdKeys - 1) / kGdKeys, warps = gd_warps(a);
+    const int perSm = std::max(1, (int)(kSmemMax / gd_smem(a, warps)));
+    return std::max(1, std::min({std::min(perSm, 16 / warps) * g_num_sms / blocks, (tiles + warps - 1) / warps, 512}));
 }
 void launch_grouped_decode(const GroupedAttnArgs& a, cudaStream_t s) {
     const int vw = a.vcache ? a.vw : a.kw;

@@ -8,12 +8,14 @@
 //
 //   k_mlstm_step     one token: a block per (32 value columns, head, sequence), a warp per four columns, key channels over the
 //                    lanes; the state is fetched before the dependency wait
-//   k_mlstm_gates    several tokens, in blocks of kTok: with b_t the sum of f within a block and a_s = i_s − b_s, the weight of
+//   k_mlstm_gates    several tokens, in blocks of 32 (or 64): with b_t the sum of f within a block and a_s = i_s − b_s, the weight of
 //                    token s in the output of token t is e^{(b_t − m_t) + a_s}, that of the state before the block
 //                    e^{b_t + m_0 − m_t}.  The sums are formed in double and handed on as two floats: they reach hundreds where
 //                    their differences matter to the last bit.
 //   k_mlstm_chunk    a block per (kCols value columns, head, sequence) walks the token blocks: outputs from the state before the
 //                    block and from the products within it, then the state after it.  fp32 FMA throughout.
+// The tensor-core form of the walk is in mlstm_mma.cu.
+#include "mlstm.cuh"
 #include "row_operand.cuh"
 
 #include <algorithm>
@@ -21,8 +23,7 @@
 namespace dj {
 namespace {
 
-constexpr int kTok = 32, kCols = 32, kMaxDim = 512;
-constexpr float kDenEps = 1e-6f;
+constexpr int kTok = kMlTok, kCols = 32, kMaxDim = 512;
 
 __device__ __forceinline__ float gate_cap_f(float x, float cap) { return cap * tanhf(x / cap); }
 __device__ __forceinline__ float log_sigmoid_f(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
@@ -71,7 +72,7 @@ __global__ void __launch_bounds__(256) k_mlstm_step(const MlstmArgs a) {
     if (lane == 0) red[warp] = nq;
     __syncthreads();
     nq = ((red[0] + red[1]) + (red[2] + red[3])) + ((red[4] + red[5]) + (red[6] + red[7]));
-    const float inv = 1.0f / (fmaxf(fabsf(nq), expf(-m)) + kDenEps);
+    const float inv = 1.0f / (fmaxf(fabsf(nq), expf(-m)) + kMlDenEps);
     float o[4];
 #pragma unroll
     for (int c = 0; c < 4; c++) {
@@ -92,66 +93,65 @@ __global__ void __launch_bounds__(256) k_mlstm_step(const MlstmArgs a) {
     }
 }
 
-__host__ __device__ __forceinline__ int token_blocks(int T) { return (T + kTok - 1) / kTok; }
-
-// What k_mlstm_gates hands on, per (sequence, head): arrays of T floats, then per token block, then the normaliser.
-struct MlGates {
-    float* rowHi; float* rowLo;      // b_t − m_t
-    float* colHi; float* colLo;      // a_s
-    float* carry;                    // e^{b_t + m_0 − m_t}: the state before the block, seen by token t
-    float* floor_;                   // e^{−m_t}
-    float* add;                      // e^{b_L + a_s − m_L}: token s in the state after the block
-    float* keep;                     // [token blocks] e^{b_L + m_0 − m_L}
-    float* n0;                       // [dim] normaliser before the call
-};
-__host__ __device__ __forceinline__ MlGates gates_at(float* ws, int B, int T, int H, int dim, size_t bh) {
-    const size_t n = (size_t)B * H * T;
-    MlGates g;
-    float* p = ws + bh * T;
-    g.rowHi = p; g.rowLo = p + n; g.colHi = p + 2 * n; g.colLo = p + 3 * n; g.carry = p + 4 * n; g.floor_ = p + 5 * n; g.add = p + 6 * n;
-    g.keep = ws + 7 * n + bh * token_blocks(T);
-    g.n0 = ws + 7 * n + (size_t)B * H * token_blocks(T) + bh * dim;
-    return g;
-}
-
-// grid (heads, sequences); a warp per token block, a lane per token.  Shared: per token block its sum of f and its largest a_s.
+// grid (heads, sequences); a warp per token block, TPL consecutive tokens per lane.  Shared: per token block its sum of f, its
+// largest a_s, and the maximum before it.
+template <int TPL>
 __global__ void __launch_bounds__(256) k_mlstm_gates(const MlstmArgs a) {
-    extern __shared__ double blk[];                          // [2][token blocks], then the maximum before each block
+    constexpr int TOK = 32 * TPL;
+    extern __shared__ double blk[];
     pdl_wait();
     pdl_launch_dependents();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, h = blockIdx.x, b = blockIdx.y, nb = token_blocks(a.T), pos = (int)a.pos[b];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, h = blockIdx.x, b = blockIdx.y, nb = ml_blocks(a.T, TOK), pos = (int)a.pos[b];
     const size_t bh = (size_t)b * a.H + h, slot = (size_t)a.B * a.H * (a.dim + 1);
-    const MlGates g = gates_at(a.ws, a.B, a.T, a.H, a.dim, bh);
+    const MlGates g = ml_gates(a.ws, a.B, a.T, a.H, a.dim, TOK, bh);
     const float* nOld = a.norm + (size_t)(pos & 1) * slot + bh * (a.dim + 1);
     const bool fresh = pos == 0;
     for (int i = threadIdx.x; i < a.dim; i += 256) g.n0[i] = fresh ? 0.0f : nOld[i];
     const double start = fresh ? 0.0 : (double)nOld[a.dim];
     double* sum = blk; double* top = blk + nb; double* before = blk + 2 * nb;
-    // b_t and a_t of this lane's token, and the running maximum of a within the block
-    auto scan = [&](int j, double& bt, double& at, double& mx) {
-        const int t = j * kTok + lane;
-        float iv = 0.0f, fv = 0.0f;
-        if (t < a.T) {
-            const float* x = a.proj + ((size_t)b * a.T + t) * a.ld;
-            iv = gate_cap_f(x[a.i_off + h], a.cap);
-            fv = log_sigmoid_f(gate_cap_f(x[a.f_off + h], a.cap));
+    // b_t and a_t of this lane's tokens, and the running maximum of a within the block
+    auto scan = [&](int j, double (&bt)[TPL], double (&at)[TPL], double (&mx)[TPL]) {
+        float iv[TPL];
+        double run = 0.0;
+#pragma unroll
+        for (int u = 0; u < TPL; u++) {
+            const int t = j * TOK + lane * TPL + u;
+            float fv = 0.0f;
+            iv[u] = 0.0f;
+            if (t < a.T) {
+                const float* x = a.proj + ((size_t)b * a.T + t) * a.ld;
+                iv[u] = gate_cap_f(x[a.i_off + h], a.cap);
+                fv = log_sigmoid_f(gate_cap_f(x[a.f_off + h], a.cap));
+            }
+            run += fv;
+            bt[u] = run;
         }
-        bt = fv;
         for (int o = 1; o < 32; o <<= 1) {
-            const double u = __shfl_up_sync(0xffffffffu, bt, o);
-            if (lane >= o) bt += u;
+            const double u = __shfl_up_sync(0xffffffffu, run, o);
+            if (lane >= o) run += u;
         }
-        at = t < a.T ? (double)iv - bt : -1e30;
-        mx = at;
+        const double ahead = run - bt[TPL - 1];              // of the lanes before
+        double best = -1e30;
+#pragma unroll
+        for (int u = 0; u < TPL; u++) {
+            bt[u] += ahead;
+            at[u] = j * TOK + lane * TPL + u < a.T ? (double)iv[u] - bt[u] : -1e30;
+            best = fmax(best, at[u]);
+            mx[u] = best;
+        }
         for (int o = 1; o < 32; o <<= 1) {
-            const double u = __shfl_up_sync(0xffffffffu, mx, o);
-            if (lane >= o) mx = fmax(mx, u);
+            const double u = __shfl_up_sync(0xffffffffu, best, o);
+            if (lane >= o) best = fmax(best, u);
         }
+        const double prev = __shfl_up_sync(0xffffffffu, best, 1);
+#pragma unroll
+        for (int u = 0; u < TPL; u++)
+            if (lane > 0) mx[u] = fmax(mx[u], prev);
     };
+    double bt[TPL], at[TPL], mx[TPL];
     for (int j = warp; j < nb; j += 8) {
-        double bt, at, mx;
         scan(j, bt, at, mx);
-        if (lane == 31) { sum[j] = bt; top[j] = mx; }
+        if (lane == 31) { sum[j] = bt[TPL - 1]; top[j] = mx[TPL - 1]; }
     }
     __syncthreads();
     if (threadIdx.x == 0) {
@@ -161,18 +161,18 @@ __global__ void __launch_bounds__(256) k_mlstm_gates(const MlstmArgs a) {
     }
     __syncthreads();
     for (int j = warp; j < nb; j += 8) {
-        const int t = j * kTok + lane;
-        double bt, at, mx;
         scan(j, bt, at, mx);
         const double m0 = before[j], end = (double)(float)(sum[j] + fmax(m0, top[j]));      // the maximum after the block
-        const double m = lane == 31 || t == a.T - 1 ? end : (double)(float)(bt + fmax(m0, mx));
-        if (t < a.T) {
-            const double row = bt - m;
+#pragma unroll
+        for (int u = 0; u < TPL; u++) {
+            const int t = j * TOK + lane * TPL + u;
+            if (t >= a.T) break;
+            const double m = (double)(float)(bt[u] + fmax(m0, mx[u])), row = bt[u] - m;
             g.rowHi[t] = (float)row; g.rowLo[t] = (float)(row - (double)(float)row);
-            g.colHi[t] = (float)at; g.colLo[t] = (float)(at - (double)(float)at);
-            g.carry[t] = expf((float)(bt + m0 - m));
+            g.colHi[t] = (float)at[u]; g.colLo[t] = (float)(at[u] - (double)(float)at[u]);
+            g.carry[t] = expf((float)(bt[u] + m0 - m));
             g.floor_[t] = expf((float)-m);
-            g.add[t] = expf((float)(sum[j] + at - end));
+            g.add[t] = expf((float)(sum[j] + at[u] - end));
         }
         if (lane == 0) g.keep[j] = expf((float)(sum[j] + m0 - end));
     }
@@ -213,13 +213,13 @@ __global__ void __launch_bounds__(256) k_mlstm_chunk(const MlstmArgs a) {
     pdl_wait();
     pdl_launch_dependents();
     const int pos = (int)a.pos[b];
-    const MlGates g = gates_at(a.ws, a.B, a.T, a.H, dim, bh);
+    const MlGates g = ml_gates(a.ws, a.B, a.T, a.H, dim, kTok, bh);
     float* st = a.state + (bh * a.vdim + c0) * dim;
     for (int i = tid; i < (kCols + 1) * P; i += 256) {
         const int c = i / P, d = i - c * P;
         S[i] = d < dim ? (c == kCols ? g.n0[d] : pos != 0 && c < nc ? st[(size_t)c * dim + d] : 0.0f) : 0.0f;
     }
-    const int tx = tid & 15, ty = tid >> 4, nb = token_blocks(a.T);
+    const int tx = tid & 15, ty = tid >> 4, nb = ml_blocks(a.T, kTok);
     for (int j = 0; j < nb; j++) {
         const int t0 = j * kTok, n = min(kTok, a.T - t0);
         __syncthreads();
@@ -232,7 +232,7 @@ __global__ void __launch_bounds__(256) k_mlstm_chunk(const MlstmArgs a) {
         }
         for (int i = tid; i < 7 * kTok; i += 256) {
             const int f = i / kTok, t = i - f * kTok;
-            gt[i] = t < n ? g.rowHi[(size_t)f * a.B * a.H * a.T + t0 + t] : 0.0f;
+            gt[i] = t < n ? g.rowHi[(size_t)f * a.B * a.H * a.T + t0 + t] : f == 0 ? -INFINITY : 0.0f;
         }
         for (int i = tid; i < kTok * kCols; i += 256) {
             const int t = i / kCols, c = i - t * kCols;
@@ -255,7 +255,7 @@ __global__ void __launch_bounds__(256) k_mlstm_chunk(const MlstmArgs a) {
             float v = 0.0f;
             for (int i = lane; i < dim; i += 32) v = fmaf(S[kCols * P + i], Q[t * P + i], v);
             v = warp_sum(fmaf(v, gt[4 * kTok + t], X[t * (kTok + 1) + lane]));
-            if (lane == 0) den[t] = 1.0f / (fmaxf(fabsf(v), gt[5 * kTok + t]) + kDenEps);
+            if (lane == 0) den[t] = 1.0f / (fmaxf(fabsf(v), gt[5 * kTok + t]) + kMlDenEps);
         }
 #pragma unroll 4
         for (int s = 0; s < kTok; s++) {
@@ -308,11 +308,12 @@ __global__ void __launch_bounds__(256) k_mlstm_chunk(const MlstmArgs a) {
 
 const char* mlstm_check(const MlstmArgs& a) {
     if (a.dim > kMaxDim) return "key size not supported";
-    if (token_blocks(a.T) > 1900) return "too many tokens";
+    if (ml_blocks(a.T, kTok) > 1900) return "too many tokens";
     return nullptr;
 }
 size_t mlstm_ws_floats(const MlstmArgs& a) {
-    return a.T == 1 ? 0 : (size_t)a.B * a.H * (7 * (size_t)a.T + token_blocks(a.T) + a.dim);
+    if (a.T == 1) return 0;
+    return mlstm_mma_fits(a) ? ml_gate_floats(a.B, a.T, a.H, a.dim, kMlTokMma) + mlstm_mma_ws_floats(a) : ml_gate_floats(a.B, a.T, a.H, a.dim, kTok);
 }
 
 void launch_mlstm(const MlstmArgs& a, cudaStream_t s) {
@@ -324,12 +325,18 @@ void launch_mlstm(const MlstmArgs& a, cudaStream_t s) {
         else launch_k(k_mlstm_step<16>, grid, dim3(256), 0, s, true, a);
         return;
     }
+    const dim3 heads((unsigned)a.H, (unsigned)a.B);
+    if (mlstm_mma_fits(a)) {
+        launch_k(k_mlstm_gates<2>, heads, dim3(256), (size_t)ml_blocks(a.T, kMlTokMma) * 24, s, true, a);
+        launch_mlstm_mma(a, a.ws + ml_gate_floats(a.B, a.T, a.H, a.dim, kMlTokMma), s);
+        return;
+    }
     static bool attr = false;
     if (!attr) {
         DJ_CUDA_CHECK(cudaFuncSetAttribute(k_mlstm_chunk, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - 64));
         attr = true;
     }
-    launch_k(k_mlstm_gates, dim3((unsigned)a.H, (unsigned)a.B), dim3(256), (size_t)token_blocks(a.T) * 24, s, true, a);
+    launch_k(k_mlstm_gates<1>, heads, dim3(256), (size_t)ml_blocks(a.T, kTok) * 24, s, true, a);
     launch_k(k_mlstm_chunk, dim3((unsigned)((a.vdim + kCols - 1) / kCols), (unsigned)a.H, (unsigned)a.B), dim3(256), chunk_smem(a.dim), s, true, a);
 }
 

@@ -2,8 +2,8 @@
 
     python bench.py --layers [--layers-case NAME] [--steps K --warmup W]
 
-Each case is a Punilix stack with random weights and the Q8 model of this package that is closest to it at equal width,
-feed-forward, heads, depth, vocabulary and context.  Times are CUDA events on the library's stream: a whole prompt chunk,
+Each case holds layer-list stacks (Punilix, Somipel) with random weights and the Q8 model of this package that is closest to
+them, at equal width, feed-forward, heads, depth, vocabulary and context.  Times are CUDA events on the library's stream: a whole prompt chunk,
 K decode steps behind it (token fed back on the device), and per op code the ops of a step or of a chunk back to back as
 their own stream.  Weights exceed L2 in every case.  Roofline of an op: the slower of its algorithmic bytes over the copy
 bandwidth and its flops over the bf16 GEMM rate.
@@ -53,19 +53,47 @@ def _stack(width, delta_heads, dim, heads, mla_dim, rot, vdim, q_rank, kv_rank, 
     return {"architecture": "Punilix", "vocab": 32000, "width": width, "norm": {"groups": 4, "eps": 1e-5}, "logit_softcap": 30.0, "layers": layers}
 
 
-# name → (configuration, closest Q8 model, prompt, context window)
+def _somipel(width, heads, kv_heads, dim, lstm_heads, lstm_dim, lstm_vdim, ff, depth, attention_only=False):
+    """Layers in fours: gated attention, the same reading its keys and values, attention whose values are its keys, recurrence."""
+    layers = []
+    for i in range(depth):
+        kind = i % 4
+        attn = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5}
+        if kind == 3 and not attention_only:
+            L = {"type": "mlstm", "mixer": {"heads": lstm_heads, "dim": lstm_dim, "vdim": lstm_vdim, "gate_cap": 15.0}}
+        elif kind == 2:
+            L = {"type": "attention_2", "mixer": dict(attn, q_temp={"coef": 0.1, "every": 1024})}
+        else:
+            L = {"type": "attention", "mixer": dict(attn, bias_max=128, **({"kv_from": i - 1} if kind == 1 else {}))}
+        layers.append(dict(L, mlp={"kind": "dense", "ff": ff}))
+    return {"architecture": "Somipel", "vocab": 32000, "width": width, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "layers": layers}
+
+
+# name → (layer-list stacks, closest Q8 model, prompt)
+_W4096, _W2048 = _stack(4096, 32, 128, 32, 128, 64, 128, 1536, 512, 11008, 8, 4), _stack(2048, 16, 128, 16, 128, 64, 128, 1024, 512, 5632, 16, 2)
+_LLAMA_4096 = DecoderConfig("llama", 32000, 2176, 4096, 32, 8, 11008)
 CASES = {
-    "w4096": (_stack(4096, 32, 128, 32, 128, 64, 128, 1536, 512, 11008, 8, 4),
-              DecoderConfig("llama", 32000, 2176, 4096, 32, 8, 11008), 2048),
-    "w2048": (_stack(2048, 16, 128, 16, 128, 64, 128, 1024, 512, 5632, 16, 2),
-              DecoderConfig("deepseek", 32000, 1280, 2048, 16, 16, 5632, 1024, 512), 1024),
-    "w2048_experts": (_stack(2048, 32, 64, 16, 128, 64, 128, 1024, 512, 5632, 16, 4, moe=(64, 4, 1408)),
+    "w4096": ({"punilix": _W4096}, _LLAMA_4096, 2048),
+    "w2048": ({"punilix": _W2048}, DecoderConfig("deepseek", 32000, 1280, 2048, 16, 16, 5632, 1024, 512), 1024),
+    "w2048_experts": ({"punilix": _stack(2048, 32, 64, 16, 128, 64, 128, 1024, 512, 5632, 16, 4, moe=(64, 4, 1408))},
                       DecoderConfig("llama", 32000, 1280, 2048, 16, 16, 5632), 1024),
+    "somipel_w4096": ({"somipel": _somipel(4096, 32, 8, 128, 16, 128, 256, 11008, 8), "punilix": _W4096}, _LLAMA_4096, 2048),
+    "somipel_w2048": ({"somipel": _somipel(2048, 32, 32, 64, 8, 128, 256, 5632, 16), "punilix": _W2048},
+                      DecoderConfig("llama", 32000, 1280, 2048, 32, 16, 5632), 1024),
 }
-
-
 # decode attention where the cache is long enough to be streamed: the context is taken as given (its rows are zeros)
-LONG = ("context32k", _stack(2048, 16, 128, 16, 128, 64, 128, 1024, 512, 5632, 4, 1), DecoderConfig("deepseek", 32000, 32832, 2048, 16, 4, 5632, 1024, 512), 32768)
+LONG_CASES = {
+    "context32k": ({"punilix": _stack(2048, 16, 128, 16, 128, 64, 128, 1024, 512, 5632, 4, 1)}, DecoderConfig("deepseek", 32000, 32832, 2048, 16, 4, 5632, 1024, 512), 32768),
+    "somipel_context32k": ({"somipel": _somipel(2048, 16, 4, 128, 8, 128, 256, 5632, 3, attention_only=True)},
+                           DecoderConfig("llama", 32000, 32832, 2048, 16, 3, 5632), 32768),
+}
+DTYPES = {"punilix": "bf16 weights and latent cache, fp32 rows", "somipel": "bf16 weights and cache, fp32 rows and state"}
+
+
+def layer_list(rec, max_seq: int) -> HybridDecoder:
+    dec = HybridDecoder(HybridConfig.parse(rec, max_seq, lambda n: 32 if n.endswith(".rel") else 64), dtype="bf16")
+    dec.load_synthetic(5, 0.02)
+    return dec
 
 
 def split_ops(stream: np.ndarray) -> List[np.ndarray]:
@@ -93,12 +121,14 @@ def op_cost(op: np.ndarray, dims: Dict[int, tuple], q8: bool, context: int, kv_b
 
     def w_bytes(k, n):
         return k * n + (k + 31) // 32 * n * 4 if q8 else 2 * k * n
-    if code in (cg.OP_Q8_LINEAR, cg.OP_Q8_LINEAR_LN, cg.OP_Q8_SWIGLU, cg.OP_BF16_LINEAR):
-        at_w, at_m = {cg.OP_Q8_LINEAR: (6, 14), cg.OP_Q8_LINEAR_LN: (7, 15), cg.OP_Q8_SWIGLU: (6, 13), cg.OP_BF16_LINEAR: (14, 21)}[code]
+    if code in (cg.OP_Q8_LINEAR, cg.OP_Q8_LINEAR_LN, cg.OP_Q8_SWIGLU, cg.OP_BF16_LINEAR, cg.OP_BF16_LINEAR_SUM):
+        at_w, at_m = {cg.OP_Q8_LINEAR: (6, 14), cg.OP_Q8_LINEAR_LN: (7, 15), cg.OP_Q8_SWIGLU: (6, 13), cg.OP_BF16_LINEAR: (14, 21),
+                      cg.OP_BF16_LINEAR_SUM: (14, 21)}[code]
         w, m = c[at_w], c[at_m]
         k, n = dims[w]
         n2 = 2 * n if code == cg.OP_Q8_SWIGLU else n
-        return w_bytes(k, n2) + 4 * m * (k + n), 2 * m * k * n2
+        sums = 8 * m * k if code == cg.OP_BF16_LINEAR_SUM and c[31] >= 0 else 0          # the residual row read, the sum written
+        return w_bytes(k, n2) + 4 * m * (k + n) + sums, 2 * m * k * n2
     if code == cg.OP_BF16_BLOCK_LINEAR:
         k, n = dims[c[5]]
         return 2 * k * n + 4 * c[11] * (c[6] * k + n), 2 * c[11] * k * n
@@ -115,6 +145,14 @@ def op_cost(op: np.ndarray, dims: Dict[int, tuple], q8: bool, context: int, kv_b
         B, T, H, dim, rot, R, vdim = c[18:25]
         pairs = B * H * (T * (context - T) + T * (T + 1) // 2)
         return B * (R + rot) * kv_bytes * context + 4 * B * T * H * (dim + rot + vdim), 2 * pairs * (dim + rot + vdim) + 2 * B * context * R * H * (dim + vdim)
+    if code == cg.OP_ATTN_GROUPED:
+        B, T, H, G, dim, vdim = c[19:25]
+        pairs = B * H * (T * (context - T) + T * (T + 1) // 2)
+        row = dim * kv_bytes + 4 if c[13] < 0 else (dim + vdim) * kv_bytes
+        return B * G * row * context + 4 * B * T * H * (dim + vdim), 2 * pairs * (dim + vdim)
+    if code == cg.OP_MLSTM:
+        B, T, H, dim, vdim = c[16:21]
+        return B * (2 * 4 * H * dim * vdim + 4 * T * H * 2 * (dim + vdim)), B * T * H * 5 * dim * vdim
     if code == cg.OP_DELTA_RULE:
         B, T, H, dim = c[16:20]
         return B * (2 * 4 * H * dim * dim + 4 * T * H * dim * 6), B * T * H * (7 * dim * dim + 2 * dim * dims[c[9]][0])
@@ -203,7 +241,7 @@ def measure_long(dec, context: int, steps: int, pk) -> Dict[str, Any]:
 def main(case: str = "", steps: int = 64, warmup: int = 8, clocks=None) -> None:
     pk = peaks()
     line: Dict[str, Any] = {"metric": "layers_prefill_and_decode", "peaks": pk, "data": "synthetic", "steps": steps, "warmup": max(3, warmup), "cases": {}}
-    for name, (rec, near, prompt) in CASES.items():
+    for name, (stacks, near, prompt) in CASES.items():
         if case and name != case:
             continue
         sampler = clocks() if clocks else None
@@ -211,25 +249,25 @@ def main(case: str = "", steps: int = 64, warmup: int = 8, clocks=None) -> None:
             sampler.start()
             sampler.wait_ready()
         res = {}
-        dec = HybridDecoder(HybridConfig.parse(rec, near.max_seq_len, lambda _n: 64), dtype="bf16")
-        dec.load_synthetic(5, 0.02)
-        res["punilix"] = measure(dec, prompt, steps, warmup, 1, pk)
-        res["punilix"]["dtype"] = "bf16 weights and latent cache, fp32 rows"
-        dec.close()
+        for label, rec in stacks.items():
+            dec = layer_list(rec, near.max_seq_len)
+            res[label] = dict(measure(dec, prompt, steps, warmup, 1, pk), dtype=DTYPES[label])
+            dec.close()
         q = Q8Decoder(near, id_base=2 << 24)
         q.load_synthetic(5, 0.02)
-        res[f"{near.kind}_q8"] = measure(q, prompt, steps, warmup, 1, pk)
-        res[f"{near.kind}_q8"]["dtype"] = "q8 weights, fp32 rows and cache"
+        res[f"{near.kind}_q8"] = dict(measure(q, prompt, steps, warmup, 1, pk), dtype="q8 weights, fp32 rows and cache")
         q.close()
         if sampler:
             res["clocks"] = sampler.stop()
         line["cases"][name] = res
-    name, rec, near, context = LONG
-    if case in ("", name):
-        dec = HybridDecoder(HybridConfig.parse(rec, near.max_seq_len, lambda _n: 64), dtype="bf16")
-        dec.load_synthetic(5, 0.02)
-        res = {"punilix": measure_long(dec, context, steps, pk)}
-        dec.close()
+    for name, (stacks, near, context) in LONG_CASES.items():
+        if case and name != case:
+            continue
+        res = {}
+        for label, rec in stacks.items():
+            dec = layer_list(rec, near.max_seq_len)
+            res[label] = measure_long(dec, context, steps, pk)
+            dec.close()
         q = Q8Decoder(near, id_base=2 << 24)
         q.load_synthetic(5, 0.02)
         res[f"{near.kind}_q8"] = measure_long(q, context, steps, pk)
