@@ -28,9 +28,10 @@ template <typename T> __device__ __forceinline__ T narrow(float v);
 template <> __device__ __forceinline__ float narrow<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 narrow<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
+// unit: factor of the scores (1, or log2 e where the exponentials are powers of two).
 // a warp per head: H query heads, then (when something is appended) G key/value heads; grid (unit groups, tokens of all sequences)
 template <typename CT, typename QT>
-__global__ void __launch_bounds__(256) k_grouped_prepare(const GroupedAttnArgs a, QT* __restrict__ qp, int qw) {
+__global__ void __launch_bounds__(256) k_grouped_prepare(const GroupedAttnArgs a, QT* __restrict__ qp, int qw, float unit) {
     pdl_wait();
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31, u = blockIdx.x * 8 + (threadIdx.x >> 5);
@@ -38,35 +39,47 @@ __global__ void __launch_bounds__(256) k_grouped_prepare(const GroupedAttnArgs a
     if (u >= a.H + (a.k_off >= 0 ? a.G : 0) || p < 0 || p >= a.maxSeq) return;
     const bool query = u < a.H, shared = a.vcache == nullptr;
     const float* x = a.proj + (size_t)row * a.ld + (query ? a.q_off + u * a.dim : a.k_off + (u - a.H) * a.dim);
-    float ss = 0.0f;
-    for (int i = lane; i < a.dim; i += 32) ss = fmaf(x[i], x[i], ss);
+    const float* gain = query ? a.qgamma : a.kgamma;
+    constexpr int NE = 4;                                    // values per lane held in registers; longer heads take another round
+    float v[NE], w[NE], ss = 0.0f;
+#pragma unroll
+    for (int e = 0; e < NE; e++) {
+        const int i = e * 32 + lane;
+        v[e] = 0.0f; w[e] = 0.0f;
+        if (i < a.dim) { v[e] = x[i]; w[e] = gain[i]; ss = fmaf(v[e], v[e], ss); }
+    }
+    for (int i = NE * 32 + lane; i < a.dim; i += 32) ss = fmaf(x[i], x[i], ss);
     for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     const float inv = 1.0f / sqrtf(ss / (float)a.dim + a.eps);
     if (query) {
         const int g = u / rep, hh = u - g * rep;
         QT* dst = qp + (((size_t)b * a.G + g) * a.T * rep + (size_t)t * rep + hh) * qw;
-        const float f = a.scale * (a.qtab ? a.qtab[p] : 1.0f);
-        for (int i = lane; i < qw; i += 32) {
-            float v = 0.0f;
-            if (i < a.dim) {
-                v = (x[i] * inv) * a.qgamma[i] * f;
-                if (shared) v *= a.kgamma[i];
-            }
-            dst[i] = narrow<QT>(v);
-        }
+        const float f = a.scale * (a.qtab ? a.qtab[p] : 1.0f) * unit;
+        auto put = [&](int i, float xv, float wv) {
+            float r = (xv * inv) * wv * f;
+            if (shared && i < a.dim) r *= a.kgamma[i];
+            dst[i] = narrow<QT>(r);
+        };
+#pragma unroll
+        for (int e = 0; e < NE; e++)
+            if (e * 32 + lane < qw) put(e * 32 + lane, v[e], w[e]);
+        for (int i = NE * 32 + lane; i < qw; i += 32) put(i, i < a.dim ? x[i] : 0.0f, i < a.dim ? gain[i] : 0.0f);
         return;
     }
     const int g = u - a.H;
     const size_t at = ((size_t)b * a.G + g) * a.maxSeq + p;
     CT* k = (CT*)a.kcache + at * a.kw;
+    auto put = [&](int i, float xv, float wv) { k[i] = narrow<CT>(shared ? xv : (xv * inv) * wv); };
+#pragma unroll
+    for (int e = 0; e < NE; e++)
+        if (e * 32 + lane < a.dim) put(e * 32 + lane, v[e], w[e]);
+    for (int i = NE * 32 + lane; i < a.dim; i += 32) put(i, x[i], gain[i]);
     if (shared) {
-        for (int i = lane; i < a.dim; i += 32) k[i] = narrow<CT>(x[i]);
         if (lane == 0) a.kscale[((size_t)b * a.G + g) * a.kpitch + p] = inv;
     } else {
-        for (int i = lane; i < a.dim; i += 32) k[i] = narrow<CT>((x[i] * inv) * a.kgamma[i]);
-        CT* v = (CT*)a.vcache + at * a.vw;
+        CT* vd = (CT*)a.vcache + at * a.vw;
         const float* src = a.proj + (size_t)row * a.ld + a.v_off + g * a.vdim;
-        for (int i = lane; i < a.vdim; i += 32) v[i] = narrow<CT>(src[i]);
+        for (int i = lane; i < a.vdim; i += 32) vd[i] = narrow<CT>(src[i]);
     }
 }
 
@@ -233,16 +246,16 @@ void launch_grouped_attn(const GroupedAttnArgs& a, cudaStream_t s) {
     const int qw = (a.dim + 15) & ~15;
     const dim3 grid((unsigned)((a.H + (a.k_off >= 0 ? a.G : 0) + 7) / 8), (unsigned)(a.B * a.T));
     if (mma) {
-        launch_k(k_grouped_prepare<__nv_bfloat16, __nv_bfloat16>, grid, dim3(256), 0, s, true, a, (__nv_bfloat16*)a.ws, qw);
+        launch_k(k_grouped_prepare<__nv_bfloat16, __nv_bfloat16>, grid, dim3(256), 0, s, true, a, (__nv_bfloat16*)a.ws, qw, 1.4426950408889634f);
         launch_grouped_prefill(a, (const __nv_bfloat16*)a.ws, qw, s);
         return;
     }
     float* part = a.ws + query_floats(a);
     if (a.bf16) {
-        launch_k(k_grouped_prepare<__nv_bfloat16, float>, grid, dim3(256), 0, s, true, a, a.ws, qw);
+        launch_k(k_grouped_prepare<__nv_bfloat16, float>, grid, dim3(256), 0, s, true, a, a.ws, qw, 1.0f);
         launch_fma<__nv_bfloat16>(a, a.ws, qw, part, s);
     } else {
-        launch_k(k_grouped_prepare<float, float>, grid, dim3(256), 0, s, true, a, a.ws, qw);
+        launch_k(k_grouped_prepare<float, float>, grid, dim3(256), 0, s, true, a, a.ws, qw, 1.0f);
         launch_fma<float>(a, a.ws, qw, part, s);
     }
 }

@@ -2,13 +2,14 @@
 //
 //   k_grouped_decode    one token per sequence.  grid (key splits, blocks of 16 query heads of a group, B·G): the heads of a group
 //                       are the rows of one 16-row operand, so a cached row is read once per group.  Eight (or four) warps walk tiles
-//                       of 16 keys, each through a private three-stage cp.async ring that starts before the dependency wait; the
+//                       of 16 keys, each through a private three-stage ring of row copies (cp.async.bulk) that starts before the dependency wait; the
 //                       block that holds the newest position norms and appends it.  Queries enter as two bf16 halves.  Warps merge
 //                       in shared memory, blocks through partials that the last one to finish (a ticket) adds up.
 //   k_grouped_prefill   prompt chunks: 128 rows (token, head in the group) per block, 16 per warp, key tiles in two stages.
-// Softmax is fp32 and its weights enter the second product as two bf16 halves (16 bits).
+// Waits for copies are bounded (codes 221, 222 in the device error word).  Softmax is fp32 and its weights enter the second product as two bf16 halves (16 bits).
 #include "mma_common.cuh"
 #include "row_operand.cuh"
+#include "tc_common.cuh"
 
 #include <algorithm>
 
@@ -19,9 +20,10 @@ constexpr float kLog2e = 1.4426950408889634f;
 constexpr int kGdKeys = 16, kGdStages = 3;
 constexpr int kGpRows = 128, kGpThreads = 256;
 
-// 16 bytes to shared memory, or zeros
-__device__ __forceinline__ void cp_async16_or_zero(void* dst, const void* src, bool on) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(on ? 16 : 0) : "memory");
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
 }
 __device__ __forceinline__ float quad_max(float v) {
     v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 1));
@@ -55,9 +57,11 @@ size_t gd_smem(const GroupedAttnArgs& a, int warps) {
 
 // VN: most output n-tiles (eight value columns each), NW: warps
 template <int VN, int NW>
-__global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArgs a, int splits) {
+__global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArgs a, int splits, int* error) {
     extern __shared__ __align__(16) unsigned char gd_raw[];
+    __shared__ __align__(8) unsigned long long s_bar[NW * kGdStages];
     __shared__ float s_newScale;
+    __shared__ volatile int s_abort;
     __shared__ int s_last;
     const bool shared = a.vcache == nullptr;
     const GdShape S = gd_shape(a.kw, a.vw, shared, kGdKeys);
@@ -77,32 +81,33 @@ __global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArg
     const __nv_bfloat16* kc = (const __nv_bfloat16*)a.kcache + (size_t)blockIdx.z * a.maxSeq * a.kw;
     const __nv_bfloat16* vc = (const __nv_bfloat16*)a.vcache + (size_t)blockIdx.z * a.maxSeq * a.vw;
     const float* ksc = a.kscale + (size_t)blockIdx.z * a.kpitch;
+    auto bar = [&](int stage) { return smem_u32(&s_bar[warp * kGdStages + stage]); };
+    if (lane == 0) {
+        for (int i = 0; i < kGdStages; i++) mbar_init(bar(i), 1);
+        if (warp == 0) s_abort = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncwarp();
+    const int side = lane >> 4;                              // lanes 0-15 fetch the key rows, 16-31 the value rows (or the norms)
+    // rows past the newest key repeat it: whatever they hold is finite, and masked
     auto load = [&](int tile, int stage) {
-        const int k0 = tile * kGdKeys, kq = a.kw / 8, vq = a.vw / 8;
-        __nv_bfloat16* K = reinterpret_cast<__nv_bfloat16*>(mine + stage * S.stage);
-        for (int i = lane; i < kGdKeys * kq; i += 32) {
-            const int j = i / kq, c = i - j * kq;
-            cp_async16_or_zero(K + j * S.LDK + c * 8, kc + (size_t)min(k0 + j, pos) * a.kw + c * 8, k0 + j <= pos);
-        }
-        if (!shared) {
-            __nv_bfloat16* V = K + kGdKeys * S.LDK;
-            for (int i = lane; i < kGdKeys * vq; i += 32) {
-                const int j = i / vq, c = i - j * vq;
-                cp_async16_or_zero(V + j * S.LDV + c * 8, vc + (size_t)min(k0 + j, pos) * a.vw + c * 8, k0 + j <= pos);
-            }
-        } else if (lane < kGdKeys / 4) cp_async16_or_zero(K + kGdKeys * S.LDK + lane * 8, ksc + k0 + lane * 4, true);      // kpitch covers whole tiles
+        const int k0 = tile * kGdKeys, row = min(k0 + (lane & 15), pos);
+        const uint32_t K = smem_u32(mine + stage * S.stage);
+        if (lane == 0) mbar_arrive_expect_tx(bar(stage), (uint32_t)(kGdKeys * 2 * (a.kw + (shared ? 2 : a.vw))));
+        __syncwarp();
+        if (side == 0) bulk_g2s(K + (uint32_t)((lane & 15) * S.LDK * 2), kc + (size_t)row * a.kw, (uint32_t)(a.kw * 2), bar(stage));
+        else if (!shared) bulk_g2s(K + (uint32_t)((kGdKeys * S.LDK + (lane & 15) * S.LDV) * 2), vc + (size_t)row * a.vw, (uint32_t)(a.vw * 2), bar(stage));
+        else if (lane == 16) bulk_g2s(K + (uint32_t)(kGdKeys * S.LDK * 2), ksc + k0, kGdKeys * 4, bar(stage));      // kpitch covers whole tiles
     };
 #pragma unroll
-    for (int i = 0; i < kGdStages - 1; i++) {
+    for (int i = 0; i < kGdStages - 1; i++)
         if (tLo + warp + i * NW < tHi) load(tLo + warp + i * NW, i);
-        cp_async_commit();
-    }
     if (a.early) { pdl_wait(); pdl_launch_dependents(); }
-    if (tLo >= tHi) { cp_async_wait<0>(); return; }
+    if (tLo >= tHi) return;
 
     // A warp norms query rows warp, warp + NW, …; the warp after those with a first row norms the new key.  Rows are loaded to
     // registers together with the gains: one round trip to L2.
-    constexpr int NE = 8;                                    // channels per lane, head size up to 256
+    constexpr int NE = VN / 4 > 4 ? 8 : 4;                   // channels per lane (checked against the head size by the launcher)
     const float* x = a.proj + (size_t)b * a.ld;
     const float qf = a.scale * (a.qtab ? __ldg(a.qtab + pos) : 1.0f) * kLog2e;
     const bool append = a.k_off >= 0 && pos / kGdKeys >= tLo && pos / kGdKeys < tHi;
@@ -114,7 +119,10 @@ __global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArg
     };
     auto fetch = [&](const float* src, int n, float (&v)[NE]) {
 #pragma unroll
-        for (int e = 0; e < NE; e++) v[e] = e * 32 + lane < n ? src[e * 32 + lane] : 0.0f;
+        for (int e = 0; e < NE; e++) {
+            v[e] = 0.0f;
+            if (e * 32 + lane < n) v[e] = src[e * 32 + lane];
+        }
     };
     if (append && warp == min(nrow, NW - 1)) {
         float k[NE], kg[NE], v[NE];
@@ -140,27 +148,26 @@ __global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArg
             if (blockIdx.y == 0) a.kscale[(size_t)blockIdx.z * a.kpitch + pos] = inv;
         }
     }
-    for (int r = warp; r < 16; r += NW) {
-        float q[NE], w[NE], kg[NE], inv = 0.0f;
-        if (r < nrow) {
-            fetch(x + a.q_off + (size_t)(h0 + r) * a.dim, a.dim, q);
-            fetch(a.qgamma, a.dim, w);
-            if (shared) fetch(a.kgamma, a.dim, kg);
-            inv = inverse_rms(q);
-        }
+    for (int r = warp; r < nrow; r += NW) {
+        float q[NE], w[NE], kg[NE];
+        fetch(x + a.q_off + (size_t)(h0 + r) * a.dim, a.dim, q);
+        fetch(a.qgamma, a.dim, w);
+        if (shared) fetch(a.kgamma, a.dim, kg);
+        const float inv = inverse_rms(q);
 #pragma unroll
         for (int e = 0; e < NE; e++) {
             const int i = e * 32 + lane;
             if (i >= a.kw) break;
-            float v = 0.0f;
-            if (r < nrow) {
-                v = (q[e] * inv) * w[e] * qf;
-                if (shared) v *= kg[e];
-            }
+            float v = (q[e] * inv) * w[e] * qf;
+            if (shared) v *= kg[e];
             const __nv_bfloat16 hi = __float2bfloat16_rn(v);
             Qh[r * S.LDK + i] = hi;
             Qh[(16 + r) * S.LDK + i] = __float2bfloat16_rn(v - __bfloat162float(hi));
         }
+    }
+    for (int i = tid; i < (16 - nrow) * S.LDK / 2; i += 32 * NW) {       // rows of no head
+        reinterpret_cast<uint32_t*>(Qh + nrow * S.LDK)[i] = 0;
+        reinterpret_cast<uint32_t*>(Qh + (16 + nrow) * S.LDK)[i] = 0;
     }
     __syncthreads();
 
@@ -175,10 +182,16 @@ __global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArg
 #pragma unroll
     for (int j = 0; j < VN; j++) { o[j][0] = 0.0f; o[j][1] = 0.0f; o[j][2] = 0.0f; o[j][3] = 0.0f; }
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;
-    int stage = 0;
+    int stage = 0, phase = 0;
     for (int tile = tLo + warp; tile < tHi; tile += NW) {
-        cp_async_wait<kGdStages - 2>();
-        __syncwarp();
+        if (!__all_sync(0xffffffffu, mbar_wait(bar(stage), phase, &s_abort, error, 221))) {
+            // let the copies in flight land before the block goes: this tile's and the next one's
+            for (unsigned w = 0; w < (1u << 16) && !mbar_try_wait(bar(stage), phase); w++) {}
+            const int nextStage = stage + 1 == kGdStages ? 0 : stage + 1, nextPhase = stage + 1 == kGdStages ? phase ^ 1 : phase;
+            if (tile + NW < tHi)
+                for (unsigned w = 0; w < (1u << 16) && !mbar_try_wait(bar(nextStage), nextPhase); w++) {}
+            break;
+        }
         const int k0 = tile * kGdKeys;
         __nv_bfloat16* K = reinterpret_cast<__nv_bfloat16*>(mine + stage * S.stage);
         __nv_bfloat16* V = shared ? K : K + kGdKeys * S.LDK;
@@ -187,12 +200,12 @@ __global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArg
             for (int i = lane; i < a.kw; i += 32) K[(pos - k0) * S.LDK + i] = newK[i];
             if (shared) { if (lane == 0) sc[pos - k0] = s_newScale; }
             else { for (int i = lane; i < a.vw; i += 32) V[(pos - k0) * S.LDV + i] = newV[i]; }
+            fence_proxy_async_smem();
             __syncwarp();
         }
         {
             const int next = tile + (kGdStages - 1) * NW;
             if (next < tHi) load(next, stage == 0 ? kGdStages - 1 : stage - 1);
-            cp_async_commit();
         }
         float s[2][4], sl[2][4];                             // by the queries' high and low halves
 #pragma unroll
@@ -213,30 +226,42 @@ __global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArg
         for (int j = 0; j < 2; j++)
 #pragma unroll
             for (int e = 0; e < 4; e++) s[j][e] += sl[j][e];
-        const bool far = a.rel == nullptr || pos - (k0 + kGdKeys - 1) >= a.relLen - 1;
         float mx0 = -INFINITY, mx1 = -INFINITY;
+        if (shared) {
+#pragma unroll
+            for (int j = 0; j < 2; j++) {
+                const float2 f = *reinterpret_cast<const float2*>(sc + j * 8 + 2 * t4);
+                s[j][0] *= f.x; s[j][1] *= f.y; s[j][2] *= f.x; s[j][3] *= f.y;
+            }
+        }
+        if (k0 + kGdKeys - 1 <= pos && (a.rel == nullptr || pos - (k0 + kGdKeys - 1) >= a.relLen - 1)) {       // the whole tile is seen, and far
+#pragma unroll
+            for (int j = 0; j < 2; j++)
+#pragma unroll
+                for (int e = 0; e < 2; e++) { s[j][e] += far0; s[j][2 + e] += far1; }
+        } else {
+#pragma unroll
+            for (int j = 0; j < 2; j++)
+#pragma unroll
+                for (int e = 0; e < 2; e++) {
+                    const int d = pos - k0 - (j * 8 + 2 * t4 + e);
+                    if (a.rel && d >= 0) { s[j][e] += bias_at(rel0, d, a.relLen); s[j][2 + e] += bias_at(rel1, d, a.relLen); }
+                    if (d < 0) { s[j][e] = -INFINITY; s[j][2 + e] = -INFINITY; }
+                }
+        }
 #pragma unroll
         for (int j = 0; j < 2; j++)
 #pragma unroll
-            for (int e = 0; e < 2; e++) {
-                const int i = j * 8 + 2 * t4 + e, d = pos - k0 - i;
-                if (shared) { s[j][e] *= sc[i]; s[j][2 + e] *= sc[i]; }
-                if (d < 0) { s[j][e] = -INFINITY; s[j][2 + e] = -INFINITY; }
-                else {
-                    s[j][e] += far ? far0 : bias_at(rel0, d, a.relLen);
-                    s[j][2 + e] += far ? far1 : bias_at(rel1, d, a.relLen);
-                }
-                mx0 = fmaxf(mx0, s[j][e]); mx1 = fmaxf(mx1, s[j][2 + e]);
-            }
+            for (int e = 0; e < 2; e++) { mx0 = fmaxf(mx0, s[j][e]); mx1 = fmaxf(mx1, s[j][2 + e]); }
         mx0 = fmaxf(m0, quad_max(mx0)); mx1 = fmaxf(m1, quad_max(mx1));      // finite: a tile's first key is always seen
-        const float c0 = exp2f(m0 - mx0), c1 = exp2f(m1 - mx1);
+        const float c0 = ex2(m0 - mx0), c1 = ex2(m1 - mx1);
         m0 = mx0; m1 = mx1;
         float ps0 = 0.0f, ps1 = 0.0f;
 #pragma unroll
         for (int j = 0; j < 2; j++)
 #pragma unroll
             for (int e = 0; e < 2; e++) {
-                s[j][e] = exp2f(s[j][e] - m0); s[j][2 + e] = exp2f(s[j][2 + e] - m1);
+                s[j][e] = ex2(s[j][e] - m0); s[j][2 + e] = ex2(s[j][2 + e] - m1);
                 ps0 += s[j][e]; ps1 += s[j][2 + e];
             }
         l0 = l0 * c0 + ps0; l1 = l1 * c1 + ps1;
@@ -260,11 +285,10 @@ __global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArg
             mma_bf16(o[c], pl, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], pl, bv[0][2], bv[0][3]);
             if (two) { mma_bf16(o[c + 2], pl, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], pl, bv[1][2], bv[1][3]); }
         }
-        if (++stage == kGdStages) stage = 0;
+        if (++stage == kGdStages) { stage = 0; phase ^= 1; }
         __syncwarp();
     }
     l0 = quad_sum(l0); l1 = quad_sum(l1);
-    cp_async_wait<0>();
     __syncthreads();                                         // the ring becomes the merge buffer: [warp][16][Vp + 4]
     float* mg = reinterpret_cast<float*>(ring);
     const int mrow = Vp + 4;
@@ -286,10 +310,10 @@ __global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArg
         float mw[NW], m = active == 1 && a.sink ? 0.0f : -INFINITY;
 #pragma unroll
         for (int w = 0; w < NW; w++) { mw[w] = mg[(w * 16 + r) * mrow + Vp]; m = fmaxf(m, mw[w]); }
-        float l = active == 1 && a.sink ? exp2f(-m) : 0.0f;
+        float l = active == 1 && a.sink ? ex2(-m) : 0.0f;
 #pragma unroll
         for (int w = 0; w < NW; w++) {
-            mw[w] = exp2f(mw[w] - m);
+            mw[w] = ex2(mw[w] - m);
             l = fmaf(mw[w], mg[(w * 16 + r) * mrow + Vp + 1], l);
         }
         float* dst = active == 1 ? a.out + (size_t)b * a.ldo + (size_t)(h0 + r) * a.vdim : part + ((size_t)r * splits + blockIdx.x) * pw;
@@ -321,9 +345,9 @@ __global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArg
         for (int s = lane; s < active; s += 32) { w[s] = __ldcg(src + (size_t)s * pw); m = fmaxf(m, w[s]); }
         for (int o2 = 16; o2 > 0; o2 >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o2));
         float l = 0.0f;
-        for (int s = lane; s < active; s += 32) { w[s] = exp2f(w[s] - m); l = fmaf(w[s], __ldcg(src + (size_t)s * pw + 1), l); }
+        for (int s = lane; s < active; s += 32) { w[s] = ex2(w[s] - m); l = fmaf(w[s], __ldcg(src + (size_t)s * pw + 1), l); }
         l = warp_sum(l);
-        if (a.sink) l += exp2f(-m);
+        if (a.sink) l += ex2(-m);
         const float inv = 1.0f / l;
         for (int s = lane; s < active; s += 32) w[s] *= inv;
     }
@@ -365,8 +389,10 @@ size_t gp_smem(const GroupedAttnArgs& a, int keys) {
 
 // VN: most output n-tiles, KEYS: keys per tile
 template <int VN, int KEYS>
-__global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const GroupedAttnArgs a, const __nv_bfloat16* __restrict__ qp) {
+__global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const GroupedAttnArgs a, const __nv_bfloat16* __restrict__ qp, int* error) {
     extern __shared__ __align__(16) unsigned char gd_raw[];
+    __shared__ __align__(8) unsigned long long s_bar[2];
+    __shared__ volatile int s_abort;
     constexpr int NT = KEYS / 8;
     const bool shared = a.vcache == nullptr;
     const GdShape S = gd_shape(a.kw, a.vw, shared, KEYS);
@@ -384,22 +410,23 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const Grouped
     const __nv_bfloat16* kc = (const __nv_bfloat16*)a.kcache + (size_t)blockIdx.y * a.maxSeq * a.kw;
     const __nv_bfloat16* vc = (const __nv_bfloat16*)a.vcache + (size_t)blockIdx.y * a.maxSeq * a.vw;
     const float* ksc = a.kscale + (size_t)blockIdx.y * a.kpitch;
-    const int kq = a.kw / 8, vq = a.vw / 8;
+    const int kq = a.kw / 8;
+    if (tid == 0) {
+        mbar_init(smem_u32(&s_bar[0]), 1); mbar_init(smem_u32(&s_bar[1]), 1);
+        s_abort = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncthreads();
+    // a thread per row; rows past the newest key repeat it: whatever they hold is finite, and masked
     auto load = [&](int tile, int stage) {
-        const int k0 = tile * KEYS;
-        __nv_bfloat16* K = reinterpret_cast<__nv_bfloat16*>(ring + stage * S.stage);
-        for (int i = tid; i < KEYS * kq; i += kGpThreads) {
-            const int j = i / kq, c = i - j * kq;
-            cp_async16_or_zero(K + j * S.LDK + c * 8, kc + (size_t)min(k0 + j, lastKey) * a.kw + c * 8, k0 + j <= lastKey);
+        const int k0 = tile * KEYS, row = min(k0 + tid % KEYS, lastKey);
+        const uint32_t K = smem_u32(ring + stage * S.stage), bar = smem_u32(&s_bar[stage]);
+        if (tid == 0) mbar_arrive_expect_tx(bar, (uint32_t)(KEYS * 2 * (a.kw + (shared ? 2 : a.vw))));
+        if (tid < KEYS) bulk_g2s(K + (uint32_t)(tid * S.LDK * 2), kc + (size_t)row * a.kw, (uint32_t)(a.kw * 2), bar);
+        else if (tid < 2 * KEYS) {
+            if (!shared) bulk_g2s(K + (uint32_t)((KEYS * S.LDK + (tid - KEYS) * S.LDV) * 2), vc + (size_t)row * a.vw, (uint32_t)(a.vw * 2), bar);
+            else if (tid == KEYS) bulk_g2s(K + (uint32_t)(KEYS * S.LDK * 2), ksc + k0, KEYS * 4, bar);
         }
-        if (!shared) {
-            __nv_bfloat16* V = K + KEYS * S.LDK;
-            for (int i = tid; i < KEYS * vq; i += kGpThreads) {
-                const int j = i / vq, c = i - j * vq;
-                cp_async16_or_zero(V + j * S.LDV + c * 8, vc + (size_t)min(k0 + j, lastKey) * a.vw + c * 8, k0 + j <= lastKey);
-            }
-        } else if (tid < KEYS / 4) cp_async16_or_zero(K + KEYS * S.LDK + tid * 8, ksc + k0 + tid * 4, true);
-        cp_async_commit();
     };
     load(0, 0);
     const __nv_bfloat16* q0 = qp + ((size_t)blockIdx.y * rows + r0) * a.kw;
@@ -424,8 +451,8 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const Grouped
     float mA = -INFINITY, mB = -INFINITY, lA = 0.0f, lB = 0.0f;
     const int tiles = lastKey / KEYS + 1;
     for (int tile = 0; tile < tiles; tile++) {
-        cp_async_wait<0>();
-        __syncthreads();                                     // this tile has landed, nobody reads the other stage any more
+        // this tile has landed, nobody reads the other stage any more
+        if (!__syncthreads_and(mbar_wait(smem_u32(&s_bar[tile & 1]), (tile >> 1) & 1, &s_abort, error, 222))) break;
         if (tile + 1 < tiles) load(tile + 1, (tile + 1) & 1);
         const int k0 = tile * KEYS;
         if (k0 > warpLast) continue;
@@ -445,33 +472,43 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const Grouped
                 mma_bf16(s[n], aq, bk[0], bk[1]); mma_bf16(s[n + 1], aq, bk[2], bk[3]);
             }
         }
-        const bool edge = k0 + KEYS - 1 > warpFirst;         // some row of the warp does not see the whole tile
-        const bool far = a.rel == nullptr || warpFirst - (k0 + KEYS - 1) >= a.relLen - 1;
+        if (shared) {
+#pragma unroll
+            for (int j = 0; j < NT; j++) {
+                const float2 f = *reinterpret_cast<const float2*>(sc + j * 8 + 2 * t4);
+                s[j][0] *= f.x; s[j][1] *= f.y; s[j][2] *= f.x; s[j][3] *= f.y;
+            }
+        }
+        const bool whole = k0 + KEYS - 1 <= warpFirst;       // every row of the warp sees the whole tile
+        if (whole && (a.rel == nullptr || warpFirst - (k0 + KEYS - 1) >= a.relLen - 1)) {
+            if (a.rel) {
+#pragma unroll
+                for (int j = 0; j < NT; j++) { s[j][0] += farA; s[j][1] += farA; s[j][2] += farB; s[j][3] += farB; }
+            }
+        } else {
+#pragma unroll
+            for (int j = 0; j < NT; j++)
+#pragma unroll
+                for (int e = 0; e < 2; e++) {
+                    const int i = j * 8 + 2 * t4 + e, dA = limA - k0 - i, dB = limB - k0 - i;
+                    if (a.rel) { s[j][e] += bias_at(relA, max(dA, 0), a.relLen); s[j][2 + e] += bias_at(relB, max(dB, 0), a.relLen); }
+                    if (dA < 0) s[j][e] = -INFINITY;
+                    if (dB < 0) s[j][2 + e] = -INFINITY;
+                }
+        }
         float xA = -INFINITY, xB = -INFINITY;
 #pragma unroll
-        for (int j = 0; j < NT; j++)
-#pragma unroll
-            for (int e = 0; e < 2; e++) {
-                const int i = j * 8 + 2 * t4 + e, dA = limA - k0 - i, dB = limB - k0 - i;
-                float vA = s[j][e], vB = s[j][2 + e];
-                if (shared) { vA *= sc[i]; vB *= sc[i]; }
-                vA = fmaf(vA, kLog2e, far ? farA : dA >= 0 ? bias_at(relA, dA, a.relLen) : 0.0f);
-                vB = fmaf(vB, kLog2e, far ? farB : dB >= 0 ? bias_at(relB, dB, a.relLen) : 0.0f);
-                if (edge && dA < 0) vA = -INFINITY;
-                if (edge && dB < 0) vB = -INFINITY;
-                s[j][e] = vA; s[j][2 + e] = vB;
-                xA = fmaxf(xA, vA); xB = fmaxf(xB, vB);
-            }
+        for (int j = 0; j < NT; j++) { xA = fmaxf(xA, fmaxf(s[j][0], s[j][1])); xB = fmaxf(xB, fmaxf(s[j][2], s[j][3])); }
         xA = fmaxf(mA, quad_max(xA)); xB = fmaxf(mB, quad_max(xB));
         const float uA = xA > -INFINITY ? xA : 0.0f, uB = xB > -INFINITY ? xB : 0.0f;      // a row that has seen no key yet
-        const float cA = exp2f(mA - uA), cB = exp2f(mB - uB);
+        const float cA = ex2(mA - uA), cB = ex2(mB - uB);
         mA = xA; mB = xB;
         float pA = 0.0f, pB = 0.0f;
 #pragma unroll
         for (int j = 0; j < NT; j++)
 #pragma unroll
             for (int e = 0; e < 2; e++) {
-                s[j][e] = exp2f(s[j][e] - uA); s[j][2 + e] = exp2f(s[j][2 + e] - uB);
+                s[j][e] = ex2(s[j][e] - uA); s[j][2 + e] = ex2(s[j][2 + e] - uB);
                 pA += s[j][e]; pB += s[j][2 + e];
             }
         lA = lA * cA + pA; lB = lB * cB + pB;
@@ -486,12 +523,17 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const Grouped
             split_bf16(s[2 * kk][0], s[2 * kk][1], ph[0], pl[0]); split_bf16(s[2 * kk][2], s[2 * kk][3], ph[1], pl[1]);
             split_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1], ph[2], pl[2]); split_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3], ph[3], pl[3]);
 #pragma unroll
-            for (int c = 0; c < VN; c += 2) {
+            for (int c = 0; c < VN; c += 4) {
                 if (c >= vt) break;
-                uint32_t bv[4];
-                ldm_x4_t(bv, vAddr + (uint32_t)(kk * 16 * ldv * 2) + c * 16);
-                mma_bf16(o[c], ph, bv[0], bv[1]); mma_bf16(o[c + 1], ph, bv[2], bv[3]);
-                mma_bf16(o[c], pl, bv[0], bv[1]); mma_bf16(o[c + 1], pl, bv[2], bv[3]);
+                uint32_t bv[2][4];
+                const bool two = c + 2 < vt;                 // value columns come in pairs of tiles
+                const uint32_t at = vAddr + (uint32_t)(kk * 16 * ldv * 2);
+                ldm_x4_t(bv[0], at + c * 16);
+                ldm_x4_t(bv[1], at + (two ? c + 2 : c) * 16);
+                mma_bf16(o[c], ph, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], ph, bv[0][2], bv[0][3]);
+                if (two) { mma_bf16(o[c + 2], ph, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], ph, bv[1][2], bv[1][3]); }
+                mma_bf16(o[c], pl, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], pl, bv[0][2], bv[0][3]);
+                if (two) { mma_bf16(o[c + 2], pl, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], pl, bv[1][2], bv[1][3]); }
             }
         }
     }
@@ -501,8 +543,8 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const Grouped
         float f = 1.0f;
         if (a.sink) {
             const float u = fmaxf(m, 0.0f);
-            f = exp2f(m - u);
-            l = l * f + exp2f(-u);
+            f = ex2(m - u);
+            l = l * f + ex2(-u);
         }
         f /= l;
         float* dst = a.out + (size_t)(b * a.T + r / rep) * a.ldo + (size_t)(g * rep + r % rep) * a.vdim;
@@ -517,7 +559,7 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const Grouped
     finish(rb, mB, lB, 2);
 }
 
-constexpr size_t kSmemMax = 227 * 1024 - 64;
+constexpr size_t kSmemMax = 226 * 1024;       // beside the static part
 template <typename K>
 void raise(K kernel, bool& done) {
     if (!done) DJ_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax));
@@ -530,7 +572,7 @@ void decode_with(const GroupedAttnArgs& a, cudaStream_t s) {
     static bool done = false;
     raise(k_grouped_decode<VN, NW>, done);
     const int splits = grouped_mma_splits(a);
-    launch_k(k_grouped_decode<VN, NW>, dim3((unsigned)splits, (unsigned)((a.H / a.G + 15) / 16), (unsigned)(a.B * a.G)), dim3(32 * NW), gd_smem(a, NW), s, true, a, splits);
+    launch_k(k_grouped_decode<VN, NW>, dim3((unsigned)splits, (unsigned)((a.H / a.G + 15) / 16), (unsigned)(a.B * a.G)), dim3(32 * NW), gd_smem(a, NW), s, true, a, splits, g_dev_error);
 }
 template <int VN>
 void decode(const GroupedAttnArgs& a, cudaStream_t s) {
@@ -542,7 +584,7 @@ void prefill(const GroupedAttnArgs& a, const __nv_bfloat16* q, cudaStream_t s) {
     static bool done = false;
     raise(k_grouped_prefill<VN, KEYS>, done);
     const unsigned blocks = (unsigned)((a.T * (a.H / a.G) + kGpRows - 1) / kGpRows);
-    launch_k(k_grouped_prefill<VN, KEYS>, dim3(blocks, (unsigned)(a.B * a.G)), dim3(kGpThreads), gp_smem(a, KEYS), s, true, a, q);
+    launch_k(k_grouped_prefill<VN, KEYS>, dim3(blocks, (unsigned)(a.B * a.G)), dim3(kGpThreads), gp_smem(a, KEYS), s, true, a, q, g_dev_error);
 }
 
 }  // namespace
@@ -557,7 +599,8 @@ int grouped_mma_splits(const GroupedAttnArgs& a) {
 }
 void launch_grouped_decode(const GroupedAttnArgs& a, cudaStream_t s) {
     const int vw = a.vcache ? a.vw : a.kw;
-    if (vw <= 64) decode<8>(a, s);
+    if (std::max(a.kw, vw) > 128) decode<32>(a, s);      // both head sizes bound the channels per lane
+    else if (vw <= 64) decode<8>(a, s);
     else if (vw <= 128) decode<16>(a, s);
     else decode<32>(a, s);
 }

@@ -25,8 +25,6 @@ namespace {
 
 constexpr int kTok = kMlTok, kCols = 32, kMaxDim = 512;
 
-__device__ __forceinline__ float gate_cap_f(float x, float cap) { return cap * tanhf(x / cap); }
-__device__ __forceinline__ float log_sigmoid_f(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float warp_sum(float v) {
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
     return v;
@@ -93,89 +91,11 @@ __global__ void __launch_bounds__(256) k_mlstm_step(const MlstmArgs a) {
     }
 }
 
-// grid (heads, sequences); a warp per token block, TPL consecutive tokens per lane.  Shared: per token block its sum of f, its
-// largest a_s, and the maximum before it.
-template <int TPL>
 __global__ void __launch_bounds__(256) k_mlstm_gates(const MlstmArgs a) {
-    constexpr int TOK = 32 * TPL;
     extern __shared__ double blk[];
     pdl_wait();
     pdl_launch_dependents();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, h = blockIdx.x, b = blockIdx.y, nb = ml_blocks(a.T, TOK), pos = (int)a.pos[b];
-    const size_t bh = (size_t)b * a.H + h, slot = (size_t)a.B * a.H * (a.dim + 1);
-    const MlGates g = ml_gates(a.ws, a.B, a.T, a.H, a.dim, TOK, bh);
-    const float* nOld = a.norm + (size_t)(pos & 1) * slot + bh * (a.dim + 1);
-    const bool fresh = pos == 0;
-    for (int i = threadIdx.x; i < a.dim; i += 256) g.n0[i] = fresh ? 0.0f : nOld[i];
-    const double start = fresh ? 0.0 : (double)nOld[a.dim];
-    double* sum = blk; double* top = blk + nb; double* before = blk + 2 * nb;
-    // b_t and a_t of this lane's tokens, and the running maximum of a within the block
-    auto scan = [&](int j, double (&bt)[TPL], double (&at)[TPL], double (&mx)[TPL]) {
-        float iv[TPL];
-        double run = 0.0;
-#pragma unroll
-        for (int u = 0; u < TPL; u++) {
-            const int t = j * TOK + lane * TPL + u;
-            float fv = 0.0f;
-            iv[u] = 0.0f;
-            if (t < a.T) {
-                const float* x = a.proj + ((size_t)b * a.T + t) * a.ld;
-                iv[u] = gate_cap_f(x[a.i_off + h], a.cap);
-                fv = log_sigmoid_f(gate_cap_f(x[a.f_off + h], a.cap));
-            }
-            run += fv;
-            bt[u] = run;
-        }
-        for (int o = 1; o < 32; o <<= 1) {
-            const double u = __shfl_up_sync(0xffffffffu, run, o);
-            if (lane >= o) run += u;
-        }
-        const double ahead = run - bt[TPL - 1];              // of the lanes before
-        double best = -1e30;
-#pragma unroll
-        for (int u = 0; u < TPL; u++) {
-            bt[u] += ahead;
-            at[u] = j * TOK + lane * TPL + u < a.T ? (double)iv[u] - bt[u] : -1e30;
-            best = fmax(best, at[u]);
-            mx[u] = best;
-        }
-        for (int o = 1; o < 32; o <<= 1) {
-            const double u = __shfl_up_sync(0xffffffffu, best, o);
-            if (lane >= o) best = fmax(best, u);
-        }
-        const double prev = __shfl_up_sync(0xffffffffu, best, 1);
-#pragma unroll
-        for (int u = 0; u < TPL; u++)
-            if (lane > 0) mx[u] = fmax(mx[u], prev);
-    };
-    double bt[TPL], at[TPL], mx[TPL];
-    for (int j = warp; j < nb; j += 8) {
-        scan(j, bt, at, mx);
-        if (lane == 31) { sum[j] = bt[TPL - 1]; top[j] = mx[TPL - 1]; }
-    }
-    __syncthreads();
-    if (threadIdx.x == 0) {
-        double m = start;
-        for (int j = 0; j < nb; j++) { before[j] = m; m = (double)(float)(sum[j] + fmax(m, top[j])); }
-        a.norm[(size_t)((pos + a.T) & 1) * slot + bh * (a.dim + 1) + a.dim] = (float)m;
-    }
-    __syncthreads();
-    for (int j = warp; j < nb; j += 8) {
-        scan(j, bt, at, mx);
-        const double m0 = before[j], end = (double)(float)(sum[j] + fmax(m0, top[j]));      // the maximum after the block
-#pragma unroll
-        for (int u = 0; u < TPL; u++) {
-            const int t = j * TOK + lane * TPL + u;
-            if (t >= a.T) break;
-            const double m = (double)(float)(bt[u] + fmax(m0, mx[u])), row = bt[u] - m;
-            g.rowHi[t] = (float)row; g.rowLo[t] = (float)(row - (double)(float)row);
-            g.colHi[t] = (float)at[u]; g.colLo[t] = (float)(at[u] - (double)(float)at[u]);
-            g.carry[t] = expf((float)(bt[u] + m0 - m));
-            g.floor_[t] = expf((float)-m);
-            g.add[t] = expf((float)(sum[j] + at[u] - end));
-        }
-        if (lane == 0) g.keep[j] = expf((float)(sum[j] + m0 - end));
-    }
+    ml_gate_block<1>(a, blockIdx.x, blockIdx.y, blk);
 }
 
 size_t chunk_smem(int dim) {
@@ -313,7 +233,7 @@ const char* mlstm_check(const MlstmArgs& a) {
 }
 size_t mlstm_ws_floats(const MlstmArgs& a) {
     if (a.T == 1) return 0;
-    return mlstm_mma_fits(a) ? ml_gate_floats(a.B, a.T, a.H, a.dim, kMlTokMma) + mlstm_mma_ws_floats(a) : ml_gate_floats(a.B, a.T, a.H, a.dim, kTok);
+    return mlstm_mma_fits(a) ? mlstm_mma_ws_floats(a) : ml_gate_floats(a.B, a.T, a.H, a.dim, kTok);
 }
 
 void launch_mlstm(const MlstmArgs& a, cudaStream_t s) {
@@ -325,18 +245,13 @@ void launch_mlstm(const MlstmArgs& a, cudaStream_t s) {
         else launch_k(k_mlstm_step<16>, grid, dim3(256), 0, s, true, a);
         return;
     }
-    const dim3 heads((unsigned)a.H, (unsigned)a.B);
-    if (mlstm_mma_fits(a)) {
-        launch_k(k_mlstm_gates<2>, heads, dim3(256), (size_t)ml_blocks(a.T, kMlTokMma) * 24, s, true, a);
-        launch_mlstm_mma(a, a.ws + ml_gate_floats(a.B, a.T, a.H, a.dim, kMlTokMma), s);
-        return;
-    }
+    if (mlstm_mma_fits(a)) { launch_mlstm_mma(a, s); return; }
     static bool attr = false;
     if (!attr) {
         DJ_CUDA_CHECK(cudaFuncSetAttribute(k_mlstm_chunk, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - 64));
         attr = true;
     }
-    launch_k(k_mlstm_gates<1>, heads, dim3(256), (size_t)ml_blocks(a.T, kTok) * 24, s, true, a);
+    launch_k(k_mlstm_gates, dim3((unsigned)a.H, (unsigned)a.B), dim3(256), (size_t)ml_blocks(a.T, kTok) * 24, s, true, a);
     launch_k(k_mlstm_chunk, dim3((unsigned)((a.vdim + kCols - 1) / kCols), (unsigned)a.H, (unsigned)a.B), dim3(256), chunk_smem(a.dim), s, true, a);
 }
 
