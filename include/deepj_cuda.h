@@ -263,7 +263,9 @@ int deepj_cuda_latent_alloc(int32_t id, int32_t batch, int32_t max_seq, int32_t 
  *                        op 80 for prompt chunks over a bf16 cache: keys and values of the context are expanded per head
  *                        (w_uk [H·dim][R], w_uv [H·vdim][R]); out = the heads' values.  Sizes multiples of eight,
  *                        dim + rot <= 256, vdim <= 128
- *  83 BF16_LINEAR_SUM   [the 29 ints of op 77, bias, pair, base, base_off, ldbase, multBits, sum, sum_off, ldsum]
+ *  83 BF16_LINEAR_SUM   [op, x, x_off, ldx, gamma, groups, epsBits, gate, gate_off, ldgate, k1, x2, x2_off, ldx2, w,
+ *                        residual, res_off, ldr, out, out_off, ldo, M, glu_row, limitBits, glu, glu_off, ldglu,
+ *                        softcapBits, exact, bias, pair, base, base_off, ldbase, multBits, sum, sum_off, ldsum]
  *                        op 77 with: a bias per plain output (or -1); pair = 1: glu = g·sigmoid(g)·u; base >= 0: the staged
  *                        row is base + mult·norm(x), a sublayer's normed output added to the residual stream, also written
  *                        to `sum` (>= 0, another buffer than base)
