@@ -2,11 +2,12 @@
 //
 //   k_grouped_decode    one token per sequence.  grid (key splits, blocks of 16 query heads of a group, B·G): the heads of a group
 //                       are the rows of one 16-row operand, so a cached row is read once per group.  Eight (or four) warps walk tiles
-//                       of 16 keys, each through a private three-stage ring of row copies (cp.async.bulk) that starts before the dependency wait; the
+//                       of 16 keys, each through a private three-stage ring of tensor copies that starts before the dependency wait; the
 //                       block that holds the newest position norms and appends it.  Queries enter as two bf16 halves.  Warps merge
 //                       in shared memory, blocks through partials that the last one to finish (a ticket) adds up.
-//   k_grouped_prefill   prompt chunks: 128 rows (token, head in the group) per block, 16 per warp, key tiles in two stages.
-// Waits for copies are bounded (codes 221, 222 in the device error word).  Softmax is fp32 and its weights enter the second product as two bf16 halves (16 bits).
+//   k_grouped_prefill   prompt chunks: 128 rows (token, head in the group) per block, 16 per warp, key tiles in three stages.
+// Key and value rows travel as 64-column boxes with 128-byte swizzle.
+// Waits for copies are bounded (codes 221-223 in the device error word).  Softmax is fp32 and its weights enter the second product as two bf16 halves (16 bits).
 #include "mma_common.cuh"
 #include "row_operand.cuh"
 #include "tc_common.cuh"
@@ -17,7 +18,7 @@ namespace dj {
 namespace {
 
 constexpr float kLog2e = 1.4426950408889634f;
-constexpr int kGdKeys = 16, kGdStages = 3;
+constexpr int kGdKeys = 16, kStages = 3, kAlone = 4;
 constexpr int kGpRows = 128, kGpThreads = 256;
 
 __device__ __forceinline__ float ex2(float x) {
@@ -41,66 +42,81 @@ __device__ __forceinline__ float warp_sum(float v) {
 // Bias of query rows (table row `rel`, fp32) at distance d, in the exponent's base-2 units.
 __device__ __forceinline__ float bias_at(const float* rel, int d, int len) { return __ldg(rel + min(d, len - 1)) * kLog2e; }
 
-struct GdShape { int Dp, LDK, LDV, stage; };       // padded head size, row pitches (halves), bytes of a stage
+struct GdParams {
+    GroupedAttnArgs a;
+    CUtensorMap k, v;                                        // rows of 64 columns × a tile's keys
+    int splits; int* error;
+};
+
+// Shared memory: tiles (1024-byte aligned), then queries, the new row, the norms of cached keys.
+struct GdShape { int kb, vb, tile, LDQ; };                   // boxes of a key and of a value row, bytes of a stage, query row pitch (halves)
 __host__ __device__ __forceinline__ GdShape gd_shape(int kw, int vw, bool shared, int keys) {
     GdShape g;
-    g.Dp = kw; g.LDK = kw + 8; g.LDV = shared ? 0 : vw + 8;
-    g.stage = keys * (g.LDK + g.LDV) * 2 + (shared ? keys * 4 : 0);
+    g.kb = (kw + 63) / 64; g.vb = shared ? 0 : (vw + 63) / 64;
+    g.tile = (g.kb + g.vb) * keys * 128; g.LDQ = kw + 8;
     return g;
 }
+// Byte offset of 16-byte column c of row r in a tile of boxes: the copy engine swaps the columns of a 128-byte row by its number.
+__device__ __forceinline__ uint32_t swizzled(int r, int c, int keys) { return (uint32_t)((c >> 3) * keys * 128 + r * 128 + (((c & 7) ^ (r & 7)) << 4)); }
+
 size_t gd_smem(const GroupedAttnArgs& a, int warps) {
     const bool shared = a.vcache == nullptr;
     const GdShape g = gd_shape(a.kw, a.vw, shared, kGdKeys);
-    const size_t ring = (size_t)warps * kGdStages * g.stage, merge = (size_t)warps * 16 * ((shared ? a.kw : a.vw) + 4) * 4;
-    return 2 * 16 * g.LDK * 2 + (size_t)(g.LDK + (shared ? 8 : g.LDV)) * 2 + std::max(ring, merge);
+    const size_t ring = (size_t)warps * kStages * g.tile, merge = (size_t)warps * 16 * ((shared ? a.kw : a.vw) + 4) * 4;
+    return 1024 + std::max(ring, merge) + (size_t)2 * 16 * g.LDQ * 2 + (size_t)(a.kw + a.vw + 16) * 2 + (size_t)warps * kStages * kGdKeys * 4;
 }
 
 // VN: most output n-tiles (eight value columns each), NW: warps
 template <int VN, int NW>
-__global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArgs a, int splits, int* error) {
-    extern __shared__ __align__(16) unsigned char gd_raw[];
-    __shared__ __align__(8) unsigned long long s_bar[NW * kGdStages];
+__global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(const __grid_constant__ GdParams p) {
+    extern __shared__ __align__(1024) unsigned char gd_raw[];
+    __shared__ __align__(8) unsigned long long s_bar[NW * kStages];
     __shared__ float s_newScale;
     __shared__ volatile int s_abort;
     __shared__ int s_last;
+    const GroupedAttnArgs& a = p.a;
+    const int splits = p.splits;
     const bool shared = a.vcache == nullptr;
     const GdShape S = gd_shape(a.kw, a.vw, shared, kGdKeys);
     const int Vp = shared ? a.kw : a.vw, vt = Vp / 8;
-    __nv_bfloat16* Qh = reinterpret_cast<__nv_bfloat16*>(gd_raw);        // [16][LDK], then the low halves
-    __nv_bfloat16* newK = Qh + 2 * 16 * S.LDK;
-    __nv_bfloat16* newV = newK + S.LDK;
-    unsigned char* ring = reinterpret_cast<unsigned char*>(newV + (shared ? 8 : S.LDV));
+    const uint32_t raw = smem_u32(gd_raw), skip = ((raw + 1023u) & ~1023u) - raw;
+    unsigned char* ring = gd_raw + skip;
+    const size_t ringBytes = max((size_t)NW * kStages * S.tile, (size_t)NW * 16 * (Vp + 4) * 4);
+    __nv_bfloat16* Qh = reinterpret_cast<__nv_bfloat16*>(ring + ringBytes);          // [16][LDQ], then the low halves
+    float* scales = reinterpret_cast<float*>(Qh + 2 * 16 * S.LDQ);                   // [warp][stage][16]
+    __nv_bfloat16* newK = reinterpret_cast<__nv_bfloat16*>(scales + NW * kStages * kGdKeys);
+    __nv_bfloat16* newV = newK + a.kw;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, rl = lane >> 2, t4 = lane & 3;
-    unsigned char* mine = ring + warp * kGdStages * S.stage;
+    unsigned char* mine = ring + warp * kStages * S.tile;
+    float* mySc = scales + warp * kStages * kGdKeys;
     const int rep = a.H / a.G, b = blockIdx.z / a.G, g = blockIdx.z - b * a.G, h0 = g * rep + blockIdx.y * 16, nrow = min(16, rep - (int)blockIdx.y * 16);
     if (!a.early) { pdl_wait(); pdl_launch_dependents(); }
     const int pos = (int)a.pos[b];
     const bool valid = pos >= 0 && pos < a.maxSeq;
-    const int tiles = valid ? pos / kGdKeys + 1 : 0, per = max(NW, (tiles + splits - 1) / splits), active = (tiles + per - 1) / per;
+    // a few tiles per warp cost less than adding up the parts of several blocks
+    const int tiles = valid ? pos / kGdKeys + 1 : 0, per = tiles <= kAlone * NW ? kAlone * NW : max(NW, (tiles + splits - 1) / splits), active = (tiles + per - 1) / per;
     const int tLo = blockIdx.x * per, tHi = min(tiles, tLo + per);
-    const __nv_bfloat16* kc = (const __nv_bfloat16*)a.kcache + (size_t)blockIdx.z * a.maxSeq * a.kw;
-    const __nv_bfloat16* vc = (const __nv_bfloat16*)a.vcache + (size_t)blockIdx.z * a.maxSeq * a.vw;
     const float* ksc = a.kscale + (size_t)blockIdx.z * a.kpitch;
-    auto bar = [&](int stage) { return smem_u32(&s_bar[warp * kGdStages + stage]); };
+    const int plane = blockIdx.z * a.maxSeq;                 // first row of this head's keys and values
+    auto bar = [&](int stage) { return smem_u32(&s_bar[warp * kStages + stage]); };
     if (lane == 0) {
-        for (int i = 0; i < kGdStages; i++) mbar_init(bar(i), 1);
+        for (int i = 0; i < kStages; i++) mbar_init(bar(i), 1);
         if (warp == 0) s_abort = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     __syncwarp();
-    const int side = lane >> 4;                              // lanes 0-15 fetch the key rows, 16-31 the value rows (or the norms)
-    // rows past the newest key repeat it: whatever they hold is finite, and masked
+    // rows past the newest key are whatever earlier requests left: finite, and masked
     auto load = [&](int tile, int stage) {
-        const int k0 = tile * kGdKeys, row = min(k0 + (lane & 15), pos);
-        const uint32_t K = smem_u32(mine + stage * S.stage);
-        if (lane == 0) mbar_arrive_expect_tx(bar(stage), (uint32_t)(kGdKeys * 2 * (a.kw + (shared ? 2 : a.vw))));
-        __syncwarp();
-        if (side == 0) bulk_g2s(K + (uint32_t)((lane & 15) * S.LDK * 2), kc + (size_t)row * a.kw, (uint32_t)(a.kw * 2), bar(stage));
-        else if (!shared) bulk_g2s(K + (uint32_t)((kGdKeys * S.LDK + (lane & 15) * S.LDV) * 2), vc + (size_t)row * a.vw, (uint32_t)(a.vw * 2), bar(stage));
-        else if (lane == 16) bulk_g2s(K + (uint32_t)(kGdKeys * S.LDK * 2), ksc + k0, kGdKeys * 4, bar(stage));      // kpitch covers whole tiles
+        if (lane != 0) return;
+        const int k0 = tile * kGdKeys;
+        uint32_t dst = smem_u32(mine + stage * S.tile);
+        mbar_arrive_expect_tx(bar(stage), (uint32_t)(S.tile + (shared ? kGdKeys * 4 : 0)));
+        for (int c = 0; c < S.kb; c++, dst += kGdKeys * 128) tma_box(dst, &p.k, c * 64, plane + k0, bar(stage));
+        for (int c = 0; c < S.vb; c++, dst += kGdKeys * 128) tma_box(dst, &p.v, c * 64, plane + k0, bar(stage));
+        if (shared) bulk_g2s(smem_u32(mySc + stage * kGdKeys), ksc + k0, kGdKeys * 4, bar(stage));      // kpitch covers whole tiles
     };
 #pragma unroll
-    for (int i = 0; i < kGdStages - 1; i++)
+    for (int i = 0; i < kStages - 1; i++)
         if (tLo + warp + i * NW < tHi) load(tLo + warp + i * NW, i);
     if (a.early) { pdl_wait(); pdl_launch_dependents(); }
     if (tLo >= tHi) return;
@@ -161,20 +177,19 @@ __global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArg
             float v = (q[e] * inv) * w[e] * qf;
             if (shared) v *= kg[e];
             const __nv_bfloat16 hi = __float2bfloat16_rn(v);
-            Qh[r * S.LDK + i] = hi;
-            Qh[(16 + r) * S.LDK + i] = __float2bfloat16_rn(v - __bfloat162float(hi));
+            Qh[r * S.LDQ + i] = hi;
+            Qh[(16 + r) * S.LDQ + i] = __float2bfloat16_rn(v - __bfloat162float(hi));
         }
     }
-    for (int i = tid; i < (16 - nrow) * S.LDK / 2; i += 32 * NW) {       // rows of no head
-        reinterpret_cast<uint32_t*>(Qh + nrow * S.LDK)[i] = 0;
-        reinterpret_cast<uint32_t*>(Qh + (16 + nrow) * S.LDK)[i] = 0;
+    for (int i = tid; i < (16 - nrow) * S.LDQ / 2; i += 32 * NW) {       // rows of no head
+        reinterpret_cast<uint32_t*>(Qh + nrow * S.LDQ)[i] = 0;
+        reinterpret_cast<uint32_t*>(Qh + (16 + nrow) * S.LDQ)[i] = 0;
     }
     __syncthreads();
 
-    const uint32_t qAddr = smem_u32(Qh) + (uint32_t)(((lane & 15) * S.LDK + (lane >> 4) * 8) * 2), qlDelta = (uint32_t)(16 * S.LDK * 2);
-    const uint32_t kLane = (uint32_t)((((lane & 7) + ((lane >> 4) << 3)) * S.LDK + ((lane >> 3) & 1) * 8) * 2);
-    const int ldv = shared ? S.LDK : S.LDV;
-    const uint32_t vLane = (uint32_t)((((lane & 7) + (((lane >> 3) & 1) << 3)) * ldv + (lane >> 4) * 8) * 2);
+    const uint32_t qAddr = smem_u32(Qh) + (uint32_t)(((lane & 15) * S.LDQ + (lane >> 4) * 8) * 2), qlDelta = (uint32_t)(16 * S.LDQ * 2);
+    const int kRow = (lane & 7) + ((lane >> 4) << 3), kHalf = (lane >> 3) & 1;       // operand B from rows of keys
+    const int vRow = (lane & 7) + (((lane >> 3) & 1) << 3), vHalf = lane >> 4;       // … read transposed
     const float* rel0 = a.rel ? a.rel + (size_t)(h0 + min(rl, nrow - 1)) * a.relLen : nullptr;
     const float* rel1 = a.rel ? a.rel + (size_t)(h0 + min(rl + 8, nrow - 1)) * a.relLen : nullptr;
     const float far0 = a.rel ? bias_at(rel0, a.relLen - 1, a.relLen) : 0.0f, far1 = a.rel ? bias_at(rel1, a.relLen - 1, a.relLen) : 0.0f;
@@ -184,41 +199,42 @@ __global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArg
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;
     int stage = 0, phase = 0;
     for (int tile = tLo + warp; tile < tHi; tile += NW) {
-        if (!__all_sync(0xffffffffu, mbar_wait(bar(stage), phase, &s_abort, error, 221))) {
+        if (!__all_sync(0xffffffffu, mbar_wait(bar(stage), phase, &s_abort, p.error, 221))) {
             // let the copies in flight land before the block goes: this tile's and the next one's
             for (unsigned w = 0; w < (1u << 16) && !mbar_try_wait(bar(stage), phase); w++) {}
-            const int nextStage = stage + 1 == kGdStages ? 0 : stage + 1, nextPhase = stage + 1 == kGdStages ? phase ^ 1 : phase;
+            const int nextStage = stage + 1 == kStages ? 0 : stage + 1, nextPhase = stage + 1 == kStages ? phase ^ 1 : phase;
             if (tile + NW < tHi)
                 for (unsigned w = 0; w < (1u << 16) && !mbar_try_wait(bar(nextStage), nextPhase); w++) {}
             break;
         }
         const int k0 = tile * kGdKeys;
-        __nv_bfloat16* K = reinterpret_cast<__nv_bfloat16*>(mine + stage * S.stage);
-        __nv_bfloat16* V = shared ? K : K + kGdKeys * S.LDK;
-        float* sc = reinterpret_cast<float*>(K + kGdKeys * S.LDK);
+        unsigned char* K = mine + stage * S.tile;
+        unsigned char* V = shared ? K : K + S.kb * kGdKeys * 128;
+        float* sc = mySc + stage * kGdKeys;
         if (append && tile == pos / kGdKeys) {               // what was fetched predates the append
-            for (int i = lane; i < a.kw; i += 32) K[(pos - k0) * S.LDK + i] = newK[i];
-            if (shared) { if (lane == 0) sc[pos - k0] = s_newScale; }
-            else { for (int i = lane; i < a.vw; i += 32) V[(pos - k0) * S.LDV + i] = newV[i]; }
+            const int r = pos - k0;
+            for (int i = lane; i < a.kw; i += 32) *reinterpret_cast<__nv_bfloat16*>(K + swizzled(r, i >> 3, kGdKeys) + (i & 7) * 2) = newK[i];
+            if (shared) { if (lane == 0) sc[r] = s_newScale; }
+            else { for (int i = lane; i < a.vw; i += 32) *reinterpret_cast<__nv_bfloat16*>(V + swizzled(r, i >> 3, kGdKeys) + (i & 7) * 2) = newV[i]; }
             fence_proxy_async_smem();
             __syncwarp();
         }
         {
-            const int next = tile + (kGdStages - 1) * NW;
-            if (next < tHi) load(next, stage == 0 ? kGdStages - 1 : stage - 1);
+            const int next = tile + (kStages - 1) * NW;
+            if (next < tHi) load(next, stage == 0 ? kStages - 1 : stage - 1);
         }
         float s[2][4], sl[2][4];                             // by the queries' high and low halves
 #pragma unroll
         for (int j = 0; j < 2; j++)
 #pragma unroll
             for (int e = 0; e < 4; e++) { s[j][e] = 0.0f; sl[j][e] = 0.0f; }
-        const uint32_t kAddr = smem_u32(K) + kLane;
+        const uint32_t kAddr = smem_u32(K);
 #pragma unroll 4
-        for (int kk = 0; kk < S.Dp / 16; kk++) {
+        for (int kk = 0; kk < a.kw / 16; kk++) {
             uint32_t ah[4], al[4], bk[4];
             ldm_x4(ah, qAddr + kk * 32);
             ldm_x4(al, qAddr + qlDelta + kk * 32);
-            ldm_x4(bk, kAddr + kk * 32);
+            ldm_x4(bk, kAddr + swizzled(kRow, kk * 2 + kHalf, kGdKeys));
             mma_bf16(s[0], ah, bk[0], bk[1]); mma_bf16(s[1], ah, bk[2], bk[3]);
             mma_bf16(sl[0], al, bk[0], bk[1]); mma_bf16(sl[1], al, bk[2], bk[3]);
         }
@@ -272,20 +288,20 @@ __global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArg
 #pragma unroll
             for (int c = 0; c < VN; c++) { o[c][0] *= c0; o[c][1] *= c0; o[c][2] *= c1; o[c][3] *= c1; }
         }
-        const uint32_t vAddr = smem_u32(V) + vLane;
+        const uint32_t vAddr = smem_u32(V);
 #pragma unroll
         for (int c = 0; c < VN; c += 4) {
             if (c >= vt) break;
             uint32_t bv[2][4];
             const bool two = c + 2 < vt;                     // value columns come in pairs of tiles
-            ldm_x4_t(bv[0], vAddr + c * 16);
-            ldm_x4_t(bv[1], vAddr + (two ? c + 2 : c) * 16);
+            ldm_x4_t(bv[0], vAddr + swizzled(vRow, c + vHalf, kGdKeys));
+            ldm_x4_t(bv[1], vAddr + swizzled(vRow, (two ? c + 2 : c) + vHalf, kGdKeys));
             mma_bf16(o[c], ph, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], ph, bv[0][2], bv[0][3]);
             if (two) { mma_bf16(o[c + 2], ph, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], ph, bv[1][2], bv[1][3]); }
             mma_bf16(o[c], pl, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], pl, bv[0][2], bv[0][3]);
             if (two) { mma_bf16(o[c + 2], pl, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], pl, bv[1][2], bv[1][3]); }
         }
-        if (++stage == kGdStages) { stage = 0; phase ^= 1; }
+        if (++stage == kStages) { stage = 0; phase ^= 1; }
         __syncwarp();
     }
     l0 = quad_sum(l0); l1 = quad_sum(l1);
@@ -327,78 +343,92 @@ __global__ void __launch_bounds__(32 * NW) k_grouped_decode(const GroupedAttnArg
         if (active > 1 && lane == 0) { dst[Vp] = m; dst[Vp + 1] = l; }
     }
     if (active == 1) return;
-    __threadfence();
     __syncthreads();
     if (tid == 0) {
+        __threadfence();                                     // the block's partials, before its ticket
         int* ticket = a.tickets + blockIdx.z * gridDim.y + blockIdx.y;
         s_last = atomicAdd(ticket, 1) == active - 1;
         if (s_last) *ticket = 0;
+        __threadfence();
     }
     __syncthreads();
     if (!s_last) return;
-    __threadfence();
-    float* wts = mg;                                         // [16][splits]: weight of every part, all over the row's sum
-    for (int r = warp; r < nrow; r += NW) {
-        const float* src = part + (size_t)r * splits * pw + Vp;
-        float* w = wts + r * splits;
-        float m = a.sink ? 0.0f : -INFINITY;
-        for (int s = lane; s < active; s += 32) { w[s] = __ldcg(src + (size_t)s * pw); m = fmaxf(m, w[s]); }
-        for (int o2 = 16; o2 > 0; o2 >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o2));
-        float l = 0.0f;
-        for (int s = lane; s < active; s += 32) { w[s] = ex2(w[s] - m); l = fmaf(w[s], __ldcg(src + (size_t)s * pw + 1), l); }
-        l = warp_sum(l);
-        if (a.sink) l += ex2(-m);
-        const float inv = 1.0f / l;
-        for (int s = lane; s < active; s += 32) w[s] *= inv;
-    }
-    __syncthreads();
-    // a thread: four columns of a row over every `share`-th part; the shares of a column sit in neighbouring lanes
+    // a thread: four columns of a row over every `share`-th part, with a running maximum of its own (maximum, sum and values of a
+    // part travel together); the shares of a column sit in neighbouring lanes
     const int items = nrow * (Vp / 4);
     int share = 1;
     while (share < 8 && items * share * 2 <= 32 * NW) share <<= 1;
     for (int u = tid / share; u < (items + 31) / 32 * 32; u += 32 * NW / share) {
-        const int r = u / (Vp / 4), c = u - r * (Vp / 4), first = tid & (share - 1);
+        const int r = min(u, items - 1) / (Vp / 4), c = min(u, items - 1) % (Vp / 4), first = tid & (share - 1);
+        const float* src = part + (size_t)r * splits * pw;
+        float M = -INFINITY, L = 0.0f;
         float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        if (u < items) {
-            const float4* src = reinterpret_cast<const float4*>(part + (size_t)r * splits * pw) + c;
-            const float* w = wts + r * splits;
-#pragma unroll 8
-            for (int s = first; s < active; s += share) {
-                const float4 p4 = __ldcg(src + (size_t)s * (pw / 4));
-                v.x = fmaf(w[s], p4.x, v.x); v.y = fmaf(w[s], p4.y, v.y); v.z = fmaf(w[s], p4.z, v.z); v.w = fmaf(w[s], p4.w, v.w);
+        constexpr int BATCH = 8;
+        for (int s0 = first; s0 < active; s0 += share * BATCH) {
+            float2 ml[BATCH];
+            float4 x4[BATCH];
+#pragma unroll
+            for (int i = 0; i < BATCH; i++) {
+                const int s = s0 + i * share;
+                ml[i] = make_float2(-INFINITY, 0.0f); x4[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                if (s < active) {
+                    ml[i] = __ldcg(reinterpret_cast<const float2*>(src + (size_t)s * pw + Vp));
+                    x4[i] = __ldcg(reinterpret_cast<const float4*>(src + (size_t)s * pw) + c);
+                }
+            }
+            float top = M;
+#pragma unroll
+            for (int i = 0; i < BATCH; i++) top = fmaxf(top, ml[i].x);
+            const float old = ex2(M - top);                  // the batch's first part is there: top is finite
+            M = top; L *= old; v.x *= old; v.y *= old; v.z *= old; v.w *= old;
+#pragma unroll
+            for (int i = 0; i < BATCH; i++) {
+                const float f = ex2(ml[i].x - top);
+                L = fmaf(f, ml[i].y, L);
+                v.x = fmaf(f, x4[i].x, v.x); v.y = fmaf(f, x4[i].y, v.y); v.z = fmaf(f, x4[i].z, v.z); v.w = fmaf(f, x4[i].w, v.w);
             }
         }
+        float top = M;
+        for (int o2 = 1; o2 < share; o2 <<= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o2));
+        if (a.sink) top = fmaxf(top, 0.0f);
+        const float f = ex2(M - top);                        // a share without parts has M = −∞ and adds nothing
+        L *= f; v.x *= f; v.y *= f; v.z *= f; v.w *= f;
         for (int o2 = 1; o2 < share; o2 <<= 1) {
+            L += __shfl_xor_sync(0xffffffffu, L, o2);
             v.x += __shfl_xor_sync(0xffffffffu, v.x, o2); v.y += __shfl_xor_sync(0xffffffffu, v.y, o2);
             v.z += __shfl_xor_sync(0xffffffffu, v.z, o2); v.w += __shfl_xor_sync(0xffffffffu, v.w, o2);
         }
+        if (a.sink) L += ex2(-top);
         if (u < items && first == 0) {
             float* dst = a.out + (size_t)b * a.ldo + (size_t)(h0 + r) * a.vdim + 4 * c;
-            const float e[4] = {v.x, v.y, v.z, v.w};
+            const float e[4] = {v.x, v.y, v.z, v.w}, inv = 1.0f / L;
 #pragma unroll
             for (int i = 0; i < 4; i++)
-                if (4 * c + i < a.vdim) dst[i] = e[i];
+                if (4 * c + i < a.vdim) dst[i] = e[i] * inv;
         }
     }
 }
 
 size_t gp_smem(const GroupedAttnArgs& a, int keys) {
     const GdShape g = gd_shape(a.kw, a.vw, a.vcache == nullptr, keys);
-    return (size_t)kGpRows * g.LDK * 2 + 2 * (size_t)g.stage;
+    return 1024 + (size_t)kStages * g.tile + (size_t)kGpRows * g.LDQ * 2 + (size_t)kStages * keys * 4;
 }
 
 // VN: most output n-tiles, KEYS: keys per tile
 template <int VN, int KEYS>
-__global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const GroupedAttnArgs a, const __nv_bfloat16* __restrict__ qp, int* error) {
-    extern __shared__ __align__(16) unsigned char gd_raw[];
-    __shared__ __align__(8) unsigned long long s_bar[2];
+__global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const __grid_constant__ GdParams p, const __nv_bfloat16* __restrict__ qp) {
+    extern __shared__ __align__(1024) unsigned char gd_raw[];
+    __shared__ __align__(8) unsigned long long s_bar[2 * kStages];
     __shared__ volatile int s_abort;
     constexpr int NT = KEYS / 8;
+    const GroupedAttnArgs& a = p.a;
     const bool shared = a.vcache == nullptr;
     const GdShape S = gd_shape(a.kw, a.vw, shared, KEYS);
     const int vt = (shared ? a.kw : a.vw) / 8;
-    __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(gd_raw);
-    unsigned char* ring = gd_raw + (size_t)kGpRows * S.LDK * 2;
+    const uint32_t raw = smem_u32(gd_raw), skip = ((raw + 1023u) & ~1023u) - raw;
+    unsigned char* ring = gd_raw + skip;
+    __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(ring + (size_t)kStages * S.tile);        // [kGpRows][LDQ]
+    float* scales = reinterpret_cast<float*>(Qs + kGpRows * S.LDQ);                               // [stage][KEYS]
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, rl = lane >> 2, t4 = lane & 3;
     const int rep = a.H / a.G, rows = a.T * rep, b = blockIdx.y / a.G, g = blockIdx.y - b * a.G;
     const int r0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * kGpRows;         // the rows with the most keys first
@@ -407,68 +437,70 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const Grouped
     const int pos0 = (int)a.pos[b];
     if (pos0 < 0 || pos0 + a.T > a.maxSeq) return;
     const int lastKey = pos0 + (min(rows, r0 + kGpRows) - 1) / rep;
-    const __nv_bfloat16* kc = (const __nv_bfloat16*)a.kcache + (size_t)blockIdx.y * a.maxSeq * a.kw;
-    const __nv_bfloat16* vc = (const __nv_bfloat16*)a.vcache + (size_t)blockIdx.y * a.maxSeq * a.vw;
     const float* ksc = a.kscale + (size_t)blockIdx.y * a.kpitch;
-    const int kq = a.kw / 8;
+    const int kq = a.kw / 8, plane = blockIdx.y * a.maxSeq, tiles = lastKey / KEYS + 1;
+    auto full = [&](int stage) { return smem_u32(&s_bar[stage]); };
+    auto empty = [&](int stage) { return smem_u32(&s_bar[kStages + stage]); };
     if (tid == 0) {
-        mbar_init(smem_u32(&s_bar[0]), 1); mbar_init(smem_u32(&s_bar[1]), 1);
+        for (int i = 0; i < kStages; i++) { mbar_init(full(i), 1); mbar_init(empty(i), kGpThreads / 32); }
         s_abort = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     __syncthreads();
-    // a thread per row; rows past the newest key repeat it: whatever they hold is finite, and masked
-    auto load = [&](int tile, int stage) {
-        const int k0 = tile * KEYS, row = min(k0 + tid % KEYS, lastKey);
-        const uint32_t K = smem_u32(ring + stage * S.stage), bar = smem_u32(&s_bar[stage]);
-        if (tid == 0) mbar_arrive_expect_tx(bar, (uint32_t)(KEYS * 2 * (a.kw + (shared ? 2 : a.vw))));
-        if (tid < KEYS) bulk_g2s(K + (uint32_t)(tid * S.LDK * 2), kc + (size_t)row * a.kw, (uint32_t)(a.kw * 2), bar);
-        else if (tid < 2 * KEYS) {
-            if (!shared) bulk_g2s(K + (uint32_t)((KEYS * S.LDK + (tid - KEYS) * S.LDV) * 2), vc + (size_t)row * a.vw, (uint32_t)(a.vw * 2), bar);
-            else if (tid == KEYS) bulk_g2s(K + (uint32_t)(KEYS * S.LDK * 2), ksc + k0, KEYS * 4, bar);
-        }
+    // by one thread; rows past the newest key are whatever earlier requests left: finite, and masked
+    auto load = [&](int tile) {
+        const int k0 = tile * KEYS, stage = tile % kStages;
+        uint32_t dst = smem_u32(ring + stage * S.tile);
+        mbar_arrive_expect_tx(full(stage), (uint32_t)(S.tile + (shared ? KEYS * 4 : 0)));
+        for (int c = 0; c < S.kb; c++, dst += KEYS * 128) tma_box(dst, &p.k, c * 64, plane + k0, full(stage));
+        for (int c = 0; c < S.vb; c++, dst += KEYS * 128) tma_box(dst, &p.v, c * 64, plane + k0, full(stage));
+        if (shared) bulk_g2s(smem_u32(scales + stage * KEYS), ksc + k0, KEYS * 4, full(stage));
     };
-    load(0, 0);
+    int issued = 0;
+    if (tid == 0)
+        for (; issued < min(kStages - 1, tiles); issued++) load(issued);
     const __nv_bfloat16* q0 = qp + ((size_t)blockIdx.y * rows + r0) * a.kw;
     for (int i = tid; i < kGpRows * kq; i += kGpThreads) {
         const int r = i / kq, c = i - r * kq;
-        *reinterpret_cast<uint4*>(Qs + r * S.LDK + c * 8) =
+        *reinterpret_cast<uint4*>(Qs + r * S.LDQ + c * 8) =
             r0 + r < rows ? *reinterpret_cast<const uint4*>(q0 + (size_t)r * a.kw + c * 8) : make_uint4(0, 0, 0, 0);
     }
+    __syncthreads();
     const int w0 = r0 + warp * 16, ra = w0 + rl, rb = ra + 8;
     const int limA = ra < rows ? pos0 + ra / rep : -1, limB = rb < rows ? pos0 + rb / rep : -1;      // newest key of a row
     const int warpLast = w0 < rows ? pos0 + (min(rows, w0 + 16) - 1) / rep : -1, warpFirst = pos0 + w0 / rep;
     const float* relA = a.rel ? a.rel + (size_t)(g * rep + ra % rep) * a.relLen : nullptr;
     const float* relB = a.rel ? a.rel + (size_t)(g * rep + rb % rep) * a.relLen : nullptr;
     const float farA = a.rel ? bias_at(relA, a.relLen - 1, a.relLen) : 0.0f, farB = a.rel ? bias_at(relB, a.relLen - 1, a.relLen) : 0.0f;
-    const uint32_t qAddr = smem_u32(Qs) + (uint32_t)(((warp * 16 + (lane & 15)) * S.LDK + (lane >> 4) * 8) * 2);
-    const uint32_t kLane = (uint32_t)((((lane & 7) + ((lane >> 4) << 3)) * S.LDK + ((lane >> 3) & 1) * 8) * 2);
-    const int ldv = shared ? S.LDK : S.LDV;
-    const uint32_t vLane = (uint32_t)((((lane & 7) + (((lane >> 3) & 1) << 3)) * ldv + (lane >> 4) * 8) * 2);
+    const uint32_t qAddr = smem_u32(Qs) + (uint32_t)(((warp * 16 + (lane & 15)) * S.LDQ + (lane >> 4) * 8) * 2);
+    const int kRow = (lane & 7) + ((lane >> 4) << 3), kHalf = (lane >> 3) & 1;       // operand B from rows of keys
+    const int vRow = (lane & 7) + (((lane >> 3) & 1) << 3), vHalf = lane >> 4;       // … read transposed
     float o[VN][4];
 #pragma unroll
     for (int j = 0; j < VN; j++) { o[j][0] = 0.0f; o[j][1] = 0.0f; o[j][2] = 0.0f; o[j][3] = 0.0f; }
     float mA = -INFINITY, mB = -INFINITY, lA = 0.0f, lB = 0.0f;
-    const int tiles = lastKey / KEYS + 1;
     for (int tile = 0; tile < tiles; tile++) {
-        // this tile has landed, nobody reads the other stage any more
-        if (!__syncthreads_and(mbar_wait(smem_u32(&s_bar[tile & 1]), (tile >> 1) & 1, &s_abort, error, 222))) break;
-        if (tile + 1 < tiles) load(tile + 1, (tile + 1) & 1);
-        const int k0 = tile * KEYS;
-        if (k0 > warpLast) continue;
-        const __nv_bfloat16* K = reinterpret_cast<const __nv_bfloat16*>(ring + (tile & 1) * S.stage);
-        const float* sc = reinterpret_cast<const float*>(K + KEYS * S.LDK);
+        const int stage = tile % kStages, k0 = tile * KEYS;
+        if (tid == 0 && issued < tiles) {                    // the tile two ahead goes where the last one was
+            if (issued < kStages || mbar_wait(empty(issued % kStages), (issued / kStages - 1) & 1, &s_abort, p.error, 223)) load(issued++);
+        }
+        __syncwarp();
+        if (!__all_sync(0xffffffffu, mbar_wait(full(stage), (tile / kStages) & 1, &s_abort, p.error, 222))) break;
+        auto release = [&] { __syncwarp(); if (lane == 0) mbar_arrive(empty(stage)); };
+        if (k0 > warpLast) { release(); continue; }
+        const unsigned char* K = ring + stage * S.tile;
+        const float* sc = scales + stage * KEYS;
         float s[NT][4];
 #pragma unroll
         for (int j = 0; j < NT; j++) { s[j][0] = 0.0f; s[j][1] = 0.0f; s[j][2] = 0.0f; s[j][3] = 0.0f; }
-        const uint32_t kAddr = smem_u32(K) + kLane;
-        for (int kk = 0; kk < S.Dp / 16; kk++) {
+        const uint32_t kAddr = smem_u32(K);
+        for (int kk = 0; kk < a.kw / 16; kk++) {
             uint32_t aq[4];
             ldm_x4(aq, qAddr + kk * 32);
 #pragma unroll
             for (int n = 0; n < NT; n += 2) {
                 uint32_t bk[4];
-                ldm_x4(bk, kAddr + (uint32_t)(n * 8 * S.LDK * 2) + kk * 32);
+                ldm_x4(bk, kAddr + (uint32_t)(n * 8 * 128) + swizzled(kRow, kk * 2 + kHalf, KEYS));
                 mma_bf16(s[n], aq, bk[0], bk[1]); mma_bf16(s[n + 1], aq, bk[2], bk[3]);
             }
         }
@@ -516,7 +548,7 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const Grouped
 #pragma unroll
             for (int c = 0; c < VN; c++) { o[c][0] *= cA; o[c][1] *= cA; o[c][2] *= cB; o[c][3] *= cB; }
         }
-        const uint32_t vAddr = smem_u32(shared ? K : K + KEYS * S.LDK) + vLane;
+        const uint32_t vAddr = smem_u32(shared ? K : K + S.kb * KEYS * 128);
 #pragma unroll
         for (int kk = 0; kk < KEYS / 16; kk++) {
             uint32_t ph[4], pl[4];
@@ -527,16 +559,20 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const Grouped
                 if (c >= vt) break;
                 uint32_t bv[2][4];
                 const bool two = c + 2 < vt;                 // value columns come in pairs of tiles
-                const uint32_t at = vAddr + (uint32_t)(kk * 16 * ldv * 2);
-                ldm_x4_t(bv[0], at + c * 16);
-                ldm_x4_t(bv[1], at + (two ? c + 2 : c) * 16);
+                const uint32_t at = vAddr + (uint32_t)(kk * 16 * 128);
+                ldm_x4_t(bv[0], at + swizzled(vRow, c + vHalf, KEYS));
+                ldm_x4_t(bv[1], at + swizzled(vRow, (two ? c + 2 : c) + vHalf, KEYS));
                 mma_bf16(o[c], ph, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], ph, bv[0][2], bv[0][3]);
                 if (two) { mma_bf16(o[c + 2], ph, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], ph, bv[1][2], bv[1][3]); }
                 mma_bf16(o[c], pl, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], pl, bv[0][2], bv[0][3]);
                 if (two) { mma_bf16(o[c + 2], pl, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], pl, bv[1][2], bv[1][3]); }
             }
         }
+        release();
     }
+    if (tid == 0 && s_abort)                                 // a wait ran out: let the copies in flight land before the block goes
+        for (int t = max(0, issued - kStages); t < issued; t++)
+            for (unsigned w = 0; w < (1u << 16) && !mbar_try_wait(full(t % kStages), (t / kStages) & 1); w++) {}
     lA = quad_sum(lA); lB = quad_sum(lB);
     auto finish = [&](int r, float m, float l, int e) {
         if (r >= rows) return;
@@ -567,12 +603,31 @@ void raise(K kernel, bool& done) {
 }
 // warps of a decode block: eight where their rings fit
 int gd_warps(const GroupedAttnArgs& a) { return gd_smem(a, 8) <= kSmemMax ? 8 : 4; }
+bool cache_map(CUtensorMap* map, const void* base, int width, size_t rows, int keys) {
+    EncodeTiledFn enc = encode_tiled_fn();
+    if (enc == nullptr) return false;
+    const cuuint64_t dims[2] = {(cuuint64_t)width, (cuuint64_t)rows};
+    const cuuint64_t strides[1] = {(cuuint64_t)width * 2};
+    const cuuint32_t box[2] = {64u, (cuuint32_t)keys};
+    const cuuint32_t estr[2] = {1u, 1u};
+    return enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
+               CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+GdParams params(const GroupedAttnArgs& a, int keys, int splits) {
+    GdParams p = {};
+    p.a = a; p.splits = splits; p.error = g_dev_error;
+    const size_t rows = (size_t)a.B * a.G * a.maxSeq;
+    if (!cache_map(&p.k, a.kcache, a.kw, rows, keys) || (a.vcache && !cache_map(&p.v, a.vcache, a.vw, rows, keys)))
+        throw std::runtime_error("grouped attention: the cache cannot be described to the copy engine");
+    return p;
+}
 template <int VN, int NW>
 void decode_with(const GroupedAttnArgs& a, cudaStream_t s) {
     static bool done = false;
     raise(k_grouped_decode<VN, NW>, done);
     const int splits = grouped_mma_splits(a);
-    launch_k(k_grouped_decode<VN, NW>, dim3((unsigned)splits, (unsigned)((a.H / a.G + 15) / 16), (unsigned)(a.B * a.G)), dim3(32 * NW), gd_smem(a, NW), s, true, a, splits, g_dev_error);
+    launch_k(k_grouped_decode<VN, NW>, dim3((unsigned)splits, (unsigned)((a.H / a.G + 15) / 16), (unsigned)(a.B * a.G)), dim3(32 * NW), gd_smem(a, NW), s, true,
+             params(a, kGdKeys, splits));
 }
 template <int VN>
 void decode(const GroupedAttnArgs& a, cudaStream_t s) {
@@ -584,18 +639,19 @@ void prefill(const GroupedAttnArgs& a, const __nv_bfloat16* q, cudaStream_t s) {
     static bool done = false;
     raise(k_grouped_prefill<VN, KEYS>, done);
     const unsigned blocks = (unsigned)((a.T * (a.H / a.G) + kGpRows - 1) / kGpRows);
-    launch_k(k_grouped_prefill<VN, KEYS>, dim3(blocks, (unsigned)(a.B * a.G)), dim3(kGpThreads), gp_smem(a, KEYS), s, true, a, q, g_dev_error);
+    launch_k(k_grouped_prefill<VN, KEYS>, dim3(blocks, (unsigned)(a.B * a.G)), dim3(kGpThreads), gp_smem(a, KEYS), s, true, params(a, KEYS, 1), q);
 }
 
 }  // namespace
 
 bool grouped_mma_fits(const GroupedAttnArgs& a) {
-    return a.bf16 && a.kw <= 256 && a.vw <= 256 && a.kw % 16 == 0 && a.vw % 16 == 0 && (a.vcache != nullptr || a.kpitch % 64 == 0);
+    return a.bf16 && (size_t)a.B * a.G * a.maxSeq < (1u << 31) && a.kw <= 256 && a.vw <= 256 && a.kw % 16 == 0 && a.vw % 16 == 0 && (a.vcache != nullptr || a.kpitch % 64 == 0);
 }
 int grouped_mma_splits(const GroupedAttnArgs& a) {
     const int blocks = a.B * a.G * ((a.H / a.G + 15) / 16), tiles = (a.maxSeq + kGdKeys - 1) / kGdKeys, warps = gd_warps(a);
-    const int perSm = std::max(1, (int)(kSmemMax / gd_smem(a, warps)));
-    return std::max(1, std::min({std::min(perSm, 16 / warps) * g_num_sms / blocks, (tiles + warps - 1) / warps, 512}));
+    // two blocks of the narrow form fit the registers of an SM
+    const int perSm = std::max(a.kw, a.vcache ? a.vw : a.kw) <= 128 && (a.vcache ? a.vw : a.kw) <= 64 ? std::min(2, std::max(1, (int)(kSmemMax / gd_smem(a, warps)))) : 1;
+    return std::max(1, std::min({perSm * g_num_sms / blocks, (tiles + warps - 1) / warps, 512}));
 }
 void launch_grouped_decode(const GroupedAttnArgs& a, cudaStream_t s) {
     const int vw = a.vcache ? a.vw : a.kw;
