@@ -2,7 +2,7 @@
 //
 //   k_grouped_decode    one token per sequence.  grid (key splits, blocks of 16 query heads of a group, B·G): the heads of a group
 //                       are the rows of one 16-row operand, so a cached row is read once per group.  Eight (or four) warps walk tiles
-//                       of 16 keys, each through a private three-stage ring of tensor copies that starts before the dependency wait; the
+//                       of 16 keys, each through a private ring of tensor copies, as deep as shared memory allows, that starts before the dependency wait; the
 //                       block that holds the newest position norms and appends it.  Queries enter as two bf16 halves.  Warps merge
 //                       in shared memory, blocks through partials that the last one to finish (a ticket) adds up.
 //   k_grouped_prefill   prompt chunks: 128 rows (token, head in the group) per block, 16 per warp, key tiles in three stages.
@@ -18,7 +18,7 @@ namespace dj {
 namespace {
 
 constexpr float kLog2e = 1.4426950408889634f;
-constexpr int kGdKeys = 16, kStages = 3, kAlone = 4;
+constexpr int kGdKeys = 16, kGpStages = 3, kGdMaxStages = 8, kAlone = 4;
 constexpr int kGpRows = 128, kGpThreads = 256;
 
 __device__ __forceinline__ float ex2(float x) {
@@ -45,7 +45,7 @@ __device__ __forceinline__ float bias_at(const float* rel, int d, int len) { ret
 struct GdParams {
     GroupedAttnArgs a;
     CUtensorMap k, v;                                        // rows of 64 columns × a tile's keys
-    int splits; int* error;
+    int splits, stages; int* error;
 };
 
 // Shared memory: tiles (1024-byte aligned), then queries, the new row, the norms of cached keys.
@@ -59,38 +59,40 @@ __host__ __device__ __forceinline__ GdShape gd_shape(int kw, int vw, bool shared
 // Byte offset of 16-byte column c of row r in a tile of boxes: the copy engine swaps the columns of a 128-byte row by its number.
 __device__ __forceinline__ uint32_t swizzled(int r, int c, int keys) { return (uint32_t)((c >> 3) * keys * 128 + r * 128 + (((c & 7) ^ (r & 7)) << 4)); }
 
-size_t gd_smem(const GroupedAttnArgs& a, int warps) {
+size_t gd_smem(const GroupedAttnArgs& a, int warps, int stages) {
     const bool shared = a.vcache == nullptr;
     const GdShape g = gd_shape(a.kw, a.vw, shared, kGdKeys);
-    const size_t ring = (size_t)warps * kStages * g.tile, merge = (size_t)warps * 16 * ((shared ? a.kw : a.vw) + 4) * 4;
-    return 1024 + std::max(ring, merge) + (size_t)2 * 16 * g.LDQ * 2 + (size_t)(a.kw + a.vw + 16) * 2 + (size_t)warps * kStages * kGdKeys * 4;
+    const size_t ring = (size_t)warps * stages * g.tile, merge = (size_t)warps * 16 * ((shared ? a.kw : a.vw) + 4) * 4;
+    return 1024 + std::max(ring, merge) + (size_t)2 * 16 * g.LDQ * 2 + (size_t)(a.kw + a.vw + 16) * 2 + (size_t)warps * stages * kGdKeys * 4;
 }
 
 // VN: most output n-tiles (eight value columns each), NW: warps
 template <int VN, int NW>
 __global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(const __grid_constant__ GdParams p) {
     extern __shared__ __align__(1024) unsigned char gd_raw[];
-    __shared__ __align__(8) unsigned long long s_bar[NW * kStages];
+    __shared__ __align__(8) unsigned long long s_bar[NW * kGdMaxStages];
     __shared__ float s_newScale;
     __shared__ volatile int s_abort;
     __shared__ int s_last;
     const GroupedAttnArgs& a = p.a;
-    const int splits = p.splits;
+    const int splits = p.splits, stages = p.stages;
     const bool shared = a.vcache == nullptr;
     const GdShape S = gd_shape(a.kw, a.vw, shared, kGdKeys);
     const int Vp = shared ? a.kw : a.vw, vt = Vp / 8;
     const uint32_t raw = smem_u32(gd_raw), skip = ((raw + 1023u) & ~1023u) - raw;
     unsigned char* ring = gd_raw + skip;
-    const size_t ringBytes = max((size_t)NW * kStages * S.tile, (size_t)NW * 16 * (Vp + 4) * 4);
+    const size_t ringBytes = max((size_t)NW * stages * S.tile, (size_t)NW * 16 * (Vp + 4) * 4);
     __nv_bfloat16* Qh = reinterpret_cast<__nv_bfloat16*>(ring + ringBytes);          // [16][LDQ], then the low halves
     float* scales = reinterpret_cast<float*>(Qh + 2 * 16 * S.LDQ);                   // [warp][stage][16]
-    __nv_bfloat16* newK = reinterpret_cast<__nv_bfloat16*>(scales + NW * kStages * kGdKeys);
+    __nv_bfloat16* newK = reinterpret_cast<__nv_bfloat16*>(scales + NW * stages * kGdKeys);
     __nv_bfloat16* newV = newK + a.kw;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, rl = lane >> 2, t4 = lane & 3;
-    unsigned char* mine = ring + warp * kStages * S.tile;
-    float* mySc = scales + warp * kStages * kGdKeys;
+    unsigned char* mine = ring + warp * stages * S.tile;
+    float* mySc = scales + warp * stages * kGdKeys;
     const int rep = a.H / a.G, b = blockIdx.z / a.G, g = blockIdx.z - b * a.G, h0 = g * rep + blockIdx.y * 16, nrow = min(16, rep - (int)blockIdx.y * 16);
-    if (!a.early) { pdl_wait(); pdl_launch_dependents(); }
+    // The next kernel is not let in early (griddepcontrol.launch_dependents): short contexts keep some SMs busy, and a projection
+    // whose blocks all go to the others streams its weights through those alone.
+    if (!a.early) pdl_wait();
     const int pos = (int)a.pos[b];
     const bool valid = pos >= 0 && pos < a.maxSeq;
     // a few tiles per warp cost less than adding up the parts of several blocks
@@ -98,9 +100,9 @@ __global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(con
     const int tLo = blockIdx.x * per, tHi = min(tiles, tLo + per);
     const float* ksc = a.kscale + (size_t)blockIdx.z * a.kpitch;
     const int plane = blockIdx.z * a.maxSeq;                 // first row of this head's keys and values
-    auto bar = [&](int stage) { return smem_u32(&s_bar[warp * kStages + stage]); };
+    auto bar = [&](int stage) { return smem_u32(&s_bar[warp * kGdMaxStages + stage]); };
     if (lane == 0) {
-        for (int i = 0; i < kStages; i++) mbar_init(bar(i), 1);
+        for (int i = 0; i < stages; i++) mbar_init(bar(i), 1);
         if (warp == 0) s_abort = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -115,10 +117,9 @@ __global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(con
         for (int c = 0; c < S.vb; c++, dst += kGdKeys * 128) tma_box(dst, &p.v, c * 64, plane + k0, bar(stage));
         if (shared) bulk_g2s(smem_u32(mySc + stage * kGdKeys), ksc + k0, kGdKeys * 4, bar(stage));      // kpitch covers whole tiles
     };
-#pragma unroll
-    for (int i = 0; i < kStages - 1; i++)
+    for (int i = 0; i < stages - 1; i++)
         if (tLo + warp + i * NW < tHi) load(tLo + warp + i * NW, i);
-    if (a.early) { pdl_wait(); pdl_launch_dependents(); }
+    if (a.early) pdl_wait();
     if (tLo >= tHi) return;
 
     // A warp norms query rows warp, warp + NW, …; the warp after those with a first row norms the new key.  Rows are loaded to
@@ -200,11 +201,12 @@ __global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(con
     int stage = 0, phase = 0;
     for (int tile = tLo + warp; tile < tHi; tile += NW) {
         if (!__all_sync(0xffffffffu, mbar_wait(bar(stage), phase, &s_abort, p.error, 221))) {
-            // let the copies in flight land before the block goes: this tile's and the next one's
+            // let the copies in flight land before the block goes
             for (unsigned w = 0; w < (1u << 16) && !mbar_try_wait(bar(stage), phase); w++) {}
-            const int nextStage = stage + 1 == kStages ? 0 : stage + 1, nextPhase = stage + 1 == kStages ? phase ^ 1 : phase;
-            if (tile + NW < tHi)
-                for (unsigned w = 0; w < (1u << 16) && !mbar_try_wait(bar(nextStage), nextPhase); w++) {}
+            for (int t = tile + NW, k = 1; t < tHi && k < stages - 1; t += NW, k++) {
+                const int st = (stage + k) % stages, ph = stage + k >= stages ? phase ^ 1 : phase;
+                for (unsigned w = 0; w < (1u << 16) && !mbar_try_wait(bar(st), ph); w++) {}
+            }
             break;
         }
         const int k0 = tile * kGdKeys;
@@ -220,8 +222,8 @@ __global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(con
             __syncwarp();
         }
         {
-            const int next = tile + (kStages - 1) * NW;
-            if (next < tHi) load(next, stage == 0 ? kStages - 1 : stage - 1);
+            const int next = tile + (stages - 1) * NW;
+            if (next < tHi) load(next, stage == 0 ? stages - 1 : stage - 1);
         }
         float s[2][4], sl[2][4];                             // by the queries' high and low halves
 #pragma unroll
@@ -301,7 +303,7 @@ __global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(con
             mma_bf16(o[c], pl, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], pl, bv[0][2], bv[0][3]);
             if (two) { mma_bf16(o[c + 2], pl, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], pl, bv[1][2], bv[1][3]); }
         }
-        if (++stage == kStages) { stage = 0; phase ^= 1; }
+        if (++stage == stages) { stage = 0; phase ^= 1; }
         __syncwarp();
     }
     l0 = quad_sum(l0); l1 = quad_sum(l1);
@@ -411,14 +413,14 @@ __global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(con
 
 size_t gp_smem(const GroupedAttnArgs& a, int keys) {
     const GdShape g = gd_shape(a.kw, a.vw, a.vcache == nullptr, keys);
-    return 1024 + (size_t)kStages * g.tile + (size_t)kGpRows * g.LDQ * 2 + (size_t)kStages * keys * 4;
+    return 1024 + (size_t)kGpStages * g.tile + (size_t)kGpRows * g.LDQ * 2 + (size_t)kGpStages * keys * 4;
 }
 
 // VN: most output n-tiles, KEYS: keys per tile
 template <int VN, int KEYS>
 __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const __grid_constant__ GdParams p, const __nv_bfloat16* __restrict__ qp) {
     extern __shared__ __align__(1024) unsigned char gd_raw[];
-    __shared__ __align__(8) unsigned long long s_bar[2 * kStages];
+    __shared__ __align__(8) unsigned long long s_bar[2 * kGpStages];
     __shared__ volatile int s_abort;
     constexpr int NT = KEYS / 8;
     const GroupedAttnArgs& a = p.a;
@@ -427,7 +429,7 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const __grid_
     const int vt = (shared ? a.kw : a.vw) / 8;
     const uint32_t raw = smem_u32(gd_raw), skip = ((raw + 1023u) & ~1023u) - raw;
     unsigned char* ring = gd_raw + skip;
-    __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(ring + (size_t)kStages * S.tile);        // [kGpRows][LDQ]
+    __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(ring + (size_t)kGpStages * S.tile);        // [kGpRows][LDQ]
     float* scales = reinterpret_cast<float*>(Qs + kGpRows * S.LDQ);                               // [stage][KEYS]
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, rl = lane >> 2, t4 = lane & 3;
     const int rep = a.H / a.G, rows = a.T * rep, b = blockIdx.y / a.G, g = blockIdx.y - b * a.G;
@@ -440,16 +442,16 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const __grid_
     const float* ksc = a.kscale + (size_t)blockIdx.y * a.kpitch;
     const int kq = a.kw / 8, plane = blockIdx.y * a.maxSeq, tiles = lastKey / KEYS + 1;
     auto full = [&](int stage) { return smem_u32(&s_bar[stage]); };
-    auto empty = [&](int stage) { return smem_u32(&s_bar[kStages + stage]); };
+    auto empty = [&](int stage) { return smem_u32(&s_bar[kGpStages + stage]); };
     if (tid == 0) {
-        for (int i = 0; i < kStages; i++) { mbar_init(full(i), 1); mbar_init(empty(i), kGpThreads / 32); }
+        for (int i = 0; i < kGpStages; i++) { mbar_init(full(i), 1); mbar_init(empty(i), kGpThreads / 32); }
         s_abort = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     __syncthreads();
     // by one thread; rows past the newest key are whatever earlier requests left: finite, and masked
     auto load = [&](int tile) {
-        const int k0 = tile * KEYS, stage = tile % kStages;
+        const int k0 = tile * KEYS, stage = tile % kGpStages;
         uint32_t dst = smem_u32(ring + stage * S.tile);
         mbar_arrive_expect_tx(full(stage), (uint32_t)(S.tile + (shared ? KEYS * 4 : 0)));
         for (int c = 0; c < S.kb; c++, dst += KEYS * 128) tma_box(dst, &p.k, c * 64, plane + k0, full(stage));
@@ -458,7 +460,7 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const __grid_
     };
     int issued = 0;
     if (tid == 0)
-        for (; issued < min(kStages - 1, tiles); issued++) load(issued);
+        for (; issued < min(kGpStages - 1, tiles); issued++) load(issued);
     const __nv_bfloat16* q0 = qp + ((size_t)blockIdx.y * rows + r0) * a.kw;
     for (int i = tid; i < kGpRows * kq; i += kGpThreads) {
         const int r = i / kq, c = i - r * kq;
@@ -480,12 +482,12 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const __grid_
     for (int j = 0; j < VN; j++) { o[j][0] = 0.0f; o[j][1] = 0.0f; o[j][2] = 0.0f; o[j][3] = 0.0f; }
     float mA = -INFINITY, mB = -INFINITY, lA = 0.0f, lB = 0.0f;
     for (int tile = 0; tile < tiles; tile++) {
-        const int stage = tile % kStages, k0 = tile * KEYS;
+        const int stage = tile % kGpStages, k0 = tile * KEYS;
         if (tid == 0 && issued < tiles) {                    // the tile two ahead goes where the last one was
-            if (issued < kStages || mbar_wait(empty(issued % kStages), (issued / kStages - 1) & 1, &s_abort, p.error, 223)) load(issued++);
+            if (issued < kGpStages || mbar_wait(empty(issued % kGpStages), (issued / kGpStages - 1) & 1, &s_abort, p.error, 223)) load(issued++);
         }
         __syncwarp();
-        if (!__all_sync(0xffffffffu, mbar_wait(full(stage), (tile / kStages) & 1, &s_abort, p.error, 222))) break;
+        if (!__all_sync(0xffffffffu, mbar_wait(full(stage), (tile / kGpStages) & 1, &s_abort, p.error, 222))) break;
         auto release = [&] { __syncwarp(); if (lane == 0) mbar_arrive(empty(stage)); };
         if (k0 > warpLast) { release(); continue; }
         const unsigned char* K = ring + stage * S.tile;
@@ -571,8 +573,8 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const __grid_
         release();
     }
     if (tid == 0 && s_abort)                                 // a wait ran out: let the copies in flight land before the block goes
-        for (int t = max(0, issued - kStages); t < issued; t++)
-            for (unsigned w = 0; w < (1u << 16) && !mbar_try_wait(full(t % kStages), (t / kStages) & 1); w++) {}
+        for (int t = max(0, issued - kGpStages); t < issued; t++)
+            for (unsigned w = 0; w < (1u << 16) && !mbar_try_wait(full(t % kGpStages), (t / kGpStages) & 1); w++) {}
     lA = quad_sum(lA); lB = quad_sum(lB);
     auto finish = [&](int r, float m, float l, int e) {
         if (r >= rows) return;
@@ -601,8 +603,6 @@ void raise(K kernel, bool& done) {
     if (!done) DJ_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax));
     done = true;
 }
-// warps of a decode block: eight where their rings fit
-int gd_warps(const GroupedAttnArgs& a) { return gd_smem(a, 8) <= kSmemMax ? 8 : 4; }
 bool cache_map(CUtensorMap* map, const void* base, int width, size_t rows, int keys) {
     EncodeTiledFn enc = encode_tiled_fn();
     if (enc == nullptr) return false;
@@ -613,21 +613,34 @@ bool cache_map(CUtensorMap* map, const void* base, int width, size_t rows, int k
     return enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
                CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
-GdParams params(const GroupedAttnArgs& a, int keys, int splits) {
+GdParams params(const GroupedAttnArgs& a, int keys) {
     GdParams p = {};
-    p.a = a; p.splits = splits; p.error = g_dev_error;
+    p.a = a; p.error = g_dev_error;
     const size_t rows = (size_t)a.B * a.G * a.maxSeq;
     if (!cache_map(&p.k, a.kcache, a.kw, rows, keys) || (a.vcache && !cache_map(&p.v, a.vcache, a.vw, rows, keys)))
         throw std::runtime_error("grouped attention: the cache cannot be described to the copy engine");
     return p;
 }
+// warps of a decode block: eight where two stages of their rings fit; blocks per SM as the registers of its form allow
+int gd_warps(const GroupedAttnArgs& a) { return gd_smem(a, 8, 2) <= kSmemMax ? 8 : 4; }
+int gd_blocks_per_sm(const GroupedAttnArgs& a) {
+    const int vw = a.vcache ? a.vw : a.kw;
+    return vw <= 64 && a.kw <= 128 && 2 * gd_smem(a, gd_warps(a), 3) <= kSmemMax ? 2 : 1;
+}
+int gd_stages(const GroupedAttnArgs& a) {
+    const int warps = gd_warps(a);
+    const size_t room = kSmemMax / gd_blocks_per_sm(a);
+    int n = kGdMaxStages;
+    while (n > 2 && gd_smem(a, warps, n) > room) n--;
+    return n;
+}
 template <int VN, int NW>
 void decode_with(const GroupedAttnArgs& a, cudaStream_t s) {
     static bool done = false;
     raise(k_grouped_decode<VN, NW>, done);
-    const int splits = grouped_mma_splits(a);
-    launch_k(k_grouped_decode<VN, NW>, dim3((unsigned)splits, (unsigned)((a.H / a.G + 15) / 16), (unsigned)(a.B * a.G)), dim3(32 * NW), gd_smem(a, NW), s, true,
-             params(a, kGdKeys, splits));
+    GdParams p = params(a, kGdKeys);
+    p.splits = grouped_mma_splits(a); p.stages = gd_stages(a);
+    launch_k(k_grouped_decode<VN, NW>, dim3((unsigned)p.splits, (unsigned)((a.H / a.G + 15) / 16), (unsigned)(a.B * a.G)), dim3(32 * NW), gd_smem(a, NW, p.stages), s, true, p);
 }
 template <int VN>
 void decode(const GroupedAttnArgs& a, cudaStream_t s) {
@@ -639,7 +652,7 @@ void prefill(const GroupedAttnArgs& a, const __nv_bfloat16* q, cudaStream_t s) {
     static bool done = false;
     raise(k_grouped_prefill<VN, KEYS>, done);
     const unsigned blocks = (unsigned)((a.T * (a.H / a.G) + kGpRows - 1) / kGpRows);
-    launch_k(k_grouped_prefill<VN, KEYS>, dim3(blocks, (unsigned)(a.B * a.G)), dim3(kGpThreads), gp_smem(a, KEYS), s, true, params(a, KEYS, 1), q);
+    launch_k(k_grouped_prefill<VN, KEYS>, dim3(blocks, (unsigned)(a.B * a.G)), dim3(kGpThreads), gp_smem(a, KEYS), s, true, params(a, KEYS), q);
 }
 
 }  // namespace
@@ -649,9 +662,7 @@ bool grouped_mma_fits(const GroupedAttnArgs& a) {
 }
 int grouped_mma_splits(const GroupedAttnArgs& a) {
     const int blocks = a.B * a.G * ((a.H / a.G + 15) / 16), tiles = (a.maxSeq + kGdKeys - 1) / kGdKeys, warps = gd_warps(a);
-    // two blocks of the narrow form fit the registers of an SM
-    const int perSm = std::max(a.kw, a.vcache ? a.vw : a.kw) <= 128 && (a.vcache ? a.vw : a.kw) <= 64 ? std::min(2, std::max(1, (int)(kSmemMax / gd_smem(a, warps)))) : 1;
-    return std::max(1, std::min({perSm * g_num_sms / blocks, (tiles + warps - 1) / warps, 512}));
+    return std::max(1, std::min({gd_blocks_per_sm(a) * g_num_sms / blocks, (tiles + warps - 1) / warps, 512}));
 }
 void launch_grouped_decode(const GroupedAttnArgs& a, cudaStream_t s) {
     const int vw = a.vcache ? a.vw : a.kw;
