@@ -53,10 +53,11 @@ struct GdShape { int kb, vb, tile, LDQ; };                   // boxes of a key a
 __host__ __device__ __forceinline__ GdShape gd_shape(int kw, int vw, bool shared, int keys) {
     GdShape g;
     g.kb = (kw + 63) / 64; g.vb = shared ? 0 : (vw + 63) / 64;
-    g.tile = (g.kb + g.vb) * keys * 128; g.LDQ = kw + 8;
+    g.tile = (g.kb + g.vb) * keys * 128; g.LDQ = g.kb * 64 + 8;
     return g;
 }
 // Byte offset of 16-byte column c of row r in a tile of boxes: the copy engine swaps the columns of a 128-byte row by its number.
+// Columns past a row's width hold zeros, in the boxes and in the query rows.
 __device__ __forceinline__ uint32_t swizzled(int r, int c, int keys) { return (uint32_t)((c >> 3) * keys * 128 + r * 128 + (((c & 7) ^ (r & 7)) << 4)); }
 
 size_t gd_smem(const GroupedAttnArgs& a, int warps, int stages) {
@@ -174,7 +175,7 @@ __global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(con
 #pragma unroll
         for (int e = 0; e < NE; e++) {
             const int i = e * 32 + lane;
-            if (i >= a.kw) break;
+            if (i >= S.kb * 64) break;
             float v = (q[e] * inv) * w[e] * qf;
             if (shared) v *= kg[e];
             const __nv_bfloat16 hi = __float2bfloat16_rn(v);
@@ -189,8 +190,12 @@ __global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(con
     __syncthreads();
 
     const uint32_t qAddr = smem_u32(Qh) + (uint32_t)(((lane & 15) * S.LDQ + (lane >> 4) * 8) * 2), qlDelta = (uint32_t)(16 * S.LDQ * 2);
-    const int kRow = (lane & 7) + ((lane >> 4) << 3), kHalf = (lane >> 3) & 1;       // operand B from rows of keys
-    const int vRow = (lane & 7) + (((lane >> 3) & 1) << 3), vHalf = lane >> 4;       // … read transposed
+    uint32_t kOff[4], vOff[4];                               // operand B, columns 16i of a box: from rows of keys, and read transposed
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        kOff[i] = swizzled((lane & 7) + ((lane >> 4) << 3), 2 * i + ((lane >> 3) & 1), 0);
+        vOff[i] = swizzled((lane & 7) + (((lane >> 3) & 1) << 3), 2 * i + (lane >> 4), 0);
+    }
     const float* rel0 = a.rel ? a.rel + (size_t)(h0 + min(rl, nrow - 1)) * a.relLen : nullptr;
     const float* rel1 = a.rel ? a.rel + (size_t)(h0 + min(rl + 8, nrow - 1)) * a.relLen : nullptr;
     const float far0 = a.rel ? bias_at(rel0, a.relLen - 1, a.relLen) : 0.0f, far1 = a.rel ? bias_at(rel1, a.relLen - 1, a.relLen) : 0.0f;
@@ -231,15 +236,16 @@ __global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(con
 #pragma unroll
             for (int e = 0; e < 4; e++) { s[j][e] = 0.0f; sl[j][e] = 0.0f; }
         const uint32_t kAddr = smem_u32(K);
-#pragma unroll 4
-        for (int kk = 0; kk < a.kw / 16; kk++) {
-            uint32_t ah[4], al[4], bk[4];
-            ldm_x4(ah, qAddr + kk * 32);
-            ldm_x4(al, qAddr + qlDelta + kk * 32);
-            ldm_x4(bk, kAddr + swizzled(kRow, kk * 2 + kHalf, kGdKeys));
-            mma_bf16(s[0], ah, bk[0], bk[1]); mma_bf16(s[1], ah, bk[2], bk[3]);
-            mma_bf16(sl[0], al, bk[0], bk[1]); mma_bf16(sl[1], al, bk[2], bk[3]);
-        }
+        for (int c = 0; c < S.kb; c++)
+#pragma unroll
+            for (int kk = 0; kk < 4; kk++) {
+                uint32_t ah[4], al[4], bk[4];
+                ldm_x4(ah, qAddr + c * 128 + kk * 32);
+                ldm_x4(al, qAddr + qlDelta + c * 128 + kk * 32);
+                ldm_x4(bk, kAddr + kOff[kk] + c * (kGdKeys * 128));
+                mma_bf16(s[0], ah, bk[0], bk[1]); mma_bf16(s[1], ah, bk[2], bk[3]);
+                mma_bf16(sl[0], al, bk[0], bk[1]); mma_bf16(sl[1], al, bk[2], bk[3]);
+            }
 #pragma unroll
         for (int j = 0; j < 2; j++)
 #pragma unroll
@@ -295,13 +301,12 @@ __global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(con
         for (int c = 0; c < VN; c += 4) {
             if (c >= vt) break;
             uint32_t bv[2][4];
-            const bool two = c + 2 < vt;                     // value columns come in pairs of tiles
-            ldm_x4_t(bv[0], vAddr + swizzled(vRow, c + vHalf, kGdKeys));
-            ldm_x4_t(bv[1], vAddr + swizzled(vRow, (two ? c + 2 : c) + vHalf, kGdKeys));
+            ldm_x4_t(bv[0], vAddr + vOff[(c & 7) / 2] + (c >> 3) * (kGdKeys * 128));
+            ldm_x4_t(bv[1], vAddr + vOff[(c & 7) / 2 + 1] + (c >> 3) * (kGdKeys * 128));
             mma_bf16(o[c], ph, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], ph, bv[0][2], bv[0][3]);
-            if (two) { mma_bf16(o[c + 2], ph, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], ph, bv[1][2], bv[1][3]); }
+            mma_bf16(o[c + 2], ph, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], ph, bv[1][2], bv[1][3]);
             mma_bf16(o[c], pl, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], pl, bv[0][2], bv[0][3]);
-            if (two) { mma_bf16(o[c + 2], pl, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], pl, bv[1][2], bv[1][3]); }
+            mma_bf16(o[c + 2], pl, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], pl, bv[1][2], bv[1][3]);
         }
         if (++stage == stages) { stage = 0; phase ^= 1; }
         __syncwarp();
@@ -462,10 +467,10 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const __grid_
     if (tid == 0)
         for (; issued < min(kGpStages - 1, tiles); issued++) load(issued);
     const __nv_bfloat16* q0 = qp + ((size_t)blockIdx.y * rows + r0) * a.kw;
-    for (int i = tid; i < kGpRows * kq; i += kGpThreads) {
-        const int r = i / kq, c = i - r * kq;
+    for (int i = tid; i < kGpRows * S.kb * 8; i += kGpThreads) {
+        const int r = i / (S.kb * 8), c = i - r * (S.kb * 8);
         *reinterpret_cast<uint4*>(Qs + r * S.LDQ + c * 8) =
-            r0 + r < rows ? *reinterpret_cast<const uint4*>(q0 + (size_t)r * a.kw + c * 8) : make_uint4(0, 0, 0, 0);
+            r0 + r < rows && c < kq ? *reinterpret_cast<const uint4*>(q0 + (size_t)r * a.kw + c * 8) : make_uint4(0, 0, 0, 0);
     }
     __syncthreads();
     const int w0 = r0 + warp * 16, ra = w0 + rl, rb = ra + 8;
@@ -475,8 +480,12 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const __grid_
     const float* relB = a.rel ? a.rel + (size_t)(g * rep + rb % rep) * a.relLen : nullptr;
     const float farA = a.rel ? bias_at(relA, a.relLen - 1, a.relLen) : 0.0f, farB = a.rel ? bias_at(relB, a.relLen - 1, a.relLen) : 0.0f;
     const uint32_t qAddr = smem_u32(Qs) + (uint32_t)(((warp * 16 + (lane & 15)) * S.LDQ + (lane >> 4) * 8) * 2);
-    const int kRow = (lane & 7) + ((lane >> 4) << 3), kHalf = (lane >> 3) & 1;       // operand B from rows of keys
-    const int vRow = (lane & 7) + (((lane >> 3) & 1) << 3), vHalf = lane >> 4;       // … read transposed
+    uint32_t kOff[4], vOff[4];                               // operand B, columns 16i of a box: from rows of keys, and read transposed
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        kOff[i] = swizzled((lane & 7) + ((lane >> 4) << 3), 2 * i + ((lane >> 3) & 1), 0);
+        vOff[i] = swizzled((lane & 7) + (((lane >> 3) & 1) << 3), 2 * i + (lane >> 4), 0);
+    }
     float o[VN][4];
 #pragma unroll
     for (int j = 0; j < VN; j++) { o[j][0] = 0.0f; o[j][1] = 0.0f; o[j][2] = 0.0f; o[j][3] = 0.0f; }
@@ -496,16 +505,18 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const __grid_
 #pragma unroll
         for (int j = 0; j < NT; j++) { s[j][0] = 0.0f; s[j][1] = 0.0f; s[j][2] = 0.0f; s[j][3] = 0.0f; }
         const uint32_t kAddr = smem_u32(K);
-        for (int kk = 0; kk < a.kw / 16; kk++) {
-            uint32_t aq[4];
-            ldm_x4(aq, qAddr + kk * 32);
+        for (int c = 0; c < S.kb; c++)
 #pragma unroll
-            for (int n = 0; n < NT; n += 2) {
-                uint32_t bk[4];
-                ldm_x4(bk, kAddr + (uint32_t)(n * 8 * 128) + swizzled(kRow, kk * 2 + kHalf, KEYS));
-                mma_bf16(s[n], aq, bk[0], bk[1]); mma_bf16(s[n + 1], aq, bk[2], bk[3]);
+            for (int kk = 0; kk < 4; kk++) {
+                uint32_t aq[4];
+                ldm_x4(aq, qAddr + c * 128 + kk * 32);
+#pragma unroll
+                for (int n = 0; n < NT; n += 2) {
+                    uint32_t bk[4];
+                    ldm_x4(bk, kAddr + kOff[kk] + c * (KEYS * 128) + n * 8 * 128);
+                    mma_bf16(s[n], aq, bk[0], bk[1]); mma_bf16(s[n + 1], aq, bk[2], bk[3]);
+                }
             }
-        }
         if (shared) {
 #pragma unroll
             for (int j = 0; j < NT; j++) {
@@ -560,14 +571,12 @@ __global__ void __launch_bounds__(kGpThreads, 1) k_grouped_prefill(const __grid_
             for (int c = 0; c < VN; c += 4) {
                 if (c >= vt) break;
                 uint32_t bv[2][4];
-                const bool two = c + 2 < vt;                 // value columns come in pairs of tiles
-                const uint32_t at = vAddr + (uint32_t)(kk * 16 * 128);
-                ldm_x4_t(bv[0], at + swizzled(vRow, c + vHalf, KEYS));
-                ldm_x4_t(bv[1], at + swizzled(vRow, (two ? c + 2 : c) + vHalf, KEYS));
+                ldm_x4_t(bv[0], vAddr + vOff[(c & 7) / 2] + (c >> 3) * (KEYS * 128) + kk * 16 * 128);
+                ldm_x4_t(bv[1], vAddr + vOff[(c & 7) / 2 + 1] + (c >> 3) * (KEYS * 128) + kk * 16 * 128);
                 mma_bf16(o[c], ph, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], ph, bv[0][2], bv[0][3]);
-                if (two) { mma_bf16(o[c + 2], ph, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], ph, bv[1][2], bv[1][3]); }
+                mma_bf16(o[c + 2], ph, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], ph, bv[1][2], bv[1][3]);
                 mma_bf16(o[c], pl, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], pl, bv[0][2], bv[0][3]);
-                if (two) { mma_bf16(o[c + 2], pl, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], pl, bv[1][2], bv[1][3]); }
+                mma_bf16(o[c + 2], pl, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], pl, bv[1][2], bv[1][3]);
             }
         }
         release();
