@@ -228,7 +228,7 @@ const char* grouped_attn_check(const GroupedAttnArgs& a) {
     if (a.H % a.G != 0) return "the key/value heads must divide the query heads";
     if (a.dim > kGaMaxDim || a.vdim > kGaMaxDim) return "head size not supported";
     if ((long)a.B * a.T > 65535 || (long)a.B * a.G > 65535 || (long)a.T * (a.H / a.G) > 65535l * kGaRows) return "too many rows";
-    if (a.B * a.G * ((a.H / a.G + 15) / 16) > kAttnTickets) return "too many heads";
+    if (a.B * a.G * ((a.H / a.G + 7) / 8) > kAttnTickets) return "too many heads";
     return nullptr;
 }
 

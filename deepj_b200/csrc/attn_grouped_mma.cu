@@ -1,9 +1,10 @@
 // Grouped attention on the tensor cores (bf16 cache); what a score is made of is described in attn_grouped.cu.
 //
-//   k_grouped_decode    one token per sequence.  grid (key splits, blocks of 16 query heads of a group, B·G): the heads of a group
-//                       are the rows of one 16-row operand, so a cached row is read once per group.  Eight (or four) warps walk tiles
+//   k_grouped_decode    one token per sequence.  grid (key splits, blocks of eight query heads of a group, B·G): the heads are the
+//                       rows of one 16-row operand, their queries (and softmax weights) as bf16 high halves in rows 0-7 and
+//                       low halves in rows 8-15, so one product takes 16 bits of them.  Eight (or four) warps walk tiles
 //                       of 16 keys, each through a private ring of tensor copies, as deep as shared memory allows, that starts before the dependency wait; the
-//                       block that holds the newest position norms and appends it.  Queries enter as two bf16 halves.  Warps merge
+//                       block that holds the newest position norms and appends it.  Warps merge
 //                       in shared memory, blocks through partials that the last one to finish (a ticket) adds up.
 //   k_grouped_prefill   prompt chunks: 128 rows (token, head in the group) per block, 16 per warp, key tiles in three stages.
 // Key and value rows travel as 64-column boxes with 128-byte swizzle.
@@ -63,8 +64,8 @@ __device__ __forceinline__ uint32_t swizzled(int r, int c, int keys) { return (u
 size_t gd_smem(const GroupedAttnArgs& a, int warps, int stages) {
     const bool shared = a.vcache == nullptr;
     const GdShape g = gd_shape(a.kw, a.vw, shared, kGdKeys);
-    const size_t ring = (size_t)warps * stages * g.tile, merge = (size_t)warps * 16 * ((shared ? a.kw : a.vw) + 4) * 4;
-    return 1024 + std::max(ring, merge) + (size_t)2 * 16 * g.LDQ * 2 + (size_t)(a.kw + a.vw + 16) * 2 + (size_t)warps * stages * kGdKeys * 4;
+    const size_t ring = (size_t)warps * stages * g.tile, merge = (size_t)warps * 8 * ((shared ? a.kw : a.vw) + 4) * 4;
+    return 1024 + std::max(ring, merge) + (size_t)16 * g.LDQ * 2 + (size_t)(a.kw + a.vw + 16) * 2 + (size_t)warps * stages * kGdKeys * 4;
 }
 
 // VN: most output n-tiles (eight value columns each), NW: warps
@@ -82,15 +83,15 @@ __global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(con
     const int Vp = shared ? a.kw : a.vw, vt = Vp / 8;
     const uint32_t raw = smem_u32(gd_raw), skip = ((raw + 1023u) & ~1023u) - raw;
     unsigned char* ring = gd_raw + skip;
-    const size_t ringBytes = max((size_t)NW * stages * S.tile, (size_t)NW * 16 * (Vp + 4) * 4);
-    __nv_bfloat16* Qh = reinterpret_cast<__nv_bfloat16*>(ring + ringBytes);          // [16][LDQ], then the low halves
-    float* scales = reinterpret_cast<float*>(Qh + 2 * 16 * S.LDQ);                   // [warp][stage][16]
+    const size_t ringBytes = max((size_t)NW * stages * S.tile, (size_t)NW * 8 * (Vp + 4) * 4);
+    __nv_bfloat16* Qh = reinterpret_cast<__nv_bfloat16*>(ring + ringBytes);          // [8][LDQ] high halves, then the low ones
+    float* scales = reinterpret_cast<float*>(Qh + 16 * S.LDQ);                   // [warp][stage][16]
     __nv_bfloat16* newK = reinterpret_cast<__nv_bfloat16*>(scales + NW * stages * kGdKeys);
     __nv_bfloat16* newV = newK + a.kw;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, rl = lane >> 2, t4 = lane & 3;
     unsigned char* mine = ring + warp * stages * S.tile;
     float* mySc = scales + warp * stages * kGdKeys;
-    const int rep = a.H / a.G, b = blockIdx.z / a.G, g = blockIdx.z - b * a.G, h0 = g * rep + blockIdx.y * 16, nrow = min(16, rep - (int)blockIdx.y * 16);
+    const int rep = a.H / a.G, b = blockIdx.z / a.G, g = blockIdx.z - b * a.G, h0 = g * rep + blockIdx.y * 8, nrow = min(8, rep - (int)blockIdx.y * 8);
     // The next kernel is not let in early (griddepcontrol.launch_dependents): short contexts keep some SMs busy, and a projection
     // whose blocks all go to the others streams its weights through those alone.
     if (!a.early) pdl_wait();
@@ -180,29 +181,28 @@ __global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(con
             if (shared) v *= kg[e];
             const __nv_bfloat16 hi = __float2bfloat16_rn(v);
             Qh[r * S.LDQ + i] = hi;
-            Qh[(16 + r) * S.LDQ + i] = __float2bfloat16_rn(v - __bfloat162float(hi));
+            Qh[(8 + r) * S.LDQ + i] = __float2bfloat16_rn(v - __bfloat162float(hi));
         }
     }
-    for (int i = tid; i < (16 - nrow) * S.LDQ / 2; i += 32 * NW) {       // rows of no head
+    for (int i = tid; i < (8 - nrow) * S.LDQ / 2; i += 32 * NW) {        // rows of no head
         reinterpret_cast<uint32_t*>(Qh + nrow * S.LDQ)[i] = 0;
-        reinterpret_cast<uint32_t*>(Qh + (16 + nrow) * S.LDQ)[i] = 0;
+        reinterpret_cast<uint32_t*>(Qh + (8 + nrow) * S.LDQ)[i] = 0;
     }
     __syncthreads();
 
-    const uint32_t qAddr = smem_u32(Qh) + (uint32_t)(((lane & 15) * S.LDQ + (lane >> 4) * 8) * 2), qlDelta = (uint32_t)(16 * S.LDQ * 2);
+    const uint32_t qAddr = smem_u32(Qh) + (uint32_t)(((lane & 15) * S.LDQ + (lane >> 4) * 8) * 2);
     uint32_t kOff[4], vOff[4];                               // operand B, columns 16i of a box: from rows of keys, and read transposed
 #pragma unroll
     for (int i = 0; i < 4; i++) {
         kOff[i] = swizzled((lane & 7) + ((lane >> 4) << 3), 2 * i + ((lane >> 3) & 1), 0);
         vOff[i] = swizzled((lane & 7) + (((lane >> 3) & 1) << 3), 2 * i + (lane >> 4), 0);
     }
-    const float* rel0 = a.rel ? a.rel + (size_t)(h0 + min(rl, nrow - 1)) * a.relLen : nullptr;
-    const float* rel1 = a.rel ? a.rel + (size_t)(h0 + min(rl + 8, nrow - 1)) * a.relLen : nullptr;
-    const float far0 = a.rel ? bias_at(rel0, a.relLen - 1, a.relLen) : 0.0f, far1 = a.rel ? bias_at(rel1, a.relLen - 1, a.relLen) : 0.0f;
-    float o[VN][4];
+    const float* rel = a.rel ? a.rel + (size_t)(h0 + min(rl, nrow - 1)) * a.relLen : nullptr;
+    const float far = a.rel ? bias_at(rel, a.relLen - 1, a.relLen) : 0.0f;
+    float o[VN][4];                                          // by the weights' high halves, and by the low ones
 #pragma unroll
     for (int j = 0; j < VN; j++) { o[j][0] = 0.0f; o[j][1] = 0.0f; o[j][2] = 0.0f; o[j][3] = 0.0f; }
-    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;
+    float m = -INFINITY, l = 0.0f;
     int stage = 0, phase = 0;
     for (int tile = tLo + warp; tile < tHi; tile += NW) {
         if (!__all_sync(0xffffffffu, mbar_wait(bar(stage), phase, &s_abort, p.error, 221))) {
@@ -230,71 +230,54 @@ __global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(con
             const int next = tile + (stages - 1) * NW;
             if (next < tHi) load(next, stage == 0 ? stages - 1 : stage - 1);
         }
-        float s[2][4], sl[2][4];                             // by the queries' high and low halves
+        float bias[2][2] = {{far, far}, {far, far}};
+        if (a.rel && pos - (k0 + kGdKeys - 1) < a.relLen - 1) {
+#pragma unroll
+            for (int j = 0; j < 2; j++)
+#pragma unroll
+                for (int e = 0; e < 2; e++) bias[j][e] = bias_at(rel, max(pos - k0 - (j * 8 + 2 * t4 + e), 0), a.relLen);
+        }
+        float s[2][4];                                       // by the queries' high halves, and by the low ones
 #pragma unroll
         for (int j = 0; j < 2; j++)
 #pragma unroll
-            for (int e = 0; e < 4; e++) { s[j][e] = 0.0f; sl[j][e] = 0.0f; }
+            for (int e = 0; e < 4; e++) s[j][e] = 0.0f;
         const uint32_t kAddr = smem_u32(K);
         for (int c = 0; c < S.kb; c++)
 #pragma unroll
             for (int kk = 0; kk < 4; kk++) {
-                uint32_t ah[4], al[4], bk[4];
-                ldm_x4(ah, qAddr + c * 128 + kk * 32);
-                ldm_x4(al, qAddr + qlDelta + c * 128 + kk * 32);
+                uint32_t aq[4], bk[4];
+                ldm_x4(aq, qAddr + c * 128 + kk * 32);
                 ldm_x4(bk, kAddr + kOff[kk] + c * (kGdKeys * 128));
-                mma_bf16(s[0], ah, bk[0], bk[1]); mma_bf16(s[1], ah, bk[2], bk[3]);
-                mma_bf16(sl[0], al, bk[0], bk[1]); mma_bf16(sl[1], al, bk[2], bk[3]);
+                mma_bf16(s[0], aq, bk[0], bk[1]); mma_bf16(s[1], aq, bk[2], bk[3]);
             }
+        float w[2][2], mx = -INFINITY;
 #pragma unroll
-        for (int j = 0; j < 2; j++)
-#pragma unroll
-            for (int e = 0; e < 4; e++) s[j][e] += sl[j][e];
-        float mx0 = -INFINITY, mx1 = -INFINITY;
-        if (shared) {
-#pragma unroll
-            for (int j = 0; j < 2; j++) {
+        for (int j = 0; j < 2; j++) {
+            w[j][0] = s[j][0] + s[j][2]; w[j][1] = s[j][1] + s[j][3];
+            if (shared) {
                 const float2 f = *reinterpret_cast<const float2*>(sc + j * 8 + 2 * t4);
-                s[j][0] *= f.x; s[j][1] *= f.y; s[j][2] *= f.x; s[j][3] *= f.y;
+                w[j][0] *= f.x; w[j][1] *= f.y;
             }
-        }
-        if (k0 + kGdKeys - 1 <= pos && (a.rel == nullptr || pos - (k0 + kGdKeys - 1) >= a.relLen - 1)) {       // the whole tile is seen, and far
-#pragma unroll
-            for (int j = 0; j < 2; j++)
-#pragma unroll
-                for (int e = 0; e < 2; e++) { s[j][e] += far0; s[j][2 + e] += far1; }
-        } else {
-#pragma unroll
-            for (int j = 0; j < 2; j++)
-#pragma unroll
-                for (int e = 0; e < 2; e++) {
-                    const int d = pos - k0 - (j * 8 + 2 * t4 + e);
-                    if (a.rel && d >= 0) { s[j][e] += bias_at(rel0, d, a.relLen); s[j][2 + e] += bias_at(rel1, d, a.relLen); }
-                    if (d < 0) { s[j][e] = -INFINITY; s[j][2 + e] = -INFINITY; }
-                }
-        }
-#pragma unroll
-        for (int j = 0; j < 2; j++)
-#pragma unroll
-            for (int e = 0; e < 2; e++) { mx0 = fmaxf(mx0, s[j][e]); mx1 = fmaxf(mx1, s[j][2 + e]); }
-        mx0 = fmaxf(m0, quad_max(mx0)); mx1 = fmaxf(m1, quad_max(mx1));      // finite: a tile's first key is always seen
-        const float c0 = ex2(m0 - mx0), c1 = ex2(m1 - mx1);
-        m0 = mx0; m1 = mx1;
-        float ps0 = 0.0f, ps1 = 0.0f;
-#pragma unroll
-        for (int j = 0; j < 2; j++)
 #pragma unroll
             for (int e = 0; e < 2; e++) {
-                s[j][e] = ex2(s[j][e] - m0); s[j][2 + e] = ex2(s[j][2 + e] - m1);
-                ps0 += s[j][e]; ps1 += s[j][2 + e];
+                w[j][e] = k0 + j * 8 + 2 * t4 + e <= pos ? w[j][e] + bias[j][e] : -INFINITY;
+                mx = fmaxf(mx, w[j][e]);
             }
-        l0 = l0 * c0 + ps0; l1 = l1 * c1 + ps1;
-        uint32_t ph[4], pl[4];
-        split_bf16(s[0][0], s[0][1], ph[0], pl[0]); split_bf16(s[0][2], s[0][3], ph[1], pl[1]);
-        split_bf16(s[1][0], s[1][1], ph[2], pl[2]); split_bf16(s[1][2], s[1][3], ph[3], pl[3]);
-        if (__any_sync(0xffffffffu, c0 != 1.0f || c1 != 1.0f)) {
+        }
+        mx = fmaxf(m, quad_max(mx));                         // finite: a tile's first key is always seen
+        const float corr = ex2(m - mx);
+        m = mx;
 #pragma unroll
-            for (int c = 0; c < VN; c++) { o[c][0] *= c0; o[c][1] *= c0; o[c][2] *= c1; o[c][3] *= c1; }
+        for (int j = 0; j < 2; j++)
+#pragma unroll
+            for (int e = 0; e < 2; e++) w[j][e] = ex2(w[j][e] - m);
+        l = l * corr + ((w[0][0] + w[0][1]) + (w[1][0] + w[1][1]));
+        uint32_t pw4[4];                                     // rows 0-7: high halves, rows 8-15: low halves
+        split_bf16(w[0][0], w[0][1], pw4[0], pw4[1]); split_bf16(w[1][0], w[1][1], pw4[2], pw4[3]);
+        if (__any_sync(0xffffffffu, corr != 1.0f)) {
+#pragma unroll
+            for (int c = 0; c < VN; c++) { o[c][0] *= corr; o[c][1] *= corr; o[c][2] *= corr; o[c][3] *= corr; }
         }
         const uint32_t vAddr = smem_u32(V);
 #pragma unroll
@@ -303,48 +286,43 @@ __global__ void __launch_bounds__(32 * NW, VN <= 8 ? 2 : 1) k_grouped_decode(con
             uint32_t bv[2][4];
             ldm_x4_t(bv[0], vAddr + vOff[(c & 7) / 2] + (c >> 3) * (kGdKeys * 128));
             ldm_x4_t(bv[1], vAddr + vOff[(c & 7) / 2 + 1] + (c >> 3) * (kGdKeys * 128));
-            mma_bf16(o[c], ph, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], ph, bv[0][2], bv[0][3]);
-            mma_bf16(o[c + 2], ph, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], ph, bv[1][2], bv[1][3]);
-            mma_bf16(o[c], pl, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], pl, bv[0][2], bv[0][3]);
-            mma_bf16(o[c + 2], pl, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], pl, bv[1][2], bv[1][3]);
+            mma_bf16(o[c], pw4, bv[0][0], bv[0][1]); mma_bf16(o[c + 1], pw4, bv[0][2], bv[0][3]);
+            mma_bf16(o[c + 2], pw4, bv[1][0], bv[1][1]); mma_bf16(o[c + 3], pw4, bv[1][2], bv[1][3]);
         }
         if (++stage == stages) { stage = 0; phase ^= 1; }
         __syncwarp();
     }
-    l0 = quad_sum(l0); l1 = quad_sum(l1);
-    __syncthreads();                                         // the ring becomes the merge buffer: [warp][16][Vp + 4]
+    l = quad_sum(l);
+    __syncthreads();                                         // the ring becomes the merge buffer: [warp][8][Vp + 4]
     float* mg = reinterpret_cast<float*>(ring);
     const int mrow = Vp + 4;
     {
-        float* d0 = mg + (warp * 16 + rl) * mrow; float* d1 = d0 + 8 * mrow;
+        float* dst = mg + (warp * 8 + rl) * mrow;
 #pragma unroll
         for (int c = 0; c < VN; c++)
-            if (c < vt) {
-                d0[c * 8 + 2 * t4] = o[c][0]; d0[c * 8 + 2 * t4 + 1] = o[c][1];
-                d1[c * 8 + 2 * t4] = o[c][2]; d1[c * 8 + 2 * t4 + 1] = o[c][3];
-            }
-        if (t4 == 0) { d0[Vp] = m0; d0[Vp + 1] = l0; d1[Vp] = m1; d1[Vp + 1] = l1; }
+            if (c < vt) *reinterpret_cast<float2*>(dst + c * 8 + 2 * t4) = make_float2(o[c][0] + o[c][2], o[c][1] + o[c][3]);
+        if (t4 == 0) { dst[Vp] = m; dst[Vp + 1] = l; }
     }
     __syncthreads();
     // partials: [row][split][pw], the maximum and the sum in the last four floats, the values padded to whole 16-byte pieces
     const int pw = Vp + 4;
-    float* part = a.ws + ((size_t)blockIdx.z * rep + blockIdx.y * 16) * splits * pw;
+    float* part = a.ws + ((size_t)blockIdx.z * rep + blockIdx.y * 8) * splits * pw;
     for (int r = warp; r < nrow; r += NW) {
         float mw[NW], m = active == 1 && a.sink ? 0.0f : -INFINITY;
 #pragma unroll
-        for (int w = 0; w < NW; w++) { mw[w] = mg[(w * 16 + r) * mrow + Vp]; m = fmaxf(m, mw[w]); }
+        for (int w = 0; w < NW; w++) { mw[w] = mg[(w * 8 + r) * mrow + Vp]; m = fmaxf(m, mw[w]); }
         float l = active == 1 && a.sink ? ex2(-m) : 0.0f;
 #pragma unroll
         for (int w = 0; w < NW; w++) {
             mw[w] = ex2(mw[w] - m);
-            l = fmaf(mw[w], mg[(w * 16 + r) * mrow + Vp + 1], l);
+            l = fmaf(mw[w], mg[(w * 8 + r) * mrow + Vp + 1], l);
         }
         float* dst = active == 1 ? a.out + (size_t)b * a.ldo + (size_t)(h0 + r) * a.vdim : part + ((size_t)r * splits + blockIdx.x) * pw;
         const float norm = active == 1 ? 1.0f / l : 1.0f;
         for (int i = lane; i < (active == 1 ? a.vdim : Vp); i += 32) {
             float v = 0.0f;
 #pragma unroll
-            for (int w = 0; w < NW; w++) v = fmaf(mw[w], mg[(w * 16 + r) * mrow + i], v);
+            for (int w = 0; w < NW; w++) v = fmaf(mw[w], mg[(w * 8 + r) * mrow + i], v);
             dst[i] = v * norm;
         }
         if (active > 1 && lane == 0) { dst[Vp] = m; dst[Vp + 1] = l; }
@@ -649,7 +627,7 @@ void decode_with(const GroupedAttnArgs& a, cudaStream_t s) {
     raise(k_grouped_decode<VN, NW>, done);
     GdParams p = params(a, kGdKeys);
     p.splits = grouped_mma_splits(a); p.stages = gd_stages(a);
-    launch_k(k_grouped_decode<VN, NW>, dim3((unsigned)p.splits, (unsigned)((a.H / a.G + 15) / 16), (unsigned)(a.B * a.G)), dim3(32 * NW), gd_smem(a, NW, p.stages), s, true, p);
+    launch_k(k_grouped_decode<VN, NW>, dim3((unsigned)p.splits, (unsigned)((a.H / a.G + 7) / 8), (unsigned)(a.B * a.G)), dim3(32 * NW), gd_smem(a, NW, p.stages), s, true, p);
 }
 template <int VN>
 void decode(const GroupedAttnArgs& a, cudaStream_t s) {
@@ -670,7 +648,7 @@ bool grouped_mma_fits(const GroupedAttnArgs& a) {
     return a.bf16 && (size_t)a.B * a.G * a.maxSeq < (1u << 31) && a.kw <= 256 && a.vw <= 256 && a.kw % 16 == 0 && a.vw % 16 == 0 && (a.vcache != nullptr || a.kpitch % 64 == 0);
 }
 int grouped_mma_splits(const GroupedAttnArgs& a) {
-    const int blocks = a.B * a.G * ((a.H / a.G + 15) / 16), tiles = (a.maxSeq + kGdKeys - 1) / kGdKeys, warps = gd_warps(a);
+    const int blocks = a.B * a.G * ((a.H / a.G + 7) / 8), tiles = (a.maxSeq + kGdKeys - 1) / kGdKeys, warps = gd_warps(a);
     return std::max(1, std::min({gd_blocks_per_sm(a) * g_num_sms / blocks, (tiles + warps - 1) / warps, 512}));
 }
 void launch_grouped_decode(const GroupedAttnArgs& a, cudaStream_t s) {
