@@ -1,4 +1,4 @@
-"""The ops over bf16 weights (77-81), each mechanism alone, against plain numpy (tests/punilix_ref.py)."""
+"""The ops over bf16 weights (77-82), each mechanism alone, against plain numpy (tests/punilix_ref.py)."""
 import numpy as np
 import pytest
 

@@ -263,7 +263,7 @@ def recurrence_data(B, T, H, dim, vdim, seed, forget):
 
 
 @pytest.mark.parametrize("exact", [1, 0])
-@pytest.mark.parametrize("H,dim,vdim,cap", [(2, 32, 64, 12.0), (3, 24, 40, 5.0), (1, 128, 96, 15.0), (2, 21, 10, 3.0), (1, 256, 48, 8.0), (1, 200, 33, 30.0), (1, 300, 16, 10.0)])
+@pytest.mark.parametrize("H,dim,vdim,cap", [(2, 48, 64, 10.0), (3, 24, 40, 5.0), (1, 128, 96, 15.0), (2, 21, 10, 3.0), (1, 256, 48, 8.0), (1, 200, 33, 30.0), (1, 300, 16, 10.0)])
 def test_recurrence(dev, exact, H, dim, vdim, cap):
     B, T = 2, 150
     tol = 2e-5 if exact else 2e-2

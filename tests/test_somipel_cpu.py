@@ -48,7 +48,7 @@ def test_recurrence_against_its_closed_form():
 def test_distance_rows():
     got = [ref.distance_bucket(n, 8, 32) for n in (0, 3, 4, 5, 6, 8, 11, 16, 31, 32, 1000)]
     assert got == [0, 3, 4, 4, 4, 5, 5, 6, 7, 7, 7]      # 4 + floor(4 · log2(n/4) / 3), whole numbers reached exactly
-    for rows, far in ((8, 32), (12, 37), (32, 128), (32, 120), (2, 5), (24, 96), (6, 400), (64, 33)):
+    for rows, far in ((8, 32), (12, 37), (32, 128), (32, 100), (2, 5), (24, 96), (6, 400), (64, 33)):
         table = distance_buckets(rows, far, 5000)
         assert table[-1] == rows - 1 and (len(table) < 2 or table[-2] < rows - 1)
         want = [ref.distance_bucket(n, rows, far) for n in range(len(table) + 50)]
